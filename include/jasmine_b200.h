@@ -222,6 +222,9 @@ jsm_status jsm_trace_end(uint64_t* h_stamps, int max_launches, int* n_launches, 
  * d_table: F32 [max_pos, d/2, 4]. Built on the host with the reference's
  * sequence of roundings and uploaded (synchronous). */
 jsm_status jsm_rope_table(float* d_table, int mode, int d, float theta, int max_pos, void* stream);
+/* Rotate-half tables: (cos, sin) of m * base^(-2i/d) for pair i = (component i, component i + d/2) at position m, computed in
+ * double precision.  d_table: F32 [max_pos, d/2, 2] (synchronous). */
+jsm_status jsm_rope_half_table(float* d_table, int d, double base, int max_pos);
 /* x, out: token-major [T, n_heads*d] (F32 or BF16); positions: I32 [T] or NULL (= t). */
 jsm_status jsm_rope_apply(const void* d_x, void* d_out, jsm_dtype dtype, const float* d_table, int d, int n_heads,
                           const int32_t* d_positions, int T, void* stream);
@@ -465,6 +468,69 @@ jsm_status jsm_llama_set_context(jsm_model* m, int seq, int context_len);
 jsm_status jsm_llama_reset(jsm_model* m);
 /* bytes of weights read by one decode step on this rank, and KV bytes per cached token */
 jsm_status jsm_llama_step_bytes(jsm_model* m, uint64_t* weight_bytes, uint64_t* kv_bytes_per_token);
+
+/* ---- decoder with a list of layers (new; not in the reference) -----------------------------------------------------
+ * Every layer names its mixer and the mixer's sizes, and optionally a feed-forward; the norm sits on the sublayer's output,
+ *     x <- x + norm1(mixer(x)),   x <- x + norm2(ff(x)),      norm(y) = y / sqrt(mean(y^2) + eps) * w,
+ * with an fp32 residual stream x.  Logits = final norm of x times the embedding table, through cap * tanh(l / cap).
+ * Mixers:
+ *  latent attention  per head `dim` unrotated and `rot_dim` rotated query / key components (rotate-half pairs, base
+ *                    rope_base) and values of `vdim`; keys and values are expanded from an RMS-normed latent of kv_rank
+ *                    components, the rotated key part is shared by the heads; softmax over the last `window` positions.
+ *  selective scan    input projection to (x, z) of `inner` channels, causal convolution of `taps` taps and silu on x,
+ *                    then S <- exp(dt A) S + dt x B, y = C S + D x with `state` states per channel and a step size dt of
+ *                    rank dt_rank, gated by silu(z).
+ * Feed-forward: g = min(Wg x, limit), u = clamp(Wu x, -limit, limit), Wd (g * sigmoid(1.702 g) * (u + 1)).
+ * Tensors: "embed" [vocab, d_model], "final.norm"; layer L: "lL.norm1", "lL.norm2" (with a feed-forward),
+ * "lL.mlp.gate|up|down", and "lL.mix." + q, dkv, dkv.norm, uk, uv, o (latent attention) or in, conv, conv.b, x, dt, dt.b,
+ * A_log, D, o (selective scan).  A layer with weights_of = J uses layer J's tensors and a cache or state of its own. */
+typedef enum jsm_mixer { JSM_MIXER_LATENT_ATTENTION = 0, JSM_MIXER_SELECTIVE_SCAN = 1 } jsm_mixer;
+typedef struct jsm_layer_config {
+    int32_t mixer, weights_of;                         /* weights_of: -1 = own tensors */
+    int32_t heads, dim, rot_dim, vdim, kv_rank, window; /* latent attention */
+    int32_t inner, state, dt_rank, taps;               /* selective scan */
+    int32_t ff;                                        /* 0 = no feed-forward */
+    float ff_limit;
+    double scale, rope_base;
+} jsm_layer_config;
+typedef struct jsm_decoder_config {
+    int32_t n_layers, d_model, vocab;
+    int32_t dtype;           /* JSM_BF16: bf16 weights and activations; JSM_F32: everything in fp32 */
+    int32_t max_batch, max_context;
+    int32_t max_step_tokens; /* tokens of one pass; longer steps are cut into passes */
+    int32_t n_pages;         /* cache pages of 64 positions; 0 = max_batch full contexts */
+    float norm_eps, logit_softcap; /* logit_softcap 0 = no cap */
+} jsm_decoder_config;
+typedef struct jsm_decoder jsm_decoder;
+
+jsm_status jsm_decoder_create(const jsm_decoder_config* cfg, const jsm_layer_config* layers, jsm_decoder** out);
+jsm_status jsm_decoder_destroy(jsm_decoder* m);
+/* A tensor from HOST memory (bf16 or f32, row-major; vectors as [n, 1]); jsm_decoder_finalize then checks the shapes, packs
+ * and uploads everything and allocates the cache, the states and the workspaces. */
+jsm_status jsm_decoder_set_weight(jsm_decoder* m, const char* name, const void* h_src, int dtype, int rows, int cols);
+jsm_status jsm_decoder_finalize(jsm_decoder* m);
+/* Continuous batching with the rules of the jsm_llama_seq_* calls (rows 0 .. n_active-1, the last row takes a retired
+ * row's place).  stream NULL = a stream of the model.  All calls synchronise it.
+ * jsm_decoder_seq_open   an empty sequence in the next free row
+ * jsm_decoder_step       counts[e] further tokens of row rows[e] for every entry (h_ids: all tokens, entry after entry):
+ *                        whole prompts, portions of prompts and single tokens in any mixture; a row at most once.  want:
+ *                        n_want places in h_ids whose logits are asked for: h_logits F32 [n_want, vocab] and h_next
+ *                        [n_want] (arg-max), either may be NULL.
+ * jsm_decoder_seq_admit  seq_open and the whole prompt; the first generated token
+ * jsm_decoder_step_active one token for every active row */
+jsm_status jsm_decoder_seq_open(jsm_decoder* m, int* row);
+jsm_status jsm_decoder_step(jsm_decoder* m, int n_entries, const int32_t* rows, const int32_t* counts, const int32_t* h_ids,
+                            int n_want, const int32_t* want, int32_t* h_next, float* h_logits, void* stream);
+jsm_status jsm_decoder_seq_admit(jsm_decoder* m, const int32_t* h_prompt, int T, int* row, int32_t* h_first_token,
+                                 float* h_logits_last, void* stream);
+jsm_status jsm_decoder_step_active(jsm_decoder* m, const int32_t* h_ids, int32_t* h_next, float* h_logits, void* stream);
+jsm_status jsm_decoder_seq_retire(jsm_decoder* m, int row, int* moved_from, void* stream);
+jsm_status jsm_decoder_pool_state(jsm_decoder* m, int* n_active, int* free_pages, int* total_pages);
+jsm_status jsm_decoder_context(jsm_decoder* m, int row, int* context_len);
+/* Debugging: the residual stream after every layer of each pass goes to d_buf (F32 [n_layers][tokens][d_model]); NULL = off. */
+jsm_status jsm_decoder_set_tap(jsm_decoder* m, float* d_buf);
+/* bytes of weights one decode step reads, and bytes of cache and state it reads and writes per sequence at a context length */
+jsm_status jsm_decoder_step_bytes(jsm_decoder* m, int context_len, uint64_t* weight_bytes, uint64_t* seq_bytes);
 
 #if defined(__GNUC__)
 #pragma GCC visibility pop

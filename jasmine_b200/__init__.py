@@ -52,6 +52,22 @@ class ModelConfig(C.Structure):
 
 ALLREDUCE_FN = C.CFUNCTYPE(C.c_int, C.c_void_p, C.c_size_t, C.c_int, C.c_void_p, C.c_void_p)
 
+class LayerConfig(C.Structure):
+    _fields_ = [("mixer", C.c_int32), ("weights_of", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32),
+                ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("kv_rank", C.c_int32), ("window", C.c_int32),
+                ("inner", C.c_int32), ("state", C.c_int32), ("dt_rank", C.c_int32), ("taps", C.c_int32),
+                ("ff", C.c_int32), ("ff_limit", C.c_float), ("scale", C.c_double), ("rope_base", C.c_double)]
+
+
+class DecoderConfig(C.Structure):
+    _fields_ = [("n_layers", C.c_int32), ("d_model", C.c_int32), ("vocab", C.c_int32), ("dtype", C.c_int32),
+                ("max_batch", C.c_int32), ("max_context", C.c_int32), ("max_step_tokens", C.c_int32), ("n_pages", C.c_int32),
+                ("norm_eps", C.c_float), ("logit_softcap", C.c_float)]
+
+
+# jsm_mixer
+MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN = 0, 1
+
 # every symbol include/jasmine_b200.h declares: (restype, argtypes)
 _vp, _i, _f, _sz, _u64, _i64 = C.c_void_p, C.c_int, C.c_float, C.c_size_t, C.c_uint64, C.c_int64
 SYMBOLS = {
@@ -84,6 +100,7 @@ SYMBOLS = {
     "jsm_linear_bf16_packed": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
     "jsm_linear_bf16_packed_chained": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
     "jsm_rope_table": (_i, [_vp, _i, _i, _f, _i, _vp]),
+    "jsm_rope_half_table": (_i, [_vp, _i, C.c_double, _i]),
     "jsm_rope_apply": (_i, [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp]),
     "jsm_rope_apply_qk": (_i, [_vp, _vp, _i, _vp, _vp, _i, _i, _vp, _i, _vp, _i, _vp]),
     "jsm_attn_prefill": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _i, _vp]),
@@ -126,6 +143,19 @@ SYMBOLS = {
     "jsm_llama_set_context": (_i, [_vp, _i, _i]),
     "jsm_llama_reset": (_i, [_vp]),
     "jsm_llama_step_bytes": (_i, [_vp, C.POINTER(_u64), C.POINTER(_u64)]),
+    "jsm_decoder_create": (_i, [C.POINTER(DecoderConfig), C.POINTER(LayerConfig), C.POINTER(_vp)]),
+    "jsm_decoder_destroy": (_i, [_vp]),
+    "jsm_decoder_set_weight": (_i, [_vp, C.c_char_p, _vp, _i, _i, _i]),
+    "jsm_decoder_finalize": (_i, [_vp]),
+    "jsm_decoder_seq_open": (_i, [_vp, C.POINTER(_i)]),
+    "jsm_decoder_step": (_i, [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp]),
+    "jsm_decoder_seq_admit": (_i, [_vp, _vp, _i, C.POINTER(_i), _vp, _vp, _vp]),
+    "jsm_decoder_step_active": (_i, [_vp, _vp, _vp, _vp, _vp]),
+    "jsm_decoder_seq_retire": (_i, [_vp, _i, C.POINTER(_i), _vp]),
+    "jsm_decoder_pool_state": (_i, [_vp, C.POINTER(_i), C.POINTER(_i), C.POINTER(_i)]),
+    "jsm_decoder_context": (_i, [_vp, _i, C.POINTER(_i)]),
+    "jsm_decoder_set_tap": (_i, [_vp, _vp]),
+    "jsm_decoder_step_bytes": (_i, [_vp, _i, C.POINTER(_u64), C.POINTER(_u64)]),
 }
 
 _lib = None

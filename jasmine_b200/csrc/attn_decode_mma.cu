@@ -18,6 +18,7 @@
 // Every mbarrier wait is bounded (tc_utils.cuh); on a timeout the kernel records an error code and returns.
 #include "attn.cuh"
 #include "tc_utils.cuh"
+#include "mma_utils.cuh"
 #include <math.h>
 
 namespace jsm {
@@ -35,28 +36,11 @@ constexpr int DM_SMEM = DM_STAGES * DM_STAGE_BYTES + 1024;
 constexpr int DM_ERR_FULL = 41, DM_ERR_EMPTY = 42;
 static_assert(DM_PAGE == 64, "one stage is one page of 64 tokens");
 
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
 __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
     uint32_t y;
     asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
     return y;
 }
-// d += a[16x16] . b[16x8], bf16 operands, fp32 accumulators
-__device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 // the cache as a matrix of 128-wide rows: row of the first key of block (page, K or V, kv head)
 __device__ __forceinline__ int dm_block_row(int page, int kv, int Hkv, int hk) { return ((page * 2 + kv) * Hkv + hk) * DM_PAGE; }
 

@@ -15,6 +15,7 @@
 // rescale of the accumulator is rare; the final division by the row sum happens in the epilogue.
 // Every wait is bounded; on a timeout the CTA unwinds, frees its TMEM and records a code for the host.
 #include "attn.cuh"
+#include "decoder_ops.cuh"
 #include "tc_utils.cuh"
 #include <stdlib.h>
 #include <math.h>
@@ -409,4 +410,9 @@ jsm_status flash_prefill_launch(const void* q, const void* k, const void* v, voi
     return JSM_OK;
 }
 
+}  // namespace jsm
+
+namespace jsm {
+bool latent_flash_usable(const LatentDims&) { return false; }
+jsm_status latent_flash_launch(const LatentDims&, const void*, const void*, const void*, long long, void*, int, int, cudaStream_t) { return JSM_UNSUPPORTED; }
 }  // namespace jsm

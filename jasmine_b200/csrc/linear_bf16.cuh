@@ -4,7 +4,8 @@
 
 namespace jsm {
 
-enum LinearEpilogue { LIN_NONE = 0, LIN_RELU = 1, LIN_GELU = 2, LIN_SILU_MUL = 3, LIN_RESIDUAL = 4 };
+enum LinearEpilogue { LIN_NONE = 0, LIN_RELU = 1, LIN_GELU = 2, LIN_SILU_MUL = 3, LIN_RESIDUAL = 4,
+                      LIN_CLAMPED_GLU = 5 /* packed weights only */ };
 
 struct LinearArgs {
     const void* X;      // [T, K] bf16
@@ -49,6 +50,7 @@ struct PackedArgs {
     int ssq_stride = 0;       // 0 = T
     float eps = 0.0f;
     float* ssq_out = nullptr;
+    float glu_alpha = 0.0f, glu_limit = 0.0f;  // LIN_CLAMPED_GLU: min(g, l) * sigmoid(alpha * min(g, l)) * (clamp(u, -l, l) + 1)
     // Tensor-parallel exchange fused into the projection (tp_comm.cu describes the protocol).
     // push: the bf16 outputs are stored into this rank's slot of EVERY rank's exchange buffer (peer stores) instead of
     // Y, and the CTA that finishes last releases the call's epoch to every peer's flag word.

@@ -39,6 +39,12 @@ constexpr int PK_MAX_STAGES = 12;
 
 __device__ __noinline__ float pk_gelu(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752440f)); }
 __device__ __forceinline__ float pk_silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }  // 2 ulp division: short code
+// gate/up pair with clamps: min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1)
+__device__ __forceinline__ float pk_clamped_glu(float g, float u, float alpha, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
 
 // 1-D bulk copy global -> shared (this CTA), completion counted in bytes on `bar`; both addresses 16-byte aligned
 __device__ __forceinline__ void bulk_load(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
@@ -91,6 +97,7 @@ struct PkParams {
     __nv_bfloat16* tp_h;
     float* tp_ssq;
     long long tp_wait;
+    float glu_alpha, glu_limit;  // LIN_CLAMPED_GLU
 };
 
 constexpr int TP_TIMEOUT_CODE = 16;  // error word code of an exchange whose peers did not arrive in time (as in tp_comm.cu)
@@ -219,15 +226,18 @@ __global__ void __launch_bounds__(PK_THREADS, 1)
     // 1 / 2 = it pushes its outputs / reduces the ranks' slots into its token operand first, with flags, 4 / 5 = the same
     // with in-band epochs.
     // PRM 5: the pushing projection (plain tiles, bf16, nothing else).
+    // PRM 6, 7, 8: decoders whose norms sit on the sublayers' outputs - 6: gate-up pairs with clamps, bf16 out; 7 / 8: plain
+    // tiles and nothing else, f32 / bf16 out.
     const bool tp_push = TPM == 1 || TPM == 4 || (TPM == 3 && P.tp_mode == 1);
     const bool tp_reduce = TPM == 2 || TPM == 5 || (TPM == 3 && P.tp_mode == 2);
     const bool tp_inband = BN == 16 && (TPM == 4 || TPM == 5 || (TPM == 3 && P.tp_inband != 0));  // (at most 16 tokens)
     constexpr bool FIX = PRM >= 2;
-    const bool paired = PRM < 0 ? P.paired != 0 : (PRM == 1 || PRM == 4);
+    const bool paired = PRM < 0 ? P.paired != 0 : (PRM == 1 || PRM == 4 || PRM == 6);
     const bool has_ssq_in = FIX ? (PRM == 2 || PRM == 4) : P.ssq_in != nullptr;
-    const bool f32o = FIX ? false : P.out_f32 != 0;
+    const bool f32o = FIX ? PRM == 7 : P.out_f32 != 0;
     const float* const biasp = FIX ? nullptr : P.bias;
     const int epi = FIX ? (PRM == 3 ? LIN_RESIDUAL : PRM == 4 ? LIN_SILU_MUL : LIN_NONE) : P.epilogue;
+    auto gate_up = [&](float g, float u) { return PRM == 6 ? pk_clamped_glu(g, u, P.glu_alpha, P.glu_limit) : pk_silu(g) * u; };
     chain_trigger();
     if (threadIdx.x == 0) PK_TRACE(0);  // CTA resident
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -652,7 +662,7 @@ __global__ void __launch_bounds__(PK_THREADS, 1)
                                 const int t = c0 + j;
                                 if (t < P.T) {
                                     const float sc = scaled ? row_scale[t] : 1.0f;
-                                    const float v = pk_silu(__uint_as_float(r[j]) * sc) * (pair_smem[f * 17 + j] * sc);
+                                    const float v = gate_up(__uint_as_float(r[j]) * sc, pair_smem[f * 17 + j] * sc);
                                     if (f32o) reinterpret_cast<float*>(P.Y)[(size_t)t * P.N + n] = v;
                                     else reinterpret_cast<__nv_bfloat16*>(P.Y)[(size_t)t * P.N + n] = __float2bfloat16_rn(v);
                                 }
@@ -845,7 +855,7 @@ __global__ void __launch_bounds__(PK_THREADS, 1)
                             if (paired) {
 #pragma unroll 1
                                 for (int j = 0; j < 4; ++j) {  // one copy of the division: the values take turns in v[0]
-                                    const float y = pk_silu(v[0]) * uu[0];
+                                    const float y = gate_up(v[0], uu[0]);
                                     v[0] = v[1]; v[1] = v[2]; v[2] = v[3]; v[3] = y;
                                     uu[0] = uu[1]; uu[1] = uu[2]; uu[2] = uu[3];
                                 }
@@ -1121,8 +1131,10 @@ jsm_status linear_packed_launch(const PackedArgs& a, cudaStream_t st) {
     if (a.K <= 0 || a.K % 8) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: K (%d) must be a positive multiple of 8", a.K);
     if (a.N % 4) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: N (%d) must be a multiple of 4", a.N);
     if (a.T > 256) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: at most 256 tokens per launch (%d)", a.T);
-    if (a.epilogue < LIN_NONE || a.epilogue > LIN_RESIDUAL) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: epilogue %d", a.epilogue);
-    const int paired = a.epilogue == LIN_SILU_MUL ? 1 : 0;
+    if (a.epilogue < LIN_NONE || a.epilogue > LIN_CLAMPED_GLU) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: epilogue %d", a.epilogue);
+    const int paired = a.epilogue == LIN_SILU_MUL || a.epilogue == LIN_CLAMPED_GLU ? 1 : 0;
+    if (a.epilogue == LIN_CLAMPED_GLU && (a.out_f32 || a.ssq_in || a.tp))
+        JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: the clamped gate/up projection writes bf16, without a fused norm or exchange");
     if (paired && a.bias) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: the gate/up projection takes no bias");
     if (a.epilogue == LIN_RESIDUAL && !a.R) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: residual epilogue without R");
     if (a.bias && (reinterpret_cast<uintptr_t>(a.bias) & 15)) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: bias must be 16-byte aligned");
@@ -1131,6 +1143,7 @@ jsm_status linear_packed_launch(const PackedArgs& a, cudaStream_t st) {
     pk_dims(a.N, a.K, paired, &P.n_tiles, &P.kbt);
     P.local_epi = 1;
     P.paired = paired; P.epilogue = a.epilogue; P.out_f32 = a.out_f32 ? 1 : 0;
+    P.glu_alpha = a.glu_alpha; P.glu_limit = a.glu_limit;
     P.bias = a.bias; P.R = (const __nv_bfloat16*)a.R; P.Y = a.Y; P.Wp = (const uint8_t*)a.Wp;
     const int grid = linear_packed_grid(a.N, a.K, paired, a.T);
     P.max_slots = linear_packed_slots(a.N, a.K, paired, a.T);
@@ -1213,6 +1226,27 @@ jsm_status linear_packed_launch(const PackedArgs& a, cudaStream_t st) {
         return with_cl ? launch_packed<BN_, true, 3>(mx, mx2, P, grid, cluster, a.chained, st)           \
                        : launch_packed<BN_, false, 3>(mx, mx2, P, grid, cluster, a.chained, st);        \
     PK_GO(BN_)
+    if (a.epilogue == LIN_CLAMPED_GLU) {
+        switch (bn) {
+            case 16: return launch_packed<16, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
+            case 32: return cluster > 1 ? launch_packed<32, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st)
+                                        : launch_packed<32, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
+            case 64: return cluster > 1 ? launch_packed<64, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st)
+                                        : launch_packed<64, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
+            case 128: return launch_packed<128, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
+            default: return launch_packed<256, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
+        }
+    }
+    // plain projections of up to 64 tokens with nothing fused
+    if (bn <= 64 && !with_tp && !paired && !a.bias && a.epilogue == LIN_NONE && !a.ssq_in && !a.ssq_out) {
+#define PK_PLAIN(BN_, CL_)                                                                             \
+    return a.out_f32 ? launch_packed<BN_, CL_, 0, 7>(mx, mx2, P, grid, cluster, a.chained, st)         \
+                     : launch_packed<BN_, CL_, 0, 8>(mx, mx2, P, grid, cluster, a.chained, st)
+        if (bn == 16) { if (!with_cl) PK_PLAIN(16, false); }
+        else if (bn == 32) { if (cluster > 1) PK_PLAIN(32, true); else PK_PLAIN(32, false); }
+        else { if (cluster > 1) PK_PLAIN(64, true); else PK_PLAIN(64, false); }
+#undef PK_PLAIN
+    }
     // the few-token launches without an exchange (the decode step of one GPU): an image per kind of tile
     if (bn == 16 && !with_cl && !with_tp) {
         const bool lean = !a.bias && !a.out_f32;  // the projections of a LLaMA-style decoder step have images of their own

@@ -13,6 +13,7 @@
 #include "common.cuh"
 #include "linear_bf16.cuh"
 #include "attn.cuh"
+#include "paged_rows.cuh"
 #include <math.h>
 #include <string.h>
 #include <stdlib.h>
@@ -91,14 +92,9 @@ struct jsm_model {
     // host-buffer decode step (jsm_llama_decode_step_host): staging buffers and one instantiated graph per batch size
     int32_t *ids_dev = nullptr, *next_dev = nullptr;
     std::map<int, cudaGraphExec_t> step_graphs;
-    // continuous batching (jsm_llama_create_paged): pages are handed out on demand from one pool; the active sequences
-    // occupy the batch rows 0 .. n_active-1 and a retiring row is refilled with the last one (its block-table row moves,
-    // its pages stay where they are)
+    // continuous batching (jsm_llama_create_paged): the rows and their pages of one shared pool
     bool paged = false;
-    int n_pool_pages = 0, n_active = 0;
-    std::vector<int32_t> free_pages;
-    std::vector<std::vector<int32_t>> row_pages;
-    std::vector<int32_t> h_ctx;
+    jsm::PagedRows rows;
     int32_t* prompt_dev = nullptr;
 };
 
@@ -741,7 +737,6 @@ static jsm_status llama_create_impl(const jsm_model_config* cfg, uint64_t seed, 
     const long long table_entries = (long long)c.max_batch * m->pages_per_seq;
     const long long n_pages = pool_pages > 0 ? pool_pages : table_entries;
     m->paged = pool_pages > 0;
-    m->n_pool_pages = (int)n_pages;
     const size_t page_elems = (size_t)2 * m->Hkv_l * JSM_PAGE_SIZE * D;
     uint64_t wbytes = 0;
     const int qdim = m->Hq_l * D;  // K of the attention output projection
@@ -806,11 +801,7 @@ static jsm_status llama_create_impl(const jsm_model_config* cfg, uint64_t seed, 
         std::vector<int32_t> bt((size_t)table_entries, 0);
         if (!m->paged)
             for (long long i = 0; i < table_entries; ++i) bt[(size_t)i] = (int32_t)i;
-        else {
-            for (int p = (int)n_pages - 1; p >= 0; --p) m->free_pages.push_back(p);  // page 0 is handed out first
-            m->row_pages.resize(c.max_batch);
-            m->h_ctx.assign(c.max_batch, 0);
-        }
+        m->rows.init(c.max_batch, (int)n_pages, m->pages_per_seq, c.max_context, m->block_table);
         cudaError_t e = cudaMemcpy(m->block_table, bt.data(), bt.size() * sizeof(int32_t), cudaMemcpyHostToDevice);
         if (e != cudaSuccess) { jsm_llama_destroy(m); JSM_FAIL(JSM_CUDA, "jsm_llama_create: block table upload: %s", cudaGetErrorString(e)); }
     }
@@ -1165,35 +1156,15 @@ jsm_status jsm_llama_decode_step_host(jsm_model* m, const int32_t* h_ids, int ba
 // ---- continuous batching over the paged cache ----------------------------------------------------------------------
 // The reference's generation loop serves one sequence at a time and recomputes it from scratch (transformer_test.hpp:
 // 231-239).  Here sequences of different lengths share one decode step; they are admitted and retired between steps.
-namespace {
-// pages for `positions` cached positions of batch row `row`; uploads the part of the row's block table that changed
-jsm_status provision(jsm_model* m, int row, int positions, cudaStream_t st) {
-    std::vector<int32_t>& pages = m->row_pages[row];
-    const int have = (int)pages.size(), need = (positions + JSM_PAGE_SIZE - 1) / JSM_PAGE_SIZE;
-    if (need <= have) return JSM_OK;
-    if (need > m->pages_per_seq) JSM_FAIL(JSM_SHAPE, "context overflow: %d positions, the model was created for %d", positions, m->c.max_context);
-    if (need - have > (int)m->free_pages.size())
-        JSM_FAIL(JSM_OOM, "page pool exhausted: %d pages needed, %zu free of %d", need - have, m->free_pages.size(), m->n_pool_pages);
-    for (int i = have; i < need; ++i) {
-        pages.push_back(m->free_pages.back());
-        m->free_pages.pop_back();
-    }
-    JSM_CUDA_CHECK(cudaMemcpyAsync(m->block_table + (size_t)row * m->pages_per_seq + have, pages.data() + have, sizeof(int32_t) * (need - have),
-                                   cudaMemcpyHostToDevice, st));
-    JSM_CUDA_CHECK(cudaStreamSynchronize(st));  // the host vector may be reallocated by the next call
-    return JSM_OK;
-}
-}  // namespace
-
 jsm_status jsm_llama_seq_admit(jsm_model* m, const int32_t* h_prompt, int T, int* row_out, int32_t* h_first_token, float* h_logits_last,
                                void* stream) {
     if (!m || !h_prompt || !row_out) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_admit: null argument");
     if (!m->paged) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_admit: the model was not created with jsm_llama_create_paged");
     if (T <= 0 || T > m->max_tokens || T >= m->c.max_context) JSM_FAIL(JSM_SHAPE, "jsm_llama_seq_admit: %d prompt tokens (1..%d)", T, std::min(m->max_tokens, m->c.max_context - 1));
-    if (m->n_active >= m->c.max_batch) JSM_FAIL(JSM_OOM, "jsm_llama_seq_admit: all %d batch rows are in use", m->c.max_batch);
+    if (m->rows.n_active >= m->c.max_batch) JSM_FAIL(JSM_OOM, "jsm_llama_seq_admit: all %d batch rows are in use", m->c.max_batch);
     cudaStream_t st = as_stream(stream);
-    const int row = m->n_active;
-    jsm_status s = provision(m, row, T, st);
+    const int row = m->rows.n_active;
+    jsm_status s = m->rows.provision(row, T, st);
     if (s != JSM_OK) return s;
     JSM_CUDA_CHECK(cudaMemcpyAsync(m->prompt_dev, h_prompt, sizeof(int32_t) * T, cudaMemcpyHostToDevice, st));
     float* lg = h_logits_last ? m->logits : nullptr;
@@ -1202,8 +1173,8 @@ jsm_status jsm_llama_seq_admit(jsm_model* m, const int32_t* h_prompt, int T, int
     if (h_first_token) JSM_CUDA_CHECK(cudaMemcpyAsync(h_first_token, m->next_dev + row, sizeof(int32_t), cudaMemcpyDeviceToHost, st));
     if (h_logits_last) JSM_CUDA_CHECK(cudaMemcpyAsync(h_logits_last, m->logits, sizeof(float) * m->c.vocab, cudaMemcpyDeviceToHost, st));
     JSM_CUDA_CHECK(cudaStreamSynchronize(st));
-    m->h_ctx[row] = T;
-    m->n_active = row + 1;
+    m->rows.h_ctx[row] = T;
+    m->rows.n_active = row + 1;
     *row_out = row;
     return JSM_OK;
 }
@@ -1211,49 +1182,32 @@ jsm_status jsm_llama_seq_admit(jsm_model* m, const int32_t* h_prompt, int T, int
 jsm_status jsm_llama_seq_retire(jsm_model* m, int row, int* moved_from, void* stream) {
     if (!m) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_retire: null model");
     if (!m->paged) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_retire: the model was not created with jsm_llama_create_paged");
-    if (row < 0 || row >= m->n_active) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_retire: row %d of %d active", row, m->n_active);
+    if (row < 0 || row >= m->rows.n_active) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_seq_retire: row %d of %d active", row, m->rows.n_active);
     cudaStream_t st = as_stream(stream);
-    for (int32_t p : m->row_pages[row]) m->free_pages.push_back(p);
-    m->row_pages[row].clear();
-    const int last = m->n_active - 1;
-    if (moved_from) *moved_from = -1;
-    if (row != last) {
-        // the last active row takes the freed place: its block-table row and context length move, its pages do not
-        m->row_pages[row] = std::move(m->row_pages[last]);
-        m->row_pages[last].clear();
-        m->h_ctx[row] = m->h_ctx[last];
-        JSM_CUDA_CHECK(cudaMemcpyAsync(m->block_table + (size_t)row * m->pages_per_seq, m->row_pages[row].data(),
-                                       sizeof(int32_t) * m->row_pages[row].size(), cudaMemcpyHostToDevice, st));
-        JSM_CUDA_CHECK(cudaMemcpyAsync(m->ctx + row, &m->h_ctx[row], sizeof(int32_t), cudaMemcpyHostToDevice, st));
-        JSM_CUDA_CHECK(cudaStreamSynchronize(st));
-        if (moved_from) *moved_from = last;
-    }
-    m->h_ctx[last] = 0;
-    m->n_active = last;
-    return JSM_OK;
+    return m->rows.retire(row, moved_from, m->ctx, st);
 }
 
 jsm_status jsm_llama_step_active(jsm_model* m, const int32_t* h_ids, int32_t* h_next, float* h_logits, void* stream) {
     if (!m || !h_ids || !h_next) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_step_active: null argument");
     if (!m->paged) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_step_active: the model was not created with jsm_llama_create_paged");
-    if (m->n_active == 0) return JSM_OK;
+    if (m->rows.n_active == 0) return JSM_OK;
     cudaStream_t st = as_stream(stream);
-    for (int row = 0; row < m->n_active; ++row) {
-        if (m->h_ctx[row] >= m->c.max_context) JSM_FAIL(JSM_SHAPE, "context overflow: row %d already holds max_context = %d tokens", row, m->c.max_context);
-        jsm_status s = provision(m, row, m->h_ctx[row] + 1, st);
+    for (int row = 0; row < m->rows.n_active; ++row) {
+        if (m->rows.h_ctx[row] >= m->c.max_context) JSM_FAIL(JSM_SHAPE, "context overflow: row %d already holds max_context = %d tokens", row, m->c.max_context);
+        jsm_status s = m->rows.provision(row, m->rows.h_ctx[row] + 1, st);
         if (s != JSM_OK) return s;
     }
-    jsm_status s = jsm_llama_decode_step_host(m, h_ids, m->n_active, h_next, h_logits, st);
+    jsm_status s = jsm_llama_decode_step_host(m, h_ids, m->rows.n_active, h_next, h_logits, st);
     if (s != JSM_OK) return s;
-    for (int row = 0; row < m->n_active; ++row) m->h_ctx[row] += 1;
+    for (int row = 0; row < m->rows.n_active; ++row) m->rows.h_ctx[row] += 1;
     return JSM_OK;
 }
 
 jsm_status jsm_llama_pool_state(jsm_model* m, int* n_active, int* free_pages, int* total_pages) {
     if (!m) JSM_FAIL(JSM_INVALID_ARG, "jsm_llama_pool_state: null model");
-    if (n_active) *n_active = m->n_active;
-    if (free_pages) *free_pages = m->paged ? (int)m->free_pages.size() : 0;
-    if (total_pages) *total_pages = m->n_pool_pages;
+    if (n_active) *n_active = m->rows.n_active;
+    if (free_pages) *free_pages = m->paged ? (int)m->rows.free_pages.size() : 0;
+    if (total_pages) *total_pages = m->rows.n_pool_pages;
     return JSM_OK;
 }
 

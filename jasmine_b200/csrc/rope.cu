@@ -255,3 +255,19 @@ jsm_status jsm::rope_apply_strided(const void* d_x, void* d_out, jsm_dtype dtype
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
+
+extern "C" jsm_status jsm_rope_half_table(float* d_table, int d, double base, int max_pos) {
+    if (!d_table) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_half_table: null pointer");
+    if (d <= 0 || d % 2 || max_pos <= 0 || !(base > 0.0)) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_half_table: d %d, base %g, %d positions", d, base, max_pos);
+    const int half = d / 2;
+    std::vector<double> freq(half);
+    for (int i = 0; i < half; ++i) freq[i] = std::pow(base, -2.0 * i / d);
+    std::vector<float> h((size_t)max_pos * d);
+    for (int m = 0; m < max_pos; ++m)
+        for (int i = 0; i < half; ++i) {
+            h[((size_t)m * half + i) * 2] = (float)std::cos(m * freq[i]);
+            h[((size_t)m * half + i) * 2 + 1] = (float)std::sin(m * freq[i]);
+        }
+    JSM_CUDA_CHECK(cudaMemcpy(d_table, h.data(), h.size() * sizeof(float), cudaMemcpyHostToDevice));
+    return JSM_OK;
+}

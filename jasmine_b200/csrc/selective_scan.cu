@@ -1,0 +1,489 @@
+// Selective scan (Mamba) with its short causal convolution, over segments of consecutive tokens of many sequences.
+//
+//   xc = silu(conv(x) + b)                              (per channel, `taps` inputs back)
+//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c xc_c B_n      dt_c = softplus(dt_raw_c + dt_b_c)
+//   y_c = (sum_n S[c, n] C_n + D_c xc_c) * silu(z_c)
+//
+// The recurrent state S and everything that enters it is fp32; x, z and y are activations (bf16 or f32).  A sequence's
+// state lives in a slot: S and the last taps - 1 inputs of the convolution.  A segment that starts at position 0 starts from
+// zeros whatever the slot holds, so a slot needs no clearing when a new sequence takes it.
+//
+// Prompts: a CTA owns 32 channels of one segment and walks its tokens in tiles of 32 that cp.async brings into a two-stage
+// ring; four threads share a channel's states, so that the chain of dependent steps is one FMA per state and the partial
+// sums of four tokens are exchanged with three shuffles.  Decode: the same split of the states, one step for several
+// sequences per CTA; the state rows are requested first and arrive while the step sizes (a small projection) are computed.
+#include "decoder_ops.cuh"
+#include "mma_utils.cuh"
+#include "tc_utils.cuh"
+#include <math.h>
+#include <algorithm>
+
+namespace jsm {
+
+using tc::smem_u32;
+
+constexpr int SC_CH = 32;       // channels per CTA
+constexpr int SC_SUB = 4;       // threads per channel
+constexpr int SC_THREADS = SC_CH * SC_SUB;
+constexpr int SC_TT = 32;       // tokens per tile
+constexpr int SC_YP = 40;       // pitch of the output tile (floats)
+
+__device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+template <typename T>
+__device__ __forceinline__ float decay(float x);  // e^x for x <= 0
+template <>
+__device__ __forceinline__ float decay<float>(float x) { return expf(x); }
+template <>
+__device__ __forceinline__ float decay<__nv_bfloat16>(float x) { return __expf(x); }
+
+template <typename T>
+struct Vec8 {
+    __device__ static void load(const T* p, float (&v)[8]);
+    __device__ static void store(T* p, const float (&v)[8]);
+};
+template <>
+struct Vec8<float> {
+    __device__ static void load(const float* p, float (&v)[8]) {
+        const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    }
+    __device__ static void store(float* p, const float (&v)[8]) {
+        reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+        reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+    }
+};
+template <>
+struct Vec8<__nv_bfloat16> {
+    __device__ static void load(const __nv_bfloat16* p, float (&v)[8]) {
+        const uint4 w = *reinterpret_cast<const uint4*>(p);
+        v[0] = bf16lo(w.x); v[1] = bf16hi(w.x); v[2] = bf16lo(w.y); v[3] = bf16hi(w.y);
+        v[4] = bf16lo(w.z); v[5] = bf16hi(w.z); v[6] = bf16lo(w.w); v[7] = bf16hi(w.w);
+    }
+    __device__ static void store(__nv_bfloat16* p, const float (&v)[8]) {
+        uint4 w;
+        w.x = pack_bf16x2(v[0], v[1]); w.y = pack_bf16x2(v[2], v[3]); w.z = pack_bf16x2(v[4], v[5]); w.w = pack_bf16x2(v[6], v[7]);
+        *reinterpret_cast<uint4*>(p) = w;
+    }
+};
+
+// ---- convolution --------------------------------------------------------------------------------------------------
+// A thread owns 8 channels of CONV_TOK consecutive tokens; TAPS 0: taps is only known at run time
+constexpr int CONV_TOK = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, const T* __restrict__ state,
+                                                        const float* __restrict__ w, const float* __restrict__ b,
+                                                        const int32_t* __restrict__ seg_start, const int32_t* __restrict__ seg_len,
+                                                        const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ seg_slot, int ip,
+                                                        int taps_rt) {
+    chain_trigger();
+    chain_wait();
+    const int taps = TAPS ? TAPS : taps_rt;
+    const int seg = blockIdx.y, vec = ip / 8;
+    const int start = seg_start[seg], len = seg_len[seg], pos0 = seg_pos0[seg];
+    const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+    const int c = (int)(i % vec) * 8, j0 = (int)(i / vec) * CONV_TOK;
+    if (j0 >= len) return;
+    const T* st = state + (long long)seg_slot[seg] * (taps - 1) * ip + c;
+    // input of the segment's token j (negative: before the segment)
+    auto input = [&](int j, float (&v)[8]) {
+        if (j >= 0) Vec8<T>::load(xz + (long long)(start + j) * 2 * ip + c, v);
+        else if (pos0 + j >= 0) Vec8<T>::load(st + (long long)(taps - 1 + j) * ip, v);
+        else
+            for (int e = 0; e < 8; ++e) v[e] = 0.0f;
+    };
+    float bias[8];
+    Vec8<float>::load(b + c, bias);
+    const int j1 = min(len, j0 + CONV_TOK);
+    if constexpr (TAPS > 0) {
+        float win[TAPS][8], wt[TAPS][8];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) Vec8<float>::load(w + (long long)k * ip + c, wt[k]);
+#pragma unroll
+        for (int k = 0; k + 1 < TAPS; ++k) input(j0 - TAPS + 1 + k, win[k + 1]);
+        for (int j = j0; j < j1; ++j) {
+#pragma unroll
+            for (int k = 0; k + 1 < TAPS; ++k)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) win[k][e] = win[k + 1][e];
+            Vec8<T>::load(xz + (long long)(start + j) * 2 * ip + c, win[TAPS - 1]);
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                float a = bias[e];
+#pragma unroll
+                for (int k = 0; k < TAPS; ++k) a = fmaf(wt[k][e], win[k][e], a);
+                o[e] = silu_f(a);
+            }
+            Vec8<T>::store(xc + (long long)(start + j) * ip + c, o);
+        }
+    } else {
+        for (int j = j0; j < j1; ++j) {
+            float o[8];
+            for (int e = 0; e < 8; ++e) o[e] = bias[e];
+            for (int k = 0; k < taps; ++k) {
+                float v[8], wk[8];
+                input(j - taps + 1 + k, v);
+                Vec8<float>::load(w + (long long)k * ip + c, wk);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[e] = fmaf(wk[e], v[e], o[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = silu_f(o[e]);
+            Vec8<T>::store(xc + (long long)(start + j) * ip + c, o);
+        }
+    }
+}
+
+// the last taps - 1 inputs after the segment: entry k is the input taps - 1 - k tokens before the next one.  One thread per
+// channel, ascending k: an entry taken from the old state lies behind every entry already written.
+template <typename T>
+__device__ __forceinline__ void carry_conv_state(T* state, const T* __restrict__ xz, int c, int ip, int taps, int start, int len, int pos0) {
+    for (int k = 0; k + 1 < taps; ++k) {
+        const int j = len - (taps - 1) + k;
+        T v = from_f32<T>(0.0f);
+        if (j >= 0) v = xz[(long long)(start + j) * 2 * ip + c];
+        else if (pos0 + j >= 0) v = state[(long long)(k + len) * ip + c];
+        state[(long long)k * ip + c] = v;
+    }
+}
+
+template <int NS>
+__device__ __forceinline__ void lds_vec(const float* p, float (&v)[NS]) {
+    if constexpr (NS % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < NS; i += 4) {
+            const float4 a = *reinterpret_cast<const float4*>(p + i);
+            v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+        }
+    } else if constexpr (NS % 2 == 0) {
+#pragma unroll
+        for (int i = 0; i < NS; i += 2) {
+            const float2 a = *reinterpret_cast<const float2*>(p + i);
+            v[i] = a.x; v[i + 1] = a.y;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < NS; ++i) v[i] = p[i];
+    }
+}
+
+// ---- scan of prompts ----------------------------------------------------------------------------------------------
+__host__ __device__ inline int scan_nb(int np, int ns) { return np > SC_SUB * ns ? np : SC_SUB * ns; }  // B / C columns per tile row
+template <typename T>
+static size_t scan_smem(int np, int ns) {
+    return 2 * (size_t)SC_TT * SC_CH * (2 * sizeof(T) + 4) + 2 * (size_t)SC_TT * 2 * scan_nb(np, ns) * 4 + (size_t)SC_TT * SC_YP * 4;
+}
+
+struct ScanArgs {
+    const float *A, *D, *dt_b, *proj, *dt_raw;
+    const void *xz, *xc, *dt_w;
+    void *y, *conv;
+    float* S;
+    const int32_t *seg_start, *seg_len, *seg_pos0, *seg_slot;
+    int ip, np, rp, state, taps, n_segs;
+};
+
+template <typename T, int NS>
+__global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
+    extern __shared__ __align__(16) uint8_t sc_dyn[];
+    const int nb = scan_nb(a.np, NS);
+    T* xs = reinterpret_cast<T*>(sc_dyn);                                   // 2 x [TT][CH]
+    T* zs = xs + 2 * SC_TT * SC_CH;                                         // 2 x [TT][CH]
+    float* dts = reinterpret_cast<float*>(zs + 2 * SC_TT * SC_CH);          // 2 x [TT][CH]
+    float* bc = dts + 2 * SC_TT * SC_CH;                                    // 2 x [TT][B: nb | C: nb]
+    float* ys = bc + 2 * SC_TT * 2 * nb;                                    // [TT][YP]
+    chain_trigger();
+    const int tid = threadIdx.x, ch = tid >> 2, sub = tid & 3;
+    const int c0 = blockIdx.x * SC_CH, c = c0 + ch;
+    const bool live = c < a.ip;
+    float A[NS], S[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+        const int n = sub * NS + i;
+        A[i] = (live && n < a.state) ? a.A[(long long)c * a.np + n] : 0.0f;
+    }
+    for (int i = tid; i < 2 * SC_TT * 2 * nb; i += SC_THREADS) bc[i] = 0.0f;  // columns behind np stay zero
+    __syncthreads();
+    chain_wait();
+    const int seg = blockIdx.y;
+    const int start = a.seg_start[seg], len = a.seg_len[seg], pos0 = a.seg_pos0[seg], slot = a.seg_slot[seg];
+    float* state = a.S + ((long long)slot * a.ip + (live ? c : 0)) * a.np;
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+        const int n = sub * NS + i;
+        S[i] = (live && n < a.state && pos0 > 0) ? state[n] : 0.0f;
+    }
+    const int pc = a.rp + 2 * a.np;
+    const T* xz = static_cast<const T*>(a.xz);
+    const T* xc = static_cast<const T*>(a.xc);
+    auto load_tile = [&](int t0, int stage) {
+        constexpr int EV = 16 / sizeof(T), XV = SC_CH / EV;  // elements per vector, vectors per row
+        for (int i = tid; i < SC_TT * XV; i += SC_THREADS) {
+            const int r = i / XV, v = (i % XV) * EV;
+            const bool ok = t0 + r < len && c0 + v < a.ip;
+            const long long t = start + (ok ? t0 + r : 0);
+            const int cc = ok ? c0 + v : 0;
+            cp_async16(smem_u32(xs + (stage * SC_TT + r) * SC_CH + v), xc + t * a.ip + cc, ok);
+            cp_async16(smem_u32(zs + (stage * SC_TT + r) * SC_CH + v), xz + t * 2 * a.ip + a.ip + cc, ok);
+        }
+        for (int i = tid; i < SC_TT * (SC_CH / 4); i += SC_THREADS) {
+            const int r = i / (SC_CH / 4), v = (i % (SC_CH / 4)) * 4;
+            const bool ok = t0 + r < len && c0 + v < a.ip;
+            cp_async16(smem_u32(dts + (stage * SC_TT + r) * SC_CH + v), a.dt_raw + (long long)(start + (ok ? t0 + r : 0)) * a.ip + (ok ? c0 + v : 0), ok);
+        }
+        const int bv = a.np / 4;
+        for (int i = tid; i < SC_TT * 2 * bv; i += SC_THREADS) {
+            const int r = i / (2 * bv), v = i % (2 * bv);
+            const bool ok = t0 + r < len;
+            const float* src = a.proj + (long long)(start + (ok ? t0 + r : 0)) * pc + a.rp + v * 4;
+            cp_async16(smem_u32(bc + ((stage * SC_TT + r) * 2 + (v >= bv)) * nb + (v % bv) * 4), src, ok);
+        }
+    };
+    load_tile(0, 0);
+    cp_async_commit();
+    const int nt = (len + SC_TT - 1) / SC_TT;
+    for (int it = 0; it < nt; ++it) {
+        const int stage = it & 1, t0 = it * SC_TT, n = min(SC_TT, len - t0);
+        if (it + 1 < nt) load_tile(t0 + SC_TT, stage ^ 1);
+        cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        float* dt = dts + stage * SC_TT * SC_CH;
+        const T* x = xs + stage * SC_TT * SC_CH;
+        for (int i = tid; i < SC_TT * SC_CH; i += SC_THREADS) {
+            const int cc = c0 + (i & (SC_CH - 1));
+            // a step size of zero leaves the state as it is: the rows behind the segment
+            dt[i] = (i / SC_CH < n && cc < a.ip) ? softplus_f(dt[i] + a.dt_b[cc]) : 0.0f;
+        }
+        __syncthreads();
+        const float* bt = bc + stage * SC_TT * 2 * nb + sub * NS;
+#pragma unroll 1
+        for (int t4 = 0; t4 < n; t4 += 4) {
+            float y[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int t = t4 + u;
+                const float d = dt[t * SC_CH + ch], dx = d * to_f32(x[t * SC_CH + ch]);
+                float B[NS], C[NS];
+                lds_vec<NS>(bt + t * 2 * nb, B);
+                lds_vec<NS>(bt + t * 2 * nb + nb, C);
+                float acc = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NS; ++i) {
+                    S[i] = fmaf(decay<T>(d * A[i]), S[i], dx * B[i]);
+                    acc = fmaf(S[i], C[i], acc);
+                }
+                y[u] = acc;
+            }
+            // four partial sums on each of four lanes -> lane `sub` holds the sum of token t4 + sub
+            const bool hi = sub & 2, odd = sub & 1;
+            float k0 = hi ? y[2] : y[0], k1 = hi ? y[3] : y[1];
+            k0 += __shfl_xor_sync(0xffffffffu, hi ? y[0] : y[2], 2);
+            k1 += __shfl_xor_sync(0xffffffffu, hi ? y[1] : y[3], 2);
+            float k = odd ? k1 : k0;
+            k += __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 1);
+            ys[(t4 + sub) * SC_YP + ch] = k;
+        }
+        __syncthreads();
+        const T* z = zs + stage * SC_TT * SC_CH;
+        for (int i = tid; i < n * (SC_CH / 8); i += SC_THREADS) {
+            const int r = i / (SC_CH / 8), v = (i % (SC_CH / 8)) * 8;
+            if (c0 + v >= a.ip) continue;
+            float xv[8], zv[8], dv[8], o[8];
+            Vec8<T>::load(x + r * SC_CH + v, xv);
+            Vec8<T>::load(z + r * SC_CH + v, zv);
+            Vec8<float>::load(a.D + c0 + v, dv);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = fmaf(dv[e], xv[e], ys[r * SC_YP + v + e]) * silu_f(zv[e]);
+            Vec8<T>::store(static_cast<T*>(a.y) + (long long)(start + t0 + r) * a.ip + c0 + v, o);
+        }
+        __syncthreads();
+    }
+    if (live)
+#pragma unroll
+        for (int i = 0; i < NS; ++i)
+            if (sub * NS + i < a.state) state[sub * NS + i] = S[i];
+    if (tid < SC_CH && c0 + tid < a.ip)
+        carry_conv_state(static_cast<T*>(a.conv) + (long long)slot * (a.taps - 1) * a.ip, xz, c0 + tid, a.ip, a.taps, start, len, pos0);
+}
+
+// ---- decode step --------------------------------------------------------------------------------------------------
+// One token of BB sequences and 32 channels per CTA.
+template <typename T, int NS, int BB>
+__global__ void __launch_bounds__(SC_THREADS) scan_step_kernel(ScanArgs a) {
+    extern __shared__ __align__(16) float st_dyn[];  // [BB][proj columns]
+    chain_trigger();
+    const int tid = threadIdx.x, ch = tid >> 2, sub = tid & 3;
+    const int c0 = blockIdx.x * SC_CH, c = c0 + ch, cl = min(c, a.ip - 1);
+    const bool live = c < a.ip;
+    const int s0 = blockIdx.y * BB, nb = min(BB, a.n_segs - s0);
+    const int pc = a.rp + 2 * a.np;
+    float A[NS];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) A[i] = sub * NS + i < a.state ? a.A[(long long)cl * a.np + sub * NS + i] : 0.0f;
+    chain_wait();
+    float S[BB][NS];
+#pragma unroll
+    for (int b = 0; b < BB; ++b) {
+        const bool on = b < nb && a.seg_pos0[s0 + min(b, nb - 1)] > 0;
+        const float* state = a.S + ((long long)a.seg_slot[s0 + min(b, nb - 1)] * a.ip + cl) * a.np;
+#pragma unroll
+        for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? state[sub * NS + i] : 0.0f;
+    }
+    for (int i = tid; i < nb * (pc / 4); i += SC_THREADS) {
+        const int b = i / (pc / 4), v = i % (pc / 4);
+        reinterpret_cast<float4*>(st_dyn)[i] = reinterpret_cast<const float4*>(a.proj + (long long)a.seg_start[s0 + b] * pc)[v];
+    }
+    __syncthreads();
+    // step sizes: four threads share a channel's row of the projection
+    float dt[BB];
+#pragma unroll
+    for (int b = 0; b < BB; ++b) dt[b] = 0.0f;
+    const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
+    for (int r = sub * 8; r < a.rp; r += 32) {
+        float wv[8];
+        Vec8<T>::load(w + r, wv);
+#pragma unroll
+        for (int b = 0; b < BB; ++b) {
+            if (b >= nb) break;
+            const float* p = st_dyn + b * pc + r;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) dt[b] = fmaf(wv[e], p[e], dt[b]);
+        }
+    }
+    const float bias = a.dt_b[cl], dv = a.D[cl];
+    const T* xz = static_cast<const T*>(a.xz);
+#pragma unroll
+    for (int b = 0; b < BB; ++b) {
+        if (b >= nb) break;
+        float d = dt[b];
+        d += __shfl_xor_sync(0xffffffffu, d, 1);
+        d += __shfl_xor_sync(0xffffffffu, d, 2);
+        d = softplus_f(d + bias);
+        const int t = a.seg_start[s0 + b];
+        const float x = to_f32(static_cast<const T*>(a.xc)[(long long)t * a.ip + cl]), dx = d * x;
+        const float* Bp = st_dyn + b * pc + a.rp + sub * NS;
+        const float* Cp = Bp + a.np;
+        float* state = a.S + ((long long)a.seg_slot[s0 + b] * a.ip + cl) * a.np + sub * NS;
+        float y = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NS; ++i) {
+            if (sub * NS + i < a.state) {
+                S[b][i] = fmaf(decay<T>(d * A[i]), S[b][i], dx * Bp[i]);
+                y = fmaf(S[b][i], Cp[i], y);
+                if (live) state[i] = S[b][i];
+            }
+        }
+        y += __shfl_xor_sync(0xffffffffu, y, 1);
+        y += __shfl_xor_sync(0xffffffffu, y, 2);
+        if (sub == (b & 3) && live) {
+            const float z = to_f32(xz[(long long)t * 2 * a.ip + a.ip + c]);
+            static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_f(z));
+        }
+    }
+    for (int i = tid; i < SC_CH * nb; i += SC_THREADS) {
+        const int b = i / SC_CH, cc = c0 + i % SC_CH;
+        if (cc < a.ip)
+            carry_conv_state(static_cast<T*>(a.conv) + (long long)a.seg_slot[s0 + b] * (a.taps - 1) * a.ip, xz, cc, a.ip, a.taps,
+                             a.seg_start[s0 + b], 1, a.seg_pos0[s0 + b]);
+    }
+}
+
+__global__ void __launch_bounds__(256) scan_dt_operand_kernel(const float* __restrict__ proj, __nv_bfloat16* __restrict__ out, int T, int rp, int pc) {
+    chain_trigger();
+    chain_wait();
+    const int vec = rp / 8;
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < (long long)T * vec; i += (long long)gridDim.x * 256) {
+        const int t = (int)(i / vec), c = (int)(i % vec) * 8;
+        float v[8];
+        Vec8<float>::load(proj + (long long)t * pc + c, v);
+        Vec8<__nv_bfloat16>::store(out + (long long)t * rp + c, v);
+    }
+}
+
+// ---- launches -----------------------------------------------------------------------------------------------------
+template <typename T>
+static jsm_status conv_typed(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, void* xc,
+                             int max_len, cudaStream_t st) {
+    const int ip = d.ip();
+    const long long n = (long long)((max_len + CONV_TOK - 1) / CONV_TOK) * (ip / 8);
+    const dim3 grid((unsigned)((n + 255) / 256), tk.n_segs);
+    auto go = [&](auto kernel) {
+        return launch_chained(kernel, grid, dim3(256), 0, st, (const T*)xz, (T*)xc, (const T*)s.conv, w.conv, w.conv_b, tk.seg_start, tk.seg_len,
+                              tk.seg_pos0, tk.seg_slot, ip, d.taps);
+    };
+    JSM_CUDA_CHECK(d.taps == 2 ? go(scan_conv_kernel<T, 2>) : d.taps == 3 ? go(scan_conv_kernel<T, 3>)
+                   : d.taps == 4 ? go(scan_conv_kernel<T, 4>) : go(scan_conv_kernel<T, 0>));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+jsm_status scan_conv_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
+                            void* xc, cudaStream_t st) {
+    return f32 ? conv_typed<float>(d, w, s, tk, xz, xc, tk.max_len, st) : conv_typed<__nv_bfloat16>(d, w, s, tk, xz, xc, tk.max_len, st);
+}
+
+static ScanArgs scan_args(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, const void* xc,
+                          const float* proj, const float* dt_raw, void* y) {
+    ScanArgs a;
+    a.A = w.A; a.D = w.D; a.dt_b = w.dt_b; a.proj = proj; a.dt_raw = dt_raw; a.xz = xz; a.xc = xc; a.dt_w = w.dt; a.y = y;
+    a.conv = s.conv; a.S = s.S;
+    a.seg_start = tk.seg_start; a.seg_len = tk.seg_len; a.seg_pos0 = tk.seg_pos0; a.seg_slot = tk.seg_slot;
+    a.ip = d.ip(); a.np = d.np(); a.rp = d.rp(); a.state = d.state; a.taps = d.taps; a.n_segs = tk.n_segs;
+    return a;
+}
+
+template <typename T, int NS>
+static jsm_status scan_go(const ScanArgs& a, cudaStream_t st) {
+    static bool attr_done = false;
+    if (!attr_done) {
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_kernel<T, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        attr_done = true;
+    }
+    JSM_CUDA_CHECK(launch_chained(scan_kernel<T, NS>, dim3((a.ip + SC_CH - 1) / SC_CH, a.n_segs), dim3(SC_THREADS), scan_smem<T>(a.np, NS), st, a));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+template <typename T, int NS>
+static jsm_status step_go(const ScanArgs& a, cudaStream_t st) {
+    constexpr int BB = NS <= 4 ? 8 : NS <= 8 ? 4 : NS <= 16 ? 2 : 1;
+    const size_t smem = (size_t)BB * (a.rp + 2 * a.np) * sizeof(float);
+    static bool attr_done = false;
+    if (!attr_done) {
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_step_kernel<T, NS, BB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        attr_done = true;
+    }
+    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NS, BB>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + BB - 1) / BB), dim3(SC_THREADS), smem, st, a));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+// the smallest instance whose four threads hold a channel's states
+#define JSM_SCAN_DISPATCH(FN, T)                                                                        \
+    (a.state <= 4 ? FN<T, 1>(a, st) : a.state <= 8 ? FN<T, 2>(a, st) : a.state <= 16 ? FN<T, 4>(a, st)  \
+     : a.state <= 24 ? FN<T, 6>(a, st) : a.state <= 32 ? FN<T, 8>(a, st) : a.state <= 64 ? FN<T, 16>(a, st) : FN<T, 32>(a, st))
+
+jsm_status scan_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
+                       const void* xc, const float* proj, const float* dt_raw, void* y, cudaStream_t st) {
+    if (d.state > 128) JSM_FAIL(JSM_UNSUPPORTED, "selective scan: %d states per channel (at most 128)", d.state);
+    const ScanArgs a = scan_args(d, w, s, tk, xz, xc, proj, dt_raw, y);
+    return f32 ? JSM_SCAN_DISPATCH(scan_go, float) : JSM_SCAN_DISPATCH(scan_go, __nv_bfloat16);
+}
+
+jsm_status scan_step_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
+                            const void* xc, const float* proj, void* y, cudaStream_t st) {
+    if (d.state > 128) JSM_FAIL(JSM_UNSUPPORTED, "selective scan: %d states per channel (at most 128)", d.state);
+    const ScanArgs a = scan_args(d, w, s, tk, xz, xc, proj, nullptr, y);
+    return f32 ? JSM_SCAN_DISPATCH(step_go, float) : JSM_SCAN_DISPATCH(step_go, __nv_bfloat16);
+}
+#undef JSM_SCAN_DISPATCH
+
+jsm_status scan_dt_operand_launch(const ScanDims& d, const float* proj, void* out, int T, cudaStream_t st) {
+    const long long n = (long long)T * (d.rp() / 8);
+    JSM_CUDA_CHECK(launch_chained(scan_dt_operand_kernel, dim3((unsigned)std::min<long long>((n + 255) / 256, 148 * 8)), dim3(256), 0, st, proj,
+                                  (__nv_bfloat16*)out, T, d.rp(), d.proj_cols()));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+}  // namespace jsm

@@ -3,7 +3,9 @@
 // norm follows the formula of layer_norm_net_t::forward (mat_net_t.hpp:209-225)
 // with eps under the square root, RMSNorm drops the mean.
 #include "common.cuh"
+#include "decoder_ops.cuh"
 #include <math.h>
+#include <algorithm>
 
 namespace jsm {
 
@@ -136,6 +138,208 @@ __global__ void __launch_bounds__(256) add_norm_kernel(int kind, const T* __rest
             VecIO<T>::store(y + base + c, o);
         }
     }
+}
+
+// ---- decoders whose residual stream is fp32 and whose norms sit on the sublayers' outputs ---------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) embed_residual_kernel(const T* __restrict__ table, const int32_t* __restrict__ ids, float* __restrict__ x,
+                                                             T* __restrict__ xa, int wp) {
+    constexpr int N = VecIO<T>::N;
+    chain_trigger();
+    chain_wait();
+    const T* src = table + (long long)ids[blockIdx.x] * wp;
+    float* dst = x + (long long)blockIdx.x * wp;
+    for (int c = threadIdx.x * N; c < wp; c += 256 * N) {
+        float v[N];
+        VecIO<T>::load(src + c, v);
+#pragma unroll
+        for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(dst + c + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+        if (xa) VecIO<T>::store(xa + (long long)blockIdx.x * wp + c, v);
+    }
+}
+
+// One CTA per token; the sublayer's output y stays in registers between the statistics and the update (MAXV > 0: wp <=
+// 2048 * MAXV), or is read twice (MAXV 0).  Padding columns of y and of the gain are zero.
+template <int MAXV>
+__global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ gain,
+                                                            float eps, __nv_bfloat16* __restrict__ xa, int d, int wp) {
+    __shared__ float smem[8];
+    chain_trigger();
+    chain_wait();
+    const long long base = (long long)blockIdx.x * wp;
+    auto load8 = [](const float* p, float (&v)[8]) {
+        const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    };
+    float keep[MAXV ? MAXV : 1][8], res[MAXV ? MAXV : 1][8];
+    float q = 0.0f;
+    if constexpr (MAXV > 0) {
+#pragma unroll
+        for (int i = 0; i < MAXV; ++i) {
+            const int c = (i * 256 + threadIdx.x) * 8;
+            if (c < wp) {
+                load8(y + base + c, keep[i]);
+                load8(x + base + c, res[i]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) q = fmaf(keep[i][e], keep[i][e], q);
+            }
+        }
+    } else {
+        for (int c = threadIdx.x * 8; c < wp; c += 2048) {
+            float v[8];
+            load8(y + base + c, v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) q = fmaf(v[e], v[e], q);
+        }
+    }
+    q = block_sum(q, smem) / (float)d;
+    const float rms = sqrtf(q + eps);
+    auto update = [&](int c, const float (&v)[8], float (&r)[8]) {
+        float g[8];
+        load8(gain + c, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) r[e] += v[e] / rms * g[e];
+        reinterpret_cast<float4*>(x + base + c)[0] = make_float4(r[0], r[1], r[2], r[3]);
+        reinterpret_cast<float4*>(x + base + c)[1] = make_float4(r[4], r[5], r[6], r[7]);
+        if (xa) VecIO<__nv_bfloat16>::store(xa + base + c, r);
+    };
+    if constexpr (MAXV > 0) {
+#pragma unroll
+        for (int i = 0; i < MAXV; ++i) {
+            const int c = (i * 256 + threadIdx.x) * 8;
+            if (c < wp) update(c, keep[i], res[i]);
+        }
+    } else {
+        for (int c = threadIdx.x * 8; c < wp; c += 2048) {
+            float v[8], r[8];
+            load8(y + base + c, v);
+            load8(x + base + c, r);
+            update(c, v, r);
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) final_norm_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, const float* __restrict__ gain,
+                                                         float eps, T* __restrict__ out, int d, int wp) {
+    __shared__ float smem[8];
+    constexpr int N = VecIO<T>::N;
+    chain_trigger();
+    chain_wait();
+    const float* src = x + (long long)rows[blockIdx.x] * wp;
+    float q = 0.0f;
+    for (int c = threadIdx.x; c < d; c += 256) q = fmaf(src[c], src[c], q);
+    q = block_sum(q, smem) / (float)d;
+    const float rms = sqrtf(q + eps);
+    for (int c = threadIdx.x * N; c < wp; c += 256 * N) {
+        float v[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = src[c + i] / rms * gain[c + i];
+        VecIO<T>::store(out + (long long)blockIdx.x * wp + c, v);
+    }
+}
+
+// Logits of one row per blockIdx.y, split over gridDim.x CTAs: the cap in place and the arg-max over the capped values.  A
+// slice's best (value, index) becomes one monotone 64-bit key that goes into the row's key with atomicMax (larger value
+// first, then the lower index); the CTA that arrives last writes the token and resets both words for the next launch.
+__global__ void __launch_bounds__(256) logits_finish_kernel(float* __restrict__ logits, int pitch, int vocab, float cap,
+                                                            unsigned long long* __restrict__ keys, int32_t* __restrict__ ctrs,
+                                                            int32_t* __restrict__ next) {
+    __shared__ unsigned long long best[8];
+    chain_trigger();
+    chain_wait();
+    const int r = blockIdx.y;
+    float* row = logits + (long long)r * pitch;
+    const int lo = (int)((long long)blockIdx.x * vocab / gridDim.x), hi = (int)((long long)(blockIdx.x + 1) * vocab / gridDim.x);
+    unsigned long long key = 0;  // below every value's key
+    for (int i = lo + threadIdx.x; i < hi; i += 256) {
+        float v = row[i];
+        if (cap > 0.0f) {
+            v = cap * tanhf(v / cap);
+            row[i] = v;
+        }
+        const uint32_t bits = __float_as_uint(v);
+        const uint32_t mono = (bits & 0x80000000u) ? ~bits : (bits | 0x80000000u);
+        const unsigned long long k = ((unsigned long long)mono << 32) | (0xffffffffu - (uint32_t)i);
+        if (v == v && k > key) key = k;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const unsigned long long other = __shfl_xor_sync(0xffffffffu, key, o);
+        if (other > key) key = other;
+    }
+    if ((threadIdx.x & 31) == 0) best[threadIdx.x >> 5] = key;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+#pragma unroll
+        for (int w = 1; w < 8; ++w)
+            if (best[w] > key) key = best[w];
+        atomicMax(keys + r, key);
+        __threadfence();
+        if (atomicAdd(ctrs + r, 1) == (int)gridDim.x - 1) {
+            __threadfence();
+            const unsigned long long top = atomicExch(keys + r, 0ull);
+            next[r] = top ? (int32_t)(0xffffffffu - (uint32_t)(top & 0xffffffffull)) : 0;
+            ctrs[r] = 0;
+        }
+    }
+}
+
+__device__ __forceinline__ float clamped_glu(float g, float u, float alpha, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+__global__ void __launch_bounds__(256) clamped_glu_f32_kernel(const float* __restrict__ gate, const float* __restrict__ up, float* __restrict__ act,
+                                                              float alpha, float limit, long long n) {
+    chain_trigger();
+    chain_wait();
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256)
+        act[i] = clamped_glu(gate[i], up[i], alpha, limit);
+}
+
+jsm_status embed_residual_launch(bool f32, const void* table, const int32_t* ids, float* x, void* xa, int T, int wp, cudaStream_t st) {
+    if (f32)
+        JSM_CUDA_CHECK(launch_chained(embed_residual_kernel<float>, dim3(T), dim3(256), 0, st, (const float*)table, ids, x, (float*)nullptr, wp));
+    else
+        JSM_CUDA_CHECK(launch_chained(embed_residual_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, (const __nv_bfloat16*)table, ids, x,
+                                      (__nv_bfloat16*)xa, wp));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+jsm_status post_norm_add_launch(const float* y, float* x, const float* gain, float eps, void* xa, int T, int d, int wp, cudaStream_t st) {
+    auto go = [&](auto kernel) { return launch_chained(kernel, dim3(T), dim3(256), 0, st, y, x, gain, eps, (__nv_bfloat16*)xa, d, wp); };
+    JSM_CUDA_CHECK(wp <= 2048 ? go(post_norm_add_kernel<1>) : wp <= 4096 ? go(post_norm_add_kernel<2>) : go(post_norm_add_kernel<0>));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+jsm_status final_norm_launch(bool f32, const float* x, const int32_t* rows, const float* gain, float eps, void* out, int n, int d, int wp,
+                             cudaStream_t st) {
+    if (n <= 0) return JSM_OK;
+    if (f32)
+        JSM_CUDA_CHECK(launch_chained(final_norm_kernel<float>, dim3(n), dim3(256), 0, st, x, rows, gain, eps, (float*)out, d, wp));
+    else
+        JSM_CUDA_CHECK(launch_chained(final_norm_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, st, x, rows, gain, eps, (__nv_bfloat16*)out, d, wp));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+jsm_status logits_finish_launch(float* logits, int pitch, int vocab, float cap, int rows, unsigned long long* keys, int32_t* ctrs, int32_t* next,
+                                cudaStream_t st) {
+    if (rows <= 0) return JSM_OK;
+    const int slices = std::max(1, std::min(16, vocab / 1024));
+    JSM_CUDA_CHECK(launch_chained(logits_finish_kernel, dim3(slices, rows), dim3(256), 0, st, logits, pitch, vocab, cap, keys, ctrs, next));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+jsm_status clamped_glu_f32_launch(const float* gate, const float* up, float* act, float alpha, float limit, long long n, cudaStream_t st) {
+    JSM_CUDA_CHECK(launch_chained(clamped_glu_f32_kernel, dim3((unsigned)std::min<long long>((n + 255) / 256, 148 * 16)), dim3(256), 0, st, gate, up, act,
+                                  alpha, limit, n));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
 }
 
 }  // namespace jsm
