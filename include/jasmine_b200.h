@@ -205,6 +205,10 @@ jsm_status jsm_linear_bf16_packed(const void* d_X, const void* d_packed, const f
  * weight requests with the predecessor's tail.  JSM_PDL=0 makes it the plain call. */
 jsm_status jsm_linear_bf16_packed_chained(const void* d_X, const void* d_packed, const float* d_bias, int epilogue,
                                           const void* d_R, void* d_Y, int out_dtype, int T, int N, int K, void* stream);
+/* Gate/up projection with clamps over weights packed with paired = 1: g = min(gate, limit), u = clamp(up, -limit, limit),
+ * Y = g * sigmoid(alpha * g) * (u + 1), bf16 [T, N]. */
+jsm_status jsm_linear_bf16_packed_glu(const void* d_X, const void* d_packed, float alpha, float limit, void* d_Y, int T, int N,
+                                      int K, void* stream);
 
 /* Timeline of the packed projections (profiling aid, off by default; the reference has no tracing).  Between
  * jsm_trace_begin and jsm_trace_end every launch of the packed projection kernel (up to max_launches, eager launches
@@ -322,6 +326,15 @@ jsm_status jsm_embedding(const void* d_table, const void* d_pos_table, const int
 jsm_status jsm_add_norm(int kind, const void* d_h, const void* d_delta, void* d_h_out, void* d_y,
                         jsm_dtype dtype, const float* d_gain, const float* d_bias, float eps, int T, int d,
                         void* stream);
+
+/* Norm on a sublayer's output, fp32 residual stream: x += y / sqrt(mean(y^2) + eps) * gain, and a bf16 copy of the new x
+ * (d_x_bf16 or NULL).  y, x: F32 [T, d], d a multiple of 8. */
+jsm_status jsm_post_norm_add(const float* d_y, float* d_x, const float* d_gain, float eps, void* d_x_bf16, int T, int d,
+                             void* stream);
+/* logits <- cap * tanh(logits / cap) in place (cap 0: unchanged) and the arg-max of every row (the first maximum).
+ * d_keys U64 [rows], d_counters I32 [rows]: zero before the first call; the kernel leaves them zero. */
+jsm_status jsm_logits_finish(float* d_logits, int pitch, int rows, int vocab, float cap, uint64_t* d_keys, int32_t* d_counters,
+                             int32_t* d_next, void* stream);
 
 /* ---- decoder-only model (new; block wiring composed from the parts above;
  *      stack loop: encoder_t::forward mat_transformer_kernel_t.hpp:103-110) -- */

@@ -99,6 +99,9 @@ SYMBOLS = {
     "jsm_linear_unpack": (_i, [_vp, _i, _i, _i, _vp, _vp]),
     "jsm_linear_bf16_packed": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
     "jsm_linear_bf16_packed_chained": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "jsm_linear_bf16_packed_glu": (_i, [_vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]),
+    "jsm_post_norm_add": (_i, [_vp, _vp, _vp, _f, _vp, _i, _i, _vp]),
+    "jsm_logits_finish": (_i, [_vp, _i, _i, _i, _f, _vp, _vp, _vp, _vp]),
     "jsm_rope_table": (_i, [_vp, _i, _i, _f, _i, _vp]),
     "jsm_rope_half_table": (_i, [_vp, _i, C.c_double, _i]),
     "jsm_rope_apply": (_i, [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp]),
@@ -179,6 +182,13 @@ def lib() -> C.CDLL:
 def check(status: int) -> None:
     if status != OK:
         raise JsmError(status, lib().jsm_last_error().decode(errors="replace"))
+
+
+def host_ptr(a):
+    """Address of a host array (numpy or torch); None stays None."""
+    if a is None:
+        return None
+    return a.data_ptr() if hasattr(a, "data_ptr") else a.ctypes.data
 
 
 # ---- torch plumbing ------------------------------------------------------------
@@ -285,6 +295,31 @@ def linear_bf16_packed(X, packed, out, bias=None, epilogue=0, residual=None, cha
     fn = lib().jsm_linear_bf16_packed_chained if chained else lib().jsm_linear_bf16_packed
     check(fn(X.data_ptr(), packed.data_ptr(), bias.data_ptr() if bias is not None else None, epilogue,
              residual.data_ptr() if residual is not None else None, out.data_ptr(), dtype_of(out), T, N, K, stream_ptr()))
+    return out
+
+
+def linear_bf16_packed_glu(X, packed, out, alpha, limit):
+    """Clamped gate/up projection over weights packed in pairs (jsm_linear_bf16_packed_glu)."""
+    check(lib().jsm_linear_bf16_packed_glu(X.data_ptr(), packed.data_ptr(), alpha, limit, out.data_ptr(), X.shape[0], out.shape[1],
+                                           X.shape[1], stream_ptr()))
+    return out
+
+
+def post_norm_add(y, x, gain, eps, x_bf16=None):
+    """x += rms_norm(y) * gain in place, optional bf16 copy of x (jsm_post_norm_add)."""
+    check(lib().jsm_post_norm_add(y.data_ptr(), x.data_ptr(), gain.data_ptr(), eps, x_bf16.data_ptr() if x_bf16 is not None else None,
+                                  y.shape[0], y.shape[1], stream_ptr()))
+    return x
+
+
+def logits_finish(logits, vocab, cap):
+    """Caps logits [rows, pitch] in place and returns the arg-max of every row (jsm_logits_finish)."""
+    torch = _torch()
+    rows, pitch = logits.shape
+    keys = torch.zeros(rows, dtype=torch.int64, device=logits.device)
+    ctrs = torch.zeros(rows, dtype=torch.int32, device=logits.device)
+    out = torch.empty(rows, dtype=torch.int32, device=logits.device)
+    check(lib().jsm_logits_finish(logits.data_ptr(), pitch, rows, vocab, cap, keys.data_ptr(), ctrs.data_ptr(), out.data_ptr(), stream_ptr()))
     return out
 
 

@@ -11,7 +11,7 @@
 // is cut into passes of at most max_step_tokens.  A pass whose rows bring one token each replays a CUDA graph.
 //
 // bf16: weights packed for the tensor-core projections, activations bf16, residual, norms, scores, recurrences and logits
-// fp32.  f32: fp32 weights, activations and products throughout (jsm_dot_f32 and the f32 forms of the kernels).
+// fp32.  f32: fp32 weights, activations and products throughout (dot_f32.cu and the f32 forms of the kernels).
 #include "common.cuh"
 #include "decoder_ops.cuh"
 #include "linear_bf16.cuh"
@@ -27,6 +27,7 @@
 namespace jsm {
 
 int* tc_error_word();
+jsm_status dot_f32_launch(const jsm_mat& A, const jsm_mat& B, const jsm_mat& C, cudaStream_t st);
 
 struct Proj {  // one projection: N outputs, K inputs, both rounded up to multiples of 8 (zero rows / columns)
     int N = 0, K = 0, paired = 0;
@@ -335,7 +336,7 @@ static jsm_status linear(jsm_decoder* m, const Proj& p, const void* X, long long
         jsm_mat A{const_cast<void*>(X), T, p.K, x_stride, 1, JSM_F32};
         jsm_mat B{p.w32, p.K, p.N, 1, p.K, JSM_F32};
         jsm_mat C{Y, T, p.N, p.N, 1, JSM_F32};
-        return jsm_dot_f32(A, B, nullptr, 0, nullptr, C, st);
+        return dot_f32_launch(A, B, C, st);
     }
     PackedArgs a;
     a.Wp = p.packed; a.bias = nullptr; a.R = nullptr; a.out_f32 = out_f32;

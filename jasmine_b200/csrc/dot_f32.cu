@@ -17,6 +17,9 @@ constexpr int TM = 64, TN = 64, TK = 16;
 
 __device__ __forceinline__ float gelu_f(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752440f)); }
 
+// ORDERED: the reference's summation order (see above).  Otherwise every block of TK products is summed with fused
+// multiply-adds before it joins the total: shorter chains of roundings, for fp32 models that have no order to match.
+template <bool ORDERED>
 __global__ void __launch_bounds__(256) dot_f32_kernel(MatD A, MatD B, MatD bias, int has_bias, int epilogue, MatD R,
                                                       float* Cp, long long crs, long long ccs, int M, int N, int K) {
     __shared__ float As[TK][TM + 1];
@@ -47,6 +50,12 @@ __global__ void __launch_bounds__(256) dot_f32_kernel(MatD A, MatD B, MatD bias,
         }
         __syncthreads();
         const int kmax = (K - k0) < TK ? (K - k0) : TK;  // never add the zero padding: -0.0 + 0.0 would flip a sign
+        float part[4][4];
+        if (!ORDERED)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) part[i][j] = 0.0f;
         for (int k = 0; k < kmax; ++k) {
             float a[4], b[4];
 #pragma unroll
@@ -56,8 +65,16 @@ __global__ void __launch_bounds__(256) dot_f32_kernel(MatD A, MatD B, MatD bias,
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = __fadd_rn(acc[i][j], __fmul_rn(a[i], b[j]));
+                for (int j = 0; j < 4; ++j) {
+                    if (ORDERED) acc[i][j] = __fadd_rn(acc[i][j], __fmul_rn(a[i], b[j]));
+                    else part[i][j] = fmaf(a[i], b[j], part[i][j]);
+                }
         }
+        if (!ORDERED)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
         __syncthreads();
     }
 #pragma unroll
@@ -83,6 +100,16 @@ static MatD to_d(const jsm_mat& m) {
     return d;
 }
 
+// C = A . B in fp32 without the reference's order (operands as in jsm_dot_f32, checked by the caller)
+jsm_status dot_f32_launch(const jsm_mat& A, const jsm_mat& B, const jsm_mat& Cm, cudaStream_t st) {
+    const dim3 grid((Cm.cols + TN - 1) / TN, (Cm.rows + TM - 1) / TM);
+    const MatD none{nullptr, 1, 1, 0, 0};
+    dot_f32_kernel<false><<<grid, 256, 0, st>>>(to_d(A), to_d(B), none, 0, 0, none, reinterpret_cast<float*>(Cm.data), Cm.row_stride, Cm.col_stride,
+                                                A.rows, B.cols, A.cols);
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
 }  // namespace jsm
 
 using namespace jsm;
@@ -104,7 +131,7 @@ extern "C" jsm_status jsm_dot_f32(jsm_mat A, jsm_mat B, const jsm_mat* bias, int
     MatD bd = bias ? to_d(*bias) : MatD{nullptr, 1, 1, 0, 0};
     MatD rd = R ? to_d(*R) : MatD{nullptr, 1, 1, 0, 0};
     dim3 grid((Cm.cols + TN - 1) / TN, (Cm.rows + TM - 1) / TM);
-    dot_f32_kernel<<<grid, 256, 0, as_stream(stream)>>>(to_d(A), to_d(B), bd, bias ? 1 : 0, epilogue, rd,
+    dot_f32_kernel<true><<<grid, 256, 0, as_stream(stream)>>>(to_d(A), to_d(B), bd, bias ? 1 : 0, epilogue, rd,
                                                         reinterpret_cast<float*>(Cm.data), Cm.row_stride, Cm.col_stride,
                                                         A.rows, B.cols, A.cols);
     JSM_LAUNCH_CHECK();

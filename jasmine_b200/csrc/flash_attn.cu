@@ -13,6 +13,8 @@
 // first half of S_t in place.  While one tile's softmax runs on the CUDA cores, the tensor cores work on the
 // other tile.  The running maximum is only raised (and O rescaled) when it grew by more than 2^8, so the
 // rescale of the accumulator is rare; the final division by the row sum happens in the epilogue.
+// Heads whose queries / keys are 64, 128 or 192 wide and whose values are 64 or 128 wide share the kernel (narrower ones are
+// zero padded by the caller), and the mask may be a sliding window: key tiles no row of a query tile sees are skipped.
 // Every wait is bounded; on a timeout the CTA unwinds, frees its TMEM and records a code for the host.
 #include "attn.cuh"
 #include "decoder_ops.cuh"
@@ -24,12 +26,11 @@ namespace jsm {
 
 using namespace tc;
 
-constexpr int FA_D = 128;          // head_dim
+constexpr int FA_D = 128;          // head_dim of the public entry point
 constexpr int FA_BM = 128;         // queries per tile (TMEM lanes)
 constexpr int FA_BN = 128;         // keys per tile
 constexpr int FA_THREADS = 320;
-constexpr int FA_KV_STAGES = 2;
-constexpr uint32_t FA_TILE_BYTES = FA_BM * FA_D * 2;  // 32 KB: two 16 KB halves of 64 columns
+constexpr uint32_t FA_SLAB = FA_BM * 64 * 2;          // 16 KB: 64 columns of a tile of 128 rows
 constexpr float FA_RESCALE_THRESHOLD = 8.0f;          // log2 domain
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -66,6 +67,8 @@ struct FlashParams {
     float scale_log2;
     __nv_bfloat16* out;
     long long out_rs;
+    int q_hs, v_dim;     // columns between the heads of q; columns of a head's output
+    int window;          // query i sees the keys i - window + 1 .. i only (WIN)
     int* err;
 };
 
@@ -92,17 +95,21 @@ __device__ __forceinline__ void ex2_poly2(uint64_t x2, float& p0, float& p1) {
 }
 
 // POLY: of every four pairs of scores, this many take ex2_poly2 instead of ex2.approx
-template <int POLY>
+// QKD / VD: columns of a query / key and of a value; VST: stages of the V ring (keys have two); WIN: the mask is a window of
+// P.window keys, and a head's output has P.v_dim columns (VD otherwise)
+template <int POLY, int QKD, int VD, int VST, bool WIN>
 __global__ void __launch_bounds__(FA_THREADS, 1)
     flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_v, FlashParams P) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    uint8_t* q_smem = tiles;                                   // 2 x 32 KB
-    uint8_t* k_smem = tiles + 2 * FA_TILE_BYTES;               // FA_KV_STAGES x 32 KB
-    uint8_t* v_smem = k_smem + FA_KV_STAGES * FA_TILE_BYTES;   // FA_KV_STAGES x 32 KB
+    constexpr int KST = 2;
+    constexpr uint32_t QK_BYTES = QKD / 64 * FA_SLAB, V_BYTES = VD / 64 * FA_SLAB;
+    uint8_t* q_smem = tiles;                      // 2 query tiles
+    uint8_t* k_smem = tiles + 2 * QK_BYTES;       // KST key tiles
+    uint8_t* v_smem = k_smem + KST * QK_BYTES;    // VST value tiles
     __shared__ __align__(8) uint64_t q_full, o_done;
-    __shared__ __align__(8) uint64_t k_full[FA_KV_STAGES], k_empty[FA_KV_STAGES], v_full[FA_KV_STAGES], v_empty[FA_KV_STAGES];
+    __shared__ __align__(8) uint64_t k_full[KST], k_empty[KST], v_full[VST], v_empty[VST];
     __shared__ __align__(8) uint64_t s_full[2], p_ready[2];
     __shared__ uint32_t tmem_base_smem;
     __shared__ int abort_flag;
@@ -113,24 +120,25 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     const int h = blockIdx.y, b = blockIdx.z, hk = h / (P.Hq / P.Hkv);
     const int q0 = qblk * 2 * FA_BM;
     const int shift = P.Tk - P.Tq;  // query i sits at position i + shift
-    // number of key tiles each query tile needs
-    int n_tiles[2];
+    // key tiles [lo, n_tiles) of each query tile
+    int n_tiles[2], lo[2];
 #pragma unroll
     for (int t = 0; t < 2; ++t) {
         const int last_row = min(q0 + (t + 1) * FA_BM, P.Tq) - 1;  // may be < first row when the tile is empty
         int kv_end = P.causal ? min(P.Tk, last_row + shift + 1) : P.Tk;
         if (q0 + t * FA_BM >= P.Tq) kv_end = 0;
         n_tiles[t] = (kv_end + FA_BN - 1) / FA_BN;
+        lo[t] = WIN ? min(n_tiles[t], max(0, q0 + t * FA_BM + shift - P.window + 1) / FA_BN) : 0;
     }
     const int n_max = max(n_tiles[0], n_tiles[1]);
+    const int j_lo = n_tiles[1] > 0 ? min(lo[0], lo[1]) : lo[0];
 
     if (threadIdx.x == 0) {
         abort_flag = 0;
         mbar_init(&q_full, 1);
         mbar_init(&o_done, 1);
-        for (int s = 0; s < FA_KV_STAGES; ++s) {
-            mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1);
-        }
+        for (int s = 0; s < KST; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
+        for (int s = 0; s < VST; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
         for (int t = 0; t < 2; ++t) { mbar_init(&s_full[t], 1); mbar_init(&p_ready[t], 128); }
         mbar_fence_init();
         tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
@@ -143,53 +151,50 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem_base = tmem_base_smem;
-    const uint32_t S_COL[2] = {0, 128}, O_COL[2] = {256, 384};
+    const uint32_t S_COL[2] = {0, 128}, O_COL[2] = {256, 256 + VD};
 
     if (warp == 0) {
         if (lane == 0) {
-            // Q: both tiles, two 64-column halves each
-            mbar_expect_tx(&q_full, 2 * FA_TILE_BYTES);
+            // Q: both tiles, in slabs of 64 columns
+            mbar_expect_tx(&q_full, 2 * QK_BYTES);
             for (int t = 0; t < 2; ++t)
-                for (int half = 0; half < 2; ++half)
-                    tma_load_2d(q_smem + t * FA_TILE_BYTES + half * (FA_TILE_BYTES / 2), &tmap_q, h * FA_D + half * 64,
-                                b * P.Tq + q0 + t * FA_BM, &q_full);
-            int issued = 0;
-            for (int j = 0; j < n_max; ++j) {
-                const int s = j % FA_KV_STAGES;
-                const uint32_t ph = (j / FA_KV_STAGES) & 1;
-                if (j >= FA_KV_STAGES && !mbar_wait(&k_empty[s], ph ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) break;
-                mbar_expect_tx(&k_full[s], FA_TILE_BYTES);
-                for (int half = 0; half < 2; ++half)
-                    tma_load_2d(k_smem + s * FA_TILE_BYTES + half * (FA_TILE_BYTES / 2), &tmap_k, hk * FA_D + half * 64,
-                                b * P.Tk + j * FA_BN, &k_full[s]);
-                if (j >= FA_KV_STAGES && !mbar_wait(&v_empty[s], ph ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) { issued = j + 1; break; }
-                mbar_expect_tx(&v_full[s], FA_TILE_BYTES);
-                for (int half = 0; half < 2; ++half)
-                    tma_load_2d(v_smem + s * FA_TILE_BYTES + half * (FA_TILE_BYTES / 2), &tmap_v, hk * FA_D + half * 64,
-                                b * P.Tk + j * FA_BN, &v_full[s]);
-                issued = j + 1;
+                for (int c = 0; c < QKD / 64; ++c)
+                    tma_load_2d(q_smem + t * QK_BYTES + c * FA_SLAB, &tmap_q, h * P.q_hs + c * 64, b * P.Tq + q0 + t * FA_BM, &q_full);
+            int k_issued = 0, v_issued = 0;
+            for (int j = j_lo; j < n_max; ++j) {
+                const int i = j - j_lo, ks = i % KST, vs = i % VST;
+                if (i >= KST && !mbar_wait(&k_empty[ks], ((i / KST) & 1) ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) break;
+                mbar_expect_tx(&k_full[ks], QK_BYTES);
+                for (int c = 0; c < QKD / 64; ++c)
+                    tma_load_2d(k_smem + ks * QK_BYTES + c * FA_SLAB, &tmap_k, hk * QKD + c * 64, b * P.Tk + j * FA_BN, &k_full[ks]);
+                k_issued = i + 1;
+                if (i >= VST && !mbar_wait(&v_empty[vs], ((i / VST) & 1) ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) break;
+                mbar_expect_tx(&v_full[vs], V_BYTES);
+                for (int c = 0; c < VD / 64; ++c)
+                    tma_load_2d(v_smem + vs * V_BYTES + c * FA_SLAB, &tmap_v, hk * VD + c * 64, b * P.Tk + j * FA_BN, &v_full[vs]);
+                v_issued = i + 1;
             }
             if (abort_flag) {  // let the copies in flight land before the CTA exits (bounded)
                 const long long t_start = clock64();
-                for (int j = max(0, issued - FA_KV_STAGES); j < issued; ++j) {
-                    while (!mbar_try_wait(&k_full[j % FA_KV_STAGES], (j / FA_KV_STAGES) & 1) && clock64() - t_start < WAIT_LIMIT_CYCLES) {}
-                    while (!mbar_try_wait(&v_full[j % FA_KV_STAGES], (j / FA_KV_STAGES) & 1) && clock64() - t_start < WAIT_LIMIT_CYCLES) {}
-                }
+                for (int i = max(0, k_issued - KST); i < k_issued; ++i)
+                    while (!mbar_try_wait(&k_full[i % KST], (i / KST) & 1) && clock64() - t_start < WAIT_LIMIT_CYCLES) {}
+                for (int i = max(0, v_issued - VST); i < v_issued; ++i)
+                    while (!mbar_try_wait(&v_full[i % VST], (i / VST) & 1) && clock64() - t_start < WAIT_LIMIT_CYCLES) {}
                 while (!mbar_try_wait(&q_full, 0) && clock64() - t_start < WAIT_LIMIT_CYCLES) {}
             }
         }
     } else if (warp == 1) {
         if (lane == 0) {
             constexpr uint32_t idesc_qk = instr_desc_bf16(FA_BM, FA_BN, 0, 0);  // both operands K-major (head_dim contiguous)
-            constexpr uint32_t idesc_pv = instr_desc_bf16(FA_BM, FA_D, 0, 1);   // V is N-contiguous: MN-major B
+            constexpr uint32_t idesc_pv = instr_desc_bf16(FA_BM, VD, 0, 1);   // V is N-contiguous: MN-major B
             bool ok = mbar_wait(&q_full, 0, &abort_flag, P.err, TC_TIMEOUT_FULL);
             // S_t(j) = Q_t . K(j)^T into the S columns of tile t (overwrites P_t(j-1): the tensor pipe runs the MMAs of
             // this thread in issue order, so the P.V product issued before it has read P by then)
             auto issue_s = [&](int t, uint32_t k_addr) {
-                const uint32_t q_addr = smem_u32(q_smem + t * FA_TILE_BYTES);
+                const uint32_t q_addr = smem_u32(q_smem + t * QK_BYTES);
 #pragma unroll
-                for (int kk = 0; kk < FA_D / 16; ++kk) {
-                    const uint32_t off = (kk / 4) * (FA_TILE_BYTES / 2);
+                for (int kk = 0; kk < QKD / 16; ++kk) {
+                    const uint32_t off = (kk / 4) * FA_SLAB;
                     mma_ss(tmem_base + S_COL[t], smem_desc_sw128(q_addr + off) + (uint64_t)((kk % 4) * 2),
                            smem_desc_sw128(k_addr + off) + (uint64_t)((kk % 4) * 2), idesc_qk, kk > 0 ? 1u : 0u);
                 }
@@ -197,45 +202,45 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
             };
             // The scores run one key tile ahead of the P.V products: S_t(j+1) is issued right after O_t += P_t(j).V(j),
             // so the softmax of one query tile overlaps the softmax of the other instead of alternating with it.
-            if (ok && n_max > 0) {
+            auto active = [&](int t, int j) { return j >= lo[t] && j < n_tiles[t]; };
+            if (ok && n_max > j_lo) {
                 ok = mbar_wait(&k_full[0], 0, &abort_flag, P.err, TC_TIMEOUT_FULL);
                 tc_fence_after();
                 if (ok) {
                     const uint32_t k_addr = smem_u32(k_smem);
 #pragma unroll
                     for (int t = 0; t < 2; ++t)
-                        if (n_tiles[t] > 0) issue_s(t, k_addr);
+                        if (active(t, j_lo)) issue_s(t, k_addr);
                     mma_commit(&k_empty[0]);
                 }
             }
-            for (int j = 0; j < n_max && ok; ++j) {
-                const int s = j % FA_KV_STAGES, s1 = (j + 1) % FA_KV_STAGES;
-                const uint32_t ph = (j / FA_KV_STAGES) & 1, ph1 = ((j + 1) / FA_KV_STAGES) & 1;
+            for (int j = j_lo; j < n_max && ok; ++j) {
+                const int i = j - j_lo, vs = i % VST, s1 = (i + 1) % KST;
                 const bool more = j + 1 < n_max;
-                if (!mbar_wait(&v_full[s], ph, &abort_flag, P.err, TC_TIMEOUT_FULL)) { ok = false; break; }
+                if (!mbar_wait(&v_full[vs], (i / VST) & 1, &abort_flag, P.err, TC_TIMEOUT_FULL)) { ok = false; break; }
                 tc_fence_after();
-                const uint32_t v_addr = smem_u32(v_smem + s * FA_TILE_BYTES);
-                const uint32_t k_addr = smem_u32(k_smem + s1 * FA_TILE_BYTES);
+                const uint32_t v_addr = smem_u32(v_smem + vs * V_BYTES);
+                const uint32_t k_addr = smem_u32(k_smem + s1 * QK_BYTES);
 #pragma unroll
                 for (int t = 0; t < 2; ++t) {
-                    if (j < n_tiles[t]) {
-                        if (!mbar_wait(&p_ready[t], j & 1, &abort_flag, P.err, TC_TIMEOUT_MISC)) { ok = false; break; }
+                    if (active(t, j)) {
+                        if (!mbar_wait(&p_ready[t], (j - lo[t]) & 1, &abort_flag, P.err, TC_TIMEOUT_MISC)) { ok = false; break; }
                         tc_fence_after();
 #pragma unroll
                         for (int kk = 0; kk < FA_BN / 16; ++kk) {
-                            // 16 keys = two 8-row groups of 1024 bytes; the two 64-column halves of V are 16 KB apart
-                            const uint64_t v_desc = smem_desc_sw128_mn(v_addr + kk * 2048, FA_TILE_BYTES / 2);
-                            mma_ts(tmem_base + O_COL[t], tmem_base + S_COL[t] + kk * 8, v_desc, idesc_pv, (j > 0 || kk > 0) ? 1u : 0u);
+                            // 16 keys = two 8-row groups of 1024 bytes; the 64-column slabs of V are 16 KB apart
+                            const uint64_t v_desc = smem_desc_sw128_mn(v_addr + kk * 2048, FA_SLAB);
+                            mma_ts(tmem_base + O_COL[t], tmem_base + S_COL[t] + kk * 8, v_desc, idesc_pv, (j > lo[t] || kk > 0) ? 1u : 0u);
                         }
                     }
                     if (t == 0 && more) {
-                        if (!mbar_wait(&k_full[s1], ph1, &abort_flag, P.err, TC_TIMEOUT_FULL)) { ok = false; break; }
+                        if (!mbar_wait(&k_full[s1], ((i + 1) / KST) & 1, &abort_flag, P.err, TC_TIMEOUT_FULL)) { ok = false; break; }
                         tc_fence_after();
                     }
-                    if (j + 1 < n_tiles[t]) issue_s(t, k_addr);
+                    if (active(t, j + 1)) issue_s(t, k_addr);
                 }
                 if (!ok) break;
-                mma_commit(&v_empty[s]);
+                mma_commit(&v_empty[vs]);
                 if (more) mma_commit(&k_empty[s1]);
             }
             if (ok) mma_commit(&o_done);
@@ -243,16 +248,18 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     } else {
         // ---- softmax / correction / epilogue: one thread per query row
         const int t = (warp - 2) / 4;       // query tile
+        const int j_begin = t ? lo[1] : lo[0], j_end = t ? n_tiles[1] : n_tiles[0];
         const int quad = warp & 3;          // TMEM lane quadrant this warp may access
         const int row = quad * 32 + lane;   // row in the tile = TMEM lane
         const int qi = q0 + t * FA_BM + row;
         const int qpos = qi + shift;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
-        const uint32_t s_addr = lane_addr + S_COL[t], o_addr = lane_addr + O_COL[t];
-        float m_ref = -INFINITY, l = 0.0f;
+        const uint32_t s_addr = lane_addr + (t ? S_COL[1] : S_COL[0]), o_addr = lane_addr + (t ? O_COL[1] : O_COL[0]);
+        // (a finite start: a window can hide a whole key tile from some rows, whose weights are then 2^-inf = 0)
+        float m_ref = -1.0e30f, l = 0.0f;
         bool ok = true;
-        for (int j = 0; j < n_tiles[t] && ok; ++j) {
-            if (!mbar_wait(&s_full[t], j & 1, &abort_flag, P.err, TC_TIMEOUT_ACC)) { ok = false; break; }
+        for (int j = j_begin; j < j_end && ok; ++j) {
+            if (!mbar_wait(&s_full[t], (j - j_begin) & 1, &abort_flag, P.err, TC_TIMEOUT_ACC)) { ok = false; break; }
             tc_fence_after();
             // the whole score row of this thread: four TMEM loads in flight, one wait
             uint32_t sr[FA_BN];
@@ -263,11 +270,18 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
 #pragma unroll
             for (int i = 0; i < FA_BN; ++i) sv[i] = __uint_as_float(sr[i]);
             const int key0 = j * FA_BN;
+            const bool low_edge = WIN && key0 < q0 + t * FA_BM + FA_BM - 1 + shift - P.window + 1;
             const bool needs_mask = (P.causal && key0 + FA_BN - 1 > q0 + t * FA_BM + shift) || key0 + FA_BN > P.Tk;
             if (needs_mask) {
 #pragma unroll
                 for (int i = 0; i < FA_BN; ++i)
                     if ((P.causal && key0 + i > qpos) || key0 + i >= P.Tk) sv[i] = -INFINITY;
+            }
+            if (low_edge) {
+                const int first = qpos - P.window + 1 - key0;  // keys before it are out of this row's window
+#pragma unroll
+                for (int i = 0; i < FA_BN; ++i)
+                    if (i < first) sv[i] = -INFINITY;
             }
             // scores stay unscaled in registers; the scale (> 0, log2 domain) is applied inside the exponent's FMA
             // eight independent chains instead of one 127-deep dependency chain (two warps per scheduler: the row needs ILP)
@@ -288,9 +302,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
             if (__any_sync(0xffffffffu, grow)) {
                 // raise the reference maximum; the accumulated O and l shrink by 2^(old - new)
                 const float alpha = grow ? ex2_approx(m_ref - mx) : 1.0f;
-                if (j > 0) {
+                if (j > j_begin) {
 #pragma unroll
-                    for (int c = 0; c < FA_D; c += 32) {
+                    for (int c = 0; c < VD; c += 32) {
                         uint32_t r[32];
                         tmem_ld32(o_addr + c, r);
                         tmem_ld_wait();
@@ -342,18 +356,20 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
             mbar_arrive(&p_ready[t]);
         }
         // epilogue: O / l -> bf16 -> global
-        if (ok && n_tiles[t] > 0) ok = mbar_wait(&o_done, 0, &abort_flag, P.err, TC_TIMEOUT_ACC);
+        if (ok && j_end > j_begin) ok = mbar_wait(&o_done, 0, &abort_flag, P.err, TC_TIMEOUT_ACC);
         tc_fence_after();
-        if (ok && n_tiles[t] > 0) {  // warp-uniform: the TMEM loads are collective, only the stores are per row
+        if (ok && j_end > j_begin) {  // warp-uniform: the TMEM loads are collective, only the stores are per row
             const float inv = 1.0f / l;
             const bool store = qi < P.Tq;
-            __nv_bfloat16* dst = P.out + (long long)(b * P.Tq + (store ? qi : 0)) * P.out_rs + (long long)h * FA_D;
+            __nv_bfloat16* dst = P.out + (long long)(b * P.Tq + (store ? qi : 0)) * P.out_rs + (long long)h * (WIN ? P.v_dim : VD);
+            const int v_dim = WIN ? P.v_dim : VD;
+            const bool vec = v_dim % 8 == 0;
 #pragma unroll
-            for (int c = 0; c < FA_D; c += 32) {
+            for (int c = 0; c < VD; c += 32) {
                 uint32_t r[32];
                 tmem_ld32(o_addr + c, r);
                 tmem_ld_wait();
-                if (store) {
+                if (store && vec) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
                         uint4 o;
@@ -361,8 +377,12 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
                         o.y = pack_bf16x2(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv);
                         o.z = pack_bf16x2(__uint_as_float(r[i + 4]) * inv, __uint_as_float(r[i + 5]) * inv);
                         o.w = pack_bf16x2(__uint_as_float(r[i + 6]) * inv, __uint_as_float(r[i + 7]) * inv);
-                        *reinterpret_cast<uint4*>(dst + c + i) = o;
+                        if (c + i < v_dim) *reinterpret_cast<uint4*>(dst + c + i) = o;
                     }
+                } else if (store) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (c + i < v_dim) dst[c + i] = __float2bfloat16_rn(__uint_as_float(r[i]) * inv);
                 }
             }
         }
@@ -373,6 +393,21 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
         tc_fence_after();
         tmem_dealloc(tmem_base, 512);
     }
+}
+
+template <int QKD, int VD, int VST, bool WIN>
+static jsm_status flash_go(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FlashParams& P, dim3 grid, cudaStream_t st) {
+    constexpr size_t smem = (size_t)(4 * (QKD / 64) + VST * (VD / 64)) * FA_SLAB + 1024;
+    static_assert(smem <= 226 * 1024, "query tiles and rings fit the shared memory");
+    // a quarter of the exponentials on the FMA pipe: the measured optimum (none: MUFU-bound, half: issue-bound)
+    static bool attr_done = false;
+    if (!attr_done) {
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(flash_prefill_kernel<1, QKD, VD, VST, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        attr_done = true;
+    }
+    flash_prefill_kernel<1, QKD, VD, VST, WIN><<<grid, FA_THREADS, smem, st>>>(mq, mk, mv, P);
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
 }
 
 jsm_status flash_prefill_launch(const void* q, const void* k, const void* v, void* out, int batch, int Tq, int Tk, int Hq, int Hkv,
@@ -396,23 +431,38 @@ jsm_status flash_prefill_launch(const void* q, const void* k, const void* v, voi
     P.scale_log2 = scale * 1.4426950408889634f;
     P.out = reinterpret_cast<__nv_bfloat16*>(out);
     P.out_rs = o_rs;
+    P.q_hs = FA_D; P.v_dim = FA_D; P.window = 0;
     P.err = tc_error_word();
-    const size_t smem = (size_t)(2 + 2 * FA_KV_STAGES) * FA_TILE_BYTES + 1024;
-    static bool attr_done = false;
-    if (!attr_done) {
-        JSM_CUDA_CHECK(cudaFuncSetAttribute(flash_prefill_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        attr_done = true;
-    }
-    dim3 grid((Tq + 2 * FA_BM - 1) / (2 * FA_BM), Hq, batch);
-    // a quarter of the exponentials on the FMA pipe: the measured optimum (none: MUFU-bound, half: issue-bound)
-    flash_prefill_kernel<1><<<grid, FA_THREADS, smem, st>>>(mq, mk, mv, P);
-    JSM_LAUNCH_CHECK();
-    return JSM_OK;
+    return flash_go<128, 128, 2, false>(mq, mk, mv, P, dim3((Tq + 2 * FA_BM - 1) / (2 * FA_BM), Hq, batch), st);
 }
 
-}  // namespace jsm
+// ---- latent attention of long segments ---------------------------------------------------------------------------------
+bool latent_flash_usable(const LatentDims& d) { return d.dkp() <= 192 && d.dvp() <= 128 && d.scale > 0.0f; }
 
-namespace jsm {
-bool latent_flash_usable(const LatentDims&) { return false; }
-jsm_status latent_flash_launch(const LatentDims&, const void*, const void*, const void*, long long, void*, int, int, cudaStream_t) { return JSM_UNSUPPORTED; }
+jsm_status latent_flash_launch(const LatentDims& d, const void* q, const void* k, const void* v, long long kv_pitch, void* out, int n_q, int n_keys,
+                               cudaStream_t st) {
+    // a head's query box may reach into the next head's columns: the key's padding columns are zero there
+    CUtensorMap mq, mk, mv;
+    jsm_status s = make_tmap_bf16_2d(&mq, q, (uint64_t)n_q, (uint64_t)d.q_cols(), (uint64_t)d.q_cols(), FA_BM, 64);
+    if (s != JSM_OK) return s;
+    s = make_tmap_bf16_2d(&mk, k, (uint64_t)n_keys, (uint64_t)d.H * d.dkp(), (uint64_t)kv_pitch, FA_BN, 64);
+    if (s != JSM_OK) return s;
+    s = make_tmap_bf16_2d(&mv, v, (uint64_t)n_keys, (uint64_t)d.H * d.dvp(), (uint64_t)kv_pitch, FA_BN, 64);
+    if (s != JSM_OK) return s;
+    FlashParams P;
+    P.Tq = n_q; P.Tk = n_keys; P.Hq = d.H; P.Hkv = d.H; P.causal = 1;
+    P.scale_log2 = d.scale * 1.4426950408889634f;
+    P.out = reinterpret_cast<__nv_bfloat16*>(out);
+    P.out_rs = d.out_cols();
+    P.q_hs = d.qh(); P.v_dim = d.vdim; P.window = d.window;
+    P.err = tc_error_word();
+    const dim3 grid((n_q + 2 * FA_BM - 1) / (2 * FA_BM), d.H, 1);
+    const int qk = d.dkp();
+    if (d.dvp() == 64)
+        return qk == 64 ? flash_go<64, 64, 2, true>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 64, 2, true>(mq, mk, mv, P, grid, st)
+                                                                                   : flash_go<192, 64, 2, true>(mq, mk, mv, P, grid, st);
+    return qk == 64 ? flash_go<64, 128, 2, true>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 128, 2, true>(mq, mk, mv, P, grid, st)
+                                                                                : flash_go<192, 128, 1, true>(mq, mk, mv, P, grid, st);
+}
+
 }  // namespace jsm

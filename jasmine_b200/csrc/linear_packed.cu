@@ -1405,7 +1405,8 @@ extern "C" jsm_status jsm_linear_unpack(const void* d_packed, int N, int K, int 
 }
 
 static jsm_status linear_bf16_packed_entry(const void* d_X, const void* d_packed, const float* d_bias, int epilogue, const void* d_R,
-                                           void* d_Y, int out_dtype, int T, int N, int K, void* stream, bool chained) {
+                                           void* d_Y, int out_dtype, int T, int N, int K, void* stream, bool chained, float glu_alpha = 0.0f,
+                                           float glu_limit = 0.0f) {
     if (out_dtype != JSM_BF16 && out_dtype != JSM_F32) JSM_FAIL(JSM_UNSUPPORTED, "jsm_linear_bf16_packed: out dtype %d", out_dtype);
     if (T <= 0 || N <= 0) return JSM_OK;
     int dev = -1;
@@ -1415,6 +1416,7 @@ static jsm_status linear_bf16_packed_entry(const void* d_X, const void* d_packed
     PackedArgs a;
     a.X = d_X; a.Wp = d_packed; a.bias = d_bias; a.epilogue = epilogue; a.R = d_R; a.out_f32 = out_dtype == JSM_F32;
     a.N = N; a.K = K; a.x_row_stride = 0; a.chained = chained;
+    a.glu_alpha = glu_alpha; a.glu_limit = glu_limit;
     {
         // the workspace of this device, sized at set-up time (jsm_linear_pack / jsm_linear_packed_reserve); the launch
         // checks its capacity and fails rather than allocate
@@ -1438,12 +1440,19 @@ static jsm_status linear_bf16_packed_entry(const void* d_X, const void* d_packed
 
 extern "C" jsm_status jsm_linear_bf16_packed(const void* d_X, const void* d_packed, const float* d_bias, int epilogue, const void* d_R,
                                              void* d_Y, int out_dtype, int T, int N, int K, void* stream) {
+    if (epilogue == LIN_CLAMPED_GLU) JSM_FAIL(JSM_INVALID_ARG, "jsm_linear_bf16_packed: epilogue %d", epilogue);
     return linear_bf16_packed_entry(d_X, d_packed, d_bias, epilogue, d_R, d_Y, out_dtype, T, N, K, stream, false);
 }
 
 extern "C" jsm_status jsm_linear_bf16_packed_chained(const void* d_X, const void* d_packed, const float* d_bias, int epilogue,
                                                      const void* d_R, void* d_Y, int out_dtype, int T, int N, int K, void* stream) {
+    if (epilogue == LIN_CLAMPED_GLU) JSM_FAIL(JSM_INVALID_ARG, "jsm_linear_bf16_packed_chained: epilogue %d", epilogue);
     return linear_bf16_packed_entry(d_X, d_packed, d_bias, epilogue, d_R, d_Y, out_dtype, T, N, K, stream, true);
+}
+
+extern "C" jsm_status jsm_linear_bf16_packed_glu(const void* d_X, const void* d_packed, float alpha, float limit, void* d_Y, int T, int N, int K,
+                                                 void* stream) {
+    return linear_bf16_packed_entry(d_X, d_packed, nullptr, LIN_CLAMPED_GLU, nullptr, d_Y, JSM_BF16, T, N, K, stream, false, alpha, limit);
 }
 
 // ---- the fused exchange on its own (what the decoder runner composes; also how the protocol is tested on one GPU) ----

@@ -387,3 +387,18 @@ extern "C" jsm_status jsm_add_norm(int kind, const void* d_h, const void* d_delt
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
+
+extern "C" jsm_status jsm_post_norm_add(const float* d_y, float* d_x, const float* d_gain, float eps, void* d_x_bf16, int T, int d, void* stream) {
+    if (T <= 0) return JSM_OK;
+    if (!d_y || !d_x || !d_gain) JSM_FAIL(JSM_INVALID_ARG, "jsm_post_norm_add: null pointer");
+    if (d <= 0 || d % 8) JSM_FAIL(JSM_UNSUPPORTED, "jsm_post_norm_add: d %d (a multiple of 8)", d);
+    return post_norm_add_launch(d_y, d_x, d_gain, eps, d_x_bf16, T, d, d, as_stream(stream));
+}
+
+extern "C" jsm_status jsm_logits_finish(float* d_logits, int pitch, int rows, int vocab, float cap, uint64_t* d_keys, int32_t* d_counters,
+                                        int32_t* d_next, void* stream) {
+    if (rows <= 0) return JSM_OK;
+    if (!d_logits || !d_keys || !d_counters || !d_next) JSM_FAIL(JSM_INVALID_ARG, "jsm_logits_finish: null pointer");
+    if (vocab <= 0 || pitch < vocab) JSM_FAIL(JSM_SHAPE, "jsm_logits_finish: rows of %d logits, pitch %d", vocab, pitch);
+    return logits_finish_launch(d_logits, pitch, vocab, cap, rows, reinterpret_cast<unsigned long long*>(d_keys), d_counters, d_next, as_stream(stream));
+}

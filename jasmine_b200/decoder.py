@@ -4,22 +4,16 @@ No torch: tokens and logits are numpy arrays in host memory, the library owns th
 of the paged Llama handle (admit / step_active / retire / pool_state), plus open / step for portions and mixed batches."""
 from __future__ import annotations
 
+import contextlib
 import ctypes as C
 
 import numpy as np
 
-from . import BF16, F32, MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN, DecoderConfig, LayerConfig, check, lib
+from . import BF16, F32, MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN, DecoderConfig, LayerConfig, check, host_ptr, lib
 
 
 def _i32(a):
     return np.ascontiguousarray(a, dtype=np.int32)
-
-
-def _ptr(a):
-    """Address of a numpy array or of a host tensor; None stays None."""
-    if a is None:
-        return None
-    return a.data_ptr() if hasattr(a, "data_ptr") else a.ctypes.data
 
 
 class Decoder:
@@ -29,6 +23,8 @@ class Decoder:
         self.max_batch, self.max_context = max_batch, max_context
         cfg = DecoderConfig(len(layers), d_model, vocab, {"bfloat16": BF16, "float32": F32}[dtype], max_batch, max_context,
                             max(max_step_tokens, max_batch), pool_pages, norm_eps, logit_softcap)
+        self.max_step_tokens = cfg.max_step_tokens
+        self.max_window = max((k.window for k in layers if k.mixer == MIXER_LATENT_ATTENTION), default=0)
         arr = (LayerConfig * len(layers))(*layers)
         self._h = C.c_void_p()
         check(lib().jsm_decoder_create(C.byref(cfg), arr, C.byref(self._h)))
@@ -62,7 +58,7 @@ class Decoder:
         h_next = np.empty(n, np.int32) if h_next is None else h_next
         h_logits = np.empty((n, self.vocab), np.float32) if h_logits is None else h_logits
         check(lib().jsm_decoder_step(self._h, len(entries), rows.ctypes.data, counts.ctypes.data, ids.ctypes.data, n,
-                                     want.ctypes.data, _ptr(h_next), _ptr(h_logits), None))
+                                     want.ctypes.data, host_ptr(h_next), host_ptr(h_logits), None))
         return h_next, h_logits
 
     def admit(self, h_prompt, h_logits_last=None):
@@ -71,17 +67,25 @@ class Decoder:
             h_prompt = _i32(h_prompt)
         n = h_prompt.numel() if hasattr(h_prompt, "numel") else h_prompt.size
         row, tok = C.c_int(), C.c_int32()
-        check(lib().jsm_decoder_seq_admit(self._h, _ptr(h_prompt), n, C.byref(row), C.addressof(tok), _ptr(h_logits_last), None))
+        check(lib().jsm_decoder_seq_admit(self._h, host_ptr(h_prompt), n, C.byref(row), C.addressof(tok), host_ptr(h_logits_last), None))
         return row.value, tok.value
 
     def step_active(self, h_ids, h_next, h_logits=None):
-        check(lib().jsm_decoder_step_active(self._h, _ptr(h_ids), _ptr(h_next), _ptr(h_logits), None))
+        check(lib().jsm_decoder_step_active(self._h, host_ptr(h_ids), host_ptr(h_next), host_ptr(h_logits), None))
 
     def retire(self, row: int) -> int:
         """Frees the row; returns the old index of the row that moved into its place, or -1."""
         moved = C.c_int()
         check(lib().jsm_decoder_seq_retire(self._h, row, C.byref(moved), None))
         return moved.value
+
+    def pages_for(self, n_tokens: int) -> int:
+        """Cache pages a sequence of n_tokens positions holds at most: pages behind every window go back to the pool."""
+        reach = min(n_tokens, self.max_window + self.max_step_tokens)
+        return min(-(-n_tokens // 64), reach // 64 + 2) if self.max_window else 0
+
+    def stream_scope(self):
+        return contextlib.nullcontext()  # the library runs the model on a stream of its own
 
     def pool_state(self):
         a, f, t = C.c_int(), C.c_int(), C.c_int()

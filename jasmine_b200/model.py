@@ -5,7 +5,7 @@ import ctypes as C
 
 import numpy as np
 
-from . import ALLREDUCE_FN, BF16, F32, ModelConfig, check, lib, stream_ptr
+from . import ALLREDUCE_FN, BF16, F32, ModelConfig, check, host_ptr, lib, stream_ptr
 
 
 class Llama:
@@ -23,21 +23,41 @@ class Llama:
 
     # ---- continuous batching (host tensors in, host values out) ----
     def admit(self, h_prompt, h_logits_last=None):
-        """Prefills a prompt (int32 host tensor) into the next free batch row; returns (row, first generated token)."""
+        """Prefills a prompt (int32 host array) into the next free batch row; returns (row, first generated token)."""
         row, tok = C.c_int(), C.c_int32()
-        check(lib().jsm_llama_seq_admit(self._h, h_prompt.data_ptr(), h_prompt.numel(), C.byref(row), C.byref(tok),
-                                        h_logits_last.data_ptr() if h_logits_last is not None else None, stream_ptr()))
+        n = h_prompt.numel() if hasattr(h_prompt, "numel") else h_prompt.size
+        check(lib().jsm_llama_seq_admit(self._h, host_ptr(h_prompt), n, C.byref(row), C.byref(tok), host_ptr(h_logits_last),
+                                        stream_ptr()))
         return row.value, tok.value
 
     def step_active(self, h_ids, h_next, h_logits=None):
-        check(lib().jsm_llama_step_active(self._h, h_ids.data_ptr(), h_next.data_ptr(),
-                                          h_logits.data_ptr() if h_logits is not None else None, stream_ptr()))
+        check(lib().jsm_llama_step_active(self._h, host_ptr(h_ids), host_ptr(h_next), host_ptr(h_logits), stream_ptr()))
 
     def retire(self, row: int) -> int:
         """Frees the row; returns the old index of the row that moved into its place, or -1."""
         moved = C.c_int()
         check(lib().jsm_llama_seq_retire(self._h, row, C.byref(moved), stream_ptr()))
         return moved.value
+
+    @property
+    def max_batch(self):
+        return self.cfg.max_batch
+
+    @property
+    def max_context(self):
+        return self.cfg.max_context
+
+    @property
+    def vocab(self):
+        return self.cfg.vocab
+
+    def pages_for(self, n_tokens: int) -> int:
+        """Cache pages a sequence of n_tokens positions holds."""
+        return -(-n_tokens // 64)
+
+    def stream_scope(self):
+        import torch
+        return torch.cuda.stream(torch.cuda.Stream())  # a captured step needs a stream of its own
 
     def pool_state(self):
         a, f, t = C.c_int(), C.c_int(), C.c_int()
