@@ -304,6 +304,148 @@ def run_kernel_workload(args, collect=False):
     return records
 
 
+# ---- the layer-list decoder beside the LLaMA shape ---------------------------------------------------------------------
+def zugolorn_config(width):
+    """Layers of a real model's proportions: latent attention (feed-forward behind it) and selective scans in turn."""
+    heads = width // 128
+    attn = {"type": "latent_attention",
+            "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "mask": {"size": 1024 if width < 4096 else 4096},
+                      "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5},
+            "mlp": {"kind": "dense", "ff": width * 43 // 16, "limit": 7.0}}
+    scan = {"type": "mamba1", "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}, "mlp": None}
+    return {"architecture": "Zugolorn", "width": width, "vocab": 32000, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [attn, scan] * 4}
+
+
+def random_tensors(cfg):
+    """(name, bf16 bits) of every tensor: slices of one pool of normal numbers, scaled by a power of two near K^-1/2."""
+    import numpy as np
+    pool = np.random.default_rng(SEED).standard_normal(1 << 24, dtype=np.float32)
+    at = [0]
+
+    def draw(shape, std, mean=0.0):
+        n = int(np.prod(shape))
+        at[0] = (at[0] + 7919) % 4096
+        x = np.resize(pool[at[0]:], n).reshape(shape) * np.float32(std) + np.float32(mean)
+        return (x.view(np.uint32) >> 16).astype(np.uint16)
+
+    d = cfg["width"]
+    yield "embed", draw((cfg["vocab"], d), 1.0)
+    yield "final.norm", draw((d,), 0.1, 1.0)
+    for i, e in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", e["mixer"]
+        yield p + "norm1", draw((d,), 0.05, 0.4)
+        if e["type"] == "latent_attention":
+            H, r = m["heads"], m["kv_rank"]
+            shapes = {"q": (H * (m["dim"] + m["rot_dim"]), d), "dkv": (r + m["rot_dim"], d), "uk": (H * m["dim"], r), "uv": (H * m["vdim"], r),
+                      "o": (d, H * m["vdim"])}
+            yield p + "mix.dkv.norm", draw((r,), 0.1, 1.0)
+        else:
+            c, n, R = m["inner"], m["state"], m["dt_rank"]
+            shapes = {"in": (2 * c, d), "x": (R + 2 * n, c), "dt": (c, R), "o": (d, c)}
+            yield p + "mix.conv", draw((c, m["conv"]), 0.5)
+            for k, (std, mean) in {"conv.b": (0.1, 0.0), "dt.b": (0.5, -4.0), "D": (0.1, 1.0)}.items():
+                yield p + "mix." + k, draw((c,), std, mean)
+            yield p + "mix.A_log", draw((c, n), 0.5)
+        for k, s in shapes.items():
+            yield p + "mix." + k, draw(s, s[1] ** -0.5)
+        if e["mlp"]:
+            f = e["mlp"]["ff"]
+            yield p + "norm2", draw((d,), 0.05, 0.4)
+            for k, s in {"gate": (f, d), "up": (f, d), "down": (d, f)}.items():
+                yield p + "mlp." + k, draw(s, s[1] ** -0.5)
+
+
+def run_decoder_workload(args):
+    """Prefill and decode throughput of the Zugolorn design at two widths and of the LLaMA shape of equal width and about
+    equal weight bytes, both through their host-buffer serving calls (token ids in, next tokens out, every step)."""
+    import numpy as np
+    import torch
+    import jasmine_b200 as jb
+    from jasmine_b200.decoder import zugolorn_model
+    from jasmine_b200.model import Llama
+    torch.cuda.set_device(0)
+    hbm, peak_kind = measured_peaks()
+    p = ROOT / "MEASURED_PEAKS.json"
+    tf_peak = float(json.loads(p.read_text())["bf16_tflops"]) if p.exists() else 1590.0
+    K, W = max(args.steps, 1), max(args.warmup, 3)
+    rng = np.random.default_rng(SEED)
+    sampler = ClockSampler(0)
+    stream = torch.cuda.Stream()
+
+    def timed(fn, n):
+        for _ in range(W):
+            fn()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record(stream)
+        for _ in range(n):
+            fn()
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    def emit(model, phase, ms, tokens, nbytes, flops, extra):
+        frac_h, frac_t = nbytes / (ms * 1e-3) / 1e9 / hbm, flops / (ms * 1e-3) / 1e12 / tf_peak
+        print(json.dumps({"metric": f"{phase}_tokens_per_s", "value": tokens / (ms * 1e-3), "unit": "tokens/s", "n_gpus": 1, "steps": K,
+                          "warmup": W, "ms_per_step": ms, "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
+                          "data": "synthetic tokens, random weights", "config": {"model": model, **extra},
+                          "roofline": {"hbm_frac": frac_h, "tensor_frac": frac_t, "peak_source": peak_kind}}), flush=True)
+
+    widths = [args.width] if args.width else [2048, 4096]
+    for width in widths:
+        sampler.start()
+        cfg = zugolorn_config(width)
+        z = zugolorn_model(cfg, max_batch=64, max_context=8192, max_step_tokens=2048, pool_pages=64 * 12 + 128)
+        for name, bits in random_tensors(cfg):
+            z.set_weight(name, bits)
+        z.finalize()
+        z.stream = stream.cuda_stream
+        wbytes = z.step_bytes(0)[0]
+        params = wbytes / 2
+        head = 32000 * width
+        # a LLaMA layer of this width: 4 d^2 + 3 d ffn
+        ffn = width * 43 // 16
+        n_llama = max(1, round((params - head) / (4 * width * width + 3 * width * ffn)))
+        llama = Llama(n_llama, width, width // 128, width // 128, ffn, 32000, max_batch=64, max_context=1024, seed=SEED, pool_pages=64 * 16)
+        lbytes = llama.step_bytes()[0]
+        names = (f"zugolorn w{width} 4 x (latent attention + ff, scan), {wbytes / 1e9:.2f} GB", f"llama w{width} {n_llama} layers, {lbytes / 1e9:.2f} GB")
+        torch.cuda.synchronize()
+        with torch.cuda.stream(stream):
+            for T in (512, 2048):
+                prompt = rng.integers(0, 32000, T).astype(np.int32)
+
+                def z_prefill():
+                    row, _ = z.admit(prompt)
+                    z.retire(row)
+                attn = sum(4.0 * min(e["mixer"]["mask"]["size"], T / 2) * T * e["mixer"]["heads"] * 160 for e in cfg["layers"] if e["type"] == "latent_attention")
+                emit(names[0], "prefill", timed(z_prefill, max(3, K // 8)), T, wbytes, 2.0 * T * (params - head) + attn, {"seq_len": T})
+                if T <= 512:
+                    def l_prefill():
+                        row, _ = llama.admit(prompt)
+                        llama.retire(row)
+                    attn = n_llama * 4.0 * T * T / 2 * width
+                    emit(names[1], "prefill", timed(l_prefill, max(3, K // 8)), T, lbytes, 2.0 * T * (lbytes / 2 - head) + attn, {"seq_len": T})
+            for B in (1, 8, 64):
+                ctx = 512
+                for m, name, nb in ((z, names[0], lambda c: wbytes + B * z.step_bytes(c)[1]), (llama, names[1], lambda c: lbytes + B * c * llama.step_bytes()[1])):
+                    for b in range(B):
+                        m.admit(rng.integers(0, 32000, ctx).astype(np.int32))
+                    ids, nxt = np.zeros(B, np.int32), np.zeros(B, np.int32)
+
+                    def step():
+                        m.step_active(ids, nxt)
+                        ids[:] = nxt
+                    ms = timed(step, K)
+                    emit(name, "decode", ms, B, nb(ctx + W + K // 2), 0.0, {"batch": B, "context": ctx + W + K // 2})
+                    for b in range(B):
+                        m.retire(0)
+        jb.check_device_errors()
+        z.close()
+        llama.close()
+        print(json.dumps({"clocks": sampler.stop()}), flush=True)
+
+
 def run_timeline(args):
     """Device timeline of the packed projections of one eager decode step (jsm_trace_begin / jsm_trace_end): for every
     projection kind the time its CTAs were resident before their predecessor finished, the main loop, the tail (last
@@ -468,9 +610,11 @@ def main():
     ap.add_argument("--layers", type=int, default=32, help="debug only: fewer layers (the result is then not a bench value)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-extras", action="store_true", help="headline only: skip the batch-1/64 legs, the kernel-level legs and the tp parity check")
-    ap.add_argument("--workload", default="decode", choices=["decode", "expr", "flash", "kvdecode", "gateup", "timeline"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "expr", "flash", "kvdecode", "gateup", "timeline", "zugolorn"],
                     help="decode = the headline; expr / flash / kvdecode = configurations 2 / 3 / 4 of the baseline "
-                         "(kernel-level lines, one JSON line per kernel)")
+                         "(kernel-level lines, one JSON line per kernel); zugolorn = prefill and decode throughput of "
+                         "that design beside the LLaMA shape")
+    ap.add_argument("--width", type=int, default=0, help="zugolorn workload only: this width instead of both")
     ap.add_argument("--tp-emulate", type=int, default=1,
                     help="timeline workload only: run ONE rank of a tensor-parallel group of this size on one GPU")
     ap.add_argument("--profile-steps", type=int, default=0,
@@ -482,6 +626,8 @@ def main():
     args.warmup = max(args.warmup, 3)
     if args.workload == "timeline":
         return run_timeline(args)
+    if args.workload == "zugolorn":
+        return run_decoder_workload(args)
     if args.workload != "decode":
         return run_kernel_workload(args)
 

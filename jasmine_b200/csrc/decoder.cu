@@ -33,6 +33,7 @@ struct Proj {  // one projection: N outputs, K inputs, both rounded up to multip
     int N = 0, K = 0, paired = 0;
     uint8_t* packed = nullptr;  // bf16 models
     float* w32 = nullptr;       // f32 models, [N][K]
+    void* rows = nullptr;       // bf16 models, projections with few outputs or few inputs: also row-major, for many tokens
 };
 
 struct DecLayer {
@@ -276,14 +277,14 @@ static jsm_status build_scan(jsm_decoder* m, DecLayer& L, const std::string& pre
             h.put_row(d.rp() + d.np() + j, *xp, d.dt_rank + d.state + j);
         }
         DEC_TRY(upload_proj(m, h, &L.xp));
+        if (!m->f32) DEC_TRY(upload_plain(m, h, &L.xp.rows));
     }
     {
         HostMatrix h(m->f32, ip, d.rp());
         for (int j = 0; j < d.inner; ++j) h.put_row(j, *dt, j);
         DEC_TRY(upload_proj(m, h, &L.dt));
-        void* p = L.dt.w32;
-        if (!m->f32) DEC_TRY(upload_plain(m, h, &p));
-        L.sw.dt = p;
+        if (!m->f32) DEC_TRY(upload_plain(m, h, &L.dt.rows));
+        L.sw.dt = m->f32 ? (void*)L.dt.w32 : L.dt.rows;
     }
     {
         HostMatrix h(m->f32, wp, ip);
@@ -345,6 +346,20 @@ static jsm_status linear(jsm_decoder* m, const Proj& p, const void* X, long long
     a.N = p.N; a.K = p.K; a.x_row_stride = x_stride;
     a.ws = m->ws; a.ws_floats = m->ws_floats; a.counters = m->counters; a.n_counters = m->n_counters;
     a.chained = true;  // the weights are constant while the model's stream runs
+    if (p.rows && T > 64 && x_stride == p.K) {
+        // the packed kernel streams the weights once per 256 tokens over all SMs, which suits wide and deep matrices; here one
+        // launch tiles outputs x tokens, split along K while that leaves SMs idle
+        const int tiles = ((p.N + 127) / 128) * ((T + 127) / 128);
+        LinearArgs r;
+        r.X = X; r.W = p.rows; r.bias = nullptr; r.epilogue = LIN_NONE; r.R = nullptr; r.Y = Y;
+        r.out_mode = out_f32 ? 1 : 0;
+        r.T = T; r.N = p.N; r.K = p.K; r.impl = 2;
+        r.splits = std::max(1, std::min(sm_count() / tiles, p.K / 512));
+        r.ws = r.splits > 1 ? m->ws : nullptr;
+        r.counters = m->counters;
+        r.chained = true;
+        return linear_bf16_launch(r, st);
+    }
     for (int t0 = 0; t0 < T; t0 += 256) {
         a.T = std::min(256, T - t0);
         a.X = static_cast<const __nv_bfloat16*>(X) + (long long)t0 * x_stride;
@@ -760,6 +775,9 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     DEC_TRY(dalloc(m, &m->keys, 8 * (size_t)m->cap_rows));
     DEC_TRY(dalloc(m, &m->key_ctrs, 4 * (size_t)m->cap_rows));
     DEC_TRY(dalloc(m, &m->next_dev, 4 * (size_t)m->cap_rows));
+    // (partials of a split row-major projection: at most one 128 x 128 tile per SM)
+    m->ws_floats = std::max(m->ws_floats, (size_t)sm_count() * 128 * 128);
+    m->n_counters = std::max(m->n_counters, sm_count());
     DEC_TRY(dalloc(m, &m->ws, 4 * m->ws_floats));
     DEC_TRY(dalloc(m, &m->counters, 4 * (size_t)m->n_counters));
     std::map<int, int> heads;

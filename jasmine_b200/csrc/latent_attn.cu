@@ -24,12 +24,30 @@ using tc::smem_u32;
 constexpr int PAGE = JSM_PAGE_SIZE;
 
 // ---- append and rotation ------------------------------------------------------------------------------------------
-// One CTA per token.  qd row: [q head 0 (qh) | ... | down: c (rank), key part (rot)].
+// qd row of a token: [q head 0 (qh) | ... | down: c (rank), key part (rot)].  Blocks (token, part): the last part makes the
+// cache entry, the others 256 groups of 8 query components each.  vec: the boundaries between the unrotated part, the two
+// halves of the rotated part and the padding are multiples of 8.
+template <typename T>
+__device__ __forceinline__ void store8(T* p, const float (&v)[8]);
+template <>
+__device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <>
+__device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restrict__ qd, LatentDims d, const float* __restrict__ gain, float eps,
                                                           T* __restrict__ pool, const int32_t* __restrict__ block_table, int max_pages,
                                                           const float2* __restrict__ rope, const int32_t* __restrict__ tok_row,
-                                                          const int32_t* __restrict__ tok_pos, T* __restrict__ q) {
+                                                          const int32_t* __restrict__ tok_pos, T* __restrict__ q, int vec) {
     __shared__ float red[8];
     chain_trigger();
     chain_wait();
@@ -38,21 +56,46 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
     const float* src = qd + (long long)t * (q_cols + cr);
     const int pos = tok_pos[t];
     const float2* cs = rope + (long long)pos * half;
-    // queries: unrotated components copied, the rest rotated (component i with i + rot/2)
-    T* qo = q + (long long)t * q_cols;
-    for (int i = threadIdx.x; i < q_cols; i += 256) {
-        const int j = i % qh;
-        float v = 0.0f;
-        if (j < d.dim) {
-            v = src[i];
-        } else if (j < d.dim + d.rot) {
-            const int r = j - d.dim, p = r < half ? r : r - half;
-            const float2 e = cs[p];
-            const float* base = src + (i - j) + d.dim;
-            const float a = base[p], b = base[p + half];
-            v = r < half ? a * e.x - b * e.y : b * e.x + a * e.y;
+    if (blockIdx.y + 1 < gridDim.y) {
+        // queries: unrotated components copied, the rest rotated (component i with i + rot/2)
+        const int i0 = (blockIdx.y * 256 + threadIdx.x) * 8;
+        if (i0 >= q_cols) return;
+        const int j0 = i0 % qh;
+        float v[8];
+        if (vec) {
+            load8(src + i0, v);
+            if (j0 >= d.dim + d.rot) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = 0.0f;
+            } else if (j0 >= d.dim) {
+                const int r = j0 - d.dim;
+                const bool lower = r < half;
+                const int p = lower ? r : r - half;
+                float o[8], c[16];
+                load8(src + (lower ? i0 + half : i0 - half), o);
+                load8(reinterpret_cast<const float*>(cs + p), reinterpret_cast<float(&)[8]>(c[0]));
+                load8(reinterpret_cast<const float*>(cs + p + 4), reinterpret_cast<float(&)[8]>(c[8]));
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = lower ? v[e] * c[2 * e] - o[e] * c[2 * e + 1] : v[e] * c[2 * e] + o[e] * c[2 * e + 1];
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int j = j0 + e;
+                v[e] = 0.0f;
+                if (j < d.dim) {
+                    v[e] = src[i0 + e];
+                } else if (j < d.dim + d.rot) {
+                    const int r = j - d.dim, p = r < half ? r : r - half;
+                    const float2 f = cs[p];
+                    const float* base = src + (i0 - j0) + d.dim;
+                    const float a = base[p], b = base[p + half];
+                    v[e] = r < half ? a * f.x - b * f.y : b * f.x + a * f.y;
+                }
+            }
         }
-        qo[i] = from_f32<T>(v);
+        store8(q + (long long)t * q_cols + i0, v);
+        return;
     }
     // latent: RMS norm, then the cache entry
     const float* down = src + q_cols;
@@ -115,24 +158,37 @@ __global__ void __launch_bounds__(256) latent_project_simt_kernel(ProjectArgs a)
 
 // bf16 on the tensor cores: the weights are the 16-row operand, eight tokens the other, so that a decode step wastes no
 // rows.  A lane's eight consecutive k of a 32-wide block feed two k16 products - both operands in the same order, so every
-// fragment is one 16-byte load straight from global memory.  Block: 4 warps x 16 output rows; up to 32 tokens per CTA.
+// fragment is one 16-byte load straight from global memory.  Four warps per CTA: 16 output rows each, or (KSPLIT) the same
+// 16 rows and a quarter of k each, added in warp order; up to 32 tokens.
+template <bool KSPLIT>
 __global__ void __launch_bounds__(128) latent_project_mma_kernel(ProjectArgs a) {
+    __shared__ float fold[KSPLIT ? 3 * 16 * 32 : 1];
     chain_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y;
-    const int n0 = blockIdx.x * 64 + warp * 16;
+    const int n0 = KSPLIT ? blockIdx.x * 16 : blockIdx.x * 64 + warp * 16;
     const int g = lane >> 2, kq = (lane & 3) * 8;
     const int t_begin = a.t0 + blockIdx.z * 32, t_end = min(a.t0 + a.T, t_begin + 32);
-    chain_wait();
-    if (n0 < a.N) {
-        const __nv_bfloat16* w0 = static_cast<const __nv_bfloat16*>(a.W) + ((long long)h * a.nw + n0 + g) * a.kw + kq;
-        const __nv_bfloat16* w1 = w0 + 8 * a.kw;
-        const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + h * a.in_hs + kq;
-        float acc[4][4];
+    const int n_blk = a.kw / 32;
+    const int b0 = KSPLIT ? n_blk * warp / 4 : 0, b1 = KSPLIT ? n_blk * (warp + 1) / 4 : n_blk;
+    const bool on = n0 < a.N;
+    const __nv_bfloat16* w0 = static_cast<const __nv_bfloat16*>(a.W) + ((long long)h * a.nw + (on ? n0 : 0) + g) * a.kw + kq;
+    const __nv_bfloat16* w1 = w0 + 8 * a.kw;
+    // the weights are constant: the first blocks are requested before the predecessor kernel has finished
+    constexpr int PRE = 4;
+    uint4 px[PRE], py[PRE];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
-#pragma unroll 4
-        for (int k = 0; k < a.kw; k += 32) {
-            const uint4 x = __ldg(reinterpret_cast<const uint4*>(w0 + k)), y = __ldg(reinterpret_cast<const uint4*>(w1 + k));
+    for (int i = 0; i < PRE; ++i)
+        if (on && b0 + i < b1) {
+            px[i] = __ldg(reinterpret_cast<const uint4*>(w0 + (b0 + i) * 32));
+            py[i] = __ldg(reinterpret_cast<const uint4*>(w1 + (b0 + i) * 32));
+        }
+    chain_wait();
+    float acc[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
+    if (on) {
+        const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + h * a.in_hs + kq;
+        auto block = [&](int k, const uint4& x, const uint4& y) {
             const uint32_t a0[4] = {x.x, y.x, x.y, y.y}, a1[4] = {x.z, y.z, x.w, y.w};
             const bool k_in = k + kq < a.K;  // the operand's pitch covers K rounded up to 8; weights beyond K are zero
 #pragma unroll
@@ -144,7 +200,30 @@ __global__ void __launch_bounds__(128) latent_project_mma_kernel(ProjectArgs a) 
                 mma_16816(acc[j], a0, b.x, b.y);
                 mma_16816(acc[j], a1, b.z, b.w);
             }
-        }
+        };
+#pragma unroll
+        for (int i = 0; i < PRE; ++i)
+            if (b0 + i < b1) block((b0 + i) * 32, px[i], py[i]);
+#pragma unroll 4
+        for (int i = b0 + PRE; i < b1; ++i)
+            block(i * 32, __ldg(reinterpret_cast<const uint4*>(w0 + i * 32)), __ldg(reinterpret_cast<const uint4*>(w1 + i * 32)));
+    }
+    if constexpr (KSPLIT) {
+        if (warp > 0)
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) fold[((warp - 1) * 16 + j * 4 + e) * 32 + lane] = acc[j][e];
+        __syncthreads();
+        if (warp == 0)
+#pragma unroll
+            for (int w = 0; w < 3; ++w)
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) acc[j][e] += fold[(w * 16 + j * 4 + e) * 32 + lane];
+    }
+    if (on && (!KSPLIT || warp == 0)) {
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + h * a.out_hs;
 #pragma unroll
         for (int j = 0; j < 4; ++j)
@@ -169,8 +248,10 @@ static jsm_status project(bool f32, const ProjectArgs& a, int H, cudaStream_t st
     if (a.T <= 0) return JSM_OK;
     if (f32)
         JSM_CUDA_CHECK(launch_chained(latent_project_simt_kernel<float>, dim3((a.out_pad + 31) / 32, H, (a.T + 7) / 8), dim3(256), 0, st, a));
+    else if (a.kw >= 256)
+        JSM_CUDA_CHECK(launch_chained(latent_project_mma_kernel<true>, dim3((a.N + 15) / 16, H, (a.T + 31) / 32), dim3(128), 0, st, a));
     else
-        JSM_CUDA_CHECK(launch_chained(latent_project_mma_kernel, dim3((a.N + 63) / 64, H, (a.T + 31) / 32), dim3(128), 0, st, a));
+        JSM_CUDA_CHECK(launch_chained(latent_project_mma_kernel<false>, dim3((a.N + 63) / 64, H, (a.T + 31) / 32), dim3(128), 0, st, a));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -242,6 +323,8 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
 constexpr int LA_ROWS = LATENT_TILE_ROWS;
 constexpr int LA_SP = 68;  // pitch of the score tile (floats)
 constexpr int LA_PP = 72;  // pitch of the weight tile (bf16)
+constexpr int LA_ML = 4;   // behind a partial row: its maximum, its sum, two unused
+constexpr int LA_MAX_SPLITS = 256;
 
 static int la_pitch(const LatentDims& d) { return pad_to(d.rank + d.rot, 16) + 8; }  // odd multiple of 16 bytes: no bank conflicts
 static size_t la_smem(const LatentDims& d) {
@@ -280,7 +363,9 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat1
     const int p_first = pos0 + r0 / d.H, p_last = pos0 + (r0 + n_rows - 1) / d.H;
     const int key_lo = max(0, p_first - d.window + 1), key_hi = p_last + 1;
     const int pg_lo = key_lo / PAGE, n_pg = (key_hi - 1) / PAGE - pg_lo + 1;
-    const int pb = pg_lo + (int)((long long)n_pg * sp / splits), pe = pg_lo + (int)((long long)n_pg * (sp + 1) / splits);
+    const int live = min(splits, n_pg);  // the grid is made for the longest context: the splits behind the pages of this one rest
+    if (sp >= live) return;
+    const int pb = pg_lo + n_pg * sp / live, pe = pg_lo + n_pg * (sp + 1) / live;
     const int32_t* bt = block_table + (long long)seg_row[seg] * max_pages;
     const int vec = cr / 8;  // 16-byte vectors per entry
     auto load_page = [&](int pg, int stage) {
@@ -334,9 +419,9 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat1
         for (int i = 0; i < LA_ROWS / 8; ++i) {  // softmax: a warp per row, two keys per lane
             const int r = warp * (LA_ROWS / 8) + i;
             const int p = pos0 + (r0 + r) / d.H, k0 = pg * PAGE + lane, k1 = k0 + 32;
-            const bool live = r < n_rows;
-            float a = (live && k0 <= p && p - k0 < d.window) ? ss[r * LA_SP + lane] * d.scale : -INFINITY;
-            float b = (live && k1 <= p && p - k1 < d.window) ? ss[r * LA_SP + lane + 32] * d.scale : -INFINITY;
+            const bool on = r < n_rows;
+            float a = (on && k0 <= p && p - k0 < d.window) ? ss[r * LA_SP + lane] * d.scale : -INFINITY;
+            float b = (on && k1 <= p && p - k1 < d.window) ? ss[r * LA_SP + lane + 32] * d.scale : -INFINITY;
             const float m_old = row_m[r], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
             const float ref = m_new == -INFINITY ? 0.0f : m_new;
             a = __expf(a - ref);
@@ -403,38 +488,57 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat1
                             pack_bf16x2(c < d.rank ? o[a][j][e] * inv : 0.0f, c + 1 < d.rank ? o[a][j][e + 1] * inv : 0.0f);
                     }
                 } else {
-                    float* out = part + (((long long)tile * splits + sp) * LA_ROWS + r) * (rp + 2);
-                    if (c < rp) { out[c] = o[a][j][e]; out[c + 1] = o[a][j][e + 1]; }
+                    float* out = part + (((long long)tile * splits + sp) * LA_ROWS + r) * (rp + LA_ML);
+                    if (c < rp) *reinterpret_cast<float2*>(out + c) = make_float2(o[a][j][e], o[a][j][e + 1]);
                     if (warp == 0 && j == 0 && (lane & 3) == 0) { out[rp] = row_m[r]; out[rp + 1] = row_l[r]; }
                 }
             }
         }
 }
 
-// merges the partials of the splits in split order; one CTA per (tile, row)
+// merges the partials of the splits in split order; one CTA per (tile, row), four columns per thread
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part, LatentDims d, const int32_t* __restrict__ seg_start,
                                                              const int32_t* __restrict__ seg_len, const int32_t* __restrict__ tile_seg,
-                                                             const int32_t* __restrict__ tile_r0, int splits, __nv_bfloat16* __restrict__ o_lat) {
+                                                             const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ tile_r0, int max_splits,
+                                                             __nv_bfloat16* __restrict__ o_lat) {
+    __shared__ float w[LA_MAX_SPLITS];
+    __shared__ float red[8];
     chain_trigger();
     chain_wait();
-    const int tile = blockIdx.x, r = blockIdx.y, rp = pad8(d.rank);
+    const int tile = blockIdx.x, r = blockIdx.y, rp = pad8(d.rank), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int seg = tile_seg[tile], g = tile_r0[tile] + r;
-    if (g >= seg_len[seg] * d.H) return;
-    const long long stride = (long long)LA_ROWS * (rp + 2);
-    const float* p = part + ((long long)tile * splits * LA_ROWS + r) * (rp + 2);
+    const int r0 = tile_r0[tile], n_all = seg_len[seg] * d.H;
+    if (g >= n_all) return;
+    // the splits that had pages (as in the attention kernel)
+    const int p_first = seg_pos0[seg] + r0 / d.H, p_last = seg_pos0[seg] + (min(r0 + LA_ROWS, n_all) - 1) / d.H;
+    const int splits = min(max_splits, p_last / PAGE - max(0, p_first - d.window + 1) / PAGE + 1);
+    const long long stride = (long long)LA_ROWS * (rp + LA_ML);
+    const float* p = part + ((long long)tile * max_splits * LA_ROWS + r) * (rp + LA_ML);
     float m = -INFINITY;
-    for (int s = 0; s < splits; ++s) m = fmaxf(m, p[s * stride + rp]);
+    for (int s = threadIdx.x; s < splits; s += 128) m = fmaxf(m, p[s * stride + rp]);
+    m = warp_max(m);
+    if (lane == 0) red[warp] = m;
+    __syncthreads();
+    m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+    for (int s = threadIdx.x; s < splits; s += 128) w[s] = __expf(p[s * stride + rp] - m);
+    __syncthreads();
     float l = 0.0f;
-    for (int s = 0; s < splits; ++s) l += p[s * stride + rp + 1] * __expf(p[s * stride + rp] - m);
-    const float inv = 1.0f / l;
+    for (int s = lane; s < splits; s += 32) l += w[s] * p[s * stride + rp + 1];  // every warp for itself
+    const float inv = 1.0f / warp_sum(l);
     __nv_bfloat16* out = o_lat + ((long long)(seg_start[seg] + g / d.H) * d.H + g % d.H) * rp;
-    for (int c = threadIdx.x; c < rp; c += 128) {
-        float acc = 0.0f;
+    for (int c = threadIdx.x * 4; c < rp; c += 512) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
         for (int s = 0; s < splits; ++s) {
-            const float w = __expf(p[s * stride + rp] - m);
-            if (w > 0.0f) acc += w * p[s * stride + c];
+            const float4 v = __ldcs(reinterpret_cast<const float4*>(p + s * stride + c));
+            const float f = w[s];  // a split without a visible key holds zeros and weighs nothing
+            acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
         }
-        out[c] = __float2bfloat16_rn(c < d.rank ? acc * inv : 0.0f);
+        const float o[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
+        uint2 u;
+        u.x = pack_bf16x2(c < d.rank ? o[0] : 0.0f, c + 1 < d.rank ? o[1] : 0.0f);
+        u.y = pack_bf16x2(c + 2 < d.rank ? o[2] : 0.0f, c + 3 < d.rank ? o[3] : 0.0f);
+        *reinterpret_cast<uint2*>(out + c) = u;
     }
 }
 
@@ -452,13 +556,15 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const __nv_bfloat16*
 // ---- launches -----------------------------------------------------------------------------------------------------
 jsm_status latent_prep_launch(bool f32, const float* qd, const LatentDims& d, const LatentWeights& w, float eps, const LatentCache& cache,
                               const StepTokens& tk, void* q, cudaStream_t st) {
+    const dim3 grid(tk.T, (d.q_cols() / 8 + 255) / 256 + 1);
+    const int vec = d.dim % 8 == 0 && d.rot % 16 == 0 ? 1 : 0;
     if (f32)
-        JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<float>, dim3(tk.T), dim3(256), 0, st, qd, d, w.down_norm, eps, (float*)cache.pool,
-                                      cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, (float*)q));
+        JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<float>, grid, dim3(256), 0, st, qd, d, w.down_norm, eps, (float*)cache.pool,
+                                      cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, (float*)q, vec));
     else
-        JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<__nv_bfloat16>, dim3(tk.T), dim3(256), 0, st, qd, d, w.down_norm, eps,
+        JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, qd, d, w.down_norm, eps,
                                       (__nv_bfloat16*)cache.pool, cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos,
-                                      (__nv_bfloat16*)q));
+                                      (__nv_bfloat16*)q, vec));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -468,9 +574,9 @@ bool latent_mma_usable(const LatentDims& d) { return d.rank <= 512 && la_smem(d)
 int latent_splits(int n_tiles, int max_keys) {
     if (n_tiles <= 0) return 1;
     const int pages = max_keys / PAGE + 2;
-    return std::max(1, std::min(sm_count() / n_tiles, pages / 2));
+    return std::max(1, std::min({sm_count() / n_tiles, pages / 2, LA_MAX_SPLITS}));
 }
-size_t latent_part_floats(const LatentDims& d) { return (size_t)sm_count() * LA_ROWS * (pad8(d.rank) + 2); }
+size_t latent_part_floats(const LatentDims& d) { return (size_t)sm_count() * LA_ROWS * (pad8(d.rank) + LA_ML); }
 
 template <int NT>
 static jsm_status launch_mma(const LatentDims& d, const LatentCache& cache, const StepTokens& tk, const LatentTiles& tl, const LatentScratch& sc,
@@ -513,7 +619,7 @@ jsm_status latent_attn_launch(bool f32, const LatentDims& d, const LatentWeights
         JSM_LAUNCH_CHECK();
     } else {
         const int splits = latent_splits(tl.n_tiles, tl.max_keys);
-        if (splits > 1 && (size_t)tl.n_tiles * splits * LA_ROWS * (rp + 2) > sc.part_floats)
+        if (splits > 1 && (size_t)tl.n_tiles * splits * LA_ROWS * (rp + LA_ML) > sc.part_floats)
             JSM_FAIL(JSM_INVALID_ARG, "latent attention: workspace of %zu floats for %d tiles in %d splits", sc.part_floats, tl.n_tiles, splits);
         s = d.rank <= 128   ? launch_mma<2>(d, cache, tk, tl, sc, splits, st)
             : d.rank <= 256 ? launch_mma<4>(d, cache, tk, tl, sc, splits, st)
@@ -522,7 +628,7 @@ jsm_status latent_attn_launch(bool f32, const LatentDims& d, const LatentWeights
         if (s != JSM_OK) return s;
         if (splits > 1) {
             JSM_CUDA_CHECK(launch_chained(latent_combine_kernel, dim3(tl.n_tiles, LA_ROWS), dim3(128), 0, st, (const float*)sc.part, d, tk.seg_start,
-                                          tk.seg_len, tl.tile_seg, tl.tile_r0, splits, (__nv_bfloat16*)sc.o_lat));
+                                          tk.seg_len, tl.tile_seg, tk.seg_pos0, tl.tile_r0, splits, (__nv_bfloat16*)sc.o_lat));
             JSM_LAUNCH_CHECK();
         }
     }

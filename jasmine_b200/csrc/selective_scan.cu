@@ -9,8 +9,8 @@
 // zeros whatever the slot holds, so a slot needs no clearing when a new sequence takes it.
 //
 // Prompts: a CTA owns 32 channels of one segment and walks its tokens in tiles of 32 that cp.async brings into a two-stage
-// ring; four threads share a channel's states, so that the chain of dependent steps is one FMA per state and the partial
-// sums of four tokens are exchanged with three shuffles.  Decode: the same split of the states, one step for several
+// ring; eight threads share a channel's states, so that the chain of dependent steps is one FMA per state and the partial
+// sums of eight tokens are exchanged with seven shuffles.  Decode: four threads per channel, one step for several
 // sequences per CTA; the state rows are requested first and arrive while the step sizes (a small projection) are computed.
 #include "decoder_ops.cuh"
 #include "mma_utils.cuh"
@@ -23,10 +23,12 @@ namespace jsm {
 using tc::smem_u32;
 
 constexpr int SC_CH = 32;       // channels per CTA
-constexpr int SC_SUB = 4;       // threads per channel
+constexpr int SC_SUB = 8;       // threads per channel (prompts)
 constexpr int SC_THREADS = SC_CH * SC_SUB;
 constexpr int SC_TT = 32;       // tokens per tile
-constexpr int SC_YP = 40;       // pitch of the output tile (floats)
+constexpr int SC_YP = 36;       // pitch of the output tile (floats)
+constexpr int ST_SUB = 4;       // threads per channel (decode step)
+constexpr int ST_THREADS = SC_CH * ST_SUB;
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
@@ -36,14 +38,30 @@ template <>
 __device__ __forceinline__ float decay<float>(float x) { return expf(x); }
 template <>
 __device__ __forceinline__ float decay<__nv_bfloat16>(float x) { return __expf(x); }
+// the forms of a bf16 model: fp32 arithmetic with the fast exponential and logarithm; ln(1 + e) by its series where 1 + e
+// would round e away
+template <typename T>
+__device__ __forceinline__ float softplus_t(float x) {
+    if constexpr (sizeof(T) == 4) return softplus_f(x);
+    const float e = __expf(x);
+    const float series = e * (1.0f - e * (0.5f - e * (0.33333333f - e * (0.25f - e * 0.2f))));
+    return x > 20.0f ? x : x < -3.0f ? series : __logf(1.0f + e);
+}
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) {
+    if constexpr (sizeof(T) == 4) return silu_f(x);
+    return __fdividef(x, 1.0f + __expf(-x));
+}
 
 template <typename T>
-struct Vec8 {
-    __device__ static void load(const T* p, float (&v)[8]);
-    __device__ static void store(T* p, const float (&v)[8]);
-};
+struct Vec8;
 template <>
 struct Vec8<float> {
+    struct Raw { float4 a, b; };
+    __device__ static Raw fetch(const float* p) { return Raw{reinterpret_cast<const float4*>(p)[0], reinterpret_cast<const float4*>(p)[1]}; }
+    __device__ static void widen(const Raw& r, float (&v)[8]) {
+        v[0] = r.a.x; v[1] = r.a.y; v[2] = r.a.z; v[3] = r.a.w; v[4] = r.b.x; v[5] = r.b.y; v[6] = r.b.z; v[7] = r.b.w;
+    }
     __device__ static void load(const float* p, float (&v)[8]) {
         const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
         v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
@@ -55,8 +73,10 @@ struct Vec8<float> {
 };
 template <>
 struct Vec8<__nv_bfloat16> {
-    __device__ static void load(const __nv_bfloat16* p, float (&v)[8]) {
-        const uint4 w = *reinterpret_cast<const uint4*>(p);
+    using Raw = uint4;
+    __device__ static Raw fetch(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+    __device__ static void load(const __nv_bfloat16* p, float (&v)[8]) { widen(fetch(p), v); }
+    __device__ static void widen(const uint4& w, float (&v)[8]) {
         v[0] = bf16lo(w.x); v[1] = bf16hi(w.x); v[2] = bf16lo(w.y); v[3] = bf16hi(w.y);
         v[4] = bf16lo(w.z); v[5] = bf16hi(w.z); v[6] = bf16lo(w.w); v[7] = bf16hi(w.w);
     }
@@ -96,24 +116,32 @@ __global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz
     Vec8<float>::load(b + c, bias);
     const int j1 = min(len, j0 + CONV_TOK);
     if constexpr (TAPS > 0) {
+        // all the thread's inputs are requested before the first is used
+        typename Vec8<T>::Raw raw[CONV_TOK];
+#pragma unroll
+        for (int u = 0; u < CONV_TOK; ++u)
+            if (j0 + u < j1) raw[u] = Vec8<T>::fetch(xz + (long long)(start + j0 + u) * 2 * ip + c);
         float win[TAPS][8], wt[TAPS][8];
 #pragma unroll
         for (int k = 0; k < TAPS; ++k) Vec8<float>::load(w + (long long)k * ip + c, wt[k]);
 #pragma unroll
         for (int k = 0; k + 1 < TAPS; ++k) input(j0 - TAPS + 1 + k, win[k + 1]);
-        for (int j = j0; j < j1; ++j) {
+#pragma unroll
+        for (int u = 0; u < CONV_TOK; ++u) {
+            const int j = j0 + u;
+            if (j >= j1) break;
 #pragma unroll
             for (int k = 0; k + 1 < TAPS; ++k)
 #pragma unroll
                 for (int e = 0; e < 8; ++e) win[k][e] = win[k + 1][e];
-            Vec8<T>::load(xz + (long long)(start + j) * 2 * ip + c, win[TAPS - 1]);
+            Vec8<T>::widen(raw[u], win[TAPS - 1]);
             float o[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
                 float a = bias[e];
 #pragma unroll
                 for (int k = 0; k < TAPS; ++k) a = fmaf(wt[k][e], win[k][e], a);
-                o[e] = silu_f(a);
+                o[e] = silu_t<T>(a);
             }
             Vec8<T>::store(xc + (long long)(start + j) * ip + c, o);
         }
@@ -194,7 +222,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     float* bc = dts + 2 * SC_TT * SC_CH;                                    // 2 x [TT][B: nb | C: nb]
     float* ys = bc + 2 * SC_TT * 2 * nb;                                    // [TT][YP]
     chain_trigger();
-    const int tid = threadIdx.x, ch = tid >> 2, sub = tid & 3;
+    const int tid = threadIdx.x, ch = tid / SC_SUB, sub = tid % SC_SUB;
     const int c0 = blockIdx.x * SC_CH, c = c0 + ch;
     const bool live = c < a.ip;
     float A[NS], S[NS];
@@ -254,16 +282,16 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
         for (int i = tid; i < SC_TT * SC_CH; i += SC_THREADS) {
             const int cc = c0 + (i & (SC_CH - 1));
             // a step size of zero leaves the state as it is: the rows behind the segment
-            dt[i] = (i / SC_CH < n && cc < a.ip) ? softplus_f(dt[i] + a.dt_b[cc]) : 0.0f;
+            dt[i] = (i / SC_CH < n && cc < a.ip) ? softplus_t<T>(dt[i] + a.dt_b[cc]) : 0.0f;
         }
         __syncthreads();
         const float* bt = bc + stage * SC_TT * 2 * nb + sub * NS;
 #pragma unroll 1
-        for (int t4 = 0; t4 < n; t4 += 4) {
-            float y[4];
+        for (int t8 = 0; t8 < n; t8 += 8) {
+            float y[8];
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const int t = t4 + u;
+            for (int u = 0; u < 8; ++u) {
+                const int t = t8 + u;
                 const float d = dt[t * SC_CH + ch], dx = d * to_f32(x[t * SC_CH + ch]);
                 float B[NS], C[NS];
                 lds_vec<NS>(bt + t * 2 * nb, B);
@@ -276,14 +304,14 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
                 }
                 y[u] = acc;
             }
-            // four partial sums on each of four lanes -> lane `sub` holds the sum of token t4 + sub
-            const bool hi = sub & 2, odd = sub & 1;
-            float k0 = hi ? y[2] : y[0], k1 = hi ? y[3] : y[1];
-            k0 += __shfl_xor_sync(0xffffffffu, hi ? y[0] : y[2], 2);
-            k1 += __shfl_xor_sync(0xffffffffu, hi ? y[1] : y[3], 2);
-            float k = odd ? k1 : k0;
-            k += __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 1);
-            ys[(t4 + sub) * SC_YP + ch] = k;
+            // eight partial sums on each of eight lanes -> lane `sub` holds the sum of token t8 + sub
+            float k4[4], k2[2];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) k4[u] = ((sub & 4) ? y[4 + u] : y[u]) + __shfl_xor_sync(0xffffffffu, (sub & 4) ? y[u] : y[4 + u], 4);
+#pragma unroll
+            for (int u = 0; u < 2; ++u) k2[u] = ((sub & 2) ? k4[2 + u] : k4[u]) + __shfl_xor_sync(0xffffffffu, (sub & 2) ? k4[u] : k4[2 + u], 2);
+            const float k = ((sub & 1) ? k2[1] : k2[0]) + __shfl_xor_sync(0xffffffffu, (sub & 1) ? k2[0] : k2[1], 1);
+            ys[(t8 + sub) * SC_YP + ch] = k;
         }
         __syncthreads();
         const T* z = zs + stage * SC_TT * SC_CH;
@@ -295,7 +323,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
             Vec8<T>::load(z + r * SC_CH + v, zv);
             Vec8<float>::load(a.D + c0 + v, dv);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o[e] = fmaf(dv[e], xv[e], ys[r * SC_YP + v + e]) * silu_f(zv[e]);
+            for (int e = 0; e < 8; ++e) o[e] = fmaf(dv[e], xv[e], ys[r * SC_YP + v + e]) * silu_t<T>(zv[e]);
             Vec8<T>::store(static_cast<T*>(a.y) + (long long)(start + t0 + r) * a.ip + c0 + v, o);
         }
         __syncthreads();
@@ -311,10 +339,10 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 // ---- decode step --------------------------------------------------------------------------------------------------
 // One token of BB sequences and 32 channels per CTA.
 template <typename T, int NS, int BB>
-__global__ void __launch_bounds__(SC_THREADS) scan_step_kernel(ScanArgs a) {
+__global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float st_dyn[];  // [BB][proj columns]
     chain_trigger();
-    const int tid = threadIdx.x, ch = tid >> 2, sub = tid & 3;
+    const int tid = threadIdx.x, ch = tid / ST_SUB, sub = tid % ST_SUB;
     const int c0 = blockIdx.x * SC_CH, c = c0 + ch, cl = min(c, a.ip - 1);
     const bool live = c < a.ip;
     const int s0 = blockIdx.y * BB, nb = min(BB, a.n_segs - s0);
@@ -331,7 +359,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_step_kernel(ScanArgs a) {
 #pragma unroll
         for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? state[sub * NS + i] : 0.0f;
     }
-    for (int i = tid; i < nb * (pc / 4); i += SC_THREADS) {
+    for (int i = tid; i < nb * (pc / 4); i += ST_THREADS) {
         const int b = i / (pc / 4), v = i % (pc / 4);
         reinterpret_cast<float4*>(st_dyn)[i] = reinterpret_cast<const float4*>(a.proj + (long long)a.seg_start[s0 + b] * pc)[v];
     }
@@ -360,7 +388,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_step_kernel(ScanArgs a) {
         float d = dt[b];
         d += __shfl_xor_sync(0xffffffffu, d, 1);
         d += __shfl_xor_sync(0xffffffffu, d, 2);
-        d = softplus_f(d + bias);
+        d = softplus_t<T>(d + bias);
         const int t = a.seg_start[s0 + b];
         const float x = to_f32(static_cast<const T*>(a.xc)[(long long)t * a.ip + cl]), dx = d * x;
         const float* Bp = st_dyn + b * pc + a.rp + sub * NS;
@@ -379,10 +407,10 @@ __global__ void __launch_bounds__(SC_THREADS) scan_step_kernel(ScanArgs a) {
         y += __shfl_xor_sync(0xffffffffu, y, 2);
         if (sub == (b & 3) && live) {
             const float z = to_f32(xz[(long long)t * 2 * a.ip + a.ip + c]);
-            static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_f(z));
+            static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(z));
         }
     }
-    for (int i = tid; i < SC_CH * nb; i += SC_THREADS) {
+    for (int i = tid; i < SC_CH * nb; i += ST_THREADS) {
         const int b = i / SC_CH, cc = c0 + i % SC_CH;
         if (cc < a.ip)
             carry_conv_state(static_cast<T*>(a.conv) + (long long)a.seg_slot[s0 + b] * (a.taps - 1) * a.ip, xz, cc, a.ip, a.taps,
@@ -454,29 +482,35 @@ static jsm_status step_go(const ScanArgs& a, cudaStream_t st) {
         JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_step_kernel<T, NS, BB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
         attr_done = true;
     }
-    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NS, BB>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + BB - 1) / BB), dim3(SC_THREADS), smem, st, a));
+    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NS, BB>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + BB - 1) / BB), dim3(ST_THREADS), smem, st, a));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
-// the smallest instance whose four threads hold a channel's states
-#define JSM_SCAN_DISPATCH(FN, T)                                                                        \
-    (a.state <= 4 ? FN<T, 1>(a, st) : a.state <= 8 ? FN<T, 2>(a, st) : a.state <= 16 ? FN<T, 4>(a, st)  \
-     : a.state <= 24 ? FN<T, 6>(a, st) : a.state <= 32 ? FN<T, 8>(a, st) : a.state <= 64 ? FN<T, 16>(a, st) : FN<T, 32>(a, st))
+// the smallest instance whose threads hold a channel's states (per thread: state / 8 in prompts, state / 4 in a decode step)
+template <typename T>
+static jsm_status scan_dispatch(const ScanArgs& a, cudaStream_t st) {
+    return a.state <= 8 ? scan_go<T, 1>(a, st) : a.state <= 16 ? scan_go<T, 2>(a, st) : a.state <= 24 ? scan_go<T, 3>(a, st)
+         : a.state <= 32 ? scan_go<T, 4>(a, st) : a.state <= 64 ? scan_go<T, 8>(a, st) : scan_go<T, 16>(a, st);
+}
+template <typename T>
+static jsm_status step_dispatch(const ScanArgs& a, cudaStream_t st) {
+    return a.state <= 8 ? step_go<T, 2>(a, st) : a.state <= 16 ? step_go<T, 4>(a, st) : a.state <= 24 ? step_go<T, 6>(a, st)
+         : a.state <= 32 ? step_go<T, 8>(a, st) : a.state <= 64 ? step_go<T, 16>(a, st) : step_go<T, 32>(a, st);
+}
 
 jsm_status scan_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
                        const void* xc, const float* proj, const float* dt_raw, void* y, cudaStream_t st) {
     if (d.state > 128) JSM_FAIL(JSM_UNSUPPORTED, "selective scan: %d states per channel (at most 128)", d.state);
     const ScanArgs a = scan_args(d, w, s, tk, xz, xc, proj, dt_raw, y);
-    return f32 ? JSM_SCAN_DISPATCH(scan_go, float) : JSM_SCAN_DISPATCH(scan_go, __nv_bfloat16);
+    return f32 ? scan_dispatch<float>(a, st) : scan_dispatch<__nv_bfloat16>(a, st);
 }
 
 jsm_status scan_step_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
                             const void* xc, const float* proj, void* y, cudaStream_t st) {
     if (d.state > 128) JSM_FAIL(JSM_UNSUPPORTED, "selective scan: %d states per channel (at most 128)", d.state);
     const ScanArgs a = scan_args(d, w, s, tk, xz, xc, proj, nullptr, y);
-    return f32 ? JSM_SCAN_DISPATCH(step_go, float) : JSM_SCAN_DISPATCH(step_go, __nv_bfloat16);
+    return f32 ? step_dispatch<float>(a, st) : step_dispatch<__nv_bfloat16>(a, st);
 }
-#undef JSM_SCAN_DISPATCH
 
 jsm_status scan_dt_operand_launch(const ScanDims& d, const float* proj, void* out, int T, cudaStream_t st) {
     const long long n = (long long)T * (d.rp() / 8);

@@ -21,6 +21,7 @@ class Decoder:
                  max_step_tokens=2048, pool_pages=0):
         self.vocab, self.d_model, self.n_layers = vocab, d_model, len(layers)
         self.max_batch, self.max_context = max_batch, max_context
+        self.stream = None  # a CUDA stream's address, or None: a stream of the model
         cfg = DecoderConfig(len(layers), d_model, vocab, {"bfloat16": BF16, "float32": F32}[dtype], max_batch, max_context,
                             max(max_step_tokens, max_batch), pool_pages, norm_eps, logit_softcap)
         self.max_step_tokens = cfg.max_step_tokens
@@ -48,17 +49,17 @@ class Decoder:
         check(lib().jsm_decoder_seq_open(self._h, C.byref(row)))
         return row.value
 
-    def step(self, entries, want=(), h_next=None, h_logits=None):
+    def step(self, entries, want=(), h_next=None, h_logits=None, logits=True):
         """entries: [(row, tokens)]; want: flat places among all tokens of the step.  Returns (next tokens, logits) of the
-        wanted places; arrays of one's own may be passed in."""
+        wanted places; arrays of one's own may be passed in, logits=False leaves the logits on the device."""
         rows, counts = _i32([r for r, _ in entries]), _i32([len(t) for _, t in entries])
         ids = _i32(np.concatenate([np.asarray(t, np.int32).reshape(-1) for _, t in entries]))
         want = _i32(want)
         n = want.size
         h_next = np.empty(n, np.int32) if h_next is None else h_next
-        h_logits = np.empty((n, self.vocab), np.float32) if h_logits is None else h_logits
+        h_logits = np.empty((n, self.vocab), np.float32) if h_logits is None and logits else h_logits
         check(lib().jsm_decoder_step(self._h, len(entries), rows.ctypes.data, counts.ctypes.data, ids.ctypes.data, n,
-                                     want.ctypes.data, host_ptr(h_next), host_ptr(h_logits), None))
+                                     want.ctypes.data, host_ptr(h_next), host_ptr(h_logits), self.stream))
         return h_next, h_logits
 
     def admit(self, h_prompt, h_logits_last=None):
@@ -67,16 +68,16 @@ class Decoder:
             h_prompt = _i32(h_prompt)
         n = h_prompt.numel() if hasattr(h_prompt, "numel") else h_prompt.size
         row, tok = C.c_int(), C.c_int32()
-        check(lib().jsm_decoder_seq_admit(self._h, host_ptr(h_prompt), n, C.byref(row), C.addressof(tok), host_ptr(h_logits_last), None))
+        check(lib().jsm_decoder_seq_admit(self._h, host_ptr(h_prompt), n, C.byref(row), C.addressof(tok), host_ptr(h_logits_last), self.stream))
         return row.value, tok.value
 
     def step_active(self, h_ids, h_next, h_logits=None):
-        check(lib().jsm_decoder_step_active(self._h, host_ptr(h_ids), host_ptr(h_next), host_ptr(h_logits), None))
+        check(lib().jsm_decoder_step_active(self._h, host_ptr(h_ids), host_ptr(h_next), host_ptr(h_logits), self.stream))
 
     def retire(self, row: int) -> int:
         """Frees the row; returns the old index of the row that moved into its place, or -1."""
         moved = C.c_int()
-        check(lib().jsm_decoder_seq_retire(self._h, row, C.byref(moved), None))
+        check(lib().jsm_decoder_seq_retire(self._h, row, C.byref(moved), self.stream))
         return moved.value
 
     def pages_for(self, n_tokens: int) -> int:
