@@ -389,9 +389,9 @@ static jsm_status latent_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaS
     const int T = P.tk.T;
     const void* xin = m->f32 ? m->x : m->xa;
     DEC_TRY(linear(m, L.qd, xin, m->wp, m->wide, true, T, st));
-    DEC_TRY(latent_prep_launch(m->f32, m->wide, d, L.lw, m->c.norm_eps, L.cache, P.tk, m->q, st));
     const bool flash = L.expand.packed != nullptr && P.n_flash > 0;
     const TileList& tl = (flash ? P.tiles_short : P.tiles_all).at(d.H);
+    DEC_TRY(latent_prep_launch(m->f32, m->wide, d, L.lw, m->c.norm_eps, L.cache, P.tk, m->q, tl.n > 0 ? m->q_lat : nullptr, st));
     if (tl.n > 0) {
         LatentTiles t;
         t.tile_seg = P.meta + tl.seg_off; t.tile_r0 = P.meta + tl.r0_off; t.n_tiles = tl.n; t.t_first = 0; t.t_count = tl.tokens;
@@ -418,7 +418,7 @@ static jsm_status scan_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaStr
     const int T = P.tk.T;
     const void* xin = m->f32 ? m->x : m->xa;
     DEC_TRY(linear(m, L.in, xin, m->wp, m->xz, false, T, st));
-    DEC_TRY(scan_conv_launch(m->f32, d, L.sw, L.state, P.tk, m->xz, m->xc, st));
+    DEC_TRY(scan_conv_launch(m->f32, d, L.sw, L.state, P.tk, m->xz, m->xc, P.decode, st));
     DEC_TRY(linear(m, L.xp, m->xc, d.ip(), m->proj, true, T, st));
     if (P.decode) {
         DEC_TRY(scan_step_launch(m->f32, d, L.sw, L.state, P.tk, m->xz, m->xc, m->proj, m->scan_y, st));

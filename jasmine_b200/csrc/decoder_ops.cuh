@@ -49,10 +49,11 @@ struct LatentCache {
     const float2* rope;      // (cos, sin) of [position][rot / 2]
 };
 // From the fused down/query projection qd (f32 [T][q_cols + down_cols]): appends [norm(c) | rotated key part] to the
-// cache and writes the queries, rotated, to q (act [T][q_cols]).
+// cache and writes the queries, rotated, to q (act [T][q_cols]); the rotated parts also go into the latent queries q_lat
+// (act [T][H][cr], behind their rank columns; may be null).
 jsm_status latent_prep_launch(bool f32, const float* qd, const LatentDims& d, const LatentWeights& w, float eps, const LatentCache& cache,
-                              const StepTokens& tk, void* q, cudaStream_t st);
-// Attention in the latent space for the tokens listed in tiles: queries are taken into the latent space (q_lat), scored
+                              const StepTokens& tk, void* q, void* q_lat, cudaStream_t st);
+// Attention in the latent space for the tokens listed in tiles: queries are taken into the latent space (the rank columns of q_lat), scored
 // against the cache, and the weighted latents (o_lat) expanded to values: out act [T][out_cols].
 struct LatentScratch {
     void* q_lat;             // act [T][H][cr]
@@ -96,9 +97,10 @@ struct ScanState {
     void* conv;    // act [slots][taps - 1][ip]: the last inputs of the convolution
     float* S;      // [slots][ip][np]
 };
-// xc = silu(conv(x) + b) over the x half of xz (act [T][2 ip]); reads the convolution state, does not change it
+// xc = silu(conv(x) + b) over the x half of xz (act [T][2 ip]); carry (one token per segment): also moves the convolution
+// state on, which otherwise the scan does
 jsm_status scan_conv_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
-                            void* xc, cudaStream_t st);
+                            void* xc, bool carry, cudaStream_t st);
 // the scan over every segment: proj f32 [T][proj_cols], dt_raw f32 [T][ip] (before bias and softplus); y act [T][ip] is
 // gated by silu(z); carries the recurrent and the convolution state
 jsm_status scan_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,

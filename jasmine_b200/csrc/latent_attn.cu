@@ -47,7 +47,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restrict__ qd, LatentDims d, const float* __restrict__ gain, float eps,
                                                           T* __restrict__ pool, const int32_t* __restrict__ block_table, int max_pages,
                                                           const float2* __restrict__ rope, const int32_t* __restrict__ tok_row,
-                                                          const int32_t* __restrict__ tok_pos, T* __restrict__ q, int vec) {
+                                                          const int32_t* __restrict__ tok_pos, T* __restrict__ q, T* __restrict__ q_lat, int vec) {
     __shared__ float red[8];
     chain_trigger();
     chain_wait();
@@ -95,6 +95,14 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
             }
         }
         store8(q + (long long)t * q_cols + i0, v);
+        if (q_lat && j0 + 8 > d.dim && j0 < d.dim + d.rot) {
+            T* dst = q_lat + ((long long)t * d.H + i0 / qh) * cr + d.rank - d.dim;  // (component j of the query -> rank + j - dim)
+            if (vec && d.rank % 8 == 0) store8(dst + j0, v);
+            else
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+                    if (j0 + e >= d.dim && j0 + e < d.dim + d.rot) dst[j0 + e] = from_f32<T>(v[e]);
+        }
         return;
     }
     // latent: RMS norm, then the cache entry
@@ -126,7 +134,6 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const float* __restric
 
 // ---- per-head projections -----------------------------------------------------------------------------------------
 // out[t][h][n] = sum_k in[t][h][k] * W[h][n][k], n < N, k < K; W rows of pitch kw (zero padded), W[h] of nw rows.
-// copy_n > 0: out[t][h][N + j] = in[t][h][copy_from + j] for j < copy_n (the rotated query part next to the latent query).
 struct ProjectArgs {
     const void* in;
     long long in_ts, in_hs;
@@ -134,7 +141,6 @@ struct ProjectArgs {
     int N, K, nw, kw;
     void* out;
     long long out_ts, out_hs;
-    int copy_from, copy_n, out_pad;  // columns N + copy_n .. out_pad - 1 of the output are set to zero
     int t0, T;
 };
 
@@ -144,15 +150,11 @@ __global__ void __launch_bounds__(256) latent_project_simt_kernel(ProjectArgs a)
     chain_wait();
     const int n = blockIdx.x * 32 + (threadIdx.x & 31), h = blockIdx.y;
     const int t = a.t0 + blockIdx.z * 8 + (threadIdx.x >> 5);
-    if (t >= a.t0 + a.T || n >= a.out_pad) return;
+    if (t >= a.t0 + a.T || n >= a.N) return;
     const T* in = static_cast<const T*>(a.in) + t * a.in_ts + h * a.in_hs;
     float acc = 0.0f;
-    if (n < a.N) {
-        const T* w = static_cast<const T*>(a.W) + ((long long)h * a.nw + n) * a.kw;
-        for (int k = 0; k < a.K; ++k) acc = fmaf(to_f32(in[k]), to_f32(w[k]), acc);
-    } else if (n < a.N + a.copy_n) {
-        acc = to_f32(in[a.copy_from + (n - a.N)]);
-    }
+    const T* w = static_cast<const T*>(a.W) + ((long long)h * a.nw + n) * a.kw;
+    for (int k = 0; k < a.K; ++k) acc = fmaf(to_f32(in[k]), to_f32(w[k]), acc);
     static_cast<T*>(a.out)[t * a.out_ts + h * a.out_hs + n] = from_f32<T>(acc);
 }
 
@@ -233,21 +235,12 @@ __global__ void __launch_bounds__(128) latent_project_mma_kernel(ProjectArgs a) 
                 if (t < t_end && n < a.N) out[t * a.out_ts + n] = __float2bfloat16_rn(acc[j][e]);
             }
     }
-    // the copied columns and the zero padding behind them, by the first block of rows
-    if (blockIdx.x == 0) {
-        const int extra = a.out_pad - a.N;
-        for (int i = threadIdx.x; i < extra * (t_end - t_begin); i += 128) {
-            const int t = t_begin + i / extra, c = i % extra;
-            static_cast<__nv_bfloat16*>(a.out)[t * a.out_ts + h * a.out_hs + a.N + c] =
-                c < a.copy_n ? static_cast<const __nv_bfloat16*>(a.in)[t * a.in_ts + h * a.in_hs + a.copy_from + c] : __float2bfloat16_rn(0.0f);
-        }
-    }
 }
 
 static jsm_status project(bool f32, const ProjectArgs& a, int H, cudaStream_t st) {
     if (a.T <= 0) return JSM_OK;
     if (f32)
-        JSM_CUDA_CHECK(launch_chained(latent_project_simt_kernel<float>, dim3((a.out_pad + 31) / 32, H, (a.T + 7) / 8), dim3(256), 0, st, a));
+        JSM_CUDA_CHECK(launch_chained(latent_project_simt_kernel<float>, dim3((a.N + 31) / 32, H, (a.T + 7) / 8), dim3(256), 0, st, a));
     else if (a.kw >= 256)
         JSM_CUDA_CHECK(launch_chained(latent_project_mma_kernel<true>, dim3((a.N + 15) / 16, H, (a.T + 31) / 32), dim3(128), 0, st, a));
     else
@@ -317,44 +310,55 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
 }
 
 // bf16 on the tensor cores.  A CTA owns 32 (token, head) rows of one segment and a run of cache pages; a page of 64 entries
-// is one stage of a two-stage cp.async ring, read once for the scores (all rank + rot components) and once for the weighted
-// sum (the first rank components).  Eight warps: scores as 2 x 4 tiles of 16 rows x 16 keys; the sum as column blocks of
-// NT x 8 latent components per warp, all 32 rows.  Scores, maxima and sums are fp32; the weights enter the sum as bf16.
+// is one stage of a two-stage ring filled by bulk copies (a row each, one warp issues them), read once for the scores (all
+// rank + rot components) and once for the weighted sum (the first rank components).  Eight warps: scores as 2 tiles of 16
+// rows x 2 halves of the components x 2 groups of 32 keys - a warp keeps its part of the queries in registers - then the sum
+// as column blocks of NT x 8 latent components per warp, all 32 rows.  Scores, maxima and sums are fp32; the weights enter the
+// sum as bf16.  Waits for copies are bounded (tc_utils.cuh).
 constexpr int LA_ROWS = LATENT_TILE_ROWS;
 constexpr int LA_SP = 68;  // pitch of the score tile (floats)
 constexpr int LA_PP = 72;  // pitch of the weight tile (bf16)
 constexpr int LA_ML = 4;   // behind a partial row: its maximum, its sum, two unused
 constexpr int LA_MAX_SPLITS = 256;
+constexpr int LA_ERR_FULL = 51;
 
 static int la_pitch(const LatentDims& d) { return pad_to(d.rank + d.rot, 16) + 8; }  // odd multiple of 16 bytes: no bank conflicts
 static size_t la_smem(const LatentDims& d) {
-    return (size_t)(LA_ROWS + 2 * PAGE) * la_pitch(d) * 2 + LA_ROWS * LA_PP * 2 + LA_ROWS * LA_SP * 4 + 3 * LA_ROWS * 4;
+    return (size_t)2 * PAGE * la_pitch(d) * 2 + LA_ROWS * LA_PP * 2 + 2 * LA_ROWS * LA_SP * 4 + 3 * LA_ROWS * 4;
 }
 
-template <int NT>
-__global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q_lat, LatentDims d,
+template <int NT>  // KS: 16-wide steps of half the components, at most
+__global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const __nv_bfloat16* __restrict__ q_lat, LatentDims d,
                                                               const __nv_bfloat16* __restrict__ pool, const int32_t* __restrict__ block_table,
                                                               int max_pages, const int32_t* __restrict__ seg_start,
                                                               const int32_t* __restrict__ seg_len, const int32_t* __restrict__ seg_pos0,
                                                               const int32_t* __restrict__ seg_row, const int32_t* __restrict__ tile_seg,
                                                               const int32_t* __restrict__ tile_r0, __nv_bfloat16* __restrict__ o_lat,
-                                                              float* __restrict__ part, int splits, int pitch) {
+                                                              float* __restrict__ part, int splits, int pitch, int* err) {
+    constexpr int KS = 2 * NT + 4;
     extern __shared__ __align__(16) uint8_t la_dyn[];
-    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(la_dyn);       // [32][pitch]
-    __nv_bfloat16* kv = qs + LA_ROWS * pitch;                           // 2 x [64][pitch]
+    __nv_bfloat16* kv = reinterpret_cast<__nv_bfloat16*>(la_dyn);       // 2 x [64][pitch]
     __nv_bfloat16* ps = kv + 2 * PAGE * pitch;                          // [32][72]
-    float* ss = reinterpret_cast<float*>(ps + LA_ROWS * LA_PP);         // [32][68]
-    float* row_m = ss + LA_ROWS * LA_SP;
+    float* ss = reinterpret_cast<float*>(ps + LA_ROWS * LA_PP);         // 2 x [32][68]: halves of the components
+    float* row_m = ss + 2 * LA_ROWS * LA_SP;
     float* row_l = row_m + LA_ROWS;
     float* row_a = row_l + LA_ROWS;
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int abort_flag;
     chain_trigger();
     const int cr = pad8(d.rank + d.rot), rp = pad8(d.rank), cr16 = pitch - 8;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        abort_flag = 0;
+        tc::mbar_init(&full[0], 1);
+        tc::mbar_init(&full[1], 1);
+        tc::mbar_fence_init();
+    }
     // columns between the entry's pitch and the next multiple of 16 take part in the products: zero once
     if (cr < cr16)
-        for (int i = threadIdx.x; i < (LA_ROWS + 2 * PAGE) * (cr16 - cr); i += 256)
-            qs[(i / (cr16 - cr)) * pitch + cr + i % (cr16 - cr)] = __float2bfloat16_rn(0.0f);
+        for (int i = threadIdx.x; i < 2 * PAGE * (cr16 - cr); i += 256) kv[(i / (cr16 - cr)) * pitch + cr + i % (cr16 - cr)] = __float2bfloat16_rn(0.0f);
     if (threadIdx.x < LA_ROWS) { row_m[threadIdx.x] = -INFINITY; row_l[threadIdx.x] = 0.0f; }
+    __syncthreads();
     chain_wait();
     const int tile = blockIdx.x, sp = blockIdx.y;
     const int seg = tile_seg[tile], r0 = tile_r0[tile];
@@ -368,60 +372,94 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat1
     const int pb = pg_lo + n_pg * sp / live, pe = pg_lo + n_pg * (sp + 1) / live;
     const int32_t* bt = block_table + (long long)seg_row[seg] * max_pages;
     const int vec = cr / 8;  // 16-byte vectors per entry
-    auto load_page = [&](int pg, int stage) {
+    auto load_page = [&](int pg, int stage) {  // warp 0
+        const int lo = max(key_lo - pg * PAGE, 0), hi = min(key_hi - pg * PAGE, PAGE);
+        if (lane == 0) tc::mbar_expect_tx(&full[stage], (uint32_t)(hi - lo) * cr * 2);
+        __syncwarp();
         const __nv_bfloat16* src = pool + (long long)bt[pg] * PAGE * cr;
-        const uint32_t dst = smem_u32(kv + stage * PAGE * pitch);
-        for (int i = threadIdx.x; i < PAGE * vec; i += 256) {
-            const int r = i / vec, c = i - r * vec, kp = pg * PAGE + r;
-            // entries outside the tile's key range are not read: their rows are zero (a weight of 0 must meet a number)
-            cp_async16(dst + (uint32_t)(r * pitch + c * 8) * 2, src + (long long)r * cr + c * 8, kp >= key_lo && kp < key_hi);
-        }
+        __nv_bfloat16* dst = kv + stage * PAGE * pitch;
+        for (int r = lo + lane; r < hi; r += 32)
+            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst + r * pitch)),
+                         "l"(reinterpret_cast<uint64_t>(src + (long long)r * cr)), "r"(cr * 2), "r"(smem_u32(&full[stage]))
+                         : "memory");
     };
+    if (warp == 0) load_page(pb, 0);
+    // the queries pass through the second stage into registers
     for (int i = threadIdx.x; i < LA_ROWS * vec; i += 256) {
         const int r = i / vec, c = i - r * vec, g = r0 + r;
         const int t = start + g / d.H, h = g % d.H;
-        cp_async16(smem_u32(qs + r * pitch + c * 8), q_lat + ((long long)(r < n_rows ? t : start) * d.H + (r < n_rows ? h : 0)) * cr + c * 8, r < n_rows);
+        cp_async16(smem_u32(kv + (PAGE + r) * pitch + c * 8), q_lat + ((long long)(r < n_rows ? t : start) * d.H + (r < n_rows ? h : 0)) * cr + c * 8, r < n_rows);
     }
-    if (pb < pe) load_page(pb, 0);
     cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    const int mt = warp & 1, kh = (warp >> 1) & 1, kg = warp >> 2;  // this warp's rows, half of the components, keys
+    const int lm = lane >> 3, lr = lane & 7;
+    const int n_ks = cr16 / 16, ks0 = kh ? (n_ks + 1) / 2 : 0, n_mine = kh ? n_ks / 2 : (n_ks + 1) / 2;
+    uint32_t qf[KS][4];
+    {
+        const uint32_t q_addr = smem_u32(kv + (PAGE + mt * 16 + (lm & 1) * 8 + lr) * pitch + (lm >> 1) * 8);
+#pragma unroll
+        for (int k = 0; k < KS; ++k)
+            if (k < n_mine) ldsm_x4(q_addr + (ks0 + k) * 32, qf[k]);
+    }
+    tc::fence_proxy_async_smem();  // the copy engine writes this stage next
+    __syncthreads();
     float o[2][NT][4];
 #pragma unroll
     for (int a = 0; a < 2; ++a)
 #pragma unroll
         for (int j = 0; j < NT; ++j) o[a][j][0] = o[a][j][1] = o[a][j][2] = o[a][j][3] = 0.0f;
-    const int mt = warp & 1, kg = warp >> 1;  // this warp's score tile: 16 rows, 16 keys
-    const int lm = lane >> 3, lr = lane & 7;
-    const uint32_t q_addr = smem_u32(qs + (mt * 16 + (lm & 1) * 8 + lr) * pitch + (lm >> 1) * 8);
+    bool ok = true;
     for (int pg = pb; pg < pe; ++pg) {
-        const int stage = (pg - pb) & 1;
-        if (pg + 1 < pe) load_page(pg + 1, stage ^ 1);
-        cp_async_commit();
-        cp_async_wait<1>();
-        __syncthreads();
-        const __nv_bfloat16* kvs = kv + stage * PAGE * pitch;
-        {   // scores
-            float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint32_t k_addr = smem_u32(kvs + (kg * 16 + (lm >> 1) * 8 + lr) * pitch + (lm & 1) * 8);
-#pragma unroll 4
-            for (int k = 0; k < cr16; k += 16) {
-                uint32_t a[4], b[4];
-                ldsm_x4(q_addr + k * 2, a);
-                ldsm_x4(k_addr + k * 2, b);
-                mma_16816(s0, a, b[0], b[1]);
-                mma_16816(s1, a, b[2], b[3]);
+        const int i = pg - pb, stage = i & 1;
+        if (warp == 0 && pg + 1 < pe) load_page(pg + 1, stage ^ 1);
+        __nv_bfloat16* kvs = kv + stage * PAGE * pitch;
+        {   // entries outside the tile's key range are not fetched: their rows are zero (a weight of 0 must meet a number)
+            const int lo = max(key_lo - pg * PAGE, 0), hi = min(key_hi - pg * PAGE, PAGE);
+            if (lo > 0 || hi < PAGE) {
+                const int n_out = lo + PAGE - hi;
+                for (int q = threadIdx.x; q < n_out * vec; q += 256) {
+                    const int r = q / vec, c = q - r * vec;
+                    *reinterpret_cast<uint4*>(kvs + (r < lo ? r : hi + r - lo) * pitch + c * 8) = make_uint4(0, 0, 0, 0);
+                }
+                tc::fence_proxy_async_smem();
             }
-            float* dst = ss + (mt * 16 + (lane >> 2)) * LA_SP + kg * 16 + (lane & 3) * 2;
-            dst[0] = s0[0]; dst[1] = s0[1]; dst[8 * LA_SP] = s0[2]; dst[8 * LA_SP + 1] = s0[3];
-            dst[8] = s1[0]; dst[9] = s1[1]; dst[8 * LA_SP + 8] = s1[2]; dst[8 * LA_SP + 9] = s1[3];
+        }
+        ok = tc::mbar_wait(&full[stage], (i >> 1) & 1, &abort_flag, err, LA_ERR_FULL);
+        if (!__syncthreads_and(ok)) { ok = false; break; }
+        {   // scores
+            float s[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
+            const uint32_t k_addr = smem_u32(kvs + (kg * 32 + (lm >> 1) * 8 + lr) * pitch + (lm & 1) * 8) + ks0 * 32;
+#pragma unroll
+            for (int k = 0; k < KS; ++k)
+                if (k < n_mine) {
+                    uint32_t b0[4], b1[4];
+                    ldsm_x4(k_addr + k * 32, b0);
+                    ldsm_x4(k_addr + 16 * pitch * 2 + k * 32, b1);
+                    mma_16816(s[0], qf[k], b0[0], b0[1]);
+                    mma_16816(s[1], qf[k], b0[2], b0[3]);
+                    mma_16816(s[2], qf[k], b1[0], b1[1]);
+                    mma_16816(s[3], qf[k], b1[2], b1[3]);
+                }
+            float* dst = ss + (kh * LA_ROWS + mt * 16 + (lane >> 2)) * LA_SP + kg * 32 + (lane & 3) * 2;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                *reinterpret_cast<float2*>(dst + j * 8) = make_float2(s[j][0], s[j][1]);
+                *reinterpret_cast<float2*>(dst + 8 * LA_SP + j * 8) = make_float2(s[j][2], s[j][3]);
+            }
         }
         __syncthreads();
 #pragma unroll
-        for (int i = 0; i < LA_ROWS / 8; ++i) {  // softmax: a warp per row, two keys per lane
-            const int r = warp * (LA_ROWS / 8) + i;
+        for (int i2 = 0; i2 < LA_ROWS / 8; ++i2) {  // softmax: a warp per row, two keys per lane
+            const int r = warp * (LA_ROWS / 8) + i2;
             const int p = pos0 + (r0 + r) / d.H, k0 = pg * PAGE + lane, k1 = k0 + 32;
             const bool on = r < n_rows;
-            float a = (on && k0 <= p && p - k0 < d.window) ? ss[r * LA_SP + lane] * d.scale : -INFINITY;
-            float b = (on && k1 <= p && p - k1 < d.window) ? ss[r * LA_SP + lane + 32] * d.scale : -INFINITY;
+            const float* sr = ss + r * LA_SP + lane;
+            float a = (on && k0 <= p && p - k0 < d.window) ? (sr[0] + sr[LA_ROWS * LA_SP]) * d.scale : -INFINITY;
+            float b = (on && k1 <= p && p - k1 < d.window) ? (sr[32] + sr[LA_ROWS * LA_SP + 32]) * d.scale : -INFINITY;
             const float m_old = row_m[r], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
             const float ref = m_new == -INFINITY ? 0.0f : m_new;
             a = __expf(a - ref);
@@ -467,8 +505,14 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(const __nv_bfloat1
         }
         __syncthreads();  // the stage and the score / weight tiles are free
     }
-    cp_async_wait<0>();
-    __syncthreads();
+    if (!ok) {  // a copy did not arrive: let the ones in flight land (bounded) and leave the result undefined; the host learns of it
+        if (threadIdx.x == 0) {
+            const long long t0 = clock64();
+            while (clock64() - t0 < tc::WAIT_LIMIT_CYCLES / 4) {}
+        }
+        __syncthreads();
+        return;
+    }
     // rows whose keys all lie in other splits have l = 0, m = -inf: they weigh nothing in the merge
 #pragma unroll
     for (int a = 0; a < 2; ++a)
@@ -555,21 +599,25 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const __nv_bfloat16*
 
 // ---- launches -----------------------------------------------------------------------------------------------------
 jsm_status latent_prep_launch(bool f32, const float* qd, const LatentDims& d, const LatentWeights& w, float eps, const LatentCache& cache,
-                              const StepTokens& tk, void* q, cudaStream_t st) {
+                              const StepTokens& tk, void* q, void* q_lat, cudaStream_t st) {
     const dim3 grid(tk.T, (d.q_cols() / 8 + 255) / 256 + 1);
     const int vec = d.dim % 8 == 0 && d.rot % 16 == 0 ? 1 : 0;
     if (f32)
         JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<float>, grid, dim3(256), 0, st, qd, d, w.down_norm, eps, (float*)cache.pool,
-                                      cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, (float*)q, vec));
+                                      cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, (float*)q, (float*)q_lat, vec));
     else
         JSM_CUDA_CHECK(launch_chained(latent_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, qd, d, w.down_norm, eps,
                                       (__nv_bfloat16*)cache.pool, cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos,
-                                      (__nv_bfloat16*)q, vec));
+                                      (__nv_bfloat16*)q, (__nv_bfloat16*)q_lat, vec));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
 
-bool latent_mma_usable(const LatentDims& d) { return d.rank <= 512 && la_smem(d) <= 226 * 1024; }
+static int la_nt(const LatentDims& d) { return d.rank <= 128 ? 2 : d.rank <= 256 ? 4 : d.rank <= 384 ? 6 : 8; }
+bool latent_mma_usable(const LatentDims& d) {
+    // a warp's half of the queries: at most 2 NT + 4 steps of 16 components
+    return d.rank <= 512 && (pad_to(d.rank + d.rot, 16) / 16 + 1) / 2 <= 2 * la_nt(d) + 4 && la_smem(d) <= 226 * 1024;
+}
 
 int latent_splits(int n_tiles, int max_keys) {
     if (n_tiles <= 0) return 1;
@@ -588,7 +636,7 @@ static jsm_status launch_mma(const LatentDims& d, const LatentCache& cache, cons
     }
     JSM_CUDA_CHECK(launch_chained(latent_attn_mma_kernel<NT>, dim3(tl.n_tiles, splits), dim3(256), la_smem(d), st, (const __nv_bfloat16*)sc.q_lat, d,
                                   (const __nv_bfloat16*)cache.pool, cache.block_table, cache.max_pages, tk.seg_start, tk.seg_len, tk.seg_pos0,
-                                  tk.seg_row, tl.tile_seg, tl.tile_r0, (__nv_bfloat16*)sc.o_lat, sc.part, splits, la_pitch(d)));
+                                  tk.seg_row, tl.tile_seg, tl.tile_r0, (__nv_bfloat16*)sc.o_lat, sc.part, splits, la_pitch(d), tc_error_word()));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -601,7 +649,6 @@ jsm_status latent_attn_launch(bool f32, const LatentDims& d, const LatentWeights
     a.in = q; a.in_ts = d.q_cols(); a.in_hs = d.qh();
     a.W = w.uk; a.N = d.rank; a.K = d.dim; a.nw = pad_to(d.rank, 16); a.kw = pad_to(d.dim, 32);
     a.out = sc.q_lat; a.out_ts = (long long)d.H * cr; a.out_hs = cr;
-    a.copy_from = d.dim; a.copy_n = d.rot; a.out_pad = cr;
     a.t0 = tl.t_first; a.T = tl.t_count;
     jsm_status s = project(f32, a, d.H, st);
     if (s != JSM_OK) return s;
@@ -621,10 +668,12 @@ jsm_status latent_attn_launch(bool f32, const LatentDims& d, const LatentWeights
         const int splits = latent_splits(tl.n_tiles, tl.max_keys);
         if (splits > 1 && (size_t)tl.n_tiles * splits * LA_ROWS * (rp + LA_ML) > sc.part_floats)
             JSM_FAIL(JSM_INVALID_ARG, "latent attention: workspace of %zu floats for %d tiles in %d splits", sc.part_floats, tl.n_tiles, splits);
-        s = d.rank <= 128   ? launch_mma<2>(d, cache, tk, tl, sc, splits, st)
-            : d.rank <= 256 ? launch_mma<4>(d, cache, tk, tl, sc, splits, st)
-            : d.rank <= 384 ? launch_mma<6>(d, cache, tk, tl, sc, splits, st)
-                            : launch_mma<8>(d, cache, tk, tl, sc, splits, st);
+        switch (la_nt(d)) {
+            case 2: s = launch_mma<2>(d, cache, tk, tl, sc, splits, st); break;
+            case 4: s = launch_mma<4>(d, cache, tk, tl, sc, splits, st); break;
+            case 6: s = launch_mma<6>(d, cache, tk, tl, sc, splits, st); break;
+            default: s = launch_mma<8>(d, cache, tk, tl, sc, splits, st); break;
+        }
         if (s != JSM_OK) return s;
         if (splits > 1) {
             JSM_CUDA_CHECK(launch_chained(latent_combine_kernel, dim3(tl.n_tiles, LA_ROWS), dim3(128), 0, st, (const float*)sc.part, d, tk.seg_start,
@@ -636,7 +685,6 @@ jsm_status latent_attn_launch(bool f32, const LatentDims& d, const LatentWeights
     a.in = sc.o_lat; a.in_ts = (long long)d.H * rp; a.in_hs = rp;
     a.W = w.uv; a.N = d.vdim; a.K = d.rank; a.nw = pad_to(d.vdim, 16); a.kw = pad_to(d.rank, 32);
     a.out = out; a.out_ts = d.out_cols(); a.out_hs = d.vdim;
-    a.copy_from = 0; a.copy_n = 0; a.out_pad = d.vdim;
     return project(f32, a, d.H, st);
 }
 

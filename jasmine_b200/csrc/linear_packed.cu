@@ -1005,8 +1005,10 @@ int linear_packed_grid(int N, int K, int paired, int T) {
         bool use;
         if (T >= 32) {
             // a power of two up to 8 (the cluster that folds through shared memory), from half of the SMs on
+            // (an even split would put more than 8 CTAs on a tile of a narrow matrix: a cluster per tile then, whatever it leaves idle)
+            use = S > 8;
             S = S >= 8 ? 8 : S >= 4 ? 4 : S >= 2 ? 2 : 1;
-            use = nt * S * 2 >= G;
+            use = use || nt * S * 2 >= G;
         } else {
             // at most 8 contributors per tile (the fold reads every slot); from four fifths of the SMs on, or whenever the
             // even split of the stream would put more than 8 CTAs on a tile

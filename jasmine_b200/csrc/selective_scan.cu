@@ -37,20 +37,20 @@ __device__ __forceinline__ float decay(float x);  // e^x for x <= 0
 template <>
 __device__ __forceinline__ float decay<float>(float x) { return expf(x); }
 template <>
-__device__ __forceinline__ float decay<__nv_bfloat16>(float x) { return __expf(x); }
+__device__ __forceinline__ float decay<__nv_bfloat16>(float x) { return fast_ex2(LOG2E * x); }
 // the forms of a bf16 model: fp32 arithmetic with the fast exponential and logarithm; ln(1 + e) by its series where 1 + e
 // would round e away
 template <typename T>
 __device__ __forceinline__ float softplus_t(float x) {
     if constexpr (sizeof(T) == 4) return softplus_f(x);
-    const float e = __expf(x);
+    const float e = fast_ex2(LOG2E * x);
     const float series = e * (1.0f - e * (0.5f - e * (0.33333333f - e * (0.25f - e * 0.2f))));
     return x > 20.0f ? x : x < -3.0f ? series : __logf(1.0f + e);
 }
 template <typename T>
 __device__ __forceinline__ float silu_t(float x) {
     if constexpr (sizeof(T) == 4) return silu_f(x);
-    return __fdividef(x, 1.0f + __expf(-x));
+    return x * fast_rcp(1.0f + fast_ex2(-LOG2E * x));
 }
 
 template <typename T>
@@ -88,14 +88,15 @@ struct Vec8<__nv_bfloat16> {
 };
 
 // ---- convolution --------------------------------------------------------------------------------------------------
-// A thread owns 8 channels of CONV_TOK consecutive tokens; TAPS 0: taps is only known at run time
+// A thread owns 8 channels of CONV_TOK consecutive tokens; TAPS 0: taps is only known at run time.  carry: every segment is
+// one token, and the state moves on by it here (otherwise the scan does that, once every CTA has read the old state)
 constexpr int CONV_TOK = 8;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, const T* __restrict__ state,
+__global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, T* state,
                                                         const float* __restrict__ w, const float* __restrict__ b,
                                                         const int32_t* __restrict__ seg_start, const int32_t* __restrict__ seg_len,
                                                         const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ seg_slot, int ip,
-                                                        int taps_rt) {
+                                                        int taps_rt, int carry) {
     chain_trigger();
     chain_wait();
     const int taps = TAPS ? TAPS : taps_rt;
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz
     const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
     const int c = (int)(i % vec) * 8, j0 = (int)(i / vec) * CONV_TOK;
     if (j0 >= len) return;
-    const T* st = state + (long long)seg_slot[seg] * (taps - 1) * ip + c;
+    T* st = state + (long long)seg_slot[seg] * (taps - 1) * ip + c;
     // input of the segment's token j (negative: before the segment)
     auto input = [&](int j, float (&v)[8]) {
         if (j >= 0) Vec8<T>::load(xz + (long long)(start + j) * 2 * ip + c, v);
@@ -145,6 +146,9 @@ __global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz
             }
             Vec8<T>::store(xc + (long long)(start + j) * ip + c, o);
         }
+        if (carry)  // one token per segment: this thread has read all there is to read of its channels' state
+#pragma unroll
+            for (int k = 0; k + 1 < TAPS; ++k) Vec8<T>::store(st + (long long)k * ip, win[k + 1]);
     } else {
         for (int j = j0; j < j1; ++j) {
             float o[8];
@@ -157,9 +161,15 @@ __global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz
                 for (int e = 0; e < 8; ++e) o[e] = fmaf(wk[e], v[e], o[e]);
             }
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o[e] = silu_f(o[e]);
+            for (int e = 0; e < 8; ++e) o[e] = silu_t<T>(o[e]);
             Vec8<T>::store(xc + (long long)(start + j) * ip + c, o);
         }
+        if (carry)
+            for (int k = 0; k + 1 < taps; ++k) {
+                float v[8];
+                input(k + 2 - taps, v);  // ascending: an entry is read before a later one takes its place
+                Vec8<T>::store(st + (long long)k * ip, v);
+            }
     }
 }
 
@@ -200,7 +210,8 @@ __device__ __forceinline__ void lds_vec(const float* p, float (&v)[NS]) {
 __host__ __device__ inline int scan_nb(int np, int ns) { return np > SC_SUB * ns ? np : SC_SUB * ns; }  // B / C columns per tile row
 template <typename T>
 static size_t scan_smem(int np, int ns) {
-    return 2 * (size_t)SC_TT * SC_CH * (2 * sizeof(T) + 4) + 2 * (size_t)SC_TT * 2 * scan_nb(np, ns) * 4 + (size_t)SC_TT * SC_YP * 4;
+    return 2 * (size_t)SC_TT * SC_CH * (2 * sizeof(T) + 4) + 2 * (size_t)SC_TT * 2 * scan_nb(np, ns) * 4 + (size_t)SC_TT * SC_YP * 4 +
+           (size_t)SC_TT * SC_CH * 16;
 }
 
 struct ScanArgs {
@@ -221,6 +232,8 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     float* dts = reinterpret_cast<float*>(zs + 2 * SC_TT * SC_CH);          // 2 x [TT][CH]
     float* bc = dts + 2 * SC_TT * SC_CH;                                    // 2 x [TT][B: nb | C: nb]
     float* ys = bc + 2 * SC_TT * 2 * nb;                                    // [TT][YP]
+    float4* dd = reinterpret_cast<float4*>(ys + SC_TT * SC_YP);             // [TT][CH]: dt, dt, dt x, dt x
+    constexpr bool PAIRS = sizeof(T) == 2 && NS % 2 == 0;                   // bf16 models: states in pairs, base-2 exponentials
     chain_trigger();
     const int tid = threadIdx.x, ch = tid / SC_SUB, sub = tid % SC_SUB;
     const int c0 = blockIdx.x * SC_CH, c = c0 + ch;
@@ -230,6 +243,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     for (int i = 0; i < NS; ++i) {
         const int n = sub * NS + i;
         A[i] = (live && n < a.state) ? a.A[(long long)c * a.np + n] : 0.0f;
+        if (PAIRS) A[i] *= LOG2E;
     }
     for (int i = tid; i < 2 * SC_TT * 2 * nb; i += SC_THREADS) bc[i] = 0.0f;  // columns behind np stay zero
     __syncthreads();
@@ -277,12 +291,13 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        float* dt = dts + stage * SC_TT * SC_CH;
+        const float* dt = dts + stage * SC_TT * SC_CH;
         const T* x = xs + stage * SC_TT * SC_CH;
         for (int i = tid; i < SC_TT * SC_CH; i += SC_THREADS) {
             const int cc = c0 + (i & (SC_CH - 1));
             // a step size of zero leaves the state as it is: the rows behind the segment
-            dt[i] = (i / SC_CH < n && cc < a.ip) ? softplus_t<T>(dt[i] + a.dt_b[cc]) : 0.0f;
+            const float d = (i / SC_CH < n && cc < a.ip) ? softplus_t<T>(dt[i] + a.dt_b[cc]) : 0.0f, dx = d * to_f32(x[i]);
+            dd[i] = make_float4(d, d, dx, dx);
         }
         __syncthreads();
         const float* bt = bc + stage * SC_TT * 2 * nb + sub * NS;
@@ -292,17 +307,35 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
                 const int t = t8 + u;
-                const float d = dt[t * SC_CH + ch], dx = d * to_f32(x[t * SC_CH + ch]);
-                float B[NS], C[NS];
-                lds_vec<NS>(bt + t * 2 * nb, B);
-                lds_vec<NS>(bt + t * 2 * nb + nb, C);
-                float acc = 0.0f;
+                if constexpr (PAIRS) {
+                    const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(dd + t * SC_CH + ch);  // (dt, dt), (dt x, dt x)
+                    const uint64_t* B = reinterpret_cast<const uint64_t*>(bt + t * 2 * nb);
+                    const uint64_t* C = reinterpret_cast<const uint64_t*>(bt + t * 2 * nb + nb);
+                    uint64_t acc = 0;
 #pragma unroll
-                for (int i = 0; i < NS; ++i) {
-                    S[i] = fmaf(decay<T>(d * A[i]), S[i], dx * B[i]);
-                    acc = fmaf(S[i], C[i], acc);
+                    for (int i = 0; i < NS / 2; ++i) {
+                        float e0, e1;
+                        f2_unpack(f2_mul(w.x, f2_pack(A[2 * i], A[2 * i + 1])), e0, e1);
+                        const uint64_t s2 = f2_fma(f2_pack(fast_ex2(e0), fast_ex2(e1)), f2_pack(S[2 * i], S[2 * i + 1]), f2_mul(w.y, B[i]));
+                        f2_unpack(s2, S[2 * i], S[2 * i + 1]);
+                        acc = i == 0 ? f2_mul(s2, C[i]) : f2_fma(s2, C[i], acc);
+                    }
+                    float lo, hi;
+                    f2_unpack(acc, lo, hi);
+                    y[u] = lo + hi;
+                } else {
+                    const float4 w = dd[t * SC_CH + ch];
+                    float B[NS], C[NS];
+                    lds_vec<NS>(bt + t * 2 * nb, B);
+                    lds_vec<NS>(bt + t * 2 * nb + nb, C);
+                    float acc = 0.0f;
+#pragma unroll
+                    for (int i = 0; i < NS; ++i) {
+                        S[i] = fmaf(decay<T>(w.x * A[i]), S[i], w.z * B[i]);
+                        acc = fmaf(S[i], C[i], acc);
+                    }
+                    y[u] = acc;
                 }
-                y[u] = acc;
             }
             // eight partial sums on each of eight lanes -> lane `sub` holds the sum of token t8 + sub
             float k4[4], k2[2];
@@ -337,7 +370,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 }
 
 // ---- decode step --------------------------------------------------------------------------------------------------
-// One token of BB sequences and 32 channels per CTA.
+// One token of BB sequences and 32 channels per CTA (the convolution has already moved its state on).
 template <typename T, int NS, int BB>
 __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float st_dyn[];  // [BB][proj columns]
@@ -347,74 +380,105 @@ __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
     const bool live = c < a.ip;
     const int s0 = blockIdx.y * BB, nb = min(BB, a.n_segs - s0);
     const int pc = a.rp + 2 * a.np;
+    // constants of the channel, before the predecessor kernel has finished
     float A[NS];
 #pragma unroll
     for (int i = 0; i < NS; ++i) A[i] = sub * NS + i < a.state ? a.A[(long long)cl * a.np + sub * NS + i] : 0.0f;
+    const float bias = a.dt_b[cl], dv = a.D[cl];
+    const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
+    constexpr int PRE = 4;
+    typename Vec8<T>::Raw wr[PRE];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+        if (sub * 8 + i * 32 < a.rp) wr[i] = Vec8<T>::fetch(w + sub * 8 + i * 32);
     chain_wait();
-    float S[BB][NS];
-#pragma unroll
-    for (int b = 0; b < BB; ++b) {
-        const bool on = b < nb && a.seg_pos0[s0 + min(b, nb - 1)] > 0;
-        const float* state = a.S + ((long long)a.seg_slot[s0 + min(b, nb - 1)] * a.ip + cl) * a.np;
-#pragma unroll
-        for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? state[sub * NS + i] : 0.0f;
-    }
     for (int i = tid; i < nb * (pc / 4); i += ST_THREADS) {
         const int b = i / (pc / 4), v = i % (pc / 4);
-        reinterpret_cast<float4*>(st_dyn)[i] = reinterpret_cast<const float4*>(a.proj + (long long)a.seg_start[s0 + b] * pc)[v];
+        cp_async16(smem_u32(st_dyn + i * 4), a.proj + (long long)a.seg_start[s0 + b] * pc + v * 4, true);
     }
+    cp_async_commit();
+    // the states and the activations are on their way while the step sizes are computed
+    float* Sp[BB];
+    float S[BB][NS];
+    T xv[BB], zv[(BB + 3) / 4];
+    const T* xz = static_cast<const T*>(a.xz);
+#pragma unroll
+    for (int b = 0; b < BB; ++b) {
+        const int sg = s0 + min(b, nb - 1);
+        const int t = a.seg_start[sg];
+        Sp[b] = a.S + ((long long)a.seg_slot[sg] * a.ip + cl) * a.np + sub * NS;
+        const bool on = a.seg_pos0[sg] > 0;
+        if (NS % 4 == 0 && sub * NS + NS <= a.state) {
+#pragma unroll
+            for (int i = 0; i < NS / 4; ++i) {
+                const float4 v = on ? reinterpret_cast<const float4*>(Sp[b])[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+                S[b][4 * i] = v.x; S[b][4 * i + 1] = v.y; S[b][4 * i + 2] = v.z; S[b][4 * i + 3] = v.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? Sp[b][i] : 0.0f;
+        }
+        xv[b] = static_cast<const T*>(a.xc)[(long long)t * a.ip + cl];
+        if ((b & 3) == sub) zv[b / 4] = xz[(long long)t * 2 * a.ip + a.ip + cl];
+    }
+    cp_async_wait<0>();
     __syncthreads();
     // step sizes: four threads share a channel's row of the projection
     float dt[BB];
 #pragma unroll
     for (int b = 0; b < BB; ++b) dt[b] = 0.0f;
-    const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
-    for (int r = sub * 8; r < a.rp; r += 32) {
+    auto dot = [&](int r, const typename Vec8<T>::Raw& raw) {
         float wv[8];
-        Vec8<T>::load(w + r, wv);
+        Vec8<T>::widen(raw, wv);
 #pragma unroll
         for (int b = 0; b < BB; ++b) {
-            if (b >= nb) break;
-            const float* p = st_dyn + b * pc + r;
-#pragma unroll
-            for (int e = 0; e < 8; ++e) dt[b] = fmaf(wv[e], p[e], dt[b]);
+            const float4* p = reinterpret_cast<const float4*>(st_dyn + min(b, nb - 1) * pc + r);
+            const float4 u = p[0], v = p[1];
+            dt[b] = fmaf(wv[0], u.x, dt[b]); dt[b] = fmaf(wv[1], u.y, dt[b]); dt[b] = fmaf(wv[2], u.z, dt[b]); dt[b] = fmaf(wv[3], u.w, dt[b]);
+            dt[b] = fmaf(wv[4], v.x, dt[b]); dt[b] = fmaf(wv[5], v.y, dt[b]); dt[b] = fmaf(wv[6], v.z, dt[b]); dt[b] = fmaf(wv[7], v.w, dt[b]);
         }
-    }
-    const float bias = a.dt_b[cl], dv = a.D[cl];
-    const T* xz = static_cast<const T*>(a.xz);
+    };
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+        if (sub * 8 + i * 32 < a.rp) dot(sub * 8 + i * 32, wr[i]);
+#pragma unroll 4
+    for (int r = sub * 8 + PRE * 32; r < a.rp; r += 32) dot(r, Vec8<T>::fetch(w + r));
+    __syncwarp();  // (the four threads of a channel may differ in their trip counts)
 #pragma unroll
     for (int b = 0; b < BB; ++b) {
-        if (b >= nb) break;
         float d = dt[b];
         d += __shfl_xor_sync(0xffffffffu, d, 1);
         d += __shfl_xor_sync(0xffffffffu, d, 2);
-        d = softplus_t<T>(d + bias);
-        const int t = a.seg_start[s0 + b];
-        const float x = to_f32(static_cast<const T*>(a.xc)[(long long)t * a.ip + cl]), dx = d * x;
-        const float* Bp = st_dyn + b * pc + a.rp + sub * NS;
+        dt[b] = softplus_t<T>(d + bias);
+    }
+#pragma unroll
+    for (int b = 0; b < BB; ++b) {
+        const float x = to_f32(xv[b]), dx = dt[b] * x;
+        const float* Bp = st_dyn + min(b, nb - 1) * pc + a.rp + sub * NS;
         const float* Cp = Bp + a.np;
-        float* state = a.S + ((long long)a.seg_slot[s0 + b] * a.ip + cl) * a.np + sub * NS;
         float y = 0.0f;
 #pragma unroll
         for (int i = 0; i < NS; ++i) {
             if (sub * NS + i < a.state) {
-                S[b][i] = fmaf(decay<T>(d * A[i]), S[b][i], dx * Bp[i]);
+                S[b][i] = fmaf(decay<T>(dt[b] * A[i]), S[b][i], dx * Bp[i]);
                 y = fmaf(S[b][i], Cp[i], y);
-                if (live) state[i] = S[b][i];
+            }
+        }
+        if (b < nb && live) {
+            if (NS % 4 == 0 && sub * NS + NS <= a.state) {
+#pragma unroll
+                for (int i = 0; i < NS / 4; ++i)
+                    reinterpret_cast<float4*>(Sp[b])[i] = make_float4(S[b][4 * i], S[b][4 * i + 1], S[b][4 * i + 2], S[b][4 * i + 3]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < NS; ++i)
+                    if (sub * NS + i < a.state) Sp[b][i] = S[b][i];
             }
         }
         y += __shfl_xor_sync(0xffffffffu, y, 1);
         y += __shfl_xor_sync(0xffffffffu, y, 2);
-        if (sub == (b & 3) && live) {
-            const float z = to_f32(xz[(long long)t * 2 * a.ip + a.ip + c]);
-            static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(z));
-        }
-    }
-    for (int i = tid; i < SC_CH * nb; i += ST_THREADS) {
-        const int b = i / SC_CH, cc = c0 + i % SC_CH;
-        if (cc < a.ip)
-            carry_conv_state(static_cast<T*>(a.conv) + (long long)a.seg_slot[s0 + b] * (a.taps - 1) * a.ip, xz, cc, a.ip, a.taps,
-                             a.seg_start[s0 + b], 1, a.seg_pos0[s0 + b]);
+        if (sub == (b & 3) && b < nb && live)
+            static_cast<T*>(a.y)[(long long)a.seg_start[s0 + b] * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(to_f32(zv[b / 4])));
     }
 }
 
@@ -433,13 +497,13 @@ __global__ void __launch_bounds__(256) scan_dt_operand_kernel(const float* __res
 // ---- launches -----------------------------------------------------------------------------------------------------
 template <typename T>
 static jsm_status conv_typed(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, void* xc,
-                             int max_len, cudaStream_t st) {
+                             bool carry, cudaStream_t st) {
     const int ip = d.ip();
-    const long long n = (long long)((max_len + CONV_TOK - 1) / CONV_TOK) * (ip / 8);
+    const long long n = (long long)((tk.max_len + CONV_TOK - 1) / CONV_TOK) * (ip / 8);
     const dim3 grid((unsigned)((n + 255) / 256), tk.n_segs);
     auto go = [&](auto kernel) {
-        return launch_chained(kernel, grid, dim3(256), 0, st, (const T*)xz, (T*)xc, (const T*)s.conv, w.conv, w.conv_b, tk.seg_start, tk.seg_len,
-                              tk.seg_pos0, tk.seg_slot, ip, d.taps);
+        return launch_chained(kernel, grid, dim3(256), 0, st, (const T*)xz, (T*)xc, (T*)s.conv, w.conv, w.conv_b, tk.seg_start, tk.seg_len,
+                              tk.seg_pos0, tk.seg_slot, ip, d.taps, carry ? 1 : 0);
     };
     JSM_CUDA_CHECK(d.taps == 2 ? go(scan_conv_kernel<T, 2>) : d.taps == 3 ? go(scan_conv_kernel<T, 3>)
                    : d.taps == 4 ? go(scan_conv_kernel<T, 4>) : go(scan_conv_kernel<T, 0>));
@@ -448,8 +512,8 @@ static jsm_status conv_typed(const ScanDims& d, const ScanWeights& w, const Scan
 }
 
 jsm_status scan_conv_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
-                            void* xc, cudaStream_t st) {
-    return f32 ? conv_typed<float>(d, w, s, tk, xz, xc, tk.max_len, st) : conv_typed<__nv_bfloat16>(d, w, s, tk, xz, xc, tk.max_len, st);
+                            void* xc, bool carry, cudaStream_t st) {
+    return f32 ? conv_typed<float>(d, w, s, tk, xz, xc, carry, st) : conv_typed<__nv_bfloat16>(d, w, s, tk, xz, xc, carry, st);
 }
 
 static ScanArgs scan_args(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, const void* xc,
