@@ -319,7 +319,7 @@ constexpr int LA_ROWS = LATENT_TILE_ROWS;
 constexpr int LA_SP = 68;  // pitch of the score tile (floats)
 constexpr int LA_PP = 72;  // pitch of the weight tile (bf16)
 constexpr int LA_ML = 4;   // behind a partial row: its maximum, its sum, two unused
-constexpr int LA_MAX_SPLITS = 256;
+constexpr int LA_MAX_SPLITS = 128;
 constexpr int LA_ERR_FULL = 51;
 
 static int la_pitch(const LatentDims& d) { return pad_to(d.rank + d.rot, 16) + 8; }  // odd multiple of 16 bytes: no bank conflicts
@@ -452,27 +452,46 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const __nv_bflo
             }
         }
         __syncthreads();
+        {   // softmax: a warp takes four rows side by side, two keys per lane
+            constexpr int R = LA_ROWS / 8;
+            float a[R], b[R], mx[R], sum[R], m_old[R], ref[R];
 #pragma unroll
-        for (int i2 = 0; i2 < LA_ROWS / 8; ++i2) {  // softmax: a warp per row, two keys per lane
-            const int r = warp * (LA_ROWS / 8) + i2;
-            const int p = pos0 + (r0 + r) / d.H, k0 = pg * PAGE + lane, k1 = k0 + 32;
-            const bool on = r < n_rows;
-            const float* sr = ss + r * LA_SP + lane;
-            float a = (on && k0 <= p && p - k0 < d.window) ? (sr[0] + sr[LA_ROWS * LA_SP]) * d.scale : -INFINITY;
-            float b = (on && k1 <= p && p - k1 < d.window) ? (sr[32] + sr[LA_ROWS * LA_SP + 32]) * d.scale : -INFINITY;
-            const float m_old = row_m[r], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
-            const float ref = m_new == -INFINITY ? 0.0f : m_new;
-            a = __expf(a - ref);
-            b = __expf(b - ref);
-            const float sum = warp_sum(a + b);
-            ps[r * LA_PP + lane] = __float2bfloat16_rn(a);
-            ps[r * LA_PP + lane + 32] = __float2bfloat16_rn(b);
-            if (lane == 0) {
-                const float al = __expf(m_old - ref);
-                row_a[r] = al;
-                row_l[r] = row_l[r] * al + sum;
-                row_m[r] = m_new;
+            for (int q = 0; q < R; ++q) {
+                const int r = warp * R + q, p = pos0 + (r0 + r) / d.H, k0 = pg * PAGE + lane, k1 = k0 + 32;
+                const bool on = r < n_rows;
+                const float* sr = ss + r * LA_SP + lane;
+                a[q] = (on && k0 <= p && p - k0 < d.window) ? (sr[0] + sr[LA_ROWS * LA_SP]) * d.scale : -INFINITY;
+                b[q] = (on && k1 <= p && p - k1 < d.window) ? (sr[32] + sr[LA_ROWS * LA_SP + 32]) * d.scale : -INFINITY;
+                mx[q] = fmaxf(a[q], b[q]);
+                m_old[q] = row_m[r];
             }
+#pragma unroll
+            for (int x = 16; x > 0; x >>= 1)
+#pragma unroll
+                for (int q = 0; q < R; ++q) mx[q] = fmaxf(mx[q], __shfl_xor_sync(0xffffffffu, mx[q], x));
+#pragma unroll
+            for (int q = 0; q < R; ++q) {
+                mx[q] = fmaxf(mx[q], m_old[q]);
+                ref[q] = mx[q] == -INFINITY ? 0.0f : mx[q];
+                a[q] = __expf(a[q] - ref[q]);
+                b[q] = __expf(b[q] - ref[q]);
+                sum[q] = a[q] + b[q];
+                ps[(warp * R + q) * LA_PP + lane] = __float2bfloat16_rn(a[q]);
+                ps[(warp * R + q) * LA_PP + lane + 32] = __float2bfloat16_rn(b[q]);
+            }
+#pragma unroll
+            for (int x = 16; x > 0; x >>= 1)
+#pragma unroll
+                for (int q = 0; q < R; ++q) sum[q] += __shfl_xor_sync(0xffffffffu, sum[q], x);
+            if (lane == 0)
+#pragma unroll
+                for (int q = 0; q < R; ++q) {
+                    const int r = warp * R + q;
+                    const float al = __expf(m_old[q] - ref[q]);
+                    row_a[r] = al;
+                    row_l[r] = row_l[r] * al + sum[q];
+                    row_m[r] = mx[q];
+                }
         }
         __syncthreads();
         // weighted sum of the latents
@@ -545,8 +564,6 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
                                                              const int32_t* __restrict__ seg_len, const int32_t* __restrict__ tile_seg,
                                                              const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ tile_r0, int max_splits,
                                                              __nv_bfloat16* __restrict__ o_lat) {
-    __shared__ float w[LA_MAX_SPLITS];
-    __shared__ float red[8];
     chain_trigger();
     chain_wait();
     const int tile = blockIdx.x, r = blockIdx.y, rp = pad8(d.rank), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -558,31 +575,47 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
     const int splits = min(max_splits, p_last / PAGE - max(0, p_first - d.window + 1) / PAGE + 1);
     const long long stride = (long long)LA_ROWS * (rp + LA_ML);
     const float* p = part + ((long long)tile * max_splits * LA_ROWS + r) * (rp + LA_ML);
-    float m = -INFINITY;
-    for (int s = threadIdx.x; s < splits; s += 128) m = fmaxf(m, p[s * stride + rp]);
+    // every warp works out the weights for itself: lane s % 32 holds those of split s
+    float ms[LA_MAX_SPLITS / 32], w[LA_MAX_SPLITS / 32], m = -INFINITY, l = 0.0f;
+#pragma unroll
+    for (int i = 0; i < LA_MAX_SPLITS / 32; ++i) {
+        ms[i] = -INFINITY; w[i] = 0.0f;
+        const int s = i * 32 + lane;
+        if (s < splits) {
+            const float2 v = *reinterpret_cast<const float2*>(p + s * stride + rp);
+            ms[i] = v.x; w[i] = v.y;
+            m = fmaxf(m, v.x);
+        }
+    }
     m = warp_max(m);
-    if (lane == 0) red[warp] = m;
-    __syncthreads();
-    m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-    for (int s = threadIdx.x; s < splits; s += 128) w[s] = __expf(p[s * stride + rp] - m);
-    __syncthreads();
-    float l = 0.0f;
-    for (int s = lane; s < splits; s += 32) l += w[s] * p[s * stride + rp + 1];  // every warp for itself
+#pragma unroll
+    for (int i = 0; i < LA_MAX_SPLITS / 32; ++i) {
+        const float e = __expf(ms[i] - m);
+        l += e * w[i];
+        w[i] = e;
+    }
     const float inv = 1.0f / warp_sum(l);
     __nv_bfloat16* out = o_lat + ((long long)(seg_start[seg] + g / d.H) * d.H + g % d.H) * rp;
-    for (int c = threadIdx.x * 4; c < rp; c += 512) {
+    for (int c0 = warp * 128; c0 < rp; c0 += 512) {  // (warp-uniform: the shuffles need every lane)
+        const int c = c0 + lane * 4, cc = min(c, rp - 4);
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < LA_MAX_SPLITS / 32; ++i) {
+            if (i * 32 >= splits) break;
+            const int n = min(32, splits - i * 32);
 #pragma unroll 8
-        for (int s = 0; s < splits; ++s) {
-            const float4 v = __ldcs(reinterpret_cast<const float4*>(p + s * stride + c));
-            const float f = w[s];  // a split without a visible key holds zeros and weighs nothing
-            acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
+            for (int s = 0; s < n; ++s) {
+                const float4 v = __ldcs(reinterpret_cast<const float4*>(p + (i * 32 + s) * stride + cc));
+                const float f = __shfl_sync(0xffffffffu, w[i], s);  // a split without a visible key holds zeros and weighs nothing
+                acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
+            }
         }
-        const float o[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
-        uint2 u;
-        u.x = pack_bf16x2(c < d.rank ? o[0] : 0.0f, c + 1 < d.rank ? o[1] : 0.0f);
-        u.y = pack_bf16x2(c + 2 < d.rank ? o[2] : 0.0f, c + 3 < d.rank ? o[3] : 0.0f);
-        *reinterpret_cast<uint2*>(out + c) = u;
+        if (c < rp) {
+            uint2 u;
+            u.x = pack_bf16x2(c < d.rank ? acc.x * inv : 0.0f, c + 1 < d.rank ? acc.y * inv : 0.0f);
+            u.y = pack_bf16x2(c + 2 < d.rank ? acc.z * inv : 0.0f, c + 3 < d.rank ? acc.w * inv : 0.0f);
+            *reinterpret_cast<uint2*>(out + c) = u;
+        }
     }
 }
 

@@ -87,6 +87,19 @@ struct Vec8<__nv_bfloat16> {
     }
 };
 
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v[0] = bf16lo(a.x); v[1] = bf16hi(a.x); v[2] = bf16lo(a.y); v[3] = bf16hi(a.y);
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+
 // ---- convolution --------------------------------------------------------------------------------------------------
 // A thread owns 8 channels of CONV_TOK consecutive tokens; TAPS 0: taps is only known at run time.  carry: every segment is
 // one token, and the state moves on by it here (otherwise the scan does that, once every CTA has read the old state)
@@ -284,6 +297,12 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     };
     load_tile(0, 0);
     cp_async_commit();
+    // every pass over a tile gives a thread the same channels: their constants stay in registers
+    static_assert(SC_THREADS % SC_CH == 0 && SC_TT * SC_CH == SC_THREADS * 4, "four elements of a tile per thread");
+    const float bias = c0 + (tid & (SC_CH - 1)) < a.ip ? a.dt_b[c0 + (tid & (SC_CH - 1))] : 0.0f;
+    const int ov = (tid & (SC_CH / 4 - 1)) * 4, orow = tid / (SC_CH / 4);  // output pass: four channels of one token
+    const bool olive = c0 + ov < a.ip;
+    const float4 Dv = olive ? *reinterpret_cast<const float4*>(a.D + c0 + ov) : make_float4(0.f, 0.f, 0.f, 0.f);
     const int nt = (len + SC_TT - 1) / SC_TT;
     for (int it = 0; it < nt; ++it) {
         const int stage = it & 1, t0 = it * SC_TT, n = min(SC_TT, len - t0);
@@ -293,10 +312,11 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
         __syncthreads();
         const float* dt = dts + stage * SC_TT * SC_CH;
         const T* x = xs + stage * SC_TT * SC_CH;
-        for (int i = tid; i < SC_TT * SC_CH; i += SC_THREADS) {
-            const int cc = c0 + (i & (SC_CH - 1));
-            // a step size of zero leaves the state as it is: the rows behind the segment
-            const float d = (i / SC_CH < n && cc < a.ip) ? softplus_t<T>(dt[i] + a.dt_b[cc]) : 0.0f, dx = d * to_f32(x[i]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int i = u * SC_THREADS + tid;
+            // a step size of zero leaves the state as it is: the rows behind the segment (and channels behind the last)
+            const float d = i / SC_CH < n ? softplus_t<T>(dt[i] + bias) : 0.0f, dx = d * to_f32(x[i]);
             dd[i] = make_float4(d, d, dx, dx);
         }
         __syncthreads();
@@ -348,16 +368,14 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
         }
         __syncthreads();
         const T* z = zs + stage * SC_TT * SC_CH;
-        for (int i = tid; i < n * (SC_CH / 8); i += SC_THREADS) {
-            const int r = i / (SC_CH / 8), v = (i % (SC_CH / 8)) * 8;
-            if (c0 + v >= a.ip) continue;
-            float xv[8], zv[8], dv[8], o[8];
-            Vec8<T>::load(x + r * SC_CH + v, xv);
-            Vec8<T>::load(z + r * SC_CH + v, zv);
-            Vec8<float>::load(a.D + c0 + v, dv);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) o[e] = fmaf(dv[e], xv[e], ys[r * SC_YP + v + e]) * silu_t<T>(zv[e]);
-            Vec8<T>::store(static_cast<T*>(a.y) + (long long)(start + t0 + r) * a.ip + c0 + v, o);
+        if (orow < n && olive) {
+            float xv[4], zv[4], o[4];
+            load4(x + orow * SC_CH + ov, xv);
+            load4(z + orow * SC_CH + ov, zv);
+            const float4 yv = *reinterpret_cast<const float4*>(ys + orow * SC_YP + ov);
+            o[0] = fmaf(Dv.x, xv[0], yv.x) * silu_t<T>(zv[0]); o[1] = fmaf(Dv.y, xv[1], yv.y) * silu_t<T>(zv[1]);
+            o[2] = fmaf(Dv.z, xv[2], yv.z) * silu_t<T>(zv[2]); o[3] = fmaf(Dv.w, xv[3], yv.w) * silu_t<T>(zv[3]);
+            store4(static_cast<T*>(a.y) + (long long)(start + t0 + orow) * a.ip + c0 + ov, o);
         }
         __syncthreads();
     }
@@ -370,115 +388,123 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 }
 
 // ---- decode step --------------------------------------------------------------------------------------------------
-// One token of BB sequences and 32 channels per CTA (the convolution has already moved its state on).
+// One token of BB (at most 8) sequences and 32 channels per CTA; the convolution has already moved its state on.  The step
+// sizes of the 32 channels x 8 sequences are one small product: bf16 models take it on the tensor cores (weights as the
+// 16-row operand, two tiles of channels x two halves of the rank over the four warps), f32 models with four threads per
+// channel.  The code is kept short: a launch fetches it cold.
 template <typename T, int NS, int BB>
 __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
-    extern __shared__ __align__(16) float st_dyn[];  // [BB][proj columns]
+    extern __shared__ __align__(16) float st_dyn[];  // [BB][B: np | C: np]; f32: [BB][proj columns]
+    __shared__ float dts[2][SC_CH][9];
+    constexpr bool MMA = sizeof(T) == 2;
     chain_trigger();
-    const int tid = threadIdx.x, ch = tid / ST_SUB, sub = tid % ST_SUB;
+    const int tid = threadIdx.x, ch = tid / ST_SUB, sub = tid % ST_SUB, warp = tid >> 5, lane = tid & 31;
     const int c0 = blockIdx.x * SC_CH, c = c0 + ch, cl = min(c, a.ip - 1);
     const bool live = c < a.ip;
     const int s0 = blockIdx.y * BB, nb = min(BB, a.n_segs - s0);
-    const int pc = a.rp + 2 * a.np;
+    const int pc = a.rp + 2 * a.np, off = MMA ? a.rp : 0, sc = pc - off;  // columns of proj that go to shared memory
     // constants of the channel, before the predecessor kernel has finished
     float A[NS];
 #pragma unroll
     for (int i = 0; i < NS; ++i) A[i] = sub * NS + i < a.state ? a.A[(long long)cl * a.np + sub * NS + i] : 0.0f;
     const float bias = a.dt_b[cl], dv = a.D[cl];
-    const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
-    constexpr int PRE = 4;
-    typename Vec8<T>::Raw wr[PRE];
-#pragma unroll
-    for (int i = 0; i < PRE; ++i)
-        if (sub * 8 + i * 32 < a.rp) wr[i] = Vec8<T>::fetch(w + sub * 8 + i * 32);
     chain_wait();
-    for (int i = tid; i < nb * (pc / 4); i += ST_THREADS) {
-        const int b = i / (pc / 4), v = i % (pc / 4);
-        cp_async16(smem_u32(st_dyn + i * 4), a.proj + (long long)a.seg_start[s0 + b] * pc + v * 4, true);
+    for (int i = tid; i < nb * (sc / 4); i += ST_THREADS) {
+        const int b = i / (sc / 4), v = i % (sc / 4);
+        cp_async16(smem_u32(st_dyn + i * 4), a.proj + (long long)a.seg_start[s0 + b] * pc + off + v * 4, true);
     }
     cp_async_commit();
-    // the states and the activations are on their way while the step sizes are computed
-    float* Sp[BB];
+    // the states are on their way while the step sizes are computed
     float S[BB][NS];
-    T xv[BB], zv[(BB + 3) / 4];
-    const T* xz = static_cast<const T*>(a.xz);
 #pragma unroll
     for (int b = 0; b < BB; ++b) {
         const int sg = s0 + min(b, nb - 1);
-        const int t = a.seg_start[sg];
-        Sp[b] = a.S + ((long long)a.seg_slot[sg] * a.ip + cl) * a.np + sub * NS;
+        const float* Sp = a.S + ((long long)a.seg_slot[sg] * a.ip + cl) * a.np + sub * NS;
         const bool on = a.seg_pos0[sg] > 0;
         if (NS % 4 == 0 && sub * NS + NS <= a.state) {
 #pragma unroll
             for (int i = 0; i < NS / 4; ++i) {
-                const float4 v = on ? reinterpret_cast<const float4*>(Sp[b])[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 v = on ? reinterpret_cast<const float4*>(Sp)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
                 S[b][4 * i] = v.x; S[b][4 * i + 1] = v.y; S[b][4 * i + 2] = v.z; S[b][4 * i + 3] = v.w;
             }
         } else {
 #pragma unroll
-            for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? Sp[b][i] : 0.0f;
+            for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? Sp[i] : 0.0f;
         }
-        xv[b] = static_cast<const T*>(a.xc)[(long long)t * a.ip + cl];
-        if ((b & 3) == sub) zv[b / 4] = xz[(long long)t * 2 * a.ip + a.ip + cl];
+    }
+    if constexpr (MMA) {
+        const int mt = warp & 1, kh = warp >> 1, g = lane >> 2, kq = (lane & 3) * 8;
+        const int n_blk = (a.rp + 31) / 32, b0 = kh ? (n_blk + 1) / 2 : 0, b1 = kh ? n_blk : (n_blk + 1) / 2;
+        const int r0 = c0 + mt * 16 + g;
+        const __nv_bfloat16* w0 = static_cast<const __nv_bfloat16*>(a.dt_w) + (long long)min(r0, a.ip - 1) * a.rp;
+        const __nv_bfloat16* w1 = static_cast<const __nv_bfloat16*>(a.dt_w) + (long long)min(r0 + 8, a.ip - 1) * a.rp;
+        const float* p = a.proj + (long long)a.seg_start[s0 + min(g, nb - 1)] * pc;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int blk = b0; blk < b1; ++blk) {
+            const int k = blk * 32 + kq;
+            uint4 x = make_uint4(0, 0, 0, 0), y = x;
+            float4 u = make_float4(0.f, 0.f, 0.f, 0.f), v = u;
+            if (k < a.rp) {
+                x = __ldg(reinterpret_cast<const uint4*>(w0 + k));
+                y = __ldg(reinterpret_cast<const uint4*>(w1 + k));
+                u = reinterpret_cast<const float4*>(p + k)[0];
+                v = reinterpret_cast<const float4*>(p + k)[1];
+            }
+            const uint32_t a0[4] = {x.x, y.x, x.y, y.y}, a1[4] = {x.z, y.z, x.w, y.w};
+            mma_16816(acc, a0, pack_bf16x2(u.x, u.y), pack_bf16x2(u.z, u.w));
+            mma_16816(acc, a1, pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+        }
+        float* d = &dts[kh][mt * 16 + g][(lane & 3) * 2];
+        d[0] = acc[0]; d[1] = acc[1]; d[8 * 9] = acc[2]; d[8 * 9 + 1] = acc[3];
     }
     cp_async_wait<0>();
     __syncthreads();
-    // step sizes: four threads share a channel's row of the projection
-    float dt[BB];
-#pragma unroll
-    for (int b = 0; b < BB; ++b) dt[b] = 0.0f;
-    auto dot = [&](int r, const typename Vec8<T>::Raw& raw) {
-        float wv[8];
-        Vec8<T>::widen(raw, wv);
-#pragma unroll
-        for (int b = 0; b < BB; ++b) {
-            const float4* p = reinterpret_cast<const float4*>(st_dyn + min(b, nb - 1) * pc + r);
-            const float4 u = p[0], v = p[1];
-            dt[b] = fmaf(wv[0], u.x, dt[b]); dt[b] = fmaf(wv[1], u.y, dt[b]); dt[b] = fmaf(wv[2], u.z, dt[b]); dt[b] = fmaf(wv[3], u.w, dt[b]);
-            dt[b] = fmaf(wv[4], v.x, dt[b]); dt[b] = fmaf(wv[5], v.y, dt[b]); dt[b] = fmaf(wv[6], v.z, dt[b]); dt[b] = fmaf(wv[7], v.w, dt[b]);
+    if constexpr (!MMA) {
+        const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
+        for (int b = 0; b < nb; ++b) {
+            float d = 0.0f;
+            for (int r = sub; r < a.rp; r += ST_SUB) d = fmaf(to_f32(w[r]), st_dyn[b * sc + r], d);
+            __syncwarp();
+            d += __shfl_xor_sync(0xffffffffu, d, 1);
+            d += __shfl_xor_sync(0xffffffffu, d, 2);
+            if (sub == 0) { dts[0][ch][b] = d; dts[1][ch][b] = 0.0f; }
         }
-    };
-#pragma unroll
-    for (int i = 0; i < PRE; ++i)
-        if (sub * 8 + i * 32 < a.rp) dot(sub * 8 + i * 32, wr[i]);
-#pragma unroll 4
-    for (int r = sub * 8 + PRE * 32; r < a.rp; r += 32) dot(r, Vec8<T>::fetch(w + r));
-    __syncwarp();  // (the four threads of a channel may differ in their trip counts)
-#pragma unroll
-    for (int b = 0; b < BB; ++b) {
-        float d = dt[b];
-        d += __shfl_xor_sync(0xffffffffu, d, 1);
-        d += __shfl_xor_sync(0xffffffffu, d, 2);
-        dt[b] = softplus_t<T>(d + bias);
+        __syncwarp();
     }
+    const T* xz = static_cast<const T*>(a.xz);
 #pragma unroll
     for (int b = 0; b < BB; ++b) {
-        const float x = to_f32(xv[b]), dx = dt[b] * x;
-        const float* Bp = st_dyn + min(b, nb - 1) * pc + a.rp + sub * NS;
+        if (b >= nb) break;
+        const int t = a.seg_start[s0 + b];
+        const float x = to_f32(static_cast<const T*>(a.xc)[(long long)t * a.ip + cl]);
+        const float z = to_f32(xz[(long long)t * 2 * a.ip + a.ip + cl]);
+        const float dt = softplus_t<T>(dts[0][ch][b] + dts[1][ch][b] + bias), dx = dt * x;
+        const float* Bp = st_dyn + b * sc + (a.rp - off) + sub * NS;
         const float* Cp = Bp + a.np;
+        float* Sp = a.S + ((long long)a.seg_slot[s0 + b] * a.ip + cl) * a.np + sub * NS;
         float y = 0.0f;
 #pragma unroll
         for (int i = 0; i < NS; ++i) {
             if (sub * NS + i < a.state) {
-                S[b][i] = fmaf(decay<T>(dt[b] * A[i]), S[b][i], dx * Bp[i]);
+                S[b][i] = fmaf(decay<T>(dt * A[i]), S[b][i], dx * Bp[i]);
                 y = fmaf(S[b][i], Cp[i], y);
             }
         }
-        if (b < nb && live) {
+        if (live) {
             if (NS % 4 == 0 && sub * NS + NS <= a.state) {
 #pragma unroll
                 for (int i = 0; i < NS / 4; ++i)
-                    reinterpret_cast<float4*>(Sp[b])[i] = make_float4(S[b][4 * i], S[b][4 * i + 1], S[b][4 * i + 2], S[b][4 * i + 3]);
+                    reinterpret_cast<float4*>(Sp)[i] = make_float4(S[b][4 * i], S[b][4 * i + 1], S[b][4 * i + 2], S[b][4 * i + 3]);
             } else {
 #pragma unroll
                 for (int i = 0; i < NS; ++i)
-                    if (sub * NS + i < a.state) Sp[b][i] = S[b][i];
+                    if (sub * NS + i < a.state) Sp[i] = S[b][i];
             }
         }
         y += __shfl_xor_sync(0xffffffffu, y, 1);
         y += __shfl_xor_sync(0xffffffffu, y, 2);
-        if (sub == (b & 3) && b < nb && live)
-            static_cast<T*>(a.y)[(long long)a.seg_start[s0 + b] * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(to_f32(zv[b / 4])));
+        if (sub == (b & 3) && live) static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(z));
     }
 }
 
