@@ -292,10 +292,10 @@ static jsm_status build_scan(jsm_decoder* m, DecLayer& L, const std::string& pre
         DEC_TRY(upload_proj(m, h, &L.out));
     }
     {
-        HostMatrix c(true, d.taps, ip), a(true, ip, d.np());
+        HostMatrix c(true, d.taps, ip), a(true, d.np() / 4, ip * 4);
         for (int j = 0; j < d.inner; ++j) {
             for (int k = 0; k < d.taps; ++k) c.set(k, j, conv->at((long long)j * d.taps + k));
-            for (int n = 0; n < d.state; ++n) a.set(j, n, (float)-exp((double)A->at((long long)j * d.state + n)));
+            for (int n = 0; n < d.state; ++n) a.set(n / 4, j * 4 + n % 4, (float)-exp((double)A->at((long long)j * d.state + n)));
         }
         void *pc = nullptr, *pa = nullptr;
         DEC_TRY(upload_plain(m, c, &pc));

@@ -88,14 +88,14 @@ struct ScanDims {
 };
 struct ScanWeights {
     const float *conv, *conv_b;  // [taps][ip], [ip]
-    const float* A;              // [ip][np]: -exp(A_log) (0 in the padding)
+    const float* A;              // [np / 4][ip][4]: -exp(A_log) (0 in the padding)
     const float* D;              // [ip]
     const float* dt_b;           // [ip]
     const void* dt;              // act dtype, [ip][rp] (the fused decode step)
 };
 struct ScanState {
     void* conv;    // act [slots][taps - 1][ip]: the last inputs of the convolution
-    float* S;      // [slots][ip][np]
+    float* S;      // [slots][np / 4][ip][4]
 };
 // xc = silu(conv(x) + b) over the x half of xz (act [T][2 ip]); carry (one token per segment): also moves the convolution
 // state on, which otherwise the scan does

@@ -310,7 +310,7 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
 }
 
 // bf16 on the tensor cores.  A CTA owns 32 (token, head) rows of one segment and a run of cache pages; a page of 64 entries
-// is one stage of a two-stage ring filled by bulk copies (a row each, one warp issues them), read once for the scores (all
+// is one stage of a two-stage ring filled by bulk copies (a row each), read once for the scores (all
 // rank + rot components) and once for the weighted sum (the first rank components).  Eight warps: scores as 2 tiles of 16
 // rows x 2 halves of the components x 2 groups of 32 keys - a warp keeps its part of the queries in registers - then the sum
 // as column blocks of NT x 8 latent components per warp, all 32 rows.  Scores, maxima and sums are fp32; the weights enter the
@@ -372,18 +372,20 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const __nv_bflo
     const int pb = pg_lo + n_pg * sp / live, pe = pg_lo + n_pg * (sp + 1) / live;
     const int32_t* bt = block_table + (long long)seg_row[seg] * max_pages;
     const int vec = cr / 8;  // 16-byte vectors per entry
-    auto load_page = [&](int pg, int stage) {  // warp 0
+    // A row per copy, issued by the first eight lanes of every warp (a thread's copies go out one after the other, and one
+    // warp would hold up the others).  A copy that lands before the expected bytes are announced cannot complete the phase:
+    // the announcement is also its only arrival.
+    auto load_page = [&](int pg, int stage) {
         const int lo = max(key_lo - pg * PAGE, 0), hi = min(key_hi - pg * PAGE, PAGE);
-        if (lane == 0) tc::mbar_expect_tx(&full[stage], (uint32_t)(hi - lo) * cr * 2);
-        __syncwarp();
-        const __nv_bfloat16* src = pool + (long long)bt[pg] * PAGE * cr;
-        __nv_bfloat16* dst = kv + stage * PAGE * pitch;
-        for (int r = lo + lane; r < hi; r += 32)
-            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst + r * pitch)),
-                         "l"(reinterpret_cast<uint64_t>(src + (long long)r * cr)), "r"(cr * 2), "r"(smem_u32(&full[stage]))
+        if (threadIdx.x == 0) tc::mbar_expect_tx(&full[stage], (uint32_t)(hi - lo) * cr * 2);
+        const int r = warp * 8 + lane;
+        if (lane < 8 && r >= lo && r < hi)
+            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                             smem_u32(kv + (stage * PAGE + r) * pitch)),
+                         "l"(reinterpret_cast<uint64_t>(pool + ((long long)bt[pg] * PAGE + r) * cr)), "r"(cr * 2), "r"(smem_u32(&full[stage]))
                          : "memory");
     };
-    if (warp == 0) load_page(pb, 0);
+    load_page(pb, 0);
     // the queries pass through the second stage into registers
     for (int i = threadIdx.x; i < LA_ROWS * vec; i += 256) {
         const int r = i / vec, c = i - r * vec, g = r0 + r;
@@ -413,7 +415,7 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const __nv_bflo
     bool ok = true;
     for (int pg = pb; pg < pe; ++pg) {
         const int i = pg - pb, stage = i & 1;
-        if (warp == 0 && pg + 1 < pe) load_page(pg + 1, stage ^ 1);
+        if (pg + 1 < pe) load_page(pg + 1, stage ^ 1);
         __nv_bfloat16* kvs = kv + stage * PAGE * pitch;
         {   // entries outside the tile's key range are not fetched: their rows are zero (a weight of 0 must meet a number)
             const int lo = max(key_lo - pg * PAGE, 0), hi = min(key_hi - pg * PAGE, PAGE);

@@ -10,8 +10,11 @@
 //
 // Prompts: a CTA owns 32 channels of one segment and walks its tokens in tiles of 32 that cp.async brings into a two-stage
 // ring; eight threads share a channel's states, so that the chain of dependent steps is one FMA per state and the partial
-// sums of eight tokens are exchanged with seven shuffles.  Decode: four threads per channel, one step for several
-// sequences per CTA; the state rows are requested first and arrive while the step sizes (a small projection) are computed.
+// sums of eight tokens are exchanged with seven shuffles.  Decode: one thread per channel and sequence, eight sequences per
+// CTA; the states are requested first and arrive while the step sizes (a small projection) are computed.
+//
+// Layout of S and A: planes of four states, [plane][channel][4], so that neighbouring threads - channels - read neighbouring
+// 16-byte vectors.
 #include "decoder_ops.cuh"
 #include "mma_utils.cuh"
 #include "tc_utils.cuh"
@@ -27,8 +30,10 @@ constexpr int SC_SUB = 8;       // threads per channel (prompts)
 constexpr int SC_THREADS = SC_CH * SC_SUB;
 constexpr int SC_TT = 32;       // tokens per tile
 constexpr int SC_YP = 36;       // pitch of the output tile (floats)
-constexpr int ST_SUB = 4;       // threads per channel (decode step)
-constexpr int ST_THREADS = SC_CH * ST_SUB;
+constexpr int ST_WARPS = 4;     // decode step: a warp per sequence
+constexpr int ST_THREADS = SC_CH * ST_WARPS;
+constexpr int ST_BB = 8;        // sequences per CTA
+__host__ __device__ inline long long plane_index(int n, int c, int ip) { return ((long long)(n >> 2) * ip + c) * 4 + (n & 3); }
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
@@ -255,7 +260,7 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 #pragma unroll
     for (int i = 0; i < NS; ++i) {
         const int n = sub * NS + i;
-        A[i] = (live && n < a.state) ? a.A[(long long)c * a.np + n] : 0.0f;
+        A[i] = (live && n < a.state) ? a.A[plane_index(n, c, a.ip)] : 0.0f;
         if (PAIRS) A[i] *= LOG2E;
     }
     for (int i = tid; i < 2 * SC_TT * 2 * nb; i += SC_THREADS) bc[i] = 0.0f;  // columns behind np stay zero
@@ -263,11 +268,11 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     chain_wait();
     const int seg = blockIdx.y;
     const int start = a.seg_start[seg], len = a.seg_len[seg], pos0 = a.seg_pos0[seg], slot = a.seg_slot[seg];
-    float* state = a.S + ((long long)slot * a.ip + (live ? c : 0)) * a.np;
+    float* state = a.S + (long long)slot * a.ip * a.np;
 #pragma unroll
     for (int i = 0; i < NS; ++i) {
         const int n = sub * NS + i;
-        S[i] = (live && n < a.state && pos0 > 0) ? state[n] : 0.0f;
+        S[i] = (live && n < a.state && pos0 > 0) ? state[plane_index(n, c, a.ip)] : 0.0f;
     }
     const int pc = a.rp + 2 * a.np;
     const T* xz = static_cast<const T*>(a.xz);
@@ -382,31 +387,34 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
     if (live)
 #pragma unroll
         for (int i = 0; i < NS; ++i)
-            if (sub * NS + i < a.state) state[sub * NS + i] = S[i];
+            if (sub * NS + i < a.state) state[plane_index(sub * NS + i, c, a.ip)] = S[i];
     if (tid < SC_CH && c0 + tid < a.ip)
         carry_conv_state(static_cast<T*>(a.conv) + (long long)slot * (a.taps - 1) * a.ip, xz, c0 + tid, a.ip, a.taps, start, len, pos0);
 }
 
 // ---- decode step --------------------------------------------------------------------------------------------------
-// One token of BB (at most 8) sequences and 32 channels per CTA; the convolution has already moved its state on.  The step
-// sizes of the 32 channels x 8 sequences are one small product: bf16 models take it on the tensor cores (weights as the
-// 16-row operand, two tiles of channels x two halves of the rank over the four warps), f32 models with four threads per
-// channel.  The code is kept short: a launch fetches it cold.
-template <typename T, int NS, int BB>
+// One token of up to 8 sequences and 32 channels per CTA: lane = channel, a warp takes two sequences; the convolution has
+// already moved its state on.  The step sizes of the 32 channels x 8 sequences are one small product: bf16 models take it on
+// the tensor cores (weights as the 16-row operand, two tiles of channels x two halves of the rank over the four warps).
+// NP: planes of four states kept in registers, requested before the step sizes are known; 0 = any number, read when needed.
+template <typename T, int NP>
 __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
-    extern __shared__ __align__(16) float st_dyn[];  // [BB][B: np | C: np]; f32: [BB][proj columns]
+    extern __shared__ __align__(16) float st_dyn[];  // bf16: [8][B: np | C: np]; f32: [8][proj columns]
     __shared__ float dts[2][SC_CH][9];
     constexpr bool MMA = sizeof(T) == 2;
+    constexpr int R = ST_BB / ST_WARPS;  // sequences per warp
     chain_trigger();
-    const int tid = threadIdx.x, ch = tid / ST_SUB, sub = tid % ST_SUB, warp = tid >> 5, lane = tid & 31;
-    const int c0 = blockIdx.x * SC_CH, c = c0 + ch, cl = min(c, a.ip - 1);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int c0 = blockIdx.x * SC_CH, c = c0 + lane, cl = min(c, a.ip - 1);
     const bool live = c < a.ip;
-    const int s0 = blockIdx.y * BB, nb = min(BB, a.n_segs - s0);
+    const int s0 = blockIdx.y * ST_BB, nb = min(ST_BB, a.n_segs - s0);
     const int pc = a.rp + 2 * a.np, off = MMA ? a.rp : 0, sc = pc - off;  // columns of proj that go to shared memory
-    // constants of the channel, before the predecessor kernel has finished
-    float A[NS];
+    const int planes = a.np / 4;
+    const float4* Ap = reinterpret_cast<const float4*>(a.A) + cl;
+    float4 A[NP ? NP : 1];
+    if (NP > 0)
 #pragma unroll
-    for (int i = 0; i < NS; ++i) A[i] = sub * NS + i < a.state ? a.A[(long long)cl * a.np + sub * NS + i] : 0.0f;
+        for (int i = 0; i < NP; ++i) A[i] = i < planes ? Ap[(long long)i * a.ip] : make_float4(0.f, 0.f, 0.f, 0.f);
     const float bias = a.dt_b[cl], dv = a.D[cl];
     chain_wait();
     for (int i = tid; i < nb * (sc / 4); i += ST_THREADS) {
@@ -414,23 +422,23 @@ __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
         cp_async16(smem_u32(st_dyn + i * 4), a.proj + (long long)a.seg_start[s0 + b] * pc + off + v * 4, true);
     }
     cp_async_commit();
-    // the states are on their way while the step sizes are computed
-    float S[BB][NS];
+    float4 S[R][NP ? NP : 1];
+    float4* Sp[R];
+    bool fresh[R];
+    int tok[R];
+    T xv[R], zv[R];
 #pragma unroll
-    for (int b = 0; b < BB; ++b) {
-        const int sg = s0 + min(b, nb - 1);
-        const float* Sp = a.S + ((long long)a.seg_slot[sg] * a.ip + cl) * a.np + sub * NS;
-        const bool on = a.seg_pos0[sg] > 0;
-        if (NS % 4 == 0 && sub * NS + NS <= a.state) {
+    for (int q = 0; q < R; ++q) {
+        const int sg = s0 + min(q * ST_WARPS + warp, nb - 1);
+        tok[q] = a.seg_start[sg];
+        fresh[q] = a.seg_pos0[sg] == 0;
+        Sp[q] = reinterpret_cast<float4*>(a.S + (long long)a.seg_slot[sg] * a.ip * a.np) + cl;
+        if (NP > 0)
 #pragma unroll
-            for (int i = 0; i < NS / 4; ++i) {
-                const float4 v = on ? reinterpret_cast<const float4*>(Sp)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
-                S[b][4 * i] = v.x; S[b][4 * i + 1] = v.y; S[b][4 * i + 2] = v.z; S[b][4 * i + 3] = v.w;
-            }
-        } else {
-#pragma unroll
-            for (int i = 0; i < NS; ++i) S[b][i] = (on && sub * NS + i < a.state) ? Sp[i] : 0.0f;
-        }
+            for (int i = 0; i < NP; ++i)
+                S[q][i] = (i < planes && !fresh[q]) ? Sp[q][(long long)i * a.ip] : make_float4(0.f, 0.f, 0.f, 0.f);
+        xv[q] = static_cast<const T*>(a.xc)[(long long)tok[q] * a.ip + cl];
+        zv[q] = static_cast<const T*>(a.xz)[(long long)tok[q] * 2 * a.ip + a.ip + cl];
     }
     if constexpr (MMA) {
         const int mt = warp & 1, kh = warp >> 1, g = lane >> 2, kq = (lane & 3) * 8;
@@ -460,51 +468,41 @@ __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
     }
     cp_async_wait<0>();
     __syncthreads();
-    if constexpr (!MMA) {
-        const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
-        for (int b = 0; b < nb; ++b) {
-            float d = 0.0f;
-            for (int r = sub; r < a.rp; r += ST_SUB) d = fmaf(to_f32(w[r]), st_dyn[b * sc + r], d);
-            __syncwarp();
-            d += __shfl_xor_sync(0xffffffffu, d, 1);
-            d += __shfl_xor_sync(0xffffffffu, d, 2);
-            if (sub == 0) { dts[0][ch][b] = d; dts[1][ch][b] = 0.0f; }
-        }
-        __syncwarp();
-    }
-    const T* xz = static_cast<const T*>(a.xz);
 #pragma unroll
-    for (int b = 0; b < BB; ++b) {
+    for (int q = 0; q < R; ++q) {
+        const int b = q * ST_WARPS + warp;
         if (b >= nb) break;
-        const int t = a.seg_start[s0 + b];
-        const float x = to_f32(static_cast<const T*>(a.xc)[(long long)t * a.ip + cl]);
-        const float z = to_f32(xz[(long long)t * 2 * a.ip + a.ip + cl]);
-        const float dt = softplus_t<T>(dts[0][ch][b] + dts[1][ch][b] + bias), dx = dt * x;
-        const float* Bp = st_dyn + b * sc + (a.rp - off) + sub * NS;
-        const float* Cp = Bp + a.np;
-        float* Sp = a.S + ((long long)a.seg_slot[s0 + b] * a.ip + cl) * a.np + sub * NS;
+        float raw = 0.0f;
+        if constexpr (MMA) {
+            raw = dts[0][lane][b] + dts[1][lane][b];
+        } else {
+            const T* w = static_cast<const T*>(a.dt_w) + (long long)cl * a.rp;
+            for (int r = 0; r < a.rp; ++r) raw = fmaf(to_f32(w[r]), st_dyn[b * sc + r], raw);
+        }
+        const float x = to_f32(xv[q]), dt = softplus_t<T>(raw + bias), dx = dt * x;
+        const float4* Bp = reinterpret_cast<const float4*>(st_dyn + b * sc + (a.rp - off));
+        const float4* Cp = Bp + planes;
         float y = 0.0f;
+        auto plane = [&](int i, const float4& Ai, float4& s) {
+            const float4 B = Bp[i], C = Cp[i];
+            s.x = fmaf(decay<T>(dt * Ai.x), s.x, dx * B.x); y = fmaf(s.x, C.x, y);
+            s.y = fmaf(decay<T>(dt * Ai.y), s.y, dx * B.y); y = fmaf(s.y, C.y, y);
+            s.z = fmaf(decay<T>(dt * Ai.z), s.z, dx * B.z); y = fmaf(s.z, C.z, y);
+            s.w = fmaf(decay<T>(dt * Ai.w), s.w, dx * B.w); y = fmaf(s.w, C.w, y);
+            if (live) Sp[q][(long long)i * a.ip] = s;
+        };
+        if constexpr (NP > 0) {
 #pragma unroll
-        for (int i = 0; i < NS; ++i) {
-            if (sub * NS + i < a.state) {
-                S[b][i] = fmaf(decay<T>(dt * A[i]), S[b][i], dx * Bp[i]);
-                y = fmaf(S[b][i], Cp[i], y);
+            for (int i = 0; i < NP; ++i)
+                if (i < planes) plane(i, A[i], S[q][i]);
+        } else {
+#pragma unroll 2
+            for (int i = 0; i < planes; ++i) {
+                float4 s = fresh[q] ? make_float4(0.f, 0.f, 0.f, 0.f) : Sp[q][(long long)i * a.ip];
+                plane(i, Ap[(long long)i * a.ip], s);
             }
         }
-        if (live) {
-            if (NS % 4 == 0 && sub * NS + NS <= a.state) {
-#pragma unroll
-                for (int i = 0; i < NS / 4; ++i)
-                    reinterpret_cast<float4*>(Sp)[i] = make_float4(S[b][4 * i], S[b][4 * i + 1], S[b][4 * i + 2], S[b][4 * i + 3]);
-            } else {
-#pragma unroll
-                for (int i = 0; i < NS; ++i)
-                    if (sub * NS + i < a.state) Sp[i] = S[b][i];
-            }
-        }
-        y += __shfl_xor_sync(0xffffffffu, y, 1);
-        y += __shfl_xor_sync(0xffffffffu, y, 2);
-        if (sub == (b & 3) && live) static_cast<T*>(a.y)[(long long)t * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(z));
+        if (live) static_cast<T*>(a.y)[(long long)tok[q] * a.ip + c] = from_f32<T>(fmaf(dv, x, y) * silu_t<T>(to_f32(zv[q])));
     }
 }
 
@@ -563,20 +561,19 @@ static jsm_status scan_go(const ScanArgs& a, cudaStream_t st) {
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
-template <typename T, int NS>
+template <typename T, int NP>
 static jsm_status step_go(const ScanArgs& a, cudaStream_t st) {
-    constexpr int BB = NS <= 4 ? 8 : NS <= 8 ? 4 : NS <= 16 ? 2 : 1;
-    const size_t smem = (size_t)BB * (a.rp + 2 * a.np) * sizeof(float);
+    const size_t smem = (size_t)ST_BB * (2 * a.np + (sizeof(T) == 2 ? 0 : a.rp)) * sizeof(float);
     static bool attr_done = false;
     if (!attr_done) {
-        JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_step_kernel<T, NS, BB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_step_kernel<T, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         attr_done = true;
     }
-    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NS, BB>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + BB - 1) / BB), dim3(ST_THREADS), smem, st, a));
+    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NP>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + ST_BB - 1) / ST_BB), dim3(ST_THREADS), smem, st, a));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
-// the smallest instance whose threads hold a channel's states (per thread: state / 8 in prompts, state / 4 in a decode step)
+// the smallest instance whose threads hold a channel's states
 template <typename T>
 static jsm_status scan_dispatch(const ScanArgs& a, cudaStream_t st) {
     return a.state <= 8 ? scan_go<T, 1>(a, st) : a.state <= 16 ? scan_go<T, 2>(a, st) : a.state <= 24 ? scan_go<T, 3>(a, st)
@@ -584,8 +581,7 @@ static jsm_status scan_dispatch(const ScanArgs& a, cudaStream_t st) {
 }
 template <typename T>
 static jsm_status step_dispatch(const ScanArgs& a, cudaStream_t st) {
-    return a.state <= 8 ? step_go<T, 2>(a, st) : a.state <= 16 ? step_go<T, 4>(a, st) : a.state <= 24 ? step_go<T, 6>(a, st)
-         : a.state <= 32 ? step_go<T, 8>(a, st) : a.state <= 64 ? step_go<T, 16>(a, st) : step_go<T, 32>(a, st);
+    return a.np <= 8 ? step_go<T, 2>(a, st) : a.np <= 16 ? step_go<T, 4>(a, st) : a.np <= 32 ? step_go<T, 8>(a, st) : step_go<T, 0>(a, st);
 }
 
 jsm_status scan_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
