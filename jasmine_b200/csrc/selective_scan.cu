@@ -8,7 +8,7 @@
 // state lives in a slot: S and the last taps - 1 inputs of the convolution.  A segment that starts at position 0 starts from
 // zeros whatever the slot holds, so a slot needs no clearing when a new sequence takes it.
 //
-// Prompts: a CTA owns 32 channels of one segment and walks its tokens in tiles of 32 that cp.async brings into a two-stage
+// Prompts: a CTA owns 16 channels of one segment and walks its tokens in tiles of 32 that cp.async brings into a two-stage
 // ring; eight threads share a channel's states, so that the chain of dependent steps is one FMA per state and the partial
 // sums of eight tokens are exchanged with seven shuffles.  Decode: one thread per channel and sequence, eight sequences per
 // CTA; the states are requested first and arrive while the step sizes (a small projection) are computed.
@@ -25,13 +25,14 @@ namespace jsm {
 
 using tc::smem_u32;
 
-constexpr int SC_CH = 32;       // channels per CTA
+constexpr int SC_CH = 16;       // channels per CTA
 constexpr int SC_SUB = 8;       // threads per channel (prompts)
 constexpr int SC_THREADS = SC_CH * SC_SUB;
 constexpr int SC_TT = 32;       // tokens per tile
-constexpr int SC_YP = 36;       // pitch of the output tile (floats)
+constexpr int SC_YP = SC_CH + 4;  // pitch of the output tile (floats)
 constexpr int ST_WARPS = 4;     // decode step: a warp per sequence
-constexpr int ST_THREADS = SC_CH * ST_WARPS;
+constexpr int ST_CH = 32;       // channels per CTA: a lane each
+constexpr int ST_THREADS = ST_CH * ST_WARPS;
 constexpr int ST_BB = 8;        // sequences per CTA
 __host__ __device__ inline long long plane_index(int n, int c, int ip) { return ((long long)(n >> 2) * ip + c) * 4 + (n & 3); }
 
@@ -110,7 +111,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
 // one token, and the state moves on by it here (otherwise the scan does that, once every CTA has read the old state)
 constexpr int CONV_TOK = 8;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, T* state,
+__global__ void __launch_bounds__(256, 2) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, T* state,
                                                         const float* __restrict__ w, const float* __restrict__ b,
                                                         const int32_t* __restrict__ seg_start, const int32_t* __restrict__ seg_len,
                                                         const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ seg_slot, int ip,
@@ -400,12 +401,12 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
 template <typename T, int NP>
 __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float st_dyn[];  // bf16: [8][B: np | C: np]; f32: [8][proj columns]
-    __shared__ float dts[2][SC_CH][9];
+    __shared__ float dts[2][ST_CH][9];
     constexpr bool MMA = sizeof(T) == 2;
     constexpr int R = ST_BB / ST_WARPS;  // sequences per warp
     chain_trigger();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int c0 = blockIdx.x * SC_CH, c = c0 + lane, cl = min(c, a.ip - 1);
+    const int c0 = blockIdx.x * ST_CH, c = c0 + lane, cl = min(c, a.ip - 1);
     const bool live = c < a.ip;
     const int s0 = blockIdx.y * ST_BB, nb = min(ST_BB, a.n_segs - s0);
     const int pc = a.rp + 2 * a.np, off = MMA ? a.rp : 0, sc = pc - off;  // columns of proj that go to shared memory
@@ -569,7 +570,7 @@ static jsm_status step_go(const ScanArgs& a, cudaStream_t st) {
         JSM_CUDA_CHECK(cudaFuncSetAttribute(scan_step_kernel<T, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         attr_done = true;
     }
-    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NP>, dim3((a.ip + SC_CH - 1) / SC_CH, (a.n_segs + ST_BB - 1) / ST_BB), dim3(ST_THREADS), smem, st, a));
+    JSM_CUDA_CHECK(launch_chained(scan_step_kernel<T, NP>, dim3((a.ip + ST_CH - 1) / ST_CH, (a.n_segs + ST_BB - 1) / ST_BB), dim3(ST_THREADS), smem, st, a));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
