@@ -248,15 +248,15 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     } else {
         // ---- softmax / correction / epilogue: one thread per query row
         const int t = (warp - 2) / 4;       // query tile
-        const int j_begin = t ? lo[1] : lo[0], j_end = t ? n_tiles[1] : n_tiles[0];
+        const int j_begin = WIN ? lo[t] : 0, j_end = n_tiles[t];
         const int quad = warp & 3;          // TMEM lane quadrant this warp may access
         const int row = quad * 32 + lane;   // row in the tile = TMEM lane
         const int qi = q0 + t * FA_BM + row;
         const int qpos = qi + shift;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
-        const uint32_t s_addr = lane_addr + (t ? S_COL[1] : S_COL[0]), o_addr = lane_addr + (t ? O_COL[1] : O_COL[0]);
+        const uint32_t s_addr = lane_addr + S_COL[t], o_addr = lane_addr + O_COL[t];
         // (a finite start: a window can hide a whole key tile from some rows, whose weights are then 2^-inf = 0)
-        float m_ref = -1.0e30f, l = 0.0f;
+        float m_ref = WIN ? -1.0e30f : -INFINITY, l = 0.0f;
         bool ok = true;
         for (int j = j_begin; j < j_end && ok; ++j) {
             if (!mbar_wait(&s_full[t], (j - j_begin) & 1, &abort_flag, P.err, TC_TIMEOUT_ACC)) { ok = false; break; }
