@@ -86,7 +86,8 @@ def layer_residual(m, toks, sizes):
 ATTENTION = [dict(), dict(heads=1, dim=8, rot_dim=2, vdim=8, kv_rank=8, window=1), dict(heads=5, dim=9, rot_dim=6, vdim=13, kv_rank=17, window=7),
              dict(heads=2, dim=33, rot_dim=10, vdim=40, kv_rank=70, window=64), dict(heads=7, dim=24, rot_dim=40, vdim=24, kv_rank=130, window=65, base=300.0, scale=0.31),
              dict(heads=4, dim=48, rot_dim=16, vdim=64, kv_rank=272, window=128), dict(heads=33, dim=16, rot_dim=16, vdim=8, kv_rank=24, window=100),
-             dict(heads=2, dim=64, rot_dim=64, vdim=96, kv_rank=400, window=90), dict(heads=2, dim=130, rot_dim=30, vdim=128, kv_rank=64, window=500)]
+             dict(heads=2, dim=64, rot_dim=64, vdim=96, kv_rank=400, window=90), dict(heads=2, dim=130, rot_dim=30, vdim=128, kv_rank=64, window=500),
+             dict(heads=2, dim=200, rot_dim=32, vdim=140, kv_rank=530, window=70), dict(heads=2, dim=24, rot_dim=136, vdim=16, kv_rank=140, window=80)]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -309,11 +310,25 @@ def test_long_prompts_take_the_flash_kernel(kw, window):
     want = []
     zo.forward(cfg, zu.oracle_weights(w), toks, want)
     m = zu.build(cfg, w, "bfloat16")
-    for sizes in ([700], [129, 300, 271], [37, 400, 3, 260]):
+    for sizes in ([700], [129, 300, 271], [37, 400, 3, 260], [690] + [1] * 10):
         got = layer_residual(m, toks, sizes)[0]
         assert_close(got, want[0], 1.5 * BF16_RTOL, str(sizes))
         assert zu.error(got, want[0]) < 0.02
     m.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_one_kind_of_mixer_only(dtype):
+    """Models without attention (no pages) and without recurrence (no states)."""
+    for layers in ([zu.mamba(ff=24), zu.mamba(inner=24)], [zu.attention(ff=24), zu.attention(window=9)]):
+        cfg = zu.config(layers)
+        w = zu.random_weights(cfg, 51)
+        m = zu.build(cfg, w, dtype, max_batch=2, max_context=100)
+        for seed in (52, 53):
+            toks = zu.tokens(90, cfg["vocab"], seed)
+            assert zu.error(zu.run_portions(m, toks, [60, 2, 1]), want_logits(cfg, w, toks)) < TOL[dtype]
+        assert generate.generate(m, [toks[:5], toks[:30]], 4)[0]
+        m.close()
 
 
 def test_steps_longer_than_a_pass_are_cut():
