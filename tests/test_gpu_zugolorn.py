@@ -52,7 +52,7 @@ def test_norm_on_the_output_joins_the_residual(T, d):
     assert torch.equal(xb, xd.bfloat16())
 
 
-@pytest.mark.parametrize("vocab,pitch,cap", [(5, 8, 2.0), (72, 72, 15.0), (5003, 5008, 3.0), (40000, 40000, 0.0)])
+@pytest.mark.parametrize("vocab,pitch,cap", [(5, 8, 2.0), (72, 72, 5.0), (5003, 5008, 3.0), (40000, 40000, 0.0)])
 def test_capped_logits_and_their_maximum(vocab, pitch, cap):
     rng = np.random.default_rng(vocab)
     x = (4 * rng.standard_normal((3, pitch))).astype(np.float32)
