@@ -229,6 +229,10 @@ jsm_status jsm_rope_table(float* d_table, int mode, int d, float theta, int max_
 /* Rotate-half tables: (cos, sin) of m * base^(-2i/d) for pair i = (component i, component i + d/2) at position m, computed in
  * double precision.  d_table: F32 [max_pos, d/2, 2] (synchronous). */
 jsm_status jsm_rope_half_table(float* d_table, int d, double base, int max_pos);
+/* The same table with YaRN scaling of the frequencies (factor, original context, turns fast / slow) and cos, sin times
+ * 0.1 ln(factor) + 1; factor 0 = no scaling. */
+jsm_status jsm_rope_scaled_table(float* d_table, int d, double base, double factor, double original, double fast, double slow,
+                                 int max_pos);
 /* x, out: token-major [T, n_heads*d] (F32 or BF16); positions: I32 [T] or NULL (= t). */
 jsm_status jsm_rope_apply(const void* d_x, void* d_out, jsm_dtype dtype, const float* d_table, int d, int n_heads,
                           const int32_t* d_positions, int T, void* stream);
@@ -331,6 +335,9 @@ jsm_status jsm_add_norm(int kind, const void* d_h, const void* d_delta, void* d_
  * (d_x_bf16 or NULL).  y, x: F32 [T, d], d a multiple of 8. */
 jsm_status jsm_post_norm_add(const float* d_y, float* d_x, const float* d_gain, float eps, void* d_x_bf16, int T, int d,
                              void* stream);
+/* Norm of the sum: s = alpha * x + y, x <- s / sqrt(mean(s^2) + eps) * gain (otherwise as jsm_post_norm_add). */
+jsm_status jsm_sum_norm(const float* d_y, float* d_x, const float* d_gain, float eps, float alpha, void* d_x_bf16, int T, int d,
+                        void* stream);
 /* logits <- cap * tanh(logits / cap) in place (cap 0: unchanged) and the arg-max of every row (the first maximum).
  * d_keys U64 [rows], d_counters I32 [rows]: zero before the first call; the kernel leaves them zero. */
 jsm_status jsm_logits_finish(float* d_logits, int pitch, int rows, int vocab, float cap, uint64_t* d_keys, int32_t* d_counters,
@@ -485,7 +492,8 @@ jsm_status jsm_llama_step_bytes(jsm_model* m, uint64_t* weight_bytes, uint64_t* 
 /* ---- decoder with a list of layers (new; not in the reference) -----------------------------------------------------
  * Every layer names its mixer and the mixer's sizes, and optionally a feed-forward; the norm sits on the sublayer's output,
  *     x <- x + norm1(mixer(x)),   x <- x + norm2(ff(x)),      norm(y) = y / sqrt(mean(y^2) + eps) * w,
- * with an fp32 residual stream x.  Logits = final norm of x times the embedding table, through cap * tanh(l / cap).
+ * or on the sum, x <- norm1(alpha x + mixer(x)), with an fp32 residual stream x = embed_scale * embedding at the start.
+ * Logits = final norm of x times the embedding table, through cap * tanh(l / cap).
  * Mixers:
  *  latent attention  per head `dim` unrotated and `rot_dim` rotated query / key components (rotate-half pairs, base
  *                    rope_base) and values of `vdim`; keys and values are expanded from an RMS-normed latent of kv_rank
@@ -493,18 +501,36 @@ jsm_status jsm_llama_step_bytes(jsm_model* m, uint64_t* weight_bytes, uint64_t* 
  *  selective scan    input projection to (x, z) of `inner` channels, causal convolution of `taps` taps and silu on x,
  *                    then S <- exp(dt A) S + dt x B, y = C S + D x with `state` states per channel and a step size dt of
  *                    rank dt_rank, gated by silu(z).
- * Feed-forward: g = min(Wg x, limit), u = clamp(Wu x, -limit, limit), Wd (g * sigmoid(1.702 g) * (u + 1)).
+ *  attention         grouped queries (`heads` over `kv_heads`), biases on q, k and v, RMS norm of queries and keys per head,
+ *                    rotation of adjacent pairs on the first rot_dim components (YaRN scaling), a mask (all keys, the last
+ *                    `window`, or those of the query's own chunk of `window` positions), a learned sink per head in the
+ *                    softmax denominator, a sigmoid gate per head on the output.  kv_from = J: the keys and values of layer J.
+ *  linear attention  q, k, v through silu; S <- decay_h S + k v^T, o = S^T q; RMS norm over all heads, sigmoid gate.
+ *  delta rule        q, k (kv_heads) and v (heads) through a causal convolution of `taps` taps and silu, unit q and k;
+ *                    S <- g S, S <- S + beta k (v - S^T k)^T, o = S^T q / sqrt(dim); RMS norm per head, silu gate.
+ * Feed-forward: g = min(Wg x, limit), u = clamp(Wu x, -limit, limit), Wd (g * sigmoid(1.702 g) * (u + 1)), or
+ * Wd (gelu_tanh(Wg x) * (Wu x)).
  * Tensors: "embed" [vocab, d_model], "final.norm"; layer L: "lL.norm1", "lL.norm2" (with a feed-forward),
  * "lL.mlp.gate|up|down", and "lL.mix." + q, dkv, dkv.norm, uk, uv, o (latent attention) or in, conv, conv.b, x, dt, dt.b,
- * A_log, D, o (selective scan).  A layer with weights_of = J uses layer J's tensors and a cache or state of its own. */
-typedef enum jsm_mixer { JSM_MIXER_LATENT_ATTENTION = 0, JSM_MIXER_SELECTIVE_SCAN = 1 } jsm_mixer;
+ * A_log, D, o (selective scan), q, q.b, q.norm, k, k.b, k.norm, v, v.b, sink, g, o (attention; no k, v with kv_from), q, k, v, g,
+ * norm, o, decay (linear attention; decay F32 [heads], a constant of the configuration), q, k, v (each with .conv), b, a, A_log,
+ * dt_bias, norm, g, o (delta rule).  A layer with weights_of = J uses layer J's tensors and a cache or state of its own. */
+typedef enum jsm_mixer {
+    JSM_MIXER_LATENT_ATTENTION = 0, JSM_MIXER_SELECTIVE_SCAN = 1, JSM_MIXER_ATTENTION = 2, JSM_MIXER_LINEAR_ATTENTION = 3, JSM_MIXER_DELTA = 4
+} jsm_mixer;
+typedef enum jsm_mask { JSM_MASK_FULL = 0, JSM_MASK_WINDOW = 1, JSM_MASK_CHUNK = 2 } jsm_mask;
+typedef enum jsm_ff { JSM_FF_CLAMPED_GLU = 0, JSM_FF_GELU_GLU = 1 } jsm_ff;
+typedef enum jsm_norm_place { JSM_NORM_OUTPUT = 0, JSM_NORM_SUM = 1 } jsm_norm_place;
 typedef struct jsm_layer_config {
     int32_t mixer, weights_of;                         /* weights_of: -1 = own tensors */
-    int32_t heads, dim, rot_dim, vdim, kv_rank, window; /* latent attention */
-    int32_t inner, state, dt_rank, taps;               /* selective scan */
+    int32_t heads, dim, rot_dim, vdim, kv_rank, window; /* attention, recurrences; window: size of the mask */
+    int32_t inner, state, dt_rank, taps;               /* selective scan; taps also of the delta rule */
     int32_t ff;                                        /* 0 = no feed-forward */
     float ff_limit;
     double scale, rope_base;
+    int32_t kv_heads, kv_from;                         /* key / value heads (delta rule: query / key heads); -1 = own keys and values */
+    int32_t mask, ff_kind;                             /* jsm_mask (attention), jsm_ff */
+    double rope_factor, rope_original, rope_fast, rope_slow; /* attention: YaRN scaling, factor 0 = none */
 } jsm_layer_config;
 typedef struct jsm_decoder_config {
     int32_t n_layers, d_model, vocab;
@@ -513,6 +539,9 @@ typedef struct jsm_decoder_config {
     int32_t max_step_tokens; /* tokens of one pass; longer steps are cut into passes */
     int32_t n_pages;         /* cache pages of 64 positions; 0 = max_batch full contexts */
     float norm_eps, logit_softcap; /* logit_softcap 0 = no cap */
+    int32_t norm_place;            /* jsm_norm_place */
+    float residual_scale;          /* alpha of JSM_NORM_SUM */
+    float embed_scale;             /* factor on the embedding; 0 = 1 */
 } jsm_decoder_config;
 typedef struct jsm_decoder jsm_decoder;
 

@@ -56,17 +56,23 @@ class LayerConfig(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("weights_of", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32),
                 ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("kv_rank", C.c_int32), ("window", C.c_int32),
                 ("inner", C.c_int32), ("state", C.c_int32), ("dt_rank", C.c_int32), ("taps", C.c_int32),
-                ("ff", C.c_int32), ("ff_limit", C.c_float), ("scale", C.c_double), ("rope_base", C.c_double)]
+                ("ff", C.c_int32), ("ff_limit", C.c_float), ("scale", C.c_double), ("rope_base", C.c_double),
+                ("kv_heads", C.c_int32), ("kv_from", C.c_int32), ("mask", C.c_int32), ("ff_kind", C.c_int32),
+                ("rope_factor", C.c_double), ("rope_original", C.c_double), ("rope_fast", C.c_double), ("rope_slow", C.c_double)]
 
 
 class DecoderConfig(C.Structure):
     _fields_ = [("n_layers", C.c_int32), ("d_model", C.c_int32), ("vocab", C.c_int32), ("dtype", C.c_int32),
                 ("max_batch", C.c_int32), ("max_context", C.c_int32), ("max_step_tokens", C.c_int32), ("n_pages", C.c_int32),
-                ("norm_eps", C.c_float), ("logit_softcap", C.c_float)]
+                ("norm_eps", C.c_float), ("logit_softcap", C.c_float), ("norm_place", C.c_int32), ("residual_scale", C.c_float),
+                ("embed_scale", C.c_float)]
 
 
-# jsm_mixer
-MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN = 0, 1
+# jsm_mixer, jsm_mask, jsm_ff, jsm_norm_place
+MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN, MIXER_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_DELTA = 0, 1, 2, 3, 4
+MASK_FULL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
+FF_CLAMPED_GLU, FF_GELU_GLU = 0, 1
+NORM_OUTPUT, NORM_SUM = 0, 1
 
 # every symbol include/jasmine_b200.h declares: (restype, argtypes)
 _vp, _i, _f, _sz, _u64, _i64 = C.c_void_p, C.c_int, C.c_float, C.c_size_t, C.c_uint64, C.c_int64
@@ -101,9 +107,11 @@ SYMBOLS = {
     "jsm_linear_bf16_packed_chained": (_i, [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
     "jsm_linear_bf16_packed_glu": (_i, [_vp, _vp, _f, _f, _vp, _i, _i, _i, _vp]),
     "jsm_post_norm_add": (_i, [_vp, _vp, _vp, _f, _vp, _i, _i, _vp]),
+    "jsm_sum_norm": (_i, [_vp, _vp, _vp, _f, _f, _vp, _i, _i, _vp]),
     "jsm_logits_finish": (_i, [_vp, _i, _i, _i, _f, _vp, _vp, _vp, _vp]),
     "jsm_rope_table": (_i, [_vp, _i, _i, _f, _i, _vp]),
     "jsm_rope_half_table": (_i, [_vp, _i, C.c_double, _i]),
+    "jsm_rope_scaled_table": (_i, [_vp, _i, C.c_double, C.c_double, C.c_double, C.c_double, C.c_double, _i]),
     "jsm_rope_apply": (_i, [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp]),
     "jsm_rope_apply_qk": (_i, [_vp, _vp, _i, _vp, _vp, _i, _i, _vp, _i, _vp, _i, _vp]),
     "jsm_attn_prefill": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _i, _vp]),
@@ -309,6 +317,13 @@ def post_norm_add(y, x, gain, eps, x_bf16=None):
     """x += rms_norm(y) * gain in place, optional bf16 copy of x (jsm_post_norm_add)."""
     check(lib().jsm_post_norm_add(y.data_ptr(), x.data_ptr(), gain.data_ptr(), eps, x_bf16.data_ptr() if x_bf16 is not None else None,
                                   y.shape[0], y.shape[1], stream_ptr()))
+    return x
+
+
+def sum_norm(y, x, gain, eps, alpha, x_bf16=None):
+    """x <- rms_norm(alpha * x + y) * gain in place, optional bf16 copy of x (jsm_sum_norm)."""
+    check(lib().jsm_sum_norm(y.data_ptr(), x.data_ptr(), gain.data_ptr(), eps, alpha, x_bf16.data_ptr() if x_bf16 is not None else None,
+                             y.shape[0], y.shape[1], stream_ptr()))
     return x
 
 

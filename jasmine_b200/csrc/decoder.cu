@@ -1,12 +1,13 @@
-// Decoder whose layers are a list: every layer names its mixer (latent attention over a sliding window, or a selective
-// scan), the mixer's sizes, and an optional gated feed-forward.  The norm sits on the sublayer's output,
+// Decoder whose layers are a list: every layer names its mixer (latent attention, grouped-query attention, a selective scan, a
+// decayed sum or the delta rule), the mixer's sizes, and an optional gated feed-forward.  The norm sits on the sublayer's output,
 //     x <- x + norm1(mixer(x)),   x <- x + norm2(ff(x)),
-// the residual stream x is fp32, the logits come from the embedding table and pass through a soft cap.  A layer may use the
-// weights of an earlier one; its cache or state is always its own.
+// or on the sum, x <- norm1(alpha x + mixer(x)); the residual stream x is fp32, the logits come from the embedding table and
+// may pass through a soft cap.  A layer may use the weights of an earlier one with a cache or state of its own, and an
+// attention layer the keys and values of an earlier one.
 //
 // Serving follows the paged LLaMA runner (llama.cu, paged_rows.cuh): the active sequences occupy the batch rows
-// 0 .. n_active-1, latent-cache pages of 64 positions come from one pool (all attention layers share the block table),
-// pages that no window reaches any more go back to the pool, and every sequence owns one recurrent-state slot.  One step
+// 0 .. n_active-1, cache pages of 64 positions come from one pool (all attention layers share the block table),
+// pages that no mask reaches any more go back to the pool, and every sequence owns one recurrent-state slot.  One step
 // function runs everything: a step brings tokens of any number of rows - a prompt, a portion of one, one token each - and
 // is cut into passes of at most max_step_tokens.  A pass whose rows bring one token each replays a CUDA graph.
 //
@@ -40,13 +41,28 @@ struct DecLayer {
     jsm_layer_config c;
     LatentDims ld{};
     ScanDims sd{};
+    AttnDims ad{};
+    RecDims rd{};
     const float *norm1 = nullptr, *norm2 = nullptr;
-    Proj qd, expand, in, xp, dt, out;  // latent: queries + down projection, key / value expansion; scan: input, [dt B C], dt; both: output
+    Proj qd, expand, in, xp, dt, out;  // latent: queries + down projection, key / value expansion; scan: input, [dt B C], dt; all: output
+                                       // attention: qd = [q | gates | k | v]; recurrences: in = [q | k | v | z], xp = [b | a]
     Proj gate, up, down;               // bf16: gate holds the gate / up pairs
     LatentWeights lw{};
     ScanWeights sw{};
     LatentCache cache{};
     ScanState state{};
+    AttnWeights aw{};
+    AttnCache ac{};
+    RecWeights rw{};
+    RecState rs{};
+    bool is_attention() const { return c.mixer == JSM_MIXER_LATENT_ATTENTION || c.mixer == JSM_MIXER_ATTENTION; }
+    bool is_recurrence() const { return c.mixer == JSM_MIXER_LINEAR_ATTENTION || c.mixer == JSM_MIXER_DELTA; }
+    bool own_kv() const { return c.kv_from < 0; }
+    // rows per token and rows per tile of the tensor-core attention kernels
+    std::pair<int, int> tiling(bool decode) const {
+        return c.mixer == JSM_MIXER_LATENT_ATTENTION ? std::make_pair(ld.H, LATENT_TILE_ROWS) : std::make_pair(ad.H / ad.G, attn_tile_rows(ad, decode));
+    }
+    KeyMask key_mask() const { return c.mixer == JSM_MIXER_LATENT_ATTENTION ? KeyMask{JSM_MASK_WINDOW, c.window} : ad.mask; }
     int ffp() const { return pad8(c.ff); }
 };
 
@@ -74,12 +90,12 @@ struct jsm_decoder {
     const float* final_norm = nullptr;
     jsm::PagedRows rows;
     std::vector<int> slot_of_row, free_slots;
-    int wp = 0, vp = 0, cap_rows = 0, max_window = 0, kv_rows = 0;
+    int wp = 0, vp = 0, cap_rows = 0, kv_rows = 0;
     bool has_attention = false;
     cudaStream_t own_stream = nullptr;
     std::vector<void*> allocs;
     // activations of one pass
-    float *x = nullptr, *y = nullptr, *wide = nullptr, *proj = nullptr, *dt_raw = nullptr, *gate32 = nullptr, *logits = nullptr, *part = nullptr;
+    float *x = nullptr, *y = nullptr, *wide = nullptr, *proj = nullptr, *dt_raw = nullptr, *gate32 = nullptr, *head_gate = nullptr, *logits = nullptr, *part = nullptr;
     void *xa = nullptr, *q = nullptr, *q_lat = nullptr, *o_lat = nullptr, *att = nullptr, *xz = nullptr, *xc = nullptr, *dt_op = nullptr,
          *scan_y = nullptr, *act = nullptr, *head_in = nullptr, *gathered = nullptr, *expanded = nullptr;
     size_t part_floats = 0;
@@ -87,6 +103,7 @@ struct jsm_decoder {
     size_t ws_floats = 0;
     int* counters = nullptr;
     int n_counters = 0;
+    int* attn_ctrs = nullptr;
     unsigned long long* keys = nullptr;
     int32_t *key_ctrs = nullptr, *next_dev = nullptr, *meta = nullptr, *h_meta = nullptr;
     size_t meta_cap = 0;
@@ -309,6 +326,152 @@ static jsm_status build_scan(jsm_decoder* m, DecLayer& L, const std::string& pre
     return JSM_OK;
 }
 
+// rows [n heads x dim] of a tensor at a pitch of `pitch` rows per head, from row r0 on
+static void put_heads(HostMatrix& h, int r0, const HostTensor& t, int n, int dim, int pitch) {
+    for (int i = 0; i < n; ++i)
+        for (int j = 0; j < dim; ++j) h.put_row(r0 + i * pitch + j, t, i * dim + j);
+}
+// a vector [n heads x dim] (or a column of a matrix) at a pitch per head
+static jsm_status upload_heads(jsm_decoder* m, const HostTensor& t, int n, int dim, int pitch, const float** out) {
+    HostTensor p;
+    p.rows = n * pitch; p.cols = 1;
+    p.v.assign((size_t)n * pitch, 0.0f);
+    for (int i = 0; i < n; ++i)
+        for (int j = 0; j < dim; ++j) p.v[(size_t)i * pitch + j] = t.at((long long)i * dim + j);
+    return upload_vec(m, p, pad8(n * pitch), out);
+}
+
+static jsm_status build_attention(jsm_decoder* m, DecLayer& L, const std::string& pre) {
+    const AttnDims& d = L.ad;
+    const int D = m->c.d_model, qh = d.qh(), vh = pad8(d.vdim);
+    const bool kv = L.own_kv();
+    const HostTensor *q, *g, *k = nullptr, *v = nullptr, *o, *t;
+    DEC_TRY(want_tensor(m, pre + "mix.q", d.H * d.dim, D, &q));
+    DEC_TRY(want_tensor(m, pre + "mix.g", d.H, D, &g));
+    DEC_TRY(want_tensor(m, pre + "mix.o", D, d.H * d.vdim, &o));
+    if (kv) {
+        DEC_TRY(want_tensor(m, pre + "mix.k", d.G * d.dim, D, &k));
+        DEC_TRY(want_tensor(m, pre + "mix.v", d.G * d.vdim, D, &v));
+    }
+    {
+        HostMatrix h(m->f32, d.wide_cols(kv), m->wp);
+        put_heads(h, 0, *q, d.H, d.dim, qh);
+        for (int i = 0; i < d.H; ++i) h.put_row(d.q_cols() + i, *g, i);
+        if (kv) {
+            put_heads(h, d.q_cols() + pad8(d.H), *k, d.G, d.dim, qh);
+            put_heads(h, d.q_cols() + pad8(d.H) + d.G * qh, *v, d.G, d.vdim, vh);
+        }
+        DEC_TRY(upload_proj(m, h, &L.qd));
+    }
+    {
+        HostMatrix h(m->f32, m->wp, d.out_cols());
+        for (int j = 0; j < D; ++j) h.put_row(j, *o, j);
+        DEC_TRY(upload_proj(m, h, &L.out));
+    }
+    DEC_TRY(want_tensor(m, pre + "mix.q.b", d.H * d.dim, 1, &t));
+    DEC_TRY(upload_heads(m, *t, d.H, d.dim, qh, &L.aw.q_bias));
+    DEC_TRY(want_tensor(m, pre + "mix.q.norm", d.dim, 1, &t));
+    DEC_TRY(upload_vec(m, *t, qh, &L.aw.q_norm));
+    DEC_TRY(want_tensor(m, pre + "mix.sink", d.H, 1, &t));
+    DEC_TRY(upload_vec(m, *t, pad8(d.H), &L.aw.sink));
+    if (kv) {
+        DEC_TRY(want_tensor(m, pre + "mix.k.b", d.G * d.dim, 1, &t));
+        DEC_TRY(upload_heads(m, *t, d.G, d.dim, qh, &L.aw.k_bias));
+        DEC_TRY(want_tensor(m, pre + "mix.k.norm", d.dim, 1, &t));
+        DEC_TRY(upload_vec(m, *t, qh, &L.aw.k_norm));
+        DEC_TRY(want_tensor(m, pre + "mix.v.b", d.G * d.vdim, 1, &t));
+        DEC_TRY(upload_heads(m, *t, d.G, d.vdim, vh, &L.aw.v_bias));
+    }
+    return JSM_OK;
+}
+
+static jsm_status build_recurrence(jsm_decoder* m, DecLayer& L, const std::string& pre) {
+    const RecDims& d = L.rd;
+    const int D = m->c.d_model, kp = d.kp(), vp = d.vp(), cc = d.conv_cols();
+    const HostTensor *q, *k, *v, *z, *o, *t;
+    DEC_TRY(want_tensor(m, pre + "mix.q", d.G * d.dk, D, &q));
+    DEC_TRY(want_tensor(m, pre + "mix.k", d.G * d.dk, D, &k));
+    DEC_TRY(want_tensor(m, pre + "mix.v", d.H * d.dv, D, &v));
+    DEC_TRY(want_tensor(m, pre + "mix.g", d.H * d.dv, D, &z));
+    DEC_TRY(want_tensor(m, pre + "mix.o", D, d.H * d.dv, &o));
+    {
+        HostMatrix h(m->f32, d.raw_cols(), m->wp);
+        put_heads(h, 0, *q, d.G, d.dk, kp);
+        put_heads(h, d.G * kp, *k, d.G, d.dk, kp);
+        put_heads(h, 2 * d.G * kp, *v, d.H, d.dv, vp);
+        put_heads(h, cc, *z, d.H, d.dv, vp);
+        DEC_TRY(upload_proj(m, h, &L.in));
+    }
+    {
+        HostMatrix h(m->f32, m->wp, d.out_cols());
+        for (int r = 0; r < D; ++r)
+            for (int i = 0; i < d.H; ++i)
+                for (int j = 0; j < d.dv; ++j) h.set(r, i * vp + j, o->at((long long)r * d.H * d.dv + i * d.dv + j));
+        DEC_TRY(upload_proj(m, h, &L.out));
+    }
+    {
+        HostMatrix c(true, d.taps, cc);
+        if (d.delta) {
+            const std::pair<const char*, int> parts[3] = {{"mix.q.conv", d.G * d.dk}, {"mix.k.conv", d.G * d.dk}, {"mix.v.conv", d.H * d.dv}};
+            for (int p = 0; p < 3; ++p) {
+                DEC_TRY(want_tensor(m, pre + parts[p].first, parts[p].second, d.taps, &t));
+                const int dim = p < 2 ? d.dk : d.dv, pitch = p < 2 ? kp : vp, at = p * d.G * kp;
+                for (int j = 0; j < parts[p].second; ++j)
+                    for (int n = 0; n < d.taps; ++n) c.set(n, at + j / dim * pitch + j % dim, t->at((long long)j * d.taps + n));
+            }
+        } else {
+            for (int j = 0; j < cc; ++j) c.set(0, j, 1.0f);  // no convolution: its activation alone
+        }
+        void* p = nullptr;
+        DEC_TRY(upload_plain(m, c, &p));
+        L.rw.conv = static_cast<float*>(p);
+    }
+    if (!d.delta) {
+        DEC_TRY(want_tensor(m, pre + "mix.norm", d.H * d.dv, 1, &t));
+        DEC_TRY(upload_heads(m, *t, d.H, d.dv, vp, &L.rw.norm));
+        DEC_TRY(want_tensor(m, pre + "mix.decay", d.H, 1, &t));
+        HostTensor lg;
+        lg.rows = d.H; lg.cols = 1;
+        for (int i = 0; i < d.H; ++i) {
+            const float g = t->at(i);
+            if (!(g >= 0.0f && g <= 1.0f)) JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder: '%smix.decay' holds %g", pre.c_str(), g);
+            lg.v.push_back(g > 0.0f ? (float)log((double)g) : -1.0e30f);
+        }
+        DEC_TRY(upload_vec(m, *t, pad8(d.H), &L.rw.decay));
+        return upload_vec(m, lg, pad8(d.H), &L.rw.log_decay);
+    }
+    DEC_TRY(want_tensor(m, pre + "mix.norm", d.dv, 1, &t));
+    DEC_TRY(upload_vec(m, *t, vp, &L.rw.norm));
+    DEC_TRY(want_tensor(m, pre + "mix.dt_bias", d.H, 1, &t));
+    DEC_TRY(upload_vec(m, *t, pad8(d.H), &L.rw.dt_bias));
+    DEC_TRY(want_tensor(m, pre + "mix.A_log", d.H, 1, &t));
+    HostTensor A;
+    A.rows = d.H; A.cols = 1;
+    for (int i = 0; i < d.H; ++i) A.v.push_back((float)-exp((double)t->at(i)));
+    DEC_TRY(upload_vec(m, A, pad8(d.H), &L.rw.A));
+    const HostTensor *b, *a;
+    DEC_TRY(want_tensor(m, pre + "mix.b", d.H, D, &b));
+    DEC_TRY(want_tensor(m, pre + "mix.a", d.H, D, &a));
+    HostMatrix h(m->f32, d.ba_cols(), m->wp);
+    for (int i = 0; i < d.H; ++i) {
+        h.put_row(i, *b, i);
+        h.put_row(d.ba_cols() / 2 + i, *a, i);
+    }
+    DEC_TRY(upload_proj(m, h, &L.xp));
+    if (!m->f32) DEC_TRY(upload_plain(m, h, &L.xp.rows));
+    L.rw.ba = m->f32 ? (void*)L.xp.w32 : L.xp.rows;
+    return JSM_OK;
+}
+
+static jsm_status build_mixer(jsm_decoder* m, DecLayer& L, const std::string& pre) {
+    switch (L.c.mixer) {
+        case JSM_MIXER_LATENT_ATTENTION: return build_latent(m, L, pre);
+        case JSM_MIXER_SELECTIVE_SCAN: return build_scan(m, L, pre);
+        case JSM_MIXER_ATTENTION: return build_attention(m, L, pre);
+        default: return build_recurrence(m, L, pre);
+    }
+}
+
 static jsm_status build_ff(jsm_decoder* m, DecLayer& L, const std::string& pre) {
     const int D = m->c.d_model, F = L.c.ff, fp = L.ffp();
     const HostTensor *g, *u, *w;
@@ -332,7 +495,7 @@ static jsm_status build_ff(jsm_decoder* m, DecLayer& L, const std::string& pre) 
 
 // Y = X . W^T; X act [T][x_stride], Y f32 (out_f32) or act [T][N]
 static jsm_status linear(jsm_decoder* m, const Proj& p, const void* X, long long x_stride, void* Y, bool out_f32, int T, cudaStream_t st,
-                         float glu_limit = 0.0f) {
+                         float glu_limit = 0.0f, int glu = LIN_CLAMPED_GLU) {
     if (m->f32) {
         jsm_mat A{const_cast<void*>(X), T, p.K, x_stride, 1, JSM_F32};
         jsm_mat B{p.w32, p.K, p.N, 1, p.K, JSM_F32};
@@ -341,7 +504,7 @@ static jsm_status linear(jsm_decoder* m, const Proj& p, const void* X, long long
     }
     PackedArgs a;
     a.Wp = p.packed; a.bias = nullptr; a.R = nullptr; a.out_f32 = out_f32;
-    a.epilogue = p.paired ? LIN_CLAMPED_GLU : LIN_NONE;
+    a.epilogue = p.paired ? glu : LIN_NONE;
     a.glu_alpha = GLU_ALPHA; a.glu_limit = glu_limit;
     a.N = p.N; a.K = p.K; a.x_row_stride = x_stride;
     a.ws = m->ws; a.ws_floats = m->ws_floats; a.counters = m->counters; a.n_counters = m->n_counters;
@@ -380,7 +543,7 @@ struct Pass {
     const int32_t* want = nullptr;
     int n_want = 0;
     bool decode = false;       // one token per segment
-    std::map<int, TileList> tiles_short, tiles_all;  // per head count
+    std::map<std::pair<int, int>, TileList> tiles_short, tiles_all;  // per (rows per token, rows per tile)
     int32_t* meta = nullptr;
 };
 
@@ -390,7 +553,7 @@ static jsm_status latent_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaS
     const void* xin = m->f32 ? m->x : m->xa;
     DEC_TRY(linear(m, L.qd, xin, m->wp, m->wide, true, T, st));
     const bool flash = L.expand.packed != nullptr && P.n_flash > 0;
-    const TileList& tl = (flash ? P.tiles_short : P.tiles_all).at(d.H);
+    const TileList& tl = (flash ? P.tiles_short : P.tiles_all).at(L.tiling(P.decode));
     DEC_TRY(latent_prep_launch(m->f32, m->wide, d, L.lw, m->c.norm_eps, L.cache, P.tk, m->q, tl.n > 0 ? m->q_lat : nullptr, st));
     if (tl.n > 0) {
         LatentTiles t;
@@ -434,26 +597,81 @@ static jsm_status scan_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaStr
     return linear(m, L.out, m->scan_y, d.ip(), m->y, true, T, st);
 }
 
+static jsm_status attention_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaStream_t st) {
+    const AttnDims& d = L.ad;
+    const int T = P.tk.T;
+    DEC_TRY(linear(m, L.qd, m->f32 ? m->x : m->xa, m->wp, m->wide, true, T, st));
+    DEC_TRY(attn_prep_launch(m->f32, m->wide, d, L.aw, m->c.norm_eps, L.ac, L.own_kv(), P.tk, m->q, m->head_gate, st));
+    const bool flash = !m->f32 && P.n_flash > 0 && attn_flash_usable(d);
+    const std::pair<int, int> shape = L.tiling(P.decode);
+    const TileList& tl = (flash ? P.tiles_short : P.tiles_all).at(shape);
+    if (tl.n > 0) {
+        const AttnTiles t{P.meta + tl.seg_off, P.meta + tl.r0_off, tl.n, shape.second, 0, tl.tokens, d.mask.reach(m->c.max_context)};
+        DEC_TRY(attn_paged_launch(m->f32, d, L.aw, L.ac, P.tk, t, m->q, m->head_gate, AttnScratch{m->part, m->part_floats, m->attn_ctrs, attn_counters()},
+                                  m->att, st));
+    }
+    if (flash)
+        for (size_t i = P.segs.size() - P.n_flash; i < P.segs.size(); ++i) {
+            const PassSeg& s = P.segs[i];
+            DEC_TRY(attn_flash_launch(d, L.aw, L.ac, s.row, s.pos0, s.len, static_cast<const __nv_bfloat16*>(m->q) + (long long)P.starts[i] * d.q_cols(),
+                                      m->head_gate + (long long)P.starts[i] * d.H, static_cast<__nv_bfloat16*>(m->att) + (long long)P.starts[i] * d.out_cols(),
+                                      st));
+        }
+    return linear(m, L.out, m->att, d.out_cols(), m->y, true, T, st);
+}
+
+static jsm_status recurrence_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaStream_t st) {
+    const RecDims& d = L.rd;
+    const int T = P.tk.T;
+    const void* xin = m->f32 ? m->x : m->xa;
+    DEC_TRY(linear(m, L.in, xin, m->wp, m->xz, false, T, st));
+    DEC_TRY(short_conv_launch(m->f32, m->xz, d.raw_cols(), d.conv_cols(), d.taps, L.rw.conv, nullptr, L.rs.conv, P.tk, m->xc, P.decode, st));
+    if (P.decode) {
+        DEC_TRY(rec_step_launch(m->f32, d, L.rw, L.rs, m->c.norm_eps, P.tk, m->xz, m->xc, xin, m->wp, m->scan_y, st));
+    } else {
+        if (d.delta) DEC_TRY(linear(m, L.xp, xin, m->wp, m->proj, true, T, st));
+        DEC_TRY(rec_scan_launch(m->f32, d, L.rw, L.rs, m->c.norm_eps, P.tk, m->xz, m->xc, m->proj, m->scan_y, st));
+        DEC_TRY(short_conv_carry_launch(m->f32, m->xz, d.raw_cols(), d.conv_cols(), d.taps, L.rs.conv, P.tk, st));
+    }
+    return linear(m, L.out, m->scan_y, d.out_cols(), m->y, true, T, st);
+}
+
+static jsm_status run_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, cudaStream_t st) {
+    switch (L.c.mixer) {
+        case JSM_MIXER_LATENT_ATTENTION: return latent_mixer(m, L, P, st);
+        case JSM_MIXER_SELECTIVE_SCAN: return scan_mixer(m, L, P, st);
+        case JSM_MIXER_ATTENTION: return attention_mixer(m, L, P, st);
+        default: return recurrence_mixer(m, L, P, st);
+    }
+}
+
+// a sublayer's output y joins the residual stream
+static jsm_status join_residual(jsm_decoder* m, const float* gain, int T, cudaStream_t st) {
+    const jsm_decoder_config& c = m->c;
+    return c.norm_place == JSM_NORM_SUM ? sum_norm_launch(m->y, m->x, gain, c.norm_eps, c.residual_scale, m->xa, T, c.d_model, m->wp, st)
+                                        : post_norm_add_launch(m->y, m->x, gain, c.norm_eps, m->xa, T, c.d_model, m->wp, st);
+}
+
 static jsm_status run_layers(jsm_decoder* m, const Pass& P, cudaStream_t st) {
     const int T = P.tk.T, D = m->c.d_model, wp = m->wp;
-    const float eps = m->c.norm_eps;
-    DEC_TRY(embed_residual_launch(m->f32, m->embed, P.tk.ids, m->x, m->xa, T, wp, st));
+    DEC_TRY(embed_residual_launch(m->f32, m->embed, P.tk.ids, m->c.embed_scale, m->x, m->xa, T, wp, st));
     for (size_t l = 0; l < m->layers.size(); ++l) {
         DecLayer& L = m->layers[l];
-        DEC_TRY(L.c.mixer == JSM_MIXER_LATENT_ATTENTION ? latent_mixer(m, L, P, st) : scan_mixer(m, L, P, st));
-        DEC_TRY(post_norm_add_launch(m->y, m->x, L.norm1, eps, m->xa, T, D, wp, st));
+        DEC_TRY(run_mixer(m, L, P, st));
+        DEC_TRY(join_residual(m, L.norm1, T, st));
         if (L.c.ff > 0) {
             const void* xin = m->f32 ? m->x : m->xa;
             if (m->f32) {
                 float* up = m->gate32 + (size_t)m->c.max_step_tokens * L.ffp();
                 DEC_TRY(linear(m, L.gate, xin, wp, m->gate32, true, T, st));
                 DEC_TRY(linear(m, L.up, xin, wp, up, true, T, st));
-                DEC_TRY(clamped_glu_f32_launch(m->gate32, up, static_cast<float*>(m->act), GLU_ALPHA, L.c.ff_limit, (long long)T * L.ffp(), st));
+                if (L.c.ff_kind == JSM_FF_GELU_GLU) DEC_TRY(gelu_glu_f32_launch(m->gate32, up, static_cast<float*>(m->act), (long long)T * L.ffp(), st));
+                else DEC_TRY(clamped_glu_f32_launch(m->gate32, up, static_cast<float*>(m->act), GLU_ALPHA, L.c.ff_limit, (long long)T * L.ffp(), st));
             } else {
-                DEC_TRY(linear(m, L.gate, xin, wp, m->act, false, T, st, L.c.ff_limit));
+                DEC_TRY(linear(m, L.gate, xin, wp, m->act, false, T, st, L.c.ff_limit, L.c.ff_kind == JSM_FF_GELU_GLU ? LIN_GELU_GLU : LIN_CLAMPED_GLU));
             }
             DEC_TRY(linear(m, L.down, m->act, L.ffp(), m->y, true, T, st));
-            DEC_TRY(post_norm_add_launch(m->y, m->x, L.norm2, eps, m->xa, T, D, wp, st));
+            DEC_TRY(join_residual(m, L.norm2, T, st));
         }
         if (m->tap)
             JSM_CUDA_CHECK(cudaMemcpy2DAsync(m->tap + l * (size_t)T * D, sizeof(float) * D, m->x, sizeof(float) * wp, sizeof(float) * D, T,
@@ -467,6 +685,14 @@ static jsm_status run_head(jsm_decoder* m, const Pass& P, int w0, int n, cudaStr
     DEC_TRY(final_norm_launch(m->f32, m->x, P.want + w0, m->final_norm, m->c.norm_eps, m->head_in, n, m->c.d_model, m->wp, st));
     DEC_TRY(linear(m, m->head, m->head_in, m->wp, m->logits, true, n, st));
     return logits_finish_launch(m->logits, m->vp, m->c.vocab, m->c.logit_softcap, n, m->keys, m->key_ctrs, m->next_dev, st);
+}
+
+// first position that a token at `pos` or later can see in any layer
+static int first_needed(const jsm_decoder* m, int pos) {
+    int first = pos;
+    for (const DecLayer& L : m->layers)
+        if (L.is_attention()) first = std::min(first, L.key_mask().first(pos));
+    return first;
 }
 
 // Runs the tokens of `segs`; want_tok / want_out: wanted places as (flat token, output row) pairs.
@@ -508,20 +734,20 @@ static jsm_status run_pass(jsm_decoder* m, std::vector<PassSeg> segs, const int3
             if (w.first >= segs[i].tok0 && w.first < segs[i].tok0 + segs[i].len) push(P.starts[i] + (w.first - segs[i].tok0));
     }
     for (const DecLayer& L : m->layers) {
-        if (L.c.mixer != JSM_MIXER_LATENT_ATTENTION || P.tiles_all.count(L.ld.H)) continue;
-        const int H = L.ld.H;
+        if (!L.is_attention() || P.tiles_all.count(L.tiling(P.decode))) continue;
+        const auto [H, rows] = L.tiling(P.decode);
         std::vector<int32_t> sg, r0;
         int n_short = 0;
         for (int i = 0; i < E; ++i) {
-            for (long long r = 0; r < (long long)segs[i].len * H; r += LATENT_TILE_ROWS) { sg.push_back(i); r0.push_back((int32_t)r); }
+            for (long long r = 0; r < (long long)segs[i].len * H; r += rows) { sg.push_back(i); r0.push_back((int32_t)r); }
             if (i + 1 == E - P.n_flash) n_short = (int)sg.size();
         }
         const size_t so = M.size();
         M.insert(M.end(), sg.begin(), sg.end());
         const size_t ro = M.size();
         M.insert(M.end(), r0.begin(), r0.end());
-        P.tiles_all[H] = TileList{so, ro, (int)sg.size(), T};
-        P.tiles_short[H] = TileList{so, ro, n_short, tok_short};
+        P.tiles_all[{H, rows}] = TileList{so, ro, (int)sg.size(), T};
+        P.tiles_short[{H, rows}] = TileList{so, ro, n_short, tok_short};
     }
     if (M.size() > m->meta_cap) JSM_FAIL(JSM_SHAPE, "jsm_decoder: step metadata of %zu words (room for %zu)", M.size(), m->meta_cap);
     memcpy(m->h_meta, M.data(), M.size() * sizeof(int32_t));
@@ -574,7 +800,7 @@ static jsm_status run_pass(jsm_decoder* m, std::vector<PassSeg> segs, const int3
     JSM_CUDA_CHECK(cudaStreamSynchronize(st));
     for (const PassSeg& s : segs) {
         m->rows.h_ctx[s.row] = s.pos0 + s.len;
-        if (m->has_attention) m->rows.release_before(s.row, std::max(0, s.pos0 + s.len - m->max_window + 1));
+        if (m->has_attention) m->rows.release_before(s.row, first_needed(m, s.pos0 + s.len));
     }
     return JSM_OK;
 }
@@ -603,16 +829,33 @@ jsm_status jsm_decoder_create(const jsm_decoder_config* cfg, const jsm_layer_con
         } else if (k.mixer == JSM_MIXER_SELECTIVE_SCAN) {
             if (k.inner <= 0 || k.state <= 0 || k.dt_rank <= 0 || k.taps <= 0) JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: sizes of the scan of layer %d", l);
             if (k.state > 128) JSM_FAIL(JSM_UNSUPPORTED, "jsm_decoder_create: %d states per channel in layer %d (at most 128)", k.state, l);
+        } else if (k.mixer == JSM_MIXER_ATTENTION) {
+            if (k.heads <= 0 || k.kv_heads <= 0 || k.heads % k.kv_heads || k.dim <= 0 || k.vdim <= 0 || k.rot_dim < 0 || k.rot_dim % 2 || k.rot_dim > k.dim ||
+                (k.rot_dim > 0 && !(k.rope_base > 0.0)) || k.mask < JSM_MASK_FULL || k.mask > JSM_MASK_CHUNK || (k.mask != JSM_MASK_FULL && k.window <= 0))
+                JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: sizes of the attention of layer %d", l);
+            if (k.kv_from >= 0) {
+                const jsm_layer_config& s = layers[std::min(k.kv_from, l)];
+                if (k.kv_from >= l || s.mixer != JSM_MIXER_ATTENTION || s.kv_from >= 0 || s.heads != k.heads || s.kv_heads != k.kv_heads || s.dim != k.dim || s.vdim != k.vdim)
+                    JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: layer %d takes the keys and values of layer %d", l, k.kv_from);
+            }
+        } else if (k.mixer == JSM_MIXER_LINEAR_ATTENTION || k.mixer == JSM_MIXER_DELTA) {
+            const bool delta = k.mixer == JSM_MIXER_DELTA;
+            if (k.heads <= 0 || k.dim <= 0 || k.vdim <= 0 || (delta && (k.kv_heads <= 0 || k.heads % k.kv_heads || k.taps <= 0)))
+                JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: sizes of the recurrence of layer %d", l);
+            if (!rec_usable(RecDims{k.heads, k.heads, k.dim, k.vdim, 1, delta}))
+                JSM_FAIL(JSM_UNSUPPORTED, "jsm_decoder_create: recurrence of layer %d with heads of %d / %d components", l, k.dim, k.vdim);
         } else {
             JSM_FAIL(JSM_UNSUPPORTED, "jsm_decoder_create: mixer %d of layer %d", k.mixer, l);
         }
-        if (k.ff < 0) JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: feed-forward of layer %d", l);
+        if (k.ff < 0 || k.ff_kind < JSM_FF_CLAMPED_GLU || k.ff_kind > JSM_FF_GELU_GLU) JSM_FAIL(JSM_INVALID_ARG, "jsm_decoder_create: feed-forward of layer %d", l);
     }
+    if (c.norm_place != JSM_NORM_OUTPUT && c.norm_place != JSM_NORM_SUM) JSM_FAIL(JSM_UNSUPPORTED, "jsm_decoder_create: norm place %d", c.norm_place);
     int ndev = 0;
     DEC_TRY(jsm_device_count(&ndev));
     if (ndev == 0) JSM_FAIL(JSM_CUDA, "jsm_decoder_create: no CUDA device");
     jsm_decoder* m = new jsm_decoder();
     m->c = c;
+    if (m->c.embed_scale == 0.0f) m->c.embed_scale = 1.0f;
     m->f32 = c.dtype == JSM_F32;
     m->wp = pad8(c.d_model);
     m->vp = pad8(c.vocab);
@@ -622,12 +865,16 @@ jsm_status jsm_decoder_create(const jsm_decoder_config* cfg, const jsm_layer_con
         L.c = layers[l];
         if (L.c.mixer == JSM_MIXER_LATENT_ATTENTION) {
             L.ld = LatentDims{L.c.heads, L.c.dim, L.c.rot_dim, L.c.vdim, L.c.kv_rank, L.c.window, (float)L.c.scale};
-            m->has_attention = true;
-            m->max_window = std::max(m->max_window, L.c.window);
+        } else if (L.c.mixer == JSM_MIXER_ATTENTION) {
+            L.ad = AttnDims{L.c.heads, L.c.kv_heads, L.c.dim, L.c.vdim, L.c.rot_dim, KeyMask{L.c.mask, L.c.window}, (float)L.c.scale, 1};
+        } else if (L.is_recurrence()) {
+            const bool delta = L.c.mixer == JSM_MIXER_DELTA;
+            L.rd = RecDims{L.c.heads, delta ? L.c.kv_heads : L.c.heads, L.c.dim, L.c.vdim, delta ? L.c.taps : 1, delta};
         } else {
             L.sd = ScanDims{L.c.inner, L.c.state, L.c.dt_rank, L.c.taps};
         }
     }
+    for (const DecLayer& L : m->layers) m->has_attention |= L.is_attention();
     if (cudaStreamCreateWithFlags(&m->own_stream, cudaStreamNonBlocking) != cudaSuccess) {
         cudaGetLastError();
         delete m;
@@ -685,7 +932,7 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
         const HostTensor* t;
         DEC_TRY(want_tensor(m, pre + "norm1", c.d_model, 1, &t));
         DEC_TRY(upload_vec(m, *t, wp, &L.norm1));
-        DEC_TRY(L.c.mixer == JSM_MIXER_LATENT_ATTENTION ? build_latent(m, L, pre) : build_scan(m, L, pre));
+        DEC_TRY(build_mixer(m, L, pre));
         if (L.c.ff > 0) {
             DEC_TRY(want_tensor(m, pre + "norm2", c.d_model, 1, &t));
             DEC_TRY(upload_vec(m, *t, wp, &L.norm2));
@@ -696,11 +943,12 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
         if (L.c.weights_of < 0) continue;
         const DecLayer& S = m->layers[L.c.weights_of];
         if ((L.c.ff > 0) != (S.c.ff > 0) || L.c.ff != S.c.ff) JSM_FAIL(JSM_SHAPE, "jsm_decoder_finalize: layers that share weights differ in their feed-forward");
-        if (memcmp(&L.ld, &S.ld, offsetof(LatentDims, window)) != 0 || memcmp(&L.sd, &S.sd, sizeof(ScanDims)) != 0)
+        if (memcmp(&L.ld, &S.ld, offsetof(LatentDims, window)) != 0 || memcmp(&L.sd, &S.sd, sizeof(ScanDims)) != 0 ||
+            memcmp(&L.ad, &S.ad, offsetof(AttnDims, mask)) != 0 || memcmp(&L.rd, &S.rd, offsetof(RecDims, delta)) != 0 || L.own_kv() != S.own_kv())
             JSM_FAIL(JSM_SHAPE, "jsm_decoder_finalize: layers that share weights differ in their sizes");
         L.norm1 = S.norm1; L.norm2 = S.norm2;
         L.qd = S.qd; L.expand = S.expand; L.in = S.in; L.xp = S.xp; L.dt = S.dt; L.out = S.out;
-        L.gate = S.gate; L.up = S.up; L.down = S.down; L.lw = S.lw; L.sw = S.sw;
+        L.gate = S.gate; L.up = S.up; L.down = S.down; L.lw = S.lw; L.sw = S.sw; L.aw = S.aw; L.rw = S.rw;
     }
     m->tensors.clear();
     // cache pages, states
@@ -711,20 +959,27 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     m->rows.init(c.max_batch, n_pages, per_row, c.max_context, bt);
     m->slot_of_row.assign(c.max_batch, 0);
     for (int i = c.max_batch - 1; i >= 0; --i) m->free_slots.push_back(i);
-    std::map<std::pair<int, double>, float2*> ropes;
-    size_t wide = 0, q = 0, qlat = 0, olat = 0, att = 0, xz = 0, xc = 0, proj = 0, rp = 0, ff = 0, part = 0, gat = 0, exp_cols = 0;
+    std::map<std::vector<double>, float2*> ropes;
+    size_t wide = 0, q = 0, qlat = 0, olat = 0, att = 0, xz = 0, xc = 0, sy = 0, dtr = 0, proj = 0, rp = 0, ff = 0, part = 0, gat = 0, exp_cols = 0, gates = 0;
+    auto rope_table = [&](const jsm_layer_config& k, const float2** out) -> jsm_status {
+        *out = nullptr;
+        if (k.rot_dim == 0) return JSM_OK;
+        float2*& table = ropes[{(double)k.rot_dim, k.rope_base, k.rope_factor, k.rope_original, k.rope_fast, k.rope_slow}];
+        if (!table) {
+            DEC_TRY(dalloc(m, &table, sizeof(float2) * (size_t)c.max_context * (k.rot_dim / 2)));
+            DEC_TRY(jsm_rope_scaled_table(reinterpret_cast<float*>(table), k.rot_dim, k.rope_base, k.rope_factor, k.rope_original, k.rope_fast, k.rope_slow,
+                                          c.max_context));
+        }
+        *out = table;
+        return JSM_OK;
+    };
     for (DecLayer& L : m->layers) {
         if (L.c.mixer == JSM_MIXER_LATENT_ATTENTION) {
             const LatentDims& d = L.ld;
             DEC_TRY(dalloc(m, &L.cache.pool, (size_t)n_pages * JSM_PAGE_SIZE * d.cr() * es));
             L.cache.block_table = bt;
             L.cache.max_pages = per_row;
-            float2*& table = ropes[{d.rot, L.c.rope_base}];
-            if (!table && d.rot > 0) {
-                DEC_TRY(dalloc(m, &table, sizeof(float2) * (size_t)c.max_context * (d.rot / 2)));
-                DEC_TRY(jsm_rope_half_table(reinterpret_cast<float*>(table), d.rot, L.c.rope_base, c.max_context));
-            }
-            L.cache.rope = table;
+            DEC_TRY(rope_table(L.c, &L.cache.rope));
             wide = std::max(wide, (size_t)d.q_cols() + d.down_cols());
             q = std::max(q, (size_t)d.q_cols());
             qlat = std::max(qlat, (size_t)d.H * d.cr());
@@ -737,12 +992,34 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
                 gat = std::max(gat, (size_t)d.cr());
                 exp_cols = std::max(exp_cols, (size_t)L.expand.N);
             }
+        } else if (L.c.mixer == JSM_MIXER_ATTENTION) {
+            const AttnDims& d = L.ad;
+            if (L.own_kv()) DEC_TRY(dalloc(m, &L.ac.pool, (size_t)n_pages * d.page_elems() * es));
+            else L.ac.pool = m->layers[L.c.kv_from].ac.pool;
+            L.ac.block_table = bt;
+            L.ac.max_pages = per_row;
+            DEC_TRY(rope_table(L.c, &L.ac.rope));
+            wide = std::max(wide, (size_t)d.wide_cols(L.own_kv()));
+            q = std::max(q, (size_t)d.q_cols());
+            att = std::max(att, (size_t)d.out_cols());
+            gates = std::max(gates, (size_t)d.H);
+            if (attn_mma_usable(d)) part = std::max(part, attn_part_floats(d));
+        } else if (L.is_recurrence()) {
+            const RecDims& d = L.rd;
+            DEC_TRY(dalloc(m, &L.rs.S, sizeof(float) * (size_t)c.max_batch * d.H * d.kp() * d.vp()));
+            DEC_TRY(dalloc(m, &L.rs.conv, es * (size_t)c.max_batch * (d.taps - 1) * d.conv_cols()));
+            xz = std::max(xz, (size_t)d.raw_cols());
+            xc = std::max(xc, (size_t)d.conv_cols());
+            sy = std::max(sy, (size_t)d.out_cols());
+            proj = std::max(proj, (size_t)d.ba_cols());
         } else {
             const ScanDims& d = L.sd;
             DEC_TRY(dalloc(m, &L.state.S, sizeof(float) * (size_t)c.max_batch * d.ip() * d.np()));
             DEC_TRY(dalloc(m, &L.state.conv, es * (size_t)c.max_batch * (d.taps - 1) * d.ip()));
             xz = std::max(xz, (size_t)2 * d.ip());
             xc = std::max(xc, (size_t)d.ip());
+            sy = std::max(sy, (size_t)d.ip());
+            dtr = std::max(dtr, (size_t)d.ip());
             proj = std::max(proj, (size_t)d.proj_cols());
             rp = std::max(rp, (size_t)d.rp());
         }
@@ -760,9 +1037,11 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     DEC_TRY(dalloc(m, &m->att, es * T * att));
     DEC_TRY(dalloc(m, &m->xz, es * T * xz));
     DEC_TRY(dalloc(m, &m->xc, es * T * xc));
-    DEC_TRY(dalloc(m, &m->scan_y, es * T * xc));
+    DEC_TRY(dalloc(m, &m->scan_y, es * T * sy));
     DEC_TRY(dalloc(m, &m->proj, 4 * T * proj));
-    DEC_TRY(dalloc(m, &m->dt_raw, 4 * T * xc));
+    DEC_TRY(dalloc(m, &m->dt_raw, 4 * T * dtr));
+    DEC_TRY(dalloc(m, &m->head_gate, 4 * T * gates));
+    DEC_TRY(dalloc(m, &m->attn_ctrs, sizeof(int) * attn_counters()));
     DEC_TRY(dalloc(m, &m->dt_op, 2 * T * rp));
     DEC_TRY(dalloc(m, &m->act, es * T * ff));
     if (m->f32) DEC_TRY(dalloc(m, &m->gate32, 2 * 4 * T * ff));
@@ -780,11 +1059,11 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     m->n_counters = std::max(m->n_counters, sm_count());
     DEC_TRY(dalloc(m, &m->ws, 4 * m->ws_floats));
     DEC_TRY(dalloc(m, &m->counters, 4 * (size_t)m->n_counters));
-    std::map<int, int> heads;
+    std::map<std::pair<int, int>, int> tilings;
     for (const DecLayer& L : m->layers)
-        if (L.c.mixer == JSM_MIXER_LATENT_ATTENTION) heads[L.ld.H] = 1;
+        if (L.is_attention()) tilings[L.tiling(false)] = tilings[L.tiling(true)] = 1;
     m->meta_cap = 4 * T + 5 * T + 64;
-    for (auto& h : heads) m->meta_cap += 2 * (T * h.first / LATENT_TILE_ROWS + T + 1);
+    for (auto& t : tilings) m->meta_cap += 2 * (T * t.first.first / t.first.second + T + 1);
     DEC_TRY(dalloc(m, &m->meta, 4 * m->meta_cap));
     JSM_CUDA_CHECK(cudaMallocHost(reinterpret_cast<void**>(&m->h_meta), 4 * m->meta_cap));
     tc_error_word();  // first use allocates the device's error word: here, not inside a captured step
@@ -794,7 +1073,7 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     for (const DecLayer& L : m->layers) {
         m->weight_bytes += pb(L.qd) + pb(L.in) + pb(L.xp) + pb(L.out) + pb(L.gate) + pb(L.up) + pb(L.down);
         if (L.c.mixer == JSM_MIXER_LATENT_ATTENTION) m->weight_bytes += (uint64_t)L.ld.H * (L.ld.dim + L.ld.vdim) * L.ld.rank * es;
-        else m->weight_bytes += pb(L.dt);
+        else if (L.c.mixer == JSM_MIXER_SELECTIVE_SCAN) m->weight_bytes += pb(L.dt);
     }
     JSM_CUDA_CHECK(cudaDeviceSynchronize());
     m->ready = true;
@@ -932,6 +1211,10 @@ jsm_status jsm_decoder_step_bytes(jsm_decoder* m, int context_len, uint64_t* wei
         *seq_bytes = 0;
         for (const DecLayer& L : m->layers) {
             if (L.c.mixer == JSM_MIXER_LATENT_ATTENTION) *seq_bytes += (uint64_t)std::min(context_len, L.ld.window) * L.ld.cr() * es;
+            else if (L.c.mixer == JSM_MIXER_ATTENTION)
+                *seq_bytes += (uint64_t)std::min(context_len, L.ad.mask.reach(context_len)) * L.ad.G * (L.ad.ks() + L.ad.vs()) * 64 * es;
+            else if (L.is_recurrence())
+                *seq_bytes += 2ull * (4ull * L.rd.H * L.rd.kp() * L.rd.vp() + es * (L.rd.taps - 1) * L.rd.conv_cols());
             else *seq_bytes += 2ull * (4ull * L.sd.ip() * L.sd.np() + es * (L.sd.taps - 1) * L.sd.ip());
         }
     }

@@ -68,8 +68,15 @@ struct FlashParams {
     __nv_bfloat16* out;
     long long out_rs;
     int q_hs, v_dim;     // columns between the heads of q; columns of a head's output
-    int window;          // query i sees the keys i - window + 1 .. i only (WIN)
+    int window;          // query i sees the keys i - window + 1 .. i only (FA_WINDOW)
     int* err;
+    // FA_PAGED: keys and values come from the blocks of a paged cache (paged_attn.cu); key 0 is position `base`, which starts a
+    // page; the mask is d.mask, the sink (log2 domain, or null) joins the denominator, gate [query][Hq] multiplies the output
+    const __nv_bfloat16* pool;
+    const int32_t* pages;   // the row's block table from base's page on
+    int n_pages, base;
+    KeyMask mask;
+    const float *sink, *gate;
 };
 
 // 2^x for a pair of scores without the special-function unit: x = n + f with n = round(x) taken from the mantissa of
@@ -95,12 +102,15 @@ __device__ __forceinline__ void ex2_poly2(uint64_t x2, float& p0, float& p1) {
 }
 
 // POLY: of every four pairs of scores, this many take ex2_poly2 instead of ex2.approx
-// QKD / VD: columns of a query / key and of a value; VST: stages of the V ring (keys have two); WIN: the mask is a window of
-// P.window keys, and a head's output has P.v_dim columns (VD otherwise)
-template <int POLY, int QKD, int VD, int VST, bool WIN>
+// QKD / VD: columns of a query / key and of a value; VST: stages of the V ring (keys have two); FA_WINDOW: the mask is a window
+// of P.window keys; FA_PAGED: any mask, a sink and a gate, keys and values in a paged cache; both: a head's output has P.v_dim
+// columns (VD otherwise)
+enum FlashMode { FA_PLAIN = 0, FA_WINDOW = 1, FA_PAGED = 2 };
+template <int POLY, int QKD, int VD, int VST, int MODE>
 __global__ void __launch_bounds__(FA_THREADS, 1)
     flash_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_v, FlashParams P) {
+    constexpr bool WIN = MODE != FA_PLAIN, PAGED = MODE == FA_PAGED;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     constexpr int KST = 2;
@@ -120,6 +130,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     const int h = blockIdx.y, b = blockIdx.z, hk = h / (P.Hq / P.Hkv);
     const int q0 = qblk * 2 * FA_BM;
     const int shift = P.Tk - P.Tq;  // query i sits at position i + shift
+    // first key that query i sees
+    auto first_key = [&](int i) { return PAGED ? P.mask.first(P.base + i + shift) - P.base : i + shift - P.window + 1; };
     // key tiles [lo, n_tiles) of each query tile
     int n_tiles[2], lo[2];
 #pragma unroll
@@ -128,7 +140,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
         int kv_end = P.causal ? min(P.Tk, last_row + shift + 1) : P.Tk;
         if (q0 + t * FA_BM >= P.Tq) kv_end = 0;
         n_tiles[t] = (kv_end + FA_BN - 1) / FA_BN;
-        lo[t] = WIN ? min(n_tiles[t], max(0, q0 + t * FA_BM + shift - P.window + 1) / FA_BN) : 0;
+        lo[t] = WIN ? min(n_tiles[t], max(0, first_key(q0 + t * FA_BM)) / FA_BN) : 0;
     }
     const int n_max = max(n_tiles[0], n_tiles[1]);
     const int j_lo = n_tiles[1] > 0 ? min(lo[0], lo[1]) : lo[0];
@@ -141,7 +153,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
         for (int s = 0; s < VST; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
         for (int t = 0; t < 2; ++t) { mbar_init(&s_full[t], 1); mbar_init(&p_ready[t], 128); }
         mbar_fence_init();
-        tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
+        tma_prefetch_desc(&tmap_q);
+        if (!PAGED) { tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v); }
     }
     if (warp == 1) {
         tmem_alloc(&tmem_base_smem, 512);
@@ -161,17 +174,27 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
                 for (int c = 0; c < QKD / 64; ++c)
                     tma_load_2d(q_smem + t * QK_BYTES + c * FA_SLAB, &tmap_q, h * P.q_hs + c * 64, b * P.Tq + q0 + t * FA_BM, &q_full);
             int k_issued = 0, v_issued = 0;
+            // paged: 64 columns of a key tile are a slab of two pages (a tile's second half behind the last page repeats it: masked)
+            auto slab = [&](uint8_t* dst, int j, int c, uint64_t* bar) {
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const long long page = P.pages[min(2 * j + half, P.n_pages - 1)];
+                    bulk_load(dst + half * (FA_SLAB / 2), P.pool + ((page * P.Hkv + hk) * ((QKD + VD) / 64) + c) * (FA_SLAB / 4), FA_SLAB / 2, bar);
+                }
+            };
             for (int j = j_lo; j < n_max; ++j) {
                 const int i = j - j_lo, ks = i % KST, vs = i % VST;
                 if (i >= KST && !mbar_wait(&k_empty[ks], ((i / KST) & 1) ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) break;
                 mbar_expect_tx(&k_full[ks], QK_BYTES);
                 for (int c = 0; c < QKD / 64; ++c)
-                    tma_load_2d(k_smem + ks * QK_BYTES + c * FA_SLAB, &tmap_k, hk * QKD + c * 64, b * P.Tk + j * FA_BN, &k_full[ks]);
+                    if (PAGED) slab(k_smem + ks * QK_BYTES + c * FA_SLAB, j, c, &k_full[ks]);
+                    else tma_load_2d(k_smem + ks * QK_BYTES + c * FA_SLAB, &tmap_k, hk * QKD + c * 64, b * P.Tk + j * FA_BN, &k_full[ks]);
                 k_issued = i + 1;
                 if (i >= VST && !mbar_wait(&v_empty[vs], ((i / VST) & 1) ^ 1, &abort_flag, P.err, TC_TIMEOUT_EMPTY)) break;
                 mbar_expect_tx(&v_full[vs], V_BYTES);
                 for (int c = 0; c < VD / 64; ++c)
-                    tma_load_2d(v_smem + vs * V_BYTES + c * FA_SLAB, &tmap_v, hk * VD + c * 64, b * P.Tk + j * FA_BN, &v_full[vs]);
+                    if (PAGED) slab(v_smem + vs * V_BYTES + c * FA_SLAB, j, QKD / 64 + c, &v_full[vs]);
+                    else tma_load_2d(v_smem + vs * V_BYTES + c * FA_SLAB, &tmap_v, hk * VD + c * 64, b * P.Tk + j * FA_BN, &v_full[vs]);
                 v_issued = i + 1;
             }
             if (abort_flag) {  // let the copies in flight land before the CTA exits (bounded)
@@ -270,7 +293,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
 #pragma unroll
             for (int i = 0; i < FA_BN; ++i) sv[i] = __uint_as_float(sr[i]);
             const int key0 = j * FA_BN;
-            const bool low_edge = WIN && key0 < q0 + t * FA_BM + FA_BM - 1 + shift - P.window + 1;
+            const bool low_edge = WIN && key0 < first_key(q0 + t * FA_BM + FA_BM - 1);
             const bool needs_mask = (P.causal && key0 + FA_BN - 1 > q0 + t * FA_BM + shift) || key0 + FA_BN > P.Tk;
             if (needs_mask) {
 #pragma unroll
@@ -278,7 +301,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
                     if ((P.causal && key0 + i > qpos) || key0 + i >= P.Tk) sv[i] = -INFINITY;
             }
             if (low_edge) {
-                const int first = qpos - P.window + 1 - key0;  // keys before it are out of this row's window
+                const int first = first_key(qi) - key0;  // keys before it are out of this row's window
 #pragma unroll
                 for (int i = 0; i < FA_BN; ++i)
                     if (i < first) sv[i] = -INFINITY;
@@ -359,8 +382,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
         if (ok && j_end > j_begin) ok = mbar_wait(&o_done, 0, &abort_flag, P.err, TC_TIMEOUT_ACC);
         tc_fence_after();
         if (ok && j_end > j_begin) {  // warp-uniform: the TMEM loads are collective, only the stores are per row
-            const float inv = 1.0f / l;
             const bool store = qi < P.Tq;
+            if (PAGED && P.sink) l += ex2_approx(P.sink[h] * 1.4426950408889634f - m_ref);
+            const float inv = (PAGED && P.gate && store ? P.gate[(long long)qi * P.Hq + h] : 1.0f) / l;
             __nv_bfloat16* dst = P.out + (long long)(b * P.Tq + (store ? qi : 0)) * P.out_rs + (long long)h * (WIN ? P.v_dim : VD);
             const int v_dim = WIN ? P.v_dim : VD;
             const bool vec = v_dim % 8 == 0;
@@ -395,17 +419,17 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     }
 }
 
-template <int QKD, int VD, int VST, bool WIN>
+template <int QKD, int VD, int VST, int MODE>
 static jsm_status flash_go(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FlashParams& P, dim3 grid, cudaStream_t st) {
     constexpr size_t smem = (size_t)(4 * (QKD / 64) + VST * (VD / 64)) * FA_SLAB + 1024;
     static_assert(smem <= 226 * 1024, "query tiles and rings fit the shared memory");
     // a quarter of the exponentials on the FMA pipe: the measured optimum (none: MUFU-bound, half: issue-bound)
     static bool attr_done = false;
     if (!attr_done) {
-        JSM_CUDA_CHECK(cudaFuncSetAttribute(flash_prefill_kernel<1, QKD, VD, VST, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(flash_prefill_kernel<1, QKD, VD, VST, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         attr_done = true;
     }
-    flash_prefill_kernel<1, QKD, VD, VST, WIN><<<grid, FA_THREADS, smem, st>>>(mq, mk, mv, P);
+    flash_prefill_kernel<1, QKD, VD, VST, MODE><<<grid, FA_THREADS, smem, st>>>(mq, mk, mv, P);
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -433,7 +457,7 @@ jsm_status flash_prefill_launch(const void* q, const void* k, const void* v, voi
     P.out_rs = o_rs;
     P.q_hs = FA_D; P.v_dim = FA_D; P.window = 0;
     P.err = tc_error_word();
-    return flash_go<128, 128, 2, false>(mq, mk, mv, P, dim3((Tq + 2 * FA_BM - 1) / (2 * FA_BM), Hq, batch), st);
+    return flash_go<128, 128, 2, FA_PLAIN>(mq, mk, mv, P, dim3((Tq + 2 * FA_BM - 1) / (2 * FA_BM), Hq, batch), st);
 }
 
 // ---- latent attention of long segments ---------------------------------------------------------------------------------
@@ -459,10 +483,39 @@ jsm_status latent_flash_launch(const LatentDims& d, const void* q, const void* k
     const dim3 grid((n_q + 2 * FA_BM - 1) / (2 * FA_BM), d.H, 1);
     const int qk = d.dkp();
     if (d.dvp() == 64)
-        return qk == 64 ? flash_go<64, 64, 2, true>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 64, 2, true>(mq, mk, mv, P, grid, st)
-                                                                                   : flash_go<192, 64, 2, true>(mq, mk, mv, P, grid, st);
-    return qk == 64 ? flash_go<64, 128, 2, true>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 128, 2, true>(mq, mk, mv, P, grid, st)
-                                                                                : flash_go<192, 128, 1, true>(mq, mk, mv, P, grid, st);
+        return qk == 64 ? flash_go<64, 64, 2, FA_WINDOW>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 64, 2, FA_WINDOW>(mq, mk, mv, P, grid, st)
+                                                                                   : flash_go<192, 64, 2, FA_WINDOW>(mq, mk, mv, P, grid, st);
+    return qk == 64 ? flash_go<64, 128, 2, FA_WINDOW>(mq, mk, mv, P, grid, st) : qk == 128 ? flash_go<128, 128, 2, FA_WINDOW>(mq, mk, mv, P, grid, st)
+                                                                                : flash_go<192, 128, 1, FA_WINDOW>(mq, mk, mv, P, grid, st);
+}
+
+// ---- long segments over a paged cache ----------------------------------------------------------------------------------
+bool attn_flash_usable(const AttnDims& d) { return d.ks() <= 3 && d.vs() <= 2 && d.scale > 0.0f; }
+
+jsm_status attn_flash_launch(const AttnDims& d, const AttnWeights& w, const AttnCache& cache, int row, int pos0, int len, const void* q, const float* gate,
+                             void* out, cudaStream_t st) {
+    CUtensorMap mq;  // (a head's query box may reach into the next head's columns: the key's padding columns are zero there)
+    jsm_status s = make_tmap_bf16_2d(&mq, q, (uint64_t)len, (uint64_t)d.q_cols(), (uint64_t)d.q_cols(), FA_BM, 64);
+    if (s != JSM_OK) return s;
+    const int base = d.mask.first(pos0) / JSM_PAGE_SIZE * JSM_PAGE_SIZE;
+    FlashParams P;
+    P.Tq = len; P.Tk = pos0 + len - base; P.Hq = d.H; P.Hkv = d.G; P.causal = 1;
+    P.scale_log2 = d.scale * 1.4426950408889634f;
+    P.out = reinterpret_cast<__nv_bfloat16*>(out);
+    P.out_rs = d.out_cols();
+    P.q_hs = d.qh(); P.v_dim = d.vdim; P.window = 0;
+    P.err = tc_error_word();
+    P.pool = static_cast<const __nv_bfloat16*>(cache.pool);
+    P.pages = cache.block_table + (long long)row * cache.max_pages + base / JSM_PAGE_SIZE;
+    P.n_pages = (P.Tk + JSM_PAGE_SIZE - 1) / JSM_PAGE_SIZE;
+    P.base = base; P.mask = d.mask; P.sink = w.sink; P.gate = d.gated ? gate : nullptr;
+    const dim3 grid((len + 2 * FA_BM - 1) / (2 * FA_BM), d.H, 1);
+    const int ks = d.ks();
+    if (d.vs() == 1)
+        return ks == 1 ? flash_go<64, 64, 2, FA_PAGED>(mq, mq, mq, P, grid, st) : ks == 2 ? flash_go<128, 64, 2, FA_PAGED>(mq, mq, mq, P, grid, st)
+                                                                                        : flash_go<192, 64, 2, FA_PAGED>(mq, mq, mq, P, grid, st);
+    return ks == 1 ? flash_go<64, 128, 2, FA_PAGED>(mq, mq, mq, P, grid, st) : ks == 2 ? flash_go<128, 128, 2, FA_PAGED>(mq, mq, mq, P, grid, st)
+                                                                                     : flash_go<192, 128, 1, FA_PAGED>(mq, mq, mq, P, grid, st);
 }
 
 }  // namespace jsm

@@ -5,7 +5,7 @@
 namespace jsm {
 
 enum LinearEpilogue { LIN_NONE = 0, LIN_RELU = 1, LIN_GELU = 2, LIN_SILU_MUL = 3, LIN_RESIDUAL = 4,
-                      LIN_CLAMPED_GLU = 5 /* packed weights only */ };
+                      LIN_CLAMPED_GLU = 5, LIN_GELU_GLU = 6 /* packed weights only */ };
 
 struct LinearArgs {
     const void* X;      // [T, K] bf16

@@ -46,12 +46,12 @@ __device__ __forceinline__ float pk_clamped_glu(float g, float u, float alpha, f
     return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
 }
 
-// 1-D bulk copy global -> shared (this CTA), completion counted in bytes on `bar`; both addresses 16-byte aligned
-__device__ __forceinline__ void bulk_load(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(smem_dst)),
-                 "l"(reinterpret_cast<uint64_t>(gsrc)), "r"(bytes), "r"(smem_u32(bar))
-                 : "memory");
+// gate/up pair with the tanh form of GELU: z (1 + tanh(y)) / 2 = z / (1 + e^(-2y)), y = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float pk_gelu_glu(float z, float u) {
+    const float y2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+    return __fdividef(z, 1.0f + __expf(-y2)) * u;
 }
+
 __device__ __forceinline__ void bulk_prefetch_l2(const void* gsrc, uint32_t bytes) {
     asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<uint64_t>(gsrc)), "r"(bytes) : "memory");
 }
@@ -227,17 +227,19 @@ __global__ void __launch_bounds__(PK_THREADS, 1)
     // with in-band epochs.
     // PRM 5: the pushing projection (plain tiles, bf16, nothing else).
     // PRM 6, 7, 8: decoders whose norms sit on the sublayers' outputs - 6: gate-up pairs with clamps, bf16 out; 7 / 8: plain
-    // tiles and nothing else, f32 / bf16 out.
+    // tiles and nothing else, f32 / bf16 out; 9: gate-up pairs with the tanh form of GELU, bf16 out.
     const bool tp_push = TPM == 1 || TPM == 4 || (TPM == 3 && P.tp_mode == 1);
     const bool tp_reduce = TPM == 2 || TPM == 5 || (TPM == 3 && P.tp_mode == 2);
     const bool tp_inband = BN == 16 && (TPM == 4 || TPM == 5 || (TPM == 3 && P.tp_inband != 0));  // (at most 16 tokens)
     constexpr bool FIX = PRM >= 2;
-    const bool paired = PRM < 0 ? P.paired != 0 : (PRM == 1 || PRM == 4 || PRM == 6);
+    const bool paired = PRM < 0 ? P.paired != 0 : (PRM == 1 || PRM == 4 || PRM == 6 || PRM == 9);
     const bool has_ssq_in = FIX ? (PRM == 2 || PRM == 4) : P.ssq_in != nullptr;
     const bool f32o = FIX ? PRM == 7 : P.out_f32 != 0;
     const float* const biasp = FIX ? nullptr : P.bias;
     const int epi = FIX ? (PRM == 3 ? LIN_RESIDUAL : PRM == 4 ? LIN_SILU_MUL : LIN_NONE) : P.epilogue;
-    auto gate_up = [&](float g, float u) { return PRM == 6 ? pk_clamped_glu(g, u, P.glu_alpha, P.glu_limit) : pk_silu(g) * u; };
+    auto gate_up = [&](float g, float u) {
+        return PRM == 6 ? pk_clamped_glu(g, u, P.glu_alpha, P.glu_limit) : PRM == 9 ? pk_gelu_glu(g, u) : pk_silu(g) * u;
+    };
     chain_trigger();
     if (threadIdx.x == 0) PK_TRACE(0);  // CTA resident
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1133,10 +1135,11 @@ jsm_status linear_packed_launch(const PackedArgs& a, cudaStream_t st) {
     if (a.K <= 0 || a.K % 8) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: K (%d) must be a positive multiple of 8", a.K);
     if (a.N % 4) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: N (%d) must be a multiple of 4", a.N);
     if (a.T > 256) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: at most 256 tokens per launch (%d)", a.T);
-    if (a.epilogue < LIN_NONE || a.epilogue > LIN_CLAMPED_GLU) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: epilogue %d", a.epilogue);
-    const int paired = a.epilogue == LIN_SILU_MUL || a.epilogue == LIN_CLAMPED_GLU ? 1 : 0;
-    if (a.epilogue == LIN_CLAMPED_GLU && (a.out_f32 || a.ssq_in || a.tp))
-        JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: the clamped gate/up projection writes bf16, without a fused norm or exchange");
+    if (a.epilogue < LIN_NONE || a.epilogue > LIN_GELU_GLU) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: epilogue %d", a.epilogue);
+    const bool glu = a.epilogue == LIN_CLAMPED_GLU || a.epilogue == LIN_GELU_GLU;
+    const int paired = a.epilogue == LIN_SILU_MUL || glu ? 1 : 0;
+    if (glu && (a.out_f32 || a.ssq_in || a.tp))
+        JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: the clamped and GELU gate/up projections write bf16, without a fused norm or exchange");
     if (paired && a.bias) JSM_FAIL(JSM_UNSUPPORTED, "linear_packed: the gate/up projection takes no bias");
     if (a.epilogue == LIN_RESIDUAL && !a.R) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: residual epilogue without R");
     if (a.bias && (reinterpret_cast<uintptr_t>(a.bias) & 15)) JSM_FAIL(JSM_INVALID_ARG, "linear_packed: bias must be 16-byte aligned");
@@ -1228,16 +1231,19 @@ jsm_status linear_packed_launch(const PackedArgs& a, cudaStream_t st) {
         return with_cl ? launch_packed<BN_, true, 3>(mx, mx2, P, grid, cluster, a.chained, st)           \
                        : launch_packed<BN_, false, 3>(mx, mx2, P, grid, cluster, a.chained, st);        \
     PK_GO(BN_)
-    if (a.epilogue == LIN_CLAMPED_GLU) {
-        switch (bn) {
-            case 16: return launch_packed<16, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
-            case 32: return cluster > 1 ? launch_packed<32, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st)
-                                        : launch_packed<32, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
-            case 64: return cluster > 1 ? launch_packed<64, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st)
-                                        : launch_packed<64, false, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
-            case 128: return launch_packed<128, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
-            default: return launch_packed<256, true, 0, 6>(mx, mx2, P, grid, cluster, a.chained, st);
-        }
+    if (glu) {
+#define PK_GLU(PRM_)                                                                                                  \
+    switch (bn) {                                                                                                      \
+        case 16: return launch_packed<16, false, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st);                   \
+        case 32: return cluster > 1 ? launch_packed<32, true, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st)       \
+                                    : launch_packed<32, false, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st);     \
+        case 64: return cluster > 1 ? launch_packed<64, true, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st)       \
+                                    : launch_packed<64, false, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st);     \
+        case 128: return launch_packed<128, true, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st);                  \
+        default: return launch_packed<256, true, 0, PRM_>(mx, mx2, P, grid, cluster, a.chained, st);                   \
+    }
+        if (a.epilogue == LIN_GELU_GLU) PK_GLU(9) else PK_GLU(6)
+#undef PK_GLU
     }
     // plain projections of up to 64 tokens with nothing fused
     if (bn <= 64 && !with_tp && !paired && !a.bias && a.epilogue == LIN_NONE && !a.ssq_in && !a.ssq_out) {

@@ -10,6 +10,7 @@
 #include "common.cuh"
 #include "attn.cuh"
 #include <cmath>
+#include <algorithm>
 #include <vector>
 
 namespace jsm {
@@ -257,16 +258,36 @@ jsm_status jsm::rope_apply_strided(const void* d_x, void* d_out, jsm_dtype dtype
 }
 
 extern "C" jsm_status jsm_rope_half_table(float* d_table, int d, double base, int max_pos) {
-    if (!d_table) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_half_table: null pointer");
-    if (d <= 0 || d % 2 || max_pos <= 0 || !(base > 0.0)) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_half_table: d %d, base %g, %d positions", d, base, max_pos);
+    return jsm_rope_scaled_table(d_table, d, base, 0.0, 0.0, 0.0, 0.0, max_pos);
+}
+
+// Scaling after YaRN (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models"): pairs that turn more
+// than `fast` times within the original context keep their frequency, pairs that turn less than `slow` times are slowed by
+// `factor`, a linear ramp over the pair index lies between.
+extern "C" jsm_status jsm_rope_scaled_table(float* d_table, int d, double base, double factor, double original, double fast, double slow,
+                                            int max_pos) {
+    if (!d_table) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_scaled_table: null pointer");
+    if (d <= 0 || d % 2 || max_pos <= 0 || !(base > 0.0)) JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_scaled_table: d %d, base %g, %d positions", d, base, max_pos);
+    if (factor != 0.0 && (!(factor > 0.0) || !(original > 0.0) || !(fast > 0.0) || !(slow > 0.0) || base == 1.0))
+        JSM_FAIL(JSM_INVALID_ARG, "jsm_rope_scaled_table: factor %g, original context %g, turns %g / %g, base %g", factor, original, fast, slow, base);
     const int half = d / 2;
     std::vector<double> freq(half);
     for (int i = 0; i < half; ++i) freq[i] = std::pow(base, -2.0 * i / d);
+    double magnitude = 1.0;
+    if (factor != 0.0) {
+        auto pair_of = [&](double turns) { return d * std::log(original / (2.0 * 3.14159265358979323846 * turns)) / (2.0 * std::log(base)); };
+        const double lo = std::max(std::floor(pair_of(fast)), 0.0), hi = std::min(std::ceil(pair_of(slow)), d - 1.0);
+        for (int i = 0; i < half; ++i) {
+            const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            freq[i] = freq[i] / factor * ramp + freq[i] * (1.0 - ramp);
+        }
+        magnitude = 0.1 * std::log(factor) + 1.0;
+    }
     std::vector<float> h((size_t)max_pos * d);
     for (int m = 0; m < max_pos; ++m)
         for (int i = 0; i < half; ++i) {
-            h[((size_t)m * half + i) * 2] = (float)std::cos(m * freq[i]);
-            h[((size_t)m * half + i) * 2 + 1] = (float)std::sin(m * freq[i]);
+            h[((size_t)m * half + i) * 2] = (float)(magnitude * std::cos(m * freq[i]));
+            h[((size_t)m * half + i) * 2 + 1] = (float)(magnitude * std::sin(m * freq[i]));
         }
     JSM_CUDA_CHECK(cudaMemcpy(d_table, h.data(), h.size() * sizeof(float), cudaMemcpyHostToDevice));
     return JSM_OK;

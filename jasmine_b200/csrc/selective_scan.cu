@@ -111,7 +111,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
 // one token, and the state moves on by it here (otherwise the scan does that, once every CTA has read the old state)
 constexpr int CONV_TOK = 8;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256, 2) scan_conv_kernel(const T* __restrict__ xz, T* __restrict__ xc, T* state,
+__global__ void __launch_bounds__(256, 2) scan_conv_kernel(const T* __restrict__ xz, long long pitch, T* __restrict__ xc, T* state,
                                                         const float* __restrict__ w, const float* __restrict__ b,
                                                         const int32_t* __restrict__ seg_start, const int32_t* __restrict__ seg_len,
                                                         const int32_t* __restrict__ seg_pos0, const int32_t* __restrict__ seg_slot, int ip,
@@ -127,20 +127,23 @@ __global__ void __launch_bounds__(256, 2) scan_conv_kernel(const T* __restrict__
     T* st = state + (long long)seg_slot[seg] * (taps - 1) * ip + c;
     // input of the segment's token j (negative: before the segment)
     auto input = [&](int j, float (&v)[8]) {
-        if (j >= 0) Vec8<T>::load(xz + (long long)(start + j) * 2 * ip + c, v);
+        if (j >= 0) Vec8<T>::load(xz + (start + j) * pitch + c, v);
         else if (pos0 + j >= 0) Vec8<T>::load(st + (long long)(taps - 1 + j) * ip, v);
         else
             for (int e = 0; e < 8; ++e) v[e] = 0.0f;
     };
     float bias[8];
-    Vec8<float>::load(b + c, bias);
+    if (b) Vec8<float>::load(b + c, bias);
+    else
+#pragma unroll
+        for (int e = 0; e < 8; ++e) bias[e] = 0.0f;
     const int j1 = min(len, j0 + CONV_TOK);
     if constexpr (TAPS > 0) {
         // all the thread's inputs are requested before the first is used
         typename Vec8<T>::Raw raw[CONV_TOK];
 #pragma unroll
         for (int u = 0; u < CONV_TOK; ++u)
-            if (j0 + u < j1) raw[u] = Vec8<T>::fetch(xz + (long long)(start + j0 + u) * 2 * ip + c);
+            if (j0 + u < j1) raw[u] = Vec8<T>::fetch(xz + (start + j0 + u) * pitch + c);
         float win[TAPS][8], wt[TAPS][8];
 #pragma unroll
         for (int k = 0; k < TAPS; ++k) Vec8<float>::load(w + (long long)k * ip + c, wt[k]);
@@ -195,11 +198,12 @@ __global__ void __launch_bounds__(256, 2) scan_conv_kernel(const T* __restrict__
 // the last taps - 1 inputs after the segment: entry k is the input taps - 1 - k tokens before the next one.  One thread per
 // channel, ascending k: an entry taken from the old state lies behind every entry already written.
 template <typename T>
-__device__ __forceinline__ void carry_conv_state(T* state, const T* __restrict__ xz, int c, int ip, int taps, int start, int len, int pos0) {
+__device__ __forceinline__ void carry_conv_state(T* state, const T* __restrict__ xz, long long pitch, int c, int ip, int taps, int start, int len,
+                                                 int pos0) {
     for (int k = 0; k + 1 < taps; ++k) {
         const int j = len - (taps - 1) + k;
         T v = from_f32<T>(0.0f);
-        if (j >= 0) v = xz[(long long)(start + j) * 2 * ip + c];
+        if (j >= 0) v = xz[(start + j) * pitch + c];
         else if (pos0 + j >= 0) v = state[(long long)(k + len) * ip + c];
         state[(long long)k * ip + c] = v;
     }
@@ -390,7 +394,8 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(ScanArgs a) {
         for (int i = 0; i < NS; ++i)
             if (sub * NS + i < a.state) state[plane_index(sub * NS + i, c, a.ip)] = S[i];
     if (tid < SC_CH && c0 + tid < a.ip)
-        carry_conv_state(static_cast<T*>(a.conv) + (long long)slot * (a.taps - 1) * a.ip, xz, c0 + tid, a.ip, a.taps, start, len, pos0);
+        carry_conv_state(static_cast<T*>(a.conv) + (long long)slot * (a.taps - 1) * a.ip, xz, 2 * a.ip, c0 + tid, a.ip, a.taps, start, len,
+                            pos0);
 }
 
 // ---- decode step --------------------------------------------------------------------------------------------------
@@ -521,24 +526,49 @@ __global__ void __launch_bounds__(256) scan_dt_operand_kernel(const float* __res
 
 // ---- launches -----------------------------------------------------------------------------------------------------
 template <typename T>
-static jsm_status conv_typed(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, void* xc,
+static jsm_status conv_typed(const void* x, long long pitch, int cp, int taps, const float* w, const float* b, void* state, const StepTokens& tk, void* out,
                              bool carry, cudaStream_t st) {
-    const int ip = d.ip();
-    const long long n = (long long)((tk.max_len + CONV_TOK - 1) / CONV_TOK) * (ip / 8);
+    const long long n = (long long)((tk.max_len + CONV_TOK - 1) / CONV_TOK) * (cp / 8);
     const dim3 grid((unsigned)((n + 255) / 256), tk.n_segs);
     auto go = [&](auto kernel) {
-        return launch_chained(kernel, grid, dim3(256), 0, st, (const T*)xz, (T*)xc, (T*)s.conv, w.conv, w.conv_b, tk.seg_start, tk.seg_len,
-                              tk.seg_pos0, tk.seg_slot, ip, d.taps, carry ? 1 : 0);
+        return launch_chained(kernel, grid, dim3(256), 0, st, (const T*)x, pitch, (T*)out, (T*)state, w, b, tk.seg_start, tk.seg_len, tk.seg_pos0,
+                              tk.seg_slot, cp, taps, carry ? 1 : 0);
     };
-    JSM_CUDA_CHECK(d.taps == 2 ? go(scan_conv_kernel<T, 2>) : d.taps == 3 ? go(scan_conv_kernel<T, 3>)
-                   : d.taps == 4 ? go(scan_conv_kernel<T, 4>) : go(scan_conv_kernel<T, 0>));
+    JSM_CUDA_CHECK(taps == 1 ? go(scan_conv_kernel<T, 1>) : taps == 2 ? go(scan_conv_kernel<T, 2>) : taps == 3 ? go(scan_conv_kernel<T, 3>)
+                   : taps == 4 ? go(scan_conv_kernel<T, 4>) : go(scan_conv_kernel<T, 0>));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
 
+jsm_status short_conv_launch(bool f32, const void* x, long long x_pitch, int cp, int taps, const float* w, const float* bias, void* state,
+                             const StepTokens& tk, void* out, bool carry, cudaStream_t st) {
+    return f32 ? conv_typed<float>(x, x_pitch, cp, taps, w, bias, state, tk, out, carry, st)
+               : conv_typed<__nv_bfloat16>(x, x_pitch, cp, taps, w, bias, state, tk, out, carry, st);
+}
+
 jsm_status scan_conv_launch(bool f32, const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz,
                             void* xc, bool carry, cudaStream_t st) {
-    return f32 ? conv_typed<float>(d, w, s, tk, xz, xc, carry, st) : conv_typed<__nv_bfloat16>(d, w, s, tk, xz, xc, carry, st);
+    return short_conv_launch(f32, xz, 2 * d.ip(), d.ip(), d.taps, w.conv, w.conv_b, s.conv, tk, xc, carry, st);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) conv_carry_kernel(const T* __restrict__ x, long long pitch, T* state, const int32_t* __restrict__ seg_start,
+                                                         const int32_t* __restrict__ seg_len, const int32_t* __restrict__ seg_pos0,
+                                                         const int32_t* __restrict__ seg_slot, int cp, int taps) {
+    chain_trigger();
+    chain_wait();
+    const int c = blockIdx.x * 256 + threadIdx.x, seg = blockIdx.y;
+    if (c < cp) carry_conv_state(state + (long long)seg_slot[seg] * (taps - 1) * cp, x, pitch, c, cp, taps, seg_start[seg], seg_len[seg], seg_pos0[seg]);
+}
+jsm_status short_conv_carry_launch(bool f32, const void* x, long long x_pitch, int cp, int taps, void* state, const StepTokens& tk, cudaStream_t st) {
+    if (taps <= 1) return JSM_OK;
+    const dim3 grid((cp + 255) / 256, tk.n_segs);
+    if (f32) JSM_CUDA_CHECK(launch_chained(conv_carry_kernel<float>, grid, dim3(256), 0, st, (const float*)x, x_pitch, (float*)state, tk.seg_start, tk.seg_len,
+                                           tk.seg_pos0, tk.seg_slot, cp, taps));
+    else JSM_CUDA_CHECK(launch_chained(conv_carry_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)x, x_pitch, (__nv_bfloat16*)state,
+                                       tk.seg_start, tk.seg_len, tk.seg_pos0, tk.seg_slot, cp, taps));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
 }
 
 static ScanArgs scan_args(const ScanDims& d, const ScanWeights& w, const ScanState& s, const StepTokens& tk, const void* xz, const void* xc,

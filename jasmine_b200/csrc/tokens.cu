@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(256) add_norm_kernel(int kind, const T* __rest
 // ---- decoders whose residual stream is fp32 and whose norms sit on the sublayers' outputs ---------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) embed_residual_kernel(const T* __restrict__ table, const int32_t* __restrict__ ids, float* __restrict__ x,
-                                                             T* __restrict__ xa, int wp) {
+                                                             T* __restrict__ xa, float scale, int wp) {
     constexpr int N = VecIO<T>::N;
     chain_trigger();
     chain_wait();
@@ -153,6 +153,8 @@ __global__ void __launch_bounds__(256) embed_residual_kernel(const T* __restrict
         float v[N];
         VecIO<T>::load(src + c, v);
 #pragma unroll
+        for (int i = 0; i < N; ++i) v[i] *= scale;
+#pragma unroll
         for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(dst + c + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
         if (xa) VecIO<T>::store(xa + (long long)blockIdx.x * wp + c, v);
     }
@@ -160,9 +162,10 @@ __global__ void __launch_bounds__(256) embed_residual_kernel(const T* __restrict
 
 // One CTA per token; the sublayer's output y stays in registers between the statistics and the update (MAXV > 0: wp <=
 // 2048 * MAXV), or is read twice (MAXV 0).  Padding columns of y and of the gain are zero.
-template <int MAXV>
+// SUM false: x <- x + norm(y); true: x <- norm(alpha x + y)
+template <int MAXV, bool SUM>
 __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ gain,
-                                                            float eps, __nv_bfloat16* __restrict__ xa, int d, int wp) {
+                                                            float eps, float alpha, __nv_bfloat16* __restrict__ xa, int d, int wp) {
     __shared__ float smem[8];
     chain_trigger();
     chain_wait();
@@ -180,14 +183,22 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restr
             if (c < wp) {
                 load8(y + base + c, keep[i]);
                 load8(x + base + c, res[i]);
+                if (SUM)
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) keep[i][e] = fmaf(alpha, res[i][e], keep[i][e]);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) q = fmaf(keep[i][e], keep[i][e], q);
             }
         }
     } else {
         for (int c = threadIdx.x * 8; c < wp; c += 2048) {
-            float v[8];
+            float v[8], r[8];
             load8(y + base + c, v);
+            if (SUM) {
+                load8(x + base + c, r);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = fmaf(alpha, r[e], v[e]);
+            }
 #pragma unroll
             for (int e = 0; e < 8; ++e) q = fmaf(v[e], v[e], q);
         }
@@ -198,7 +209,7 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restr
         float g[8];
         load8(gain + c, g);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) r[e] += v[e] / rms * g[e];
+        for (int e = 0; e < 8; ++e) r[e] = SUM ? v[e] / rms * g[e] : r[e] + v[e] / rms * g[e];
         reinterpret_cast<float4*>(x + base + c)[0] = make_float4(r[0], r[1], r[2], r[3]);
         reinterpret_cast<float4*>(x + base + c)[1] = make_float4(r[4], r[5], r[6], r[7]);
         if (xa) VecIO<__nv_bfloat16>::store(xa + base + c, r);
@@ -214,6 +225,9 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restr
             float v[8], r[8];
             load8(y + base + c, v);
             load8(x + base + c, r);
+            if (SUM)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = fmaf(alpha, r[e], v[e]);
             update(c, v, r);
         }
     }
@@ -298,21 +312,29 @@ __global__ void __launch_bounds__(256) clamped_glu_f32_kernel(const float* __res
         act[i] = clamped_glu(gate[i], up[i], alpha, limit);
 }
 
-jsm_status embed_residual_launch(bool f32, const void* table, const int32_t* ids, float* x, void* xa, int T, int wp, cudaStream_t st) {
+jsm_status embed_residual_launch(bool f32, const void* table, const int32_t* ids, float scale, float* x, void* xa, int T, int wp, cudaStream_t st) {
     if (f32)
-        JSM_CUDA_CHECK(launch_chained(embed_residual_kernel<float>, dim3(T), dim3(256), 0, st, (const float*)table, ids, x, (float*)nullptr, wp));
+        JSM_CUDA_CHECK(launch_chained(embed_residual_kernel<float>, dim3(T), dim3(256), 0, st, (const float*)table, ids, x, (float*)nullptr, scale,
+                                      wp));
     else
         JSM_CUDA_CHECK(launch_chained(embed_residual_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, (const __nv_bfloat16*)table, ids, x,
-                                      (__nv_bfloat16*)xa, wp));
+                                      (__nv_bfloat16*)xa, scale, wp));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
 
-jsm_status post_norm_add_launch(const float* y, float* x, const float* gain, float eps, void* xa, int T, int d, int wp, cudaStream_t st) {
-    auto go = [&](auto kernel) { return launch_chained(kernel, dim3(T), dim3(256), 0, st, y, x, gain, eps, (__nv_bfloat16*)xa, d, wp); };
-    JSM_CUDA_CHECK(wp <= 2048 ? go(post_norm_add_kernel<1>) : wp <= 4096 ? go(post_norm_add_kernel<2>) : go(post_norm_add_kernel<0>));
+template <bool SUM>
+static jsm_status norm_residual(const float* y, float* x, const float* gain, float eps, float alpha, void* xa, int T, int d, int wp, cudaStream_t st) {
+    auto go = [&](auto kernel) { return launch_chained(kernel, dim3(T), dim3(256), 0, st, y, x, gain, eps, alpha, (__nv_bfloat16*)xa, d, wp); };
+    JSM_CUDA_CHECK(wp <= 2048 ? go(post_norm_add_kernel<1, SUM>) : wp <= 4096 ? go(post_norm_add_kernel<2, SUM>) : go(post_norm_add_kernel<0, SUM>));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
+}
+jsm_status post_norm_add_launch(const float* y, float* x, const float* gain, float eps, void* xa, int T, int d, int wp, cudaStream_t st) {
+    return norm_residual<false>(y, x, gain, eps, 1.0f, xa, T, d, wp, st);
+}
+jsm_status sum_norm_launch(const float* y, float* x, const float* gain, float eps, float alpha, void* xa, int T, int d, int wp, cudaStream_t st) {
+    return norm_residual<true>(y, x, gain, eps, alpha, xa, T, d, wp, st);
 }
 
 jsm_status final_norm_launch(bool f32, const float* x, const int32_t* rows, const float* gain, float eps, void* out, int n, int d, int wp,
@@ -331,6 +353,20 @@ jsm_status logits_finish_launch(float* logits, int pitch, int vocab, float cap, 
     if (rows <= 0) return JSM_OK;
     const int slices = std::max(1, std::min(16, vocab / 1024));
     JSM_CUDA_CHECK(launch_chained(logits_finish_kernel, dim3(slices, rows), dim3(256), 0, st, logits, pitch, vocab, cap, keys, ctrs, next));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+
+__global__ void __launch_bounds__(256) gelu_glu_f32_kernel(const float* __restrict__ gate, const float* __restrict__ up, float* __restrict__ act, long long n) {
+    chain_trigger();
+    chain_wait();
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
+        const float z = gate[i];
+        act[i] = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) * up[i];
+    }
+}
+jsm_status gelu_glu_f32_launch(const float* gate, const float* up, float* act, long long n, cudaStream_t st) {
+    JSM_CUDA_CHECK(launch_chained(gelu_glu_f32_kernel, dim3((unsigned)std::min<long long>((n + 255) / 256, 148 * 16)), dim3(256), 0, st, gate, up, act, n));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -393,6 +429,13 @@ extern "C" jsm_status jsm_post_norm_add(const float* d_y, float* d_x, const floa
     if (!d_y || !d_x || !d_gain) JSM_FAIL(JSM_INVALID_ARG, "jsm_post_norm_add: null pointer");
     if (d <= 0 || d % 8) JSM_FAIL(JSM_UNSUPPORTED, "jsm_post_norm_add: d %d (a multiple of 8)", d);
     return post_norm_add_launch(d_y, d_x, d_gain, eps, d_x_bf16, T, d, d, as_stream(stream));
+}
+
+extern "C" jsm_status jsm_sum_norm(const float* d_y, float* d_x, const float* d_gain, float eps, float alpha, void* d_x_bf16, int T, int d, void* stream) {
+    if (T <= 0) return JSM_OK;
+    if (!d_y || !d_x || !d_gain) JSM_FAIL(JSM_INVALID_ARG, "jsm_sum_norm: null pointer");
+    if (d <= 0 || d % 8) JSM_FAIL(JSM_UNSUPPORTED, "jsm_sum_norm: d %d (a multiple of 8)", d);
+    return sum_norm_launch(d_y, d_x, d_gain, eps, alpha, d_x_bf16, T, d, d, as_stream(stream));
 }
 
 extern "C" jsm_status jsm_logits_finish(float* d_logits, int pitch, int rows, int vocab, float cap, uint64_t* d_keys, int32_t* d_counters,

@@ -1,4 +1,4 @@
-"""Host-side handle of the layer-list decoder of libjasmine_b200.so (jsm_decoder_*), and the Zugolorn configuration.
+"""Host-side handle of the layer-list decoder of libjasmine_b200.so (jsm_decoder_*), and the Zugolorn and Vagonex configurations.
 
 No torch: tokens and logits are numpy arrays in host memory, the library owns the device side.  The serving calls are those
 of the paged Llama handle (admit / step_active / retire / pool_state), plus open / step for portions and mixed batches."""
@@ -9,7 +9,8 @@ import ctypes as C
 
 import numpy as np
 
-from . import BF16, F32, MIXER_LATENT_ATTENTION, MIXER_SELECTIVE_SCAN, DecoderConfig, LayerConfig, check, host_ptr, lib
+from . import (BF16, F32, FF_GELU_GLU, MASK_CHUNK, MASK_FULL, MIXER_ATTENTION, MIXER_DELTA, MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION,
+               MIXER_SELECTIVE_SCAN, NORM_OUTPUT, NORM_SUM, DecoderConfig, LayerConfig, check, host_ptr, lib)
 
 
 def _i32(a):
@@ -18,14 +19,17 @@ def _i32(a):
 
 class Decoder:
     def __init__(self, d_model, vocab, layers, norm_eps, logit_softcap=0.0, dtype="bfloat16", max_batch=8, max_context=4096,
-                 max_step_tokens=2048, pool_pages=0):
+                 max_step_tokens=2048, pool_pages=0, norm_place=NORM_OUTPUT, residual_scale=1.0, embed_scale=1.0):
         self.vocab, self.d_model, self.n_layers = vocab, d_model, len(layers)
         self.max_batch, self.max_context = max_batch, max_context
         self.stream = None  # a CUDA stream's address, or None: a stream of the model
         cfg = DecoderConfig(len(layers), d_model, vocab, {"bfloat16": BF16, "float32": F32}[dtype], max_batch, max_context,
-                            max(max_step_tokens, max_batch), pool_pages, norm_eps, logit_softcap)
+                            max(max_step_tokens, max_batch), pool_pages, norm_eps, logit_softcap, norm_place,
+                            residual_scale, embed_scale)
         self.max_step_tokens = cfg.max_step_tokens
-        self.max_window = max((k.window for k in layers if k.mixer == MIXER_LATENT_ATTENTION), default=0)
+        # most positions back that any layer looks (0: none has keys)
+        self.max_window = max((max_context if k.mixer == MIXER_ATTENTION and k.mask == MASK_FULL else k.window
+                               for k in layers if k.mixer in (MIXER_LATENT_ATTENTION, MIXER_ATTENTION)), default=0)
         arr = (LayerConfig * len(layers))(*layers)
         self._h = C.c_void_p()
         check(lib().jsm_decoder_create(C.byref(cfg), arr, C.byref(self._h)))
@@ -81,7 +85,7 @@ class Decoder:
         return moved.value
 
     def pages_for(self, n_tokens: int) -> int:
-        """Cache pages a sequence of n_tokens positions holds at most: pages behind every window go back to the pool."""
+        """Cache pages a sequence of n_tokens positions holds at most: pages behind every mask go back to the pool."""
         reach = min(n_tokens, self.max_window + self.max_step_tokens)
         return min(-(-n_tokens // 64), reach // 64 + 2) if self.max_window else 0
 
@@ -160,3 +164,54 @@ def zugolorn_model(config: dict, **serving) -> Decoder:
     """A Zugolorn decoder without its weights (set_weight for every tensor, then finalize)."""
     return Decoder(config["width"], config["vocab"], zugolorn_layers(config), config["norm"]["eps"],
                    config.get("logit_softcap") or 0.0, **serving)
+
+
+# ---- Vagonex ----------------------------------------------------------------------------------------------------------
+def _vagonex_attention(mix):
+    rot, mask = mix.get("rot") or {}, mix.get("mask") or {}
+    kv_from = mix.get("kv_from")
+    kw = dict(mixer=MIXER_ATTENTION, heads=mix["heads"], kv_heads=mix["kv_heads"], dim=mix["dim"], vdim=mix["vdim"], scale=mix["scale"],
+              rot_dim=rot.get("dims", 0), rope_base=rot.get("base", 1.0), mask=MASK_CHUNK if mask.get("size") else MASK_FULL,
+              window=mask.get("size") or 0, kv_from=-1 if kv_from is None else kv_from)
+    if rot.get("scaling"):
+        kw.update({f"rope_{k}": float(rot["scaling"][k]) for k in ("factor", "original", "fast", "slow")})
+    return kw
+
+
+def _lightning(mix):
+    if len(mix["decay"]) != mix["heads"]:
+        raise ValueError(f"lightning: {len(mix['decay'])} decays for {mix['heads']} heads")
+    return dict(mixer=MIXER_LINEAR_ATTENTION, heads=mix["heads"], dim=mix["dim"], vdim=mix["vdim"], kv_from=-1)
+
+
+def _delta(mix):
+    return dict(mixer=MIXER_DELTA, heads=mix["heads"], kv_heads=mix["kv_heads"], dim=mix["dim"], vdim=mix["vdim"], taps=mix["conv"], kv_from=-1)
+
+
+VAGONEX_MIXERS = {"attention": _vagonex_attention, "lightning": _lightning, "delta": _delta}
+
+
+def vagonex_layers(config: dict):
+    """The layer list of a Vagonex config.json as LayerConfig structures."""
+    out = []
+    for i, e in enumerate(config["layers"]):
+        if e["type"] not in VAGONEX_MIXERS:
+            raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+        kw = VAGONEX_MIXERS[e["type"]](e["mixer"])
+        mlp = e.get("mlp")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            kw.update(ff=mlp["ff"], ff_kind=FF_GELU_GLU)
+        out.append(LayerConfig(weights_of=-1, **kw))
+    return out
+
+
+def vagonex_model(config: dict, **serving) -> Decoder:
+    """A Vagonex decoder without its weights (set_weight for every tensor, then finalize)."""
+    m = Decoder(config["width"], config["vocab"], vagonex_layers(config), config["norm"]["eps"], norm_place=NORM_SUM,
+                residual_scale=config["postln_alpha"], embed_scale=config["embedding"]["scale"], **serving)
+    for i, e in enumerate(config["layers"]):
+        if e["type"] == "lightning":
+            m.set_weight(f"l{i}.mix.decay", np.asarray(e["mixer"]["decay"], np.float32))
+    return m

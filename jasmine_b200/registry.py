@@ -33,10 +33,9 @@ def load_model(folder, dtype="bfloat16", **serving):
     return ARCHITECTURES[name](Path(folder), config, dtype, serving)
 
 
-@register("Zugolorn")
-def _zugolorn(folder, config, dtype, serving):
-    from .decoder import zugolorn_model
-    model = zugolorn_model(config, dtype=dtype, **serving)
+def _layer_list(make, folder, config, dtype, serving):
+    """A layer-list decoder (decoder.py) with the tensors of model.safetensors."""
+    model = make(config, dtype=dtype, **serving)
     weights = SafeTensors(folder / "model.safetensors")
     for name in weights:
         kind, array = weights.get(name)
@@ -44,6 +43,18 @@ def _zugolorn(folder, config, dtype, serving):
             raise JsmError(UNSUPPORTED, f"tensor {name}: dtype {kind}")
         model.set_weight(name, array)
     return model.finalize()
+
+
+@register("Zugolorn")
+def _zugolorn(folder, config, dtype, serving):
+    from .decoder import zugolorn_model
+    return _layer_list(zugolorn_model, folder, config, dtype, serving)
+
+
+@register("Vagonex")
+def _vagonex(folder, config, dtype, serving):
+    from .decoder import vagonex_model
+    return _layer_list(vagonex_model, folder, config, dtype, serving)
 
 
 @register("Llama")
