@@ -317,6 +317,39 @@ def zugolorn_config(width):
             "layers": [attn, scan] * 4}
 
 
+def vagonex_config(width):
+    """Layers of a real model's proportions: two delta-rule layers, a decayed sum and chunked attention, twice; the second
+    attention layer uses the keys and values of the first."""
+    heads, ff = width // 128, {"kind": "dense", "ff": width * 43 // 16}
+    delta = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}, "mlp": ff}
+    light = {"type": "lightning", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-3 - 7 * h / heads) for h in range(heads)]}, "mlp": ff}
+    mix = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024 if width < 4096 else 4096},
+           "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 4096}}}
+    return {"architecture": "Vagonex", "width": width, "vocab": 32000, "norm": {"eps": 1e-5}, "postln_alpha": 2.0, "embedding": {"scale": 1.0},
+            "layers": [delta, delta, light, {"type": "attention", "mixer": mix, "mlp": ff},
+                       delta, delta, light, {"type": "attention", "mixer": {**mix, "kv_from": 3}, "mlp": ff}]}
+
+
+def vagonex_tensors(e):
+    """Matrices and vectors (shape, std, mean) of one Vagonex layer's mixer."""
+    m, H, n, v = e["mixer"], e["mixer"]["heads"], e["mixer"]["dim"], e["mixer"]["vdim"]
+    G = m.get("kv_heads", H)
+    rows, vecs = {"q": H * n, "g": H * v}, {}
+    if e["type"] == "attention":
+        rows["g"] = H
+        vecs = {"q.b": (H * n, 0.1, 0.0), "q.norm": (n, 0.1, 1.0), "sink": (H, 0.5, 0.0)}
+        if m.get("kv_from") is None:
+            rows.update(k=G * n, v=G * v)
+            vecs.update({"k.b": (G * n, 0.1, 0.0), "k.norm": (n, 0.1, 1.0), "v.b": (G * v, 0.1, 0.0)})
+    elif e["type"] == "lightning":
+        rows.update(k=H * n, v=H * v)
+        vecs = {"norm": (H * v, 0.1, 1.0)}
+    else:
+        rows.update(q=G * n, k=G * n, v=H * v, b=H, a=H)
+        vecs = {"A_log": (H, 0.5, 0.0), "dt_bias": (H, 0.5, -3.0), "norm": (v, 0.1, 1.0)}
+    return rows, vecs
+
+
 def random_tensors(cfg):
     """(name, bf16 bits) of every tensor: slices of one pool of normal numbers, scaled by a power of two near K^-1/2."""
     import numpy as np
@@ -335,7 +368,16 @@ def random_tensors(cfg):
     for i, e in enumerate(cfg["layers"]):
         p, m = f"l{i}.", e["mixer"]
         yield p + "norm1", draw((d,), 0.05, 0.4)
-        if e["type"] == "latent_attention":
+        if cfg["architecture"] == "Vagonex":
+            rows, vecs = vagonex_tensors(e)
+            shapes = {k: (r, d) for k, r in rows.items()}
+            shapes["o"] = (d, m["heads"] * m["vdim"])
+            for k, (n, std, mean) in vecs.items():
+                yield p + "mix." + k, draw((n,), std, mean)
+            if e["type"] == "delta":
+                for k in "qkv":
+                    yield p + f"mix.{k}.conv", draw((rows[k], m["conv"]), 0.5)
+        elif e["type"] == "latent_attention":
             H, r = m["heads"], m["kv_rank"]
             shapes = {"q": (H * (m["dim"] + m["rot_dim"]), d), "dkv": (r + m["rot_dim"], d), "uk": (H * m["dim"], r), "uv": (H * m["vdim"], r),
                       "o": (d, H * m["vdim"])}
@@ -357,12 +399,13 @@ def random_tensors(cfg):
 
 
 def run_decoder_workload(args):
-    """Prefill and decode throughput of the Zugolorn design at two widths and of the LLaMA shape of equal width and about
-    equal weight bytes, both through their host-buffer serving calls (token ids in, next tokens out, every step)."""
+    """Prefill and decode throughput of a layer-list design (zugolorn / vagonex) at two widths and of the LLaMA shape of equal
+    width and about equal weight bytes, both through their host-buffer serving calls (token ids in, next tokens out, every
+    step); vagonex: also of the Zugolorn design."""
     import numpy as np
     import torch
     import jasmine_b200 as jb
-    from jasmine_b200.decoder import zugolorn_model
+    from jasmine_b200.decoder import vagonex_model, zugolorn_model
     from jasmine_b200.model import Llama
     torch.cuda.set_device(0)
     hbm, peak_kind = measured_peaks()
@@ -395,40 +438,48 @@ def run_decoder_workload(args):
     widths = [args.width] if args.width else [2048, 4096]
     for width in widths:
         sampler.start()
-        cfg = zugolorn_config(width)
-        z = zugolorn_model(cfg, max_batch=64, max_context=8192, max_step_tokens=2048, pool_pages=64 * 12 + 128)
-        for name, bits in random_tensors(cfg):
-            z.set_weight(name, bits)
-        z.finalize()
-        z.stream = stream.cuda_stream
-        wbytes = z.step_bytes(0)[0]
-        params = wbytes / 2
         head = 32000 * width
+        designs = []  # (model, name, weight bytes, attention FLOPs of a prompt)
+        for design in (["vagonex", "zugolorn"] if args.workload == "vagonex" else ["zugolorn"]):
+            cfg = vagonex_config(width) if design == "vagonex" else zugolorn_config(width)
+            z = (vagonex_model if design == "vagonex" else zugolorn_model)(cfg, max_batch=64, max_context=8192, max_step_tokens=2048, pool_pages=64 * 12 + 128)
+            for name, bits in random_tensors(cfg):
+                z.set_weight(name, bits)
+            z.finalize()
+            z.stream = stream.cuda_stream
+            nb = z.step_bytes(0)[0]
+            layers = "2 x (2 delta, decayed sum, attention), ff" if design == "vagonex" else "4 x (latent attention + ff, scan)"
+            seen = [(e["mixer"]["mask"]["size"], e["mixer"]["heads"] * (e["mixer"]["dim"] + e["mixer"]["vdim"] + e["mixer"].get("rot_dim", 0)))
+                    for e in cfg["layers"] if "mask" in e["mixer"]]
+            designs.append((z, f"{design} w{width} {layers}, {nb / 1e9:.2f} GB", nb, lambda T, seen=seen: sum(2.0 * min(s, T / 2) * T * c for s, c in seen)))
+        wbytes = designs[0][2]
+        params = wbytes / 2
         # a LLaMA layer of this width: 4 d^2 + 3 d ffn
         ffn = width * 43 // 16
         n_llama = max(1, round((params - head) / (4 * width * width + 3 * width * ffn)))
         llama = Llama(n_llama, width, width // 128, width // 128, ffn, 32000, max_batch=64, max_context=1024, seed=SEED, pool_pages=64 * 16)
         lbytes = llama.step_bytes()[0]
-        names = (f"zugolorn w{width} 4 x (latent attention + ff, scan), {wbytes / 1e9:.2f} GB", f"llama w{width} {n_llama} layers, {lbytes / 1e9:.2f} GB")
+        llama_name = f"llama w{width} {n_llama} layers, {lbytes / 1e9:.2f} GB"
         torch.cuda.synchronize()
         with torch.cuda.stream(stream):
             for T in (512, 2048):
                 prompt = rng.integers(0, 32000, T).astype(np.int32)
 
-                def z_prefill():
-                    row, _ = z.admit(prompt)
-                    z.retire(row)
-                attn = sum(4.0 * min(e["mixer"]["mask"]["size"], T / 2) * T * e["mixer"]["heads"] * 160 for e in cfg["layers"] if e["type"] == "latent_attention")
-                emit(names[0], "prefill", timed(z_prefill, max(3, K // 8)), T, wbytes, 2.0 * T * (params - head) + attn, {"seq_len": T})
+                for z, name, nb, attn in designs:
+                    def z_prefill():
+                        row, _ = z.admit(prompt)
+                        z.retire(row)
+                    emit(name, "prefill", timed(z_prefill, max(3, K // 8)), T, nb, 2.0 * T * (nb / 2 - head) + attn(T), {"seq_len": T})
                 if T <= 512:
                     def l_prefill():
                         row, _ = llama.admit(prompt)
                         llama.retire(row)
                     attn = n_llama * 4.0 * T * T / 2 * width
-                    emit(names[1], "prefill", timed(l_prefill, max(3, K // 8)), T, lbytes, 2.0 * T * (lbytes / 2 - head) + attn, {"seq_len": T})
+                    emit(llama_name, "prefill", timed(l_prefill, max(3, K // 8)), T, lbytes, 2.0 * T * (lbytes / 2 - head) + attn, {"seq_len": T})
             for B in (1, 8, 64):
                 ctx = 512
-                for m, name, nb in ((z, names[0], lambda c: wbytes + B * z.step_bytes(c)[1]), (llama, names[1], lambda c: lbytes + B * c * llama.step_bytes()[1])):
+                runs = [(z, name, lambda c, z=z, nb=nb: nb + B * z.step_bytes(c)[1]) for z, name, nb, _ in designs]
+                for m, name, nb in runs + [(llama, llama_name, lambda c: lbytes + B * c * llama.step_bytes()[1])]:
                     for b in range(B):
                         m.admit(rng.integers(0, 32000, ctx).astype(np.int32))
                     ids, nxt = np.zeros(B, np.int32), np.zeros(B, np.int32)
@@ -441,7 +492,8 @@ def run_decoder_workload(args):
                     for b in range(B):
                         m.retire(0)
         jb.check_device_errors()
-        z.close()
+        for z, *_ in designs:
+            z.close()
         llama.close()
         print(json.dumps({"clocks": sampler.stop()}), flush=True)
 
@@ -610,11 +662,11 @@ def main():
     ap.add_argument("--layers", type=int, default=32, help="debug only: fewer layers (the result is then not a bench value)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-extras", action="store_true", help="headline only: skip the batch-1/64 legs, the kernel-level legs and the tp parity check")
-    ap.add_argument("--workload", default="decode", choices=["decode", "expr", "flash", "kvdecode", "gateup", "timeline", "zugolorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "expr", "flash", "kvdecode", "gateup", "timeline", "zugolorn", "vagonex"],
                     help="decode = the headline; expr / flash / kvdecode = configurations 2 / 3 / 4 of the baseline "
-                         "(kernel-level lines, one JSON line per kernel); zugolorn = prefill and decode throughput of "
+                         "(kernel-level lines, one JSON line per kernel); zugolorn, vagonex = prefill and decode throughput of "
                          "that design beside the LLaMA shape")
-    ap.add_argument("--width", type=int, default=0, help="zugolorn workload only: this width instead of both")
+    ap.add_argument("--width", type=int, default=0, help="zugolorn, vagonex workloads only: this width instead of both")
     ap.add_argument("--tp-emulate", type=int, default=1,
                     help="timeline workload only: run ONE rank of a tensor-parallel group of this size on one GPU")
     ap.add_argument("--profile-steps", type=int, default=0,
@@ -626,7 +678,7 @@ def main():
     args.warmup = max(args.warmup, 3)
     if args.workload == "timeline":
         return run_timeline(args)
-    if args.workload == "zugolorn":
+    if args.workload in ("zugolorn", "vagonex"):
         return run_decoder_workload(args)
     if args.workload != "decode":
         return run_kernel_workload(args)

@@ -98,7 +98,8 @@ struct jsm_decoder {
     float *x = nullptr, *y = nullptr, *wide = nullptr, *proj = nullptr, *dt_raw = nullptr, *gate32 = nullptr, *head_gate = nullptr, *logits = nullptr, *part = nullptr;
     void *xa = nullptr, *q = nullptr, *q_lat = nullptr, *o_lat = nullptr, *att = nullptr, *xz = nullptr, *xc = nullptr, *dt_op = nullptr,
          *scan_y = nullptr, *act = nullptr, *head_in = nullptr, *gathered = nullptr, *expanded = nullptr;
-    size_t part_floats = 0;
+    size_t part_floats = 0, chunk_bytes = 0;
+    void* chunk_ws = nullptr;
     float* ws = nullptr;
     size_t ws_floats = 0;
     int* counters = nullptr;
@@ -544,6 +545,7 @@ struct Pass {
     int n_want = 0;
     bool decode = false;       // one token per segment
     std::map<std::pair<int, int>, TileList> tiles_short, tiles_all;  // per (rows per token, rows per tile)
+    RecChunks chunks;          // of the passes that are no decode steps
     int32_t* meta = nullptr;
 };
 
@@ -630,7 +632,7 @@ static jsm_status recurrence_mixer(jsm_decoder* m, DecLayer& L, const Pass& P, c
         DEC_TRY(rec_step_launch(m->f32, d, L.rw, L.rs, m->c.norm_eps, P.tk, m->xz, m->xc, xin, m->wp, m->scan_y, st));
     } else {
         if (d.delta) DEC_TRY(linear(m, L.xp, xin, m->wp, m->proj, true, T, st));
-        DEC_TRY(rec_scan_launch(m->f32, d, L.rw, L.rs, m->c.norm_eps, P.tk, m->xz, m->xc, m->proj, m->scan_y, st));
+        DEC_TRY(rec_scan_launch(m->f32, d, L.rw, L.rs, m->c.norm_eps, P.tk, P.chunks, m->xz, m->xc, m->proj, m->scan_y, st));
         DEC_TRY(short_conv_carry_launch(m->f32, m->xz, d.raw_cols(), d.conv_cols(), d.taps, L.rs.conv, P.tk, st));
     }
     return linear(m, L.out, m->scan_y, d.out_cols(), m->y, true, T, st);
@@ -749,6 +751,16 @@ static jsm_status run_pass(jsm_decoder* m, std::vector<PassSeg> segs, const int3
         P.tiles_all[{H, rows}] = TileList{so, ro, (int)sg.size(), T};
         P.tiles_short[{H, rows}] = TileList{so, ro, n_short, tok_short};
     }
+    const size_t chunk_off = M.size();
+    if (m->chunk_bytes > 0 && !P.decode) {
+        std::vector<int32_t> seg, t0, first;
+        for (int i = 0; i < E; ++i) {
+            first.push_back((int32_t)seg.size());
+            for (int t = 0; t < segs[i].len; t += REC_CHUNK) { seg.push_back(i); t0.push_back(t); }
+        }
+        P.chunks.n_chunks = (int)seg.size();
+        for (const auto* v : {&seg, &t0, &first}) M.insert(M.end(), v->begin(), v->end());
+    }
     if (M.size() > m->meta_cap) JSM_FAIL(JSM_SHAPE, "jsm_decoder: step metadata of %zu words (room for %zu)", M.size(), m->meta_cap);
     memcpy(m->h_meta, M.data(), M.size() * sizeof(int32_t));
     JSM_CUDA_CHECK(cudaMemcpyAsync(m->meta, m->h_meta, M.size() * sizeof(int32_t), cudaMemcpyHostToDevice, st));
@@ -758,6 +770,9 @@ static jsm_status run_pass(jsm_decoder* m, std::vector<PassSeg> segs, const int3
     P.tk.seg_start = m->meta + seg_off; P.tk.seg_len = P.tk.seg_start + E; P.tk.seg_pos0 = P.tk.seg_len + E;
     P.tk.seg_row = P.tk.seg_pos0 + E; P.tk.seg_slot = P.tk.seg_row + E;
     P.want = m->meta + want_off;
+    P.chunks.chunk_seg = m->meta + chunk_off; P.chunks.chunk_t0 = P.chunks.chunk_seg + P.chunks.n_chunks;
+    P.chunks.seg_chunk0 = P.chunks.chunk_t0 + P.chunks.n_chunks;
+    P.chunks.ws = m->chunk_ws;
 
     const int n_head = std::min(P.n_want, m->cap_rows);
     const bool graph = P.decode && !m->tap && (P.n_want == 0 || (P.n_want == E && E <= m->cap_rows));
@@ -1012,6 +1027,7 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
             xc = std::max(xc, (size_t)d.conv_cols());
             sy = std::max(sy, (size_t)d.out_cols());
             proj = std::max(proj, (size_t)d.ba_cols());
+            if (!m->f32 && rec_chunk_usable(d)) m->chunk_bytes = std::max(m->chunk_bytes, rec_chunk_bytes(d));
         } else {
             const ScanDims& d = L.sd;
             DEC_TRY(dalloc(m, &L.state.S, sizeof(float) * (size_t)c.max_batch * d.ip() * d.np()));
@@ -1063,6 +1079,11 @@ jsm_status jsm_decoder_finalize(jsm_decoder* m) {
     for (const DecLayer& L : m->layers)
         if (L.is_attention()) tilings[L.tiling(false)] = tilings[L.tiling(true)] = 1;
     m->meta_cap = 4 * T + 5 * T + 64;
+    const size_t max_chunks = T / REC_CHUNK + c.max_batch;
+    if (m->chunk_bytes > 0) {
+        DEC_TRY(dalloc(m, &m->chunk_ws, m->chunk_bytes * max_chunks));
+        m->meta_cap += 2 * max_chunks + c.max_batch;
+    }
     for (auto& t : tilings) m->meta_cap += 2 * (T * t.first.first / t.first.second + T + 1);
     DEC_TRY(dalloc(m, &m->meta, 4 * m->meta_cap));
     JSM_CUDA_CHECK(cudaMallocHost(reinterpret_cast<void**>(&m->h_meta), 4 * m->meta_cap));

@@ -192,10 +192,20 @@ struct RecState {
     void* conv = nullptr;  // act [slots][taps - 1][conv cols]
     float* S = nullptr;    // [slots][H][kp][vp]
 };
+constexpr int REC_CHUNK = 64;  // tokens of a chunk of the tensor-core kernels
+// The chunks of a pass: segment by segment, the last one of a segment may be short.  ws: rec_chunk_bytes per chunk.
+struct RecChunks {
+    const int32_t *chunk_seg = nullptr, *chunk_t0 = nullptr;  // [n_chunks] segment, first token within it
+    const int32_t* seg_chunk0 = nullptr;                      // [n_segs] first chunk
+    int n_chunks = 0;
+    void* ws = nullptr;
+};
 bool rec_usable(const RecDims& d);
+bool rec_chunk_usable(const RecDims& d);
+size_t rec_chunk_bytes(const RecDims& d);
 // raw: the input projection; qkv: its first columns after the convolution; ba f32 [T][ba cols]; out act [T][H vp]: normed, gated
-jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const void* raw,
-                           const void* qkv, const float* ba, void* out, cudaStream_t st);
+jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const RecChunks& ch,
+                           const void* raw, const void* qkv, const float* ba, void* out, cudaStream_t st);
 // the same for one token per segment; b and a come from the layer's input x (act [T][x_pitch])
 jsm_status rec_step_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const void* raw,
                            const void* qkv, const void* x, int x_pitch, void* out, cudaStream_t st);

@@ -9,14 +9,24 @@
 // state and all of this arithmetic is fp32; q, k, v, o and the gates z are activations (bf16 or f32).  A sequence's state lives
 // in a slot; a segment that starts at position 0 starts from zeros whatever the slot holds.
 //
+// Prompts of bf16 models run on the tensor cores in chunks of 64 tokens (rec_chunk_prep, rec_chunk): with G the running sum of
+// log g in the chunk and S0 the state before it,
+//     (I + A) U = diag(beta) (V - diag(e^G) K S0),   A[t][j] = beta_t e^(G_t - G_j) (k_t . k_j), j < t   (decayed sum: U = V)
+//     O = diag(e^G) Q S0 + P U,                      P[t][j] = e^(G_t - G_j) (q_t . k_j), j <= t
+//     S = e^(G_end) S0 + sum_j e^(G_end - G_j) k_j u_j^T.
+// f32 models and heads of more than 128 key components walk the tokens one by one (rec_scan), as does a decode step (rec_step).
+//
 // Row of the input projection: [q: G heads | k: G heads | v: H heads | z: H heads], heads at pitches padded to 8; head h uses
 // query / key head h / (H / G).  State: [slot][head][kp][vp].
 #include "decoder_ops.cuh"
 #include "mma_utils.cuh"
+#include "tc_utils.cuh"
 #include <math.h>
 #include <algorithm>
 
 namespace jsm {
+
+using tc::smem_u32;
 
 constexpr float UNIT_EPS = 1e-6f;
 
@@ -110,6 +120,407 @@ __global__ void __launch_bounds__(RS_THREADS) rec_scan_kernel(RecArgs a, RecDims
 #pragma unroll
         for (int i = 0; i < NS; ++i)
             if (sub + 8 * i < kp) state[(long long)(sub + 8 * i) * vp] = S[i];
+}
+
+// ---- prompts on the tensor cores ----------------------------------------------------------------------------------
+// The matrix operands are the bf16 activations themselves: unit norms, decays and beta are fp32 factors per token around the
+// products.  fp32 operands (the state, U and its right-hand side, the inverse of I + A) enter as a sum of two bf16 numbers, so
+// that what feeds the state keeps 16 bits; P enters as bf16, as attention weights do.
+constexpr int RC_C = REC_CHUNK;       // tokens per chunk
+constexpr int RC_P = RC_C + 8;        // pitch of a chunk matrix (bf16)
+constexpr int RC_MAT = RC_C * RC_P * 2;
+constexpr int RC_SCAL = 4 * RC_C * 4 + 16;  // per token: factors of v, K S0, Q S0 and k u^T; the chunk's decay
+constexpr int RC_ERR_FULL = 71;
+constexpr float LOG_MIN = -120.0f;    // e^-120 is 0 in fp32
+__host__ __device__ inline int rc_block(bool delta) { return (delta ? 3 : 1) * RC_MAT + RC_SCAL; }  // bytes per (chunk, head): [T hi | T lo |] P | factors
+
+// Per (chunk, head): the factors, P, and the inverse T of I + A.  Eight warps.
+template <bool DELTA>
+__global__ void __launch_bounds__(256) rec_chunk_prep_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ chunk_seg, const int32_t* __restrict__ chunk_t0,
+                                                             uint8_t* __restrict__ ws, int kw) {
+    extern __shared__ __align__(16) uint8_t rc_dyn[];
+    const int pitch = kw + 8;  // kw: key components rounded up to 16
+    __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(rc_dyn);          // [64][pitch]
+    __nv_bfloat16* qs = ks + RC_C * pitch;                                 // [64][pitch]
+    float* As = reinterpret_cast<float*>(qs + RC_C * pitch);               // [64][68], strictly lower
+    float* Xs = As + RC_C * 68;                                            // [64][68]: the inverse
+    __shared__ float G[RC_C], rk[RC_C], rq[RC_C], beta[RC_C], half_sum;
+    chain_trigger();
+    chain_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int seg = chunk_seg[blockIdx.x], t0 = chunk_t0[blockIdx.x], h = blockIdx.y, g = h / (d.H / d.G);
+    const int n = min(RC_C, a.seg_len[seg] - t0), kp = d.kp(), vec = kw / 8;
+    const long long first = a.seg_start[seg] + t0;
+    const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(a.qkv) + first * d.conv_cols() + g * kp;
+    for (int i = tid; i < RC_C * vec; i += 256) {
+        const int r = i / vec, c = (i - r * vec) * 8;
+        uint4 k = make_uint4(0, 0, 0, 0), q = k;
+        if (r < n && c < kp) {
+            const __nv_bfloat16* row = qkv + (long long)r * d.conv_cols() + c;
+            q = *reinterpret_cast<const uint4*>(row);
+            k = *reinterpret_cast<const uint4*>(row + d.G * kp);
+        }
+        *reinterpret_cast<uint4*>(ks + r * pitch + c) = k;
+        *reinterpret_cast<uint4*>(qs + r * pitch + c) = q;
+    }
+    // running sum of the log decays
+    if (tid < RC_C) {
+        float lg = 0.0f, b = 0.0f;
+        if (tid < n) {
+            if (DELTA) {
+                const float* ba = a.ba + (first + tid) * d.ba_cols();
+                b = rec_sigmoid(ba[h]);
+                lg = fmaxf(a.A[h] * rec_softplus(ba[d.ba_cols() / 2 + h] + a.dt_bias[h]), LOG_MIN);
+            } else {
+                lg = fmaxf(a.log_decay[h], LOG_MIN);
+            }
+        }
+        beta[tid] = b;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float v = __shfl_up_sync(0xffffffffu, lg, o);
+            if (lane >= o) lg += v;
+        }
+        G[tid] = lg;
+        if (tid == 31) half_sum = lg;
+    }
+    __syncthreads();
+    if (tid >= 32 && tid < RC_C) G[tid] += half_sum;
+    if (DELTA) {  // lengths: four threads per row of k, then of q
+        for (int m = 0; m < 2; ++m) {
+            const __nv_bfloat16* row = (m ? qs : ks) + (tid >> 2) * pitch;
+            float ss = 0.0f;
+            for (int c = (tid & 3) * 8; c < kw; c += 32) {
+                float v[8];
+                load_f32x8(row + c, v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+            }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            if ((tid & 3) == 0) (m ? rq : rk)[tid >> 2] = (m ? a.q_scale : 1.0f) / sqrtf(ss + UNIT_EPS);
+        }
+    } else if (tid < RC_C) {
+        rk[tid] = rq[tid] = 1.0f;
+    }
+    __syncthreads();
+    uint8_t* out = ws + ((long long)blockIdx.x * d.H + h) * rc_block(DELTA);
+    __nv_bfloat16* Pm = reinterpret_cast<__nv_bfloat16*>(out + (DELTA ? 2 * RC_MAT : 0));
+    // products with the keys: warps 0-3 k . k (16 rows each), warps 4-7 q . k
+    if (DELTA || warp >= 4) {
+        const bool is_q = warp >= 4;
+        const int mt = warp & 3, lm = lane >> 3, lr = lane & 7;
+        float acc[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.0f;
+        const uint32_t a_addr = smem_u32((is_q ? qs : ks) + (mt * 16 + (lm & 1) * 8 + lr) * pitch + (lm >> 1) * 8);
+        const uint32_t b_addr = smem_u32(ks + ((lm >> 1) * 8 + lr) * pitch + (lm & 1) * 8);
+        for (int k = 0; k < kw; k += 16) {
+            uint32_t af[4];
+            ldsm_x4(a_addr + k * 2, af);
+#pragma unroll
+            for (int jp = 0; jp < 4; ++jp) {
+                if (jp > mt) break;
+                uint32_t bf[4];
+                ldsm_x4(b_addr + (jp * 16 * pitch + k) * 2, bf);
+                mma_16816(acc[2 * jp], af, bf[0], bf[1]);
+                mma_16816(acc[2 * jp + 1], af, bf[2], bf[3]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+                const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, c = j * 8 + (lane & 3) * 2;
+                float v[2];
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const bool on = is_q ? c + x <= t : c + x < t;
+                    v[x] = on ? acc[j][e + x] * rk[c + x] * (is_q ? rq[t] : beta[t] * rk[t]) * expf(G[t] - G[c + x]) : 0.0f;
+                }
+                if (is_q) *reinterpret_cast<uint32_t*>(Pm + t * RC_P + c) = pack_bf16x2(v[0], v[1]);
+                else *reinterpret_cast<float2*>(As + t * 68 + c) = make_float2(v[0], v[1]);
+            }
+    }
+    if (tid < RC_C) {
+        float* f = reinterpret_cast<float*>(out + (DELTA ? 3 : 1) * RC_MAT);
+        const bool on = tid < n;
+        const float e = expf(G[tid]), last = G[RC_C - 1];
+        f[tid] = !on ? 0.0f : DELTA ? beta[tid] : 1.0f;
+        f[RC_C + tid] = on ? beta[tid] * e * rk[tid] : 0.0f;
+        f[2 * RC_C + tid] = on ? e * rq[tid] : 0.0f;
+        f[3 * RC_C + tid] = on ? expf(last - G[tid]) * rk[tid] : 0.0f;
+        if (tid == 0) f[4 * RC_C] = expf(last);
+    }
+    if (!DELTA) return;
+    __syncthreads();
+    // column j of the inverse by forward substitution, x_t = [t = j] - sum_{i < t} A[t][i] x_i; four threads per column: thread p
+    // holds the rows 16 q + 4 p + e
+    const int j = tid >> 2, p = tid & 3;
+    float x[4][4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[q][e] = 0.0f;
+#pragma unroll
+    for (int tq = 0; tq < 4; ++tq)
+#pragma unroll
+        for (int tr = 0; tr < 16; ++tr) {
+            const int t = tq * 16 + tr;
+            float s = 0.0f;
+#pragma unroll
+            for (int q = 0; q <= tq; ++q) {
+                const float4 r = *reinterpret_cast<const float4*>(As + t * 68 + q * 16 + p * 4);
+                s = fmaf(r.x, x[q][0], s); s = fmaf(r.y, x[q][1], s); s = fmaf(r.z, x[q][2], s); s = fmaf(r.w, x[q][3], s);
+            }
+            s += __shfl_xor_sync(0xffffffffu, s, 1);
+            s += __shfl_xor_sync(0xffffffffu, s, 2);
+            if (p == tr / 4) x[tq][tr % 4] = (t == j ? 1.0f : 0.0f) - s;
+        }
+#pragma unroll
+    for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) Xs[(q * 16 + p * 4 + e) * 68 + j] = x[q][e];
+    __syncthreads();
+    __nv_bfloat16* Th = reinterpret_cast<__nv_bfloat16*>(out);
+    for (int i = tid; i < RC_C * 8; i += 256) {
+        const int r = i >> 3, c = (i & 7) * 8;
+        float v[8], lo[8];
+        load_f32x8(Xs + r * 68 + c, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) lo[e] = v[e] - __bfloat162float(__float2bfloat16_rn(v[e]));
+        store_f32x8(Th + r * RC_P + c, v);
+        store_f32x8(Th + RC_MAT / 2 + r * RC_P + c, lo);
+    }
+}
+
+// two fp32 numbers as bf16 pairs: hi + lo
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16x2(a, b);
+    lo = pack_bf16x2(a - bf16lo(hi), b - bf16hi(hi));
+}
+__device__ __forceinline__ uint32_t rc_movmatrix(uint32_t x) {
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
+}
+
+// A warp owns 16 columns of one head's state, transposed (columns x key components) in accumulator registers, and walks the
+// segment's chunks: every product has the warp's columns as rows, so that results turn into operands in registers and the
+// warps of a CTA only share the tiles of K, Q, V and the chunk matrices.  Two stages, filled by bulk copies (a row each; the
+// chunk matrices in one); waits are bounded.  KT: 16-wide steps of the key components.
+template <int KT, bool DELTA>
+__global__ void __launch_bounds__(128) rec_chunk_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
+    constexpr int KP = KT * 16 + 8;
+    extern __shared__ __align__(16) uint8_t rc_dyn[];
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int abort_flag;
+    chain_trigger();
+    const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nw = nthr / 32;
+    const int vpitch = nw * 16 + 8, block = rc_block(DELTA);
+    const int stage_bytes = 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + block;
+    for (int i = tid; i < 2 * stage_bytes / 16; i += nthr) reinterpret_cast<uint4*>(rc_dyn)[i] = make_uint4(0, 0, 0, 0);  // rows and columns that no copy fills
+    if (tid == 0) {
+        abort_flag = 0;
+        tc::mbar_init(&full[0], 1);
+        tc::mbar_init(&full[1], 1);
+        tc::mbar_fence_init();
+    }
+    tc::fence_proxy_async_smem();
+    __syncthreads();
+    chain_wait();
+    const int h = blockIdx.y, g = h / (d.H / d.G), seg = blockIdx.z, kp = d.kp(), vp = d.vp(), cc = d.conv_cols();
+    const int c0 = blockIdx.x * nw * 16, n_cols = min(nw * 16, vp - c0);
+    const int start = a.seg_start[seg], len = a.seg_len[seg], n_chunks = (len + RC_C - 1) / RC_C;
+    const uint8_t* blocks = ws + ((long long)seg_chunk0[seg] * d.H + h) * block;
+    const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(a.qkv) + (long long)start * cc;
+    auto load = [&](int ci) {
+        uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
+        const int n = min(RC_C, len - ci * RC_C);
+        if (tid == 0) {
+            tc::mbar_expect_tx(&full[ci & 1], (uint32_t)(n * (2 * kp + n_cols) * 2 + block));
+            tc::bulk_load(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2, blocks + (long long)ci * d.H * block, block, &full[ci & 1]);
+        }
+        for (int i = tid; i < 3 * n; i += nthr) {
+            const int m = i / n, r = i - m * n;  // k, q, v
+            const __nv_bfloat16* row = qkv + (long long)(ci * RC_C + r) * cc;
+            if (m < 2) tc::bulk_load(st + (m * RC_C + r) * KP * 2, row + (m == 0 ? d.G * kp : 0) + g * kp, kp * 2, &full[ci & 1]);
+            else tc::bulk_load(st + 2 * RC_C * KP * 2 + r * vpitch * 2, row + 2 * d.G * kp + h * vp + c0, n_cols * 2, &full[ci & 1]);
+        }
+    };
+    load(0);
+    // state: rows (lane / 4, + 8) of this warp's columns, key components 8 j + (lane % 4) * 2, + 1
+    float* state = a.S + ((long long)a.seg_slot[seg] * d.H + h) * kp * vp;
+    const bool fresh = a.seg_pos0[seg] == 0;
+    const int cr = c0 + warp * 16 + (lane >> 2), kc = (lane & 3) * 2;
+    float S[2 * KT][4];
+#pragma unroll
+    for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int k = j * 8 + kc + (e & 1), c = cr + (e >> 1) * 8;
+            S[j][e] = !fresh && k < kp && c < vp ? state[(long long)k * vp + c] : 0.0f;
+        }
+    const int lm = lane >> 3, lr = lane & 7;
+    bool ok = true;
+    for (int ci = 0; ci < n_chunks; ++ci) {
+        if (ci > 0) __syncthreads();  // the other stage has been used up
+        if (ci + 1 < n_chunks) load(ci + 1);
+        ok = tc::mbar_wait(&full[ci & 1], (ci >> 1) & 1, &abort_flag, err, RC_ERR_FULL);
+        if (!__syncthreads_and(ok)) { ok = false; break; }
+        const uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
+        const uint32_t kb = smem_u32(st), qb = kb + RC_C * KP * 2, vb = qb + RC_C * KP * 2, tb = vb + RC_C * vpitch * 2;
+        const uint32_t pm = tb + (DELTA ? 2 * RC_MAT : 0);
+        const float* f = reinterpret_cast<const float*>(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + (DELTA ? 3 : 1) * RC_MAT);
+        float u[8][4], o[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.0f;
+            o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
+        }
+        // S0^T K^T and S0^T Q^T
+        const uint32_t n_off = ((lm >> 1) * 8 + lr) * KP * 2 + (lm & 1) * 16;  // matrices: tokens 0-7 / 8-15 (lm >> 1), components + 8 (lm & 1)
+#pragma unroll
+        for (int kk = 0; kk < KT; ++kk) {
+            uint32_t hi[4], lo[4];
+            split2(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
+            split2(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
+            split2(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
+            split2(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+            for (int jp = 0; jp < 4; ++jp) {
+                uint32_t b[4];
+                if (DELTA) {
+                    ldsm_x4(kb + n_off + jp * 16 * KP * 2 + kk * 32, b);
+                    mma_16816(u[2 * jp], hi, b[0], b[1]);
+                    mma_16816(u[2 * jp + 1], hi, b[2], b[3]);
+                    mma_16816(u[2 * jp], lo, b[0], b[1]);
+                    mma_16816(u[2 * jp + 1], lo, b[2], b[3]);
+                }
+                ldsm_x4(qb + n_off + jp * 16 * KP * 2 + kk * 32, b);
+                mma_16816(o[2 * jp], hi, b[0], b[1]);
+                mma_16816(o[2 * jp + 1], hi, b[2], b[3]);
+                mma_16816(o[2 * jp], lo, b[0], b[1]);
+                mma_16816(o[2 * jp + 1], lo, b[2], b[3]);
+            }
+        }
+        // right-hand side: f0 v - f1 (K S0), or the values themselves
+#pragma unroll
+        for (int jp = 0; jp < 4; ++jp) {
+            uint32_t v[4];  // matrices: tokens 0-7 / 8-15 (lm >> 1), columns + 8 (lm & 1); transposed
+            ldsm_x4_trans(vb + (jp * 16 + (lm >> 1) * 8 + lr) * vpitch * 2 + warp * 32 + (lm & 1) * 16, v);
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int j = 2 * jp + x;
+                const float2 fv = *reinterpret_cast<const float2*>(f + j * 8 + kc);
+                float2 fk = make_float2(0.0f, 0.0f);
+                if (DELTA) fk = *reinterpret_cast<const float2*>(f + RC_C + j * 8 + kc);
+                u[j][0] = fv.x * bf16lo(v[2 * x]) - fk.x * u[j][0];
+                u[j][1] = fv.y * bf16hi(v[2 * x]) - fk.y * u[j][1];
+                u[j][2] = fv.x * bf16lo(v[2 * x + 1]) - fk.x * u[j][2];
+                u[j][3] = fv.y * bf16hi(v[2 * x + 1]) - fk.y * u[j][3];
+            }
+        }
+        const uint32_t m_off = ((lm >> 1) * 8 + lr) * RC_P * 2 + (lm & 1) * 16;
+        if (DELTA) {  // U = T R
+            float w[8][4];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.0f;
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                uint32_t hi[4], lo[4];
+                split2(u[2 * kk][0], u[2 * kk][1], hi[0], lo[0]);
+                split2(u[2 * kk][2], u[2 * kk][3], hi[1], lo[1]);
+                split2(u[2 * kk + 1][0], u[2 * kk + 1][1], hi[2], lo[2]);
+                split2(u[2 * kk + 1][2], u[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+                for (int jp = kk; jp < 4; ++jp) {  // (lower triangle)
+                    uint32_t b[4], c[4];
+                    ldsm_x4(tb + m_off + jp * 16 * RC_P * 2 + kk * 32, b);
+                    ldsm_x4(tb + RC_MAT + m_off + jp * 16 * RC_P * 2 + kk * 32, c);
+                    mma_16816(w[2 * jp], hi, b[0], b[1]);
+                    mma_16816(w[2 * jp + 1], hi, b[2], b[3]);
+                    mma_16816(w[2 * jp], lo, b[0], b[1]);
+                    mma_16816(w[2 * jp + 1], lo, b[2], b[3]);
+                    mma_16816(w[2 * jp], hi, c[0], c[1]);
+                    mma_16816(w[2 * jp + 1], hi, c[2], c[3]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) u[j][e] = w[j][e];
+        }
+        // O = f2 (Q S0) + P U
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float2 fq = *reinterpret_cast<const float2*>(f + 2 * RC_C + j * 8 + kc);
+            o[j][0] *= fq.x; o[j][1] *= fq.y; o[j][2] *= fq.x; o[j][3] *= fq.y;
+        }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            const uint32_t hi[4] = {pack_bf16x2(u[2 * kk][0], u[2 * kk][1]), pack_bf16x2(u[2 * kk][2], u[2 * kk][3]),
+                                    pack_bf16x2(u[2 * kk + 1][0], u[2 * kk + 1][1]), pack_bf16x2(u[2 * kk + 1][2], u[2 * kk + 1][3])};
+#pragma unroll
+            for (int jp = kk; jp < 4; ++jp) {
+                uint32_t b[4];
+                ldsm_x4(pm + m_off + jp * 16 * RC_P * 2 + kk * 32, b);
+                mma_16816(o[2 * jp], hi, b[0], b[1]);
+                mma_16816(o[2 * jp + 1], hi, b[2], b[3]);
+            }
+        }
+        // S = decay S0 + (f3 U)^T K
+        const float decay = f[4 * RC_C];
+#pragma unroll
+        for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) S[j][e] *= decay;
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            const float2 f0 = *reinterpret_cast<const float2*>(f + 3 * RC_C + kk * 16 + kc), f1 = *reinterpret_cast<const float2*>(f + 3 * RC_C + kk * 16 + 8 + kc);
+            uint32_t hi[4], lo[4];
+            split2(u[2 * kk][0] * f0.x, u[2 * kk][1] * f0.y, hi[0], lo[0]);
+            split2(u[2 * kk][2] * f0.x, u[2 * kk][3] * f0.y, hi[1], lo[1]);
+            split2(u[2 * kk + 1][0] * f1.x, u[2 * kk + 1][1] * f1.y, hi[2], lo[2]);
+            split2(u[2 * kk + 1][2] * f1.x, u[2 * kk + 1][3] * f1.y, hi[3], lo[3]);
+#pragma unroll
+            for (int jp = 0; jp < KT; ++jp) {
+                uint32_t b[4];  // matrices: tokens 0-7 / 8-15 (lm & 1), components + 8 (lm >> 1); transposed
+                ldsm_x4_trans(kb + (kk * 16 + (lm & 1) * 8 + lr) * KP * 2 + jp * 32 + (lm >> 1) * 16, b);
+                mma_16816(S[2 * jp], hi, b[0], b[1]);
+                mma_16816(S[2 * jp + 1], hi, b[2], b[3]);
+                mma_16816(S[2 * jp], lo, b[0], b[1]);
+                mma_16816(S[2 * jp + 1], lo, b[2], b[3]);
+            }
+        }
+        // output rows: token, this warp's columns
+        const int n = len - ci * RC_C, col = c0 + warp * 16 + kc;
+        __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (long long)(start + ci * RC_C) * d.H * vp + h * vp + col;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const uint32_t w0 = rc_movmatrix(pack_bf16x2(o[j][0], o[j][1])), w1 = rc_movmatrix(pack_bf16x2(o[j][2], o[j][3]));
+            const int t = j * 8 + (lane >> 2);
+            if (t < n) {
+                if (col < vp) *reinterpret_cast<uint32_t*>(out + (long long)t * d.H * vp) = w0;
+                if (col + 8 < vp) *reinterpret_cast<uint32_t*>(out + (long long)t * d.H * vp + 8) = w1;
+            }
+        }
+    }
+    if (!ok) {  // a copy did not arrive: let the ones in flight land (bounded); the host learns of it
+        if (tid == 0) {
+            const long long t = clock64();
+            while (clock64() - t < tc::WAIT_LIMIT_CYCLES / 4) {}
+        }
+        __syncthreads();
+        return;
+    }
+#pragma unroll
+    for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int k = j * 8 + kc + (e & 1), c = cr + (e >> 1) * 8;
+            if (k < kp && c < vp) state[(long long)k * vp + c] = S[j][e];
+        }
 }
 
 // ---- decode step: one token per segment ---------------------------------------------------------------------------
@@ -338,12 +749,48 @@ static jsm_status norm_typed(const RecDims& d, const RecArgs& a, int n_tok, cuda
 
 bool rec_usable(const RecDims& d) { return d.dk <= 256 && d.dv <= 1024; }
 
-jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const void* raw,
-                           const void* qkv, const float* ba, void* out, cudaStream_t st) {
+// the chunk kernels: key components in 16-wide steps, rounded up to an instance
+static int chunk_kt(const RecDims& d) { return d.kp() <= 32 ? 2 : d.kp() <= 64 ? 4 : 8; }
+bool rec_chunk_usable(const RecDims& d) { return d.dk <= 128 && d.dv <= 1024; }
+size_t rec_chunk_bytes(const RecDims& d) { return (size_t)d.H * rc_block(d.delta); }
+
+template <int KT, bool DELTA>
+static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, cudaStream_t st) {
+    static bool attr_done = false;
+    if (!attr_done) {
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_prep_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024));
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_kernel<KT, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+        attr_done = true;
+    }
+    const int kw = KT * 16;
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_prep_kernel<DELTA>, dim3(ch.n_chunks, d.H), dim3(256), (size_t)2 * RC_C * (kw + 8) * 2 + 2 * RC_C * 68 * 4, st, a, d,
+                                  ch.chunk_seg, ch.chunk_t0, static_cast<uint8_t*>(ch.ws), kw));
+    JSM_LAUNCH_CHECK();
+    // warps per CTA: a warp keeps a scheduler busy, so two while the SMs suffice and four beyond
+    const int warps = (d.vp() + 15) / 16, nw = std::min(warps, (long long)n_segs * d.H * ((warps + 1) / 2) > 2 * sm_count() ? 4 : 2);
+    const size_t smem = 2 * ((size_t)2 * RC_C * (kw + 8) * 2 + RC_C * (nw * 16 + 8) * 2 + rc_block(DELTA));
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((warps + nw - 1) / nw, d.H, n_segs), dim3(nw * 32), smem, st, a, d, ch.seg_chunk0,
+                                  static_cast<const uint8_t*>(ch.ws), tc_error_word()));
+    JSM_LAUNCH_CHECK();
+    return JSM_OK;
+}
+template <bool DELTA>
+static jsm_status chunk_sized(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, cudaStream_t st) {
+    switch (chunk_kt(d)) {
+        case 2: return chunk_go<2, DELTA>(a, d, ch, n_segs, st);
+        case 4: return chunk_go<4, DELTA>(a, d, ch, n_segs, st);
+        default: return chunk_go<8, DELTA>(a, d, ch, n_segs, st);
+    }
+}
+
+jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const RecChunks& ch,
+                           const void* raw, const void* qkv, const float* ba, void* out, cudaStream_t st) {
     if (!rec_usable(d)) JSM_FAIL(JSM_UNSUPPORTED, "linear recurrence: heads of %d / %d components (at most 256 / 1024)", d.dk, d.dv);
     RecArgs a = rec_args(f32, d, w, s, tk, raw, qkv, out, eps);
     a.ba = ba;
-    jsm_status r = f32 ? (d.delta ? scan_sized<float, true>(a, d, tk.n_segs, st) : scan_sized<float, false>(a, d, tk.n_segs, st))
+    jsm_status r;
+    if (!f32 && rec_chunk_usable(d)) r = d.delta ? chunk_sized<true>(a, d, ch, tk.n_segs, st) : chunk_sized<false>(a, d, ch, tk.n_segs, st);
+    else r = f32 ? (d.delta ? scan_sized<float, true>(a, d, tk.n_segs, st) : scan_sized<float, false>(a, d, tk.n_segs, st))
                        : (d.delta ? scan_sized<__nv_bfloat16, true>(a, d, tk.n_segs, st) : scan_sized<__nv_bfloat16, false>(a, d, tk.n_segs, st));
     if (r != JSM_OK) return r;
     return f32 ? norm_typed<float>(d, a, tk.T, st) : norm_typed<__nv_bfloat16>(d, a, tk.T, st);
