@@ -134,6 +134,11 @@ constexpr int RC_ERR_FULL = 71;
 constexpr float LOG_MIN = -120.0f;    // e^-120 is 0 in fp32
 __host__ __device__ inline int rc_block(bool delta) { return (delta ? 3 : 1) * RC_MAT + RC_SCAL; }  // bytes per (chunk, head): [T hi | T lo |] P | factors
 
+__host__ __device__ inline int rc_prep_tiles(int kw, bool delta) {  // bytes of the tiles of K and Q, and of the inverse behind them
+    const int tiles = 2 * RC_C * (kw + 8) * 2, x = delta ? RC_C * 68 * 4 : 0;
+    return tiles > x ? tiles : x;
+}
+
 // Per (chunk, head): the factors, P, and the inverse T of I + A.  Eight warps.
 template <bool DELTA>
 __global__ void __launch_bounds__(256) rec_chunk_prep_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ chunk_seg, const int32_t* __restrict__ chunk_t0,
@@ -142,8 +147,8 @@ __global__ void __launch_bounds__(256) rec_chunk_prep_kernel(RecArgs a, RecDims 
     const int pitch = kw + 8;  // kw: key components rounded up to 16
     __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(rc_dyn);          // [64][pitch]
     __nv_bfloat16* qs = ks + RC_C * pitch;                                 // [64][pitch]
-    float* As = reinterpret_cast<float*>(qs + RC_C * pitch);               // [64][68], strictly lower
-    float* Xs = As + RC_C * 68;                                            // [64][68]: the inverse
+    float* As = reinterpret_cast<float*>(rc_dyn + rc_prep_tiles(kw, DELTA));  // [64][68], strictly lower
+    float* Xs = reinterpret_cast<float*>(rc_dyn);                          // [64][68]: the inverse, where the tiles were
     __shared__ float G[RC_C], rk[RC_C], rq[RC_C], beta[RC_C], half_sum;
     chain_trigger();
     chain_wait();
@@ -305,32 +310,39 @@ __device__ __forceinline__ uint32_t rc_movmatrix(uint32_t x) {
     return y;
 }
 
-// A warp owns 16 columns of one head's state, transposed (columns x key components) in accumulator registers, and walks the
-// segment's chunks: every product has the warp's columns as rows, so that results turn into operands in registers and the
-// warps of a CTA only share the tiles of K, Q, V and the chunk matrices.  Two stages, filled by bulk copies (a row each; the
-// chunk matrices in one); waits are bounded.  KT: 16-wide steps of the key components.
+// A CTA owns 16 or 32 columns of one head's state and walks the segment's chunks.  Every product is taken transposed - rows are
+// state columns, 16 per group of four warps - so that the state, U and its right-hand side turn from accumulators into
+// left operands without a change of order: they pass through shared memory as bf16 pairs (hi, lo).  The four warps of a group
+// share the tokens of a chunk (16 each) for O and U and the key components (a quarter each) for the state, whose fp32 values
+// stay in their registers.  K, Q, V (16-byte copies by all threads) and the chunk matrices (one bulk copy, the wait for it is
+// bounded) come in two stages.  KT: 16-wide steps of the key components.
 template <int KT, bool DELTA>
-__global__ void __launch_bounds__(128) rec_chunk_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
-    constexpr int KP = KT * 16 + 8;
+__global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
+    constexpr int KP = KT * 16 + 8, PAIRS = KT >= 4 ? KT / 4 : 1;  // pairs of 8 key components of the state per warp
     extern __shared__ __align__(16) uint8_t rc_dyn[];
     __shared__ __align__(8) uint64_t full[2];
     __shared__ int abort_flag;
     chain_trigger();
-    const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nw = nthr / 32;
-    const int vpitch = nw * 16 + 8, block = rc_block(DELTA);
+    const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, cols = nthr / 8;
+    const int vpitch = cols + 8, block = rc_block(DELTA);
     const int stage_bytes = 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + block;
-    for (int i = tid; i < 2 * stage_bytes / 16; i += nthr) reinterpret_cast<uint4*>(rc_dyn)[i] = make_uint4(0, 0, 0, 0);  // rows and columns that no copy fills
+    __nv_bfloat16* Sh = reinterpret_cast<__nv_bfloat16*>(rc_dyn + 2 * stage_bytes);  // [cols][KP]: state, hi
+    __nv_bfloat16* Sl = Sh + cols * KP;
+    __nv_bfloat16* Uh = Sl + cols * KP;      // [cols][RC_P]: U
+    __nv_bfloat16* Wh = Uh + cols * RC_P;    // f3 U, hi and lo
+    __nv_bfloat16* Wl = Wh + cols * RC_P;
+    __nv_bfloat16* Rh = Wl + cols * RC_P;    // right-hand side of U, hi and lo (delta rule)
+    __nv_bfloat16* Rl = Rh + cols * RC_P;
     if (tid == 0) {
         abort_flag = 0;
         tc::mbar_init(&full[0], 1);
         tc::mbar_init(&full[1], 1);
         tc::mbar_fence_init();
     }
-    tc::fence_proxy_async_smem();
     __syncthreads();
     chain_wait();
     const int h = blockIdx.y, g = h / (d.H / d.G), seg = blockIdx.z, kp = d.kp(), vp = d.vp(), cc = d.conv_cols();
-    const int c0 = blockIdx.x * nw * 16, n_cols = min(nw * 16, vp - c0);
+    const int c0 = blockIdx.x * cols, n_cols = min(cols, vp - c0);
     const int start = a.seg_start[seg], len = a.seg_len[seg], n_chunks = (len + RC_C - 1) / RC_C;
     const uint8_t* blocks = ws + ((long long)seg_chunk0[seg] * d.H + h) * block;
     const __nv_bfloat16* qkv = static_cast<const __nv_bfloat16*>(a.qkv) + (long long)start * cc;
@@ -338,168 +350,188 @@ __global__ void __launch_bounds__(128) rec_chunk_kernel(RecArgs a, RecDims d, co
         uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
         const int n = min(RC_C, len - ci * RC_C);
         if (tid == 0) {
-            tc::mbar_expect_tx(&full[ci & 1], (uint32_t)(n * (2 * kp + n_cols) * 2 + block));
+            tc::mbar_expect_tx(&full[ci & 1], (uint32_t)block);
             tc::bulk_load(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2, blocks + (long long)ci * d.H * block, block, &full[ci & 1]);
         }
-        for (int i = tid; i < 3 * n; i += nthr) {
-            const int m = i / n, r = i - m * n;  // k, q, v
-            const __nv_bfloat16* row = qkv + (long long)(ci * RC_C + r) * cc;
-            if (m < 2) tc::bulk_load(st + (m * RC_C + r) * KP * 2, row + (m == 0 ? d.G * kp : 0) + g * kp, kp * 2, &full[ci & 1]);
-            else tc::bulk_load(st + 2 * RC_C * KP * 2 + r * vpitch * 2, row + 2 * d.G * kp + h * vp + c0, n_cols * 2, &full[ci & 1]);
+        // (rows behind the segment and columns behind the head become zeros)
+        const __nv_bfloat16* rows = qkv + (long long)ci * RC_C * cc;
+#pragma unroll 4
+        for (int i = tid; i < 2 * RC_C * KT * 2; i += nthr) {  // k, then q
+            const int r = i / (KT * 2), c = i % (KT * 2) * 8;
+            const bool on = (r & (RC_C - 1)) < n && c < kp;
+            cp_async16(smem_u32(st + (r * KP + c) * 2), on ? rows + (long long)(r & (RC_C - 1)) * cc + (r < RC_C ? d.G * kp : 0) + g * kp + c : rows, on);
         }
+        for (int i = tid; i < RC_C * (cols / 8); i += nthr) {
+            const int r = i / (cols / 8), c = i % (cols / 8) * 8;
+            const bool on = r < n && c < n_cols;
+            cp_async16(smem_u32(st + 2 * RC_C * KP * 2 + (r * vpitch + c) * 2), on ? rows + (long long)r * cc + 2 * d.G * kp + h * vp + c0 + c : rows, on);
+        }
+        cp_async_commit();
     };
     load(0);
-    // state: rows (lane / 4, + 8) of this warp's columns, key components 8 j + (lane % 4) * 2, + 1
+    const int mt = warp >> 2, w = warp & 3;
+    const int jp = mt & 1 ? 3 - w : w;  // this warp's tokens of a chunk: 16 jp .. 16 jp + 15 (the triangles even out over the schedulers)
+    const int lm = lane >> 3, lr = lane & 7, kc = (lane & 3) * 2, ar = mt * 16 + (lane >> 2);
+    // accumulators: row (lane / 4, + 8) = state column, columns (lane % 4) * 2, + 1 = token or key component
     float* state = a.S + ((long long)a.seg_slot[seg] * d.H + h) * kp * vp;
-    const bool fresh = a.seg_pos0[seg] == 0;
-    const int cr = c0 + warp * 16 + (lane >> 2), kc = (lane & 3) * 2;
-    float S[2 * KT][4];
+    const bool fresh = a.seg_pos0[seg] == 0, keeps = w * PAIRS < KT;
+    float S[2 * PAIRS][4];
 #pragma unroll
-    for (int j = 0; j < 2 * KT; ++j)
+    for (int j = 0; j < 2 * PAIRS; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int k = j * 8 + kc + (e & 1), c = cr + (e >> 1) * 8;
-            S[j][e] = !fresh && k < kp && c < vp ? state[(long long)k * vp + c] : 0.0f;
+            const int k = (w * 2 * PAIRS + j) * 8 + kc + (e & 1), c = c0 + ar + (e >> 1) * 8;
+            S[j][e] = keeps && !fresh && k < kp && c < vp ? state[(long long)k * vp + c] : 0.0f;
         }
-    const int lm = lane >> 3, lr = lane & 7;
+    auto publish = [&](__nv_bfloat16* hi, __nv_bfloat16* lo, int pitch, int col, const float (&v)[4]) {
+        uint32_t h0, l0, h1, l1;
+        split2(v[0], v[1], h0, l0);
+        split2(v[2], v[3], h1, l1);
+        *reinterpret_cast<uint32_t*>(hi + ar * pitch + col + kc) = h0;
+        *reinterpret_cast<uint32_t*>(hi + (ar + 8) * pitch + col + kc) = h1;
+        *reinterpret_cast<uint32_t*>(lo + ar * pitch + col + kc) = l0;
+        *reinterpret_cast<uint32_t*>(lo + (ar + 8) * pitch + col + kc) = l1;
+    };
+    auto publish_state = [&]() {
+        if (keeps)
+#pragma unroll
+            for (int j = 0; j < 2 * PAIRS; ++j) publish(Sh, Sl, KP, (w * 2 * PAIRS + j) * 8, S[j]);
+    };
+    publish_state();
+    const int a_row = mt * 16 + (lm & 1) * 8 + lr, a_col = (lm >> 1) * 8;   // left operand: matrices = rows 0-7 / 8-15 (lm & 1), columns + 8 (lm >> 1)
+    const int b_row = (lm >> 1) * 8 + lr, b_col = (lm & 1) * 8;             // right operand, row = output column
+    const uint32_t sh = smem_u32(Sh + a_row * KP + a_col), sl = smem_u32(Sl + a_row * KP + a_col);
+    const uint32_t uh = smem_u32(Uh + a_row * RC_P + a_col), wh = smem_u32(Wh + a_row * RC_P + a_col), wl = smem_u32(Wl + a_row * RC_P + a_col);
+    const uint32_t rh = smem_u32(Rh + a_row * RC_P + a_col), rl = smem_u32(Rl + a_row * RC_P + a_col);
     bool ok = true;
     for (int ci = 0; ci < n_chunks; ++ci) {
-        if (ci > 0) __syncthreads();  // the other stage has been used up
+        cp_async_wait<0>();
+        __syncthreads();  // K, Q, V are here, the state is published, the other stage used up
         if (ci + 1 < n_chunks) load(ci + 1);
         ok = tc::mbar_wait(&full[ci & 1], (ci >> 1) & 1, &abort_flag, err, RC_ERR_FULL);
-        if (!__syncthreads_and(ok)) { ok = false; break; }
         const uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
         const uint32_t kb = smem_u32(st), qb = kb + RC_C * KP * 2, vb = qb + RC_C * KP * 2, tb = vb + RC_C * vpitch * 2;
-        const uint32_t pm = tb + (DELTA ? 2 * RC_MAT : 0);
+        const uint32_t pm = tb + (DELTA ? 2 * RC_MAT : 0) + ((jp * 16 + b_row) * RC_P + b_col) * 2;
         const float* f = reinterpret_cast<const float*>(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + (DELTA ? 3 : 1) * RC_MAT);
-        float u[8][4], o[8][4];
+        float u[2][4], o[2][4];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.0f;
-            o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
+        for (int x = 0; x < 2; ++x) {
+            u[x][0] = u[x][1] = u[x][2] = u[x][3] = 0.0f;
+            o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.0f;
         }
-        // S0^T K^T and S0^T Q^T
-        const uint32_t n_off = ((lm >> 1) * 8 + lr) * KP * 2 + (lm & 1) * 16;  // matrices: tokens 0-7 / 8-15 (lm >> 1), components + 8 (lm & 1)
+        // S0^T K^T and S0^T Q^T of this warp's tokens
+        const uint32_t k_addr = kb + ((jp * 16 + b_row) * KP + b_col) * 2, q_addr = qb + ((jp * 16 + b_row) * KP + b_col) * 2;
 #pragma unroll
         for (int kk = 0; kk < KT; ++kk) {
-            uint32_t hi[4], lo[4];
-            split2(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
-            split2(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
-            split2(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
-            split2(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
-#pragma unroll
-            for (int jp = 0; jp < 4; ++jp) {
-                uint32_t b[4];
-                if (DELTA) {
-                    ldsm_x4(kb + n_off + jp * 16 * KP * 2 + kk * 32, b);
-                    mma_16816(u[2 * jp], hi, b[0], b[1]);
-                    mma_16816(u[2 * jp + 1], hi, b[2], b[3]);
-                    mma_16816(u[2 * jp], lo, b[0], b[1]);
-                    mma_16816(u[2 * jp + 1], lo, b[2], b[3]);
-                }
-                ldsm_x4(qb + n_off + jp * 16 * KP * 2 + kk * 32, b);
-                mma_16816(o[2 * jp], hi, b[0], b[1]);
-                mma_16816(o[2 * jp + 1], hi, b[2], b[3]);
-                mma_16816(o[2 * jp], lo, b[0], b[1]);
-                mma_16816(o[2 * jp + 1], lo, b[2], b[3]);
+            uint32_t hi[4], lo[4], b[4];
+            ldsm_x4(sh + kk * 32, hi);
+            ldsm_x4(sl + kk * 32, lo);
+            ldsm_x4(q_addr + kk * 32, b);
+            mma_16816(o[0], hi, b[0], b[1]);
+            mma_16816(o[1], hi, b[2], b[3]);
+            mma_16816(o[0], lo, b[0], b[1]);
+            mma_16816(o[1], lo, b[2], b[3]);
+            if (DELTA) {
+                ldsm_x4(k_addr + kk * 32, b);
+                mma_16816(u[0], hi, b[0], b[1]);
+                mma_16816(u[1], hi, b[2], b[3]);
+                mma_16816(u[0], lo, b[0], b[1]);
+                mma_16816(u[1], lo, b[2], b[3]);
             }
         }
-        // right-hand side: f0 v - f1 (K S0), or the values themselves
-#pragma unroll
-        for (int jp = 0; jp < 4; ++jp) {
-            uint32_t v[4];  // matrices: tokens 0-7 / 8-15 (lm >> 1), columns + 8 (lm & 1); transposed
-            ldsm_x4_trans(vb + (jp * 16 + (lm >> 1) * 8 + lr) * vpitch * 2 + warp * 32 + (lm & 1) * 16, v);
+        {   // right-hand side: f0 v - f1 (K S0); the decayed sum has U = v
+            uint32_t v[4];  // matrices: tokens 0-7 / 8-15 (lm >> 1), state columns + 8 (lm & 1); transposed
+            ldsm_x4_trans(vb + (jp * 16 + b_row) * vpitch * 2 + mt * 32 + b_col * 2, v);
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
-                const int j = 2 * jp + x;
-                const float2 fv = *reinterpret_cast<const float2*>(f + j * 8 + kc);
+                const int t = jp * 16 + x * 8;
                 float2 fk = make_float2(0.0f, 0.0f);
-                if (DELTA) fk = *reinterpret_cast<const float2*>(f + RC_C + j * 8 + kc);
-                u[j][0] = fv.x * bf16lo(v[2 * x]) - fk.x * u[j][0];
-                u[j][1] = fv.y * bf16hi(v[2 * x]) - fk.y * u[j][1];
-                u[j][2] = fv.x * bf16lo(v[2 * x + 1]) - fk.x * u[j][2];
-                u[j][3] = fv.y * bf16hi(v[2 * x + 1]) - fk.y * u[j][3];
+                const float2 fv = *reinterpret_cast<const float2*>(f + t + kc);
+                if (DELTA) fk = *reinterpret_cast<const float2*>(f + RC_C + t + kc);
+                u[x][0] = fv.x * bf16lo(v[2 * x]) - fk.x * u[x][0];
+                u[x][1] = fv.y * bf16hi(v[2 * x]) - fk.y * u[x][1];
+                u[x][2] = fv.x * bf16lo(v[2 * x + 1]) - fk.x * u[x][2];
+                u[x][3] = fv.y * bf16hi(v[2 * x + 1]) - fk.y * u[x][3];
+                if (DELTA) publish(Rh, Rl, RC_P, t, u[x]);
             }
         }
-        const uint32_t m_off = ((lm >> 1) * 8 + lr) * RC_P * 2 + (lm & 1) * 16;
         if (DELTA) {  // U = T R
-            float w[8][4];
+            if (!__syncthreads_and(ok)) { ok = false; break; }
+            const uint32_t t_addr = tb + ((jp * 16 + b_row) * RC_P + b_col) * 2;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.0f;
+            for (int x = 0; x < 2; ++x) u[x][0] = u[x][1] = u[x][2] = u[x][3] = 0.0f;
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                if (kk > jp) break;  // (lower triangle)
+                uint32_t hi[4], lo[4], b[4], c[4];
+                ldsm_x4(rh + kk * 32, hi);
+                ldsm_x4(rl + kk * 32, lo);
+                ldsm_x4(t_addr + kk * 32, b);
+                ldsm_x4(t_addr + RC_MAT + kk * 32, c);
+                mma_16816(u[0], hi, b[0], b[1]);
+                mma_16816(u[1], hi, b[2], b[3]);
+                mma_16816(u[0], lo, b[0], b[1]);
+                mma_16816(u[1], lo, b[2], b[3]);
+                mma_16816(u[0], hi, c[0], c[1]);
+                mma_16816(u[1], hi, c[2], c[3]);
+            }
+        }
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const int t = jp * 16 + x * 8;
+            const float2 fs = *reinterpret_cast<const float2*>(f + 3 * RC_C + t + kc);
+            *reinterpret_cast<uint32_t*>(Uh + ar * RC_P + t + kc) = pack_bf16x2(u[x][0], u[x][1]);
+            *reinterpret_cast<uint32_t*>(Uh + (ar + 8) * RC_P + t + kc) = pack_bf16x2(u[x][2], u[x][3]);
+            const float scaled[4] = {u[x][0] * fs.x, u[x][1] * fs.y, u[x][2] * fs.x, u[x][3] * fs.y};
+            publish(Wh, Wl, RC_P, t, scaled);
+        }
+        if (!__syncthreads_and(ok)) { ok = false; break; }
+        // S = decay S0 + (f3 U)^T K, this warp's key components
+        if (keeps) {
+            const float decay = f[4 * RC_C];
+#pragma unroll
+            for (int j = 0; j < 2 * PAIRS; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) S[j][e] *= decay;
 #pragma unroll
             for (int kk = 0; kk < 4; ++kk) {
                 uint32_t hi[4], lo[4];
-                split2(u[2 * kk][0], u[2 * kk][1], hi[0], lo[0]);
-                split2(u[2 * kk][2], u[2 * kk][3], hi[1], lo[1]);
-                split2(u[2 * kk + 1][0], u[2 * kk + 1][1], hi[2], lo[2]);
-                split2(u[2 * kk + 1][2], u[2 * kk + 1][3], hi[3], lo[3]);
+                ldsm_x4(wh + kk * 32, hi);
+                ldsm_x4(wl + kk * 32, lo);
 #pragma unroll
-                for (int jp = kk; jp < 4; ++jp) {  // (lower triangle)
-                    uint32_t b[4], c[4];
-                    ldsm_x4(tb + m_off + jp * 16 * RC_P * 2 + kk * 32, b);
-                    ldsm_x4(tb + RC_MAT + m_off + jp * 16 * RC_P * 2 + kk * 32, c);
-                    mma_16816(w[2 * jp], hi, b[0], b[1]);
-                    mma_16816(w[2 * jp + 1], hi, b[2], b[3]);
-                    mma_16816(w[2 * jp], lo, b[0], b[1]);
-                    mma_16816(w[2 * jp + 1], lo, b[2], b[3]);
-                    mma_16816(w[2 * jp], hi, c[0], c[1]);
-                    mma_16816(w[2 * jp + 1], hi, c[2], c[3]);
+                for (int i = 0; i < PAIRS; ++i) {
+                    uint32_t b[4];  // matrices: tokens 0-7 / 8-15 (lm & 1), components + 8 (lm >> 1); transposed
+                    ldsm_x4_trans(kb + (kk * 16 + (lm & 1) * 8 + lr) * KP * 2 + (w * PAIRS + i) * 32 + (lm >> 1) * 16, b);
+                    mma_16816(S[2 * i], hi, b[0], b[1]);
+                    mma_16816(S[2 * i + 1], hi, b[2], b[3]);
+                    mma_16816(S[2 * i], lo, b[0], b[1]);
+                    mma_16816(S[2 * i + 1], lo, b[2], b[3]);
                 }
             }
-#pragma unroll
-            for (int j = 0; j < 8; ++j)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) u[j][e] = w[j][e];
+            publish_state();
         }
         // O = f2 (Q S0) + P U
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float2 fq = *reinterpret_cast<const float2*>(f + 2 * RC_C + j * 8 + kc);
-            o[j][0] *= fq.x; o[j][1] *= fq.y; o[j][2] *= fq.x; o[j][3] *= fq.y;
+        for (int x = 0; x < 2; ++x) {
+            const float2 fq = *reinterpret_cast<const float2*>(f + 2 * RC_C + jp * 16 + x * 8 + kc);
+            o[x][0] *= fq.x; o[x][1] *= fq.y; o[x][2] *= fq.x; o[x][3] *= fq.y;
         }
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {
-            const uint32_t hi[4] = {pack_bf16x2(u[2 * kk][0], u[2 * kk][1]), pack_bf16x2(u[2 * kk][2], u[2 * kk][3]),
-                                    pack_bf16x2(u[2 * kk + 1][0], u[2 * kk + 1][1]), pack_bf16x2(u[2 * kk + 1][2], u[2 * kk + 1][3])};
-#pragma unroll
-            for (int jp = kk; jp < 4; ++jp) {
-                uint32_t b[4];
-                ldsm_x4(pm + m_off + jp * 16 * RC_P * 2 + kk * 32, b);
-                mma_16816(o[2 * jp], hi, b[0], b[1]);
-                mma_16816(o[2 * jp + 1], hi, b[2], b[3]);
-            }
+            if (kk > jp) break;
+            uint32_t hi[4], b[4];
+            ldsm_x4(uh + kk * 32, hi);
+            ldsm_x4(pm + kk * 32, b);
+            mma_16816(o[0], hi, b[0], b[1]);
+            mma_16816(o[1], hi, b[2], b[3]);
         }
-        // S = decay S0 + (f3 U)^T K
-        const float decay = f[4 * RC_C];
-#pragma unroll
-        for (int j = 0; j < 2 * KT; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) S[j][e] *= decay;
-#pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
-            const float2 f0 = *reinterpret_cast<const float2*>(f + 3 * RC_C + kk * 16 + kc), f1 = *reinterpret_cast<const float2*>(f + 3 * RC_C + kk * 16 + 8 + kc);
-            uint32_t hi[4], lo[4];
-            split2(u[2 * kk][0] * f0.x, u[2 * kk][1] * f0.y, hi[0], lo[0]);
-            split2(u[2 * kk][2] * f0.x, u[2 * kk][3] * f0.y, hi[1], lo[1]);
-            split2(u[2 * kk + 1][0] * f1.x, u[2 * kk + 1][1] * f1.y, hi[2], lo[2]);
-            split2(u[2 * kk + 1][2] * f1.x, u[2 * kk + 1][3] * f1.y, hi[3], lo[3]);
-#pragma unroll
-            for (int jp = 0; jp < KT; ++jp) {
-                uint32_t b[4];  // matrices: tokens 0-7 / 8-15 (lm & 1), components + 8 (lm >> 1); transposed
-                ldsm_x4_trans(kb + (kk * 16 + (lm & 1) * 8 + lr) * KP * 2 + jp * 32 + (lm >> 1) * 16, b);
-                mma_16816(S[2 * jp], hi, b[0], b[1]);
-                mma_16816(S[2 * jp + 1], hi, b[2], b[3]);
-                mma_16816(S[2 * jp], lo, b[0], b[1]);
-                mma_16816(S[2 * jp + 1], lo, b[2], b[3]);
-            }
-        }
-        // output rows: token, this warp's columns
-        const int n = len - ci * RC_C, col = c0 + warp * 16 + kc;
+        // output rows: tokens, this group's columns
+        const int n = len - ci * RC_C, col = c0 + mt * 16 + kc;
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (long long)(start + ci * RC_C) * d.H * vp + h * vp + col;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const uint32_t w0 = rc_movmatrix(pack_bf16x2(o[j][0], o[j][1])), w1 = rc_movmatrix(pack_bf16x2(o[j][2], o[j][3]));
-            const int t = j * 8 + (lane >> 2);
+        for (int x = 0; x < 2; ++x) {
+            const uint32_t w0 = rc_movmatrix(pack_bf16x2(o[x][0], o[x][1])), w1 = rc_movmatrix(pack_bf16x2(o[x][2], o[x][3]));
+            const int t = jp * 16 + x * 8 + (lane >> 2);
             if (t < n) {
                 if (col < vp) *reinterpret_cast<uint32_t*>(out + (long long)t * d.H * vp) = w0;
                 if (col + 8 < vp) *reinterpret_cast<uint32_t*>(out + (long long)t * d.H * vp + 8) = w1;
@@ -514,47 +546,61 @@ __global__ void __launch_bounds__(128) rec_chunk_kernel(RecArgs a, RecDims d, co
         __syncthreads();
         return;
     }
+    if (keeps)
 #pragma unroll
-    for (int j = 0; j < 2 * KT; ++j)
+        for (int j = 0; j < 2 * PAIRS; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int k = j * 8 + kc + (e & 1), c = cr + (e >> 1) * 8;
-            if (k < kp && c < vp) state[(long long)k * vp + c] = S[j][e];
-        }
+            for (int e = 0; e < 4; ++e) {
+                const int k = (w * 2 * PAIRS + j) * 8 + kc + (e & 1), c = c0 + ar + (e >> 1) * 8;
+                if (k < kp && c < vp) state[(long long)k * vp + c] = S[j][e];
+            }
 }
 
 // ---- decode step: one token per segment ---------------------------------------------------------------------------
-// A CTA per (head, sequence).  A thread owns four columns of NR rows of the state (0: any number, read twice); the state is
-// requested before the predecessor kernel ends - only this kernel writes it, and passes are separated by the host.  Both
-// products S^T k and S^T q come from one pass over the old state:
+// A CTA per (head, sequence).  The state passes through shared memory, in and out by one bulk copy each (IN_SMEM; larger states
+// are read twice from global memory); it is requested before the predecessor kernel ends - only this kernel writes it, and
+// passes are separated by the host.  Both products S^T k and S^T q come from one pass over the old state:
 //     S^T k of the decayed state = g (S^T k),   o = g (S^T q) + (k . q) u.
 // The delta rule's CTA has the whole head: it also takes beta and the decay from the layer's input x (two dot products) and
 // applies the norm and the gate, so that its output is the operand of the output projection.
 constexpr int RT_THREADS = 256;
+constexpr int RT_ERR_FULL = 72;
+constexpr int RT_MAX_SMEM = 200 * 1024;
 
-template <typename T, int NR, bool DELTA>
-__global__ void __launch_bounds__(RT_THREADS) rec_step_kernel(RecArgs a, RecDims d, int lpr) {
-    extern __shared__ float rt_sm[];  // q [kp], k [kp], partial sums [2][row groups][vp], o [vp]
+template <typename T, bool IN_SMEM, bool DELTA>
+__global__ void __launch_bounds__(RT_THREADS, 3) rec_step_kernel(RecArgs a, RecDims d, int lpr, int* err) {
+    extern __shared__ __align__(16) float rt_sm[];  // [state [kp][vp] |] partial sums [2][row groups][vp], q [kp], k [kp], o [vp]
     __shared__ float red[RT_THREADS / 32][5], tot[5];
+    __shared__ __align__(8) uint64_t full;
+    __shared__ int abort_flag;
     const int kp = d.kp(), vp = d.vp(), groups = RT_THREADS / lpr;
-    float *qs = rt_sm, *ks = qs + kp, *pk = ks + kp, *pq = pk + groups * vp, *os = pq + groups * vp;
+    float *pk = rt_sm + (IN_SMEM ? kp * vp : 0), *pq = pk + groups * vp, *qs = pq + groups * vp, *ks = qs + kp, *os = ks + kp;
     chain_trigger();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x, g = h / (d.H / d.G), seg = blockIdx.y;
     const int rg = tid / lpr, c = (tid % lpr) * 4;
     const bool on = c < vp;
     const bool fresh = a.seg_pos0[seg] == 0;
-    float* state = a.S + ((long long)a.seg_slot[seg] * d.H + h) * kp * vp + c;
-    float4 S[NR ? NR : 1];
-    if (NR > 0)
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int r = rg + i * groups;
-            S[i] = on && r < kp && !fresh ? *reinterpret_cast<const float4*>(state + (long long)r * vp) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float* state = a.S + ((long long)a.seg_slot[seg] * d.H + h) * kp * vp;
+    if (IN_SMEM) {
+        if (fresh) {
+            for (int i = tid; i < kp * vp / 4; i += RT_THREADS) reinterpret_cast<float4*>(rt_sm)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        } else if (tid == 0) {
+            abort_flag = 0;
+            tc::mbar_init(&full, 1);
+            tc::mbar_fence_init();
+            tc::mbar_expect_tx(&full, (uint32_t)(kp * vp * 4));
+            tc::bulk_load(rt_sm, state, (uint32_t)(kp * vp * 4), &full);
         }
+    }
+    const float A = DELTA ? a.A[h] : a.decay[h], dt_bias = DELTA ? a.dt_bias[h] : 0.0f;
+    const float gain = DELTA && tid < vp ? a.norm[tid] : 0.0f;
     chain_wait();
-    const int t = a.seg_start[seg];
+    const int t = seg;  // every segment is one token
     const T* row = static_cast<const T*>(a.qkv) + (long long)t * d.conv_cols();
+    const T* z = static_cast<const T*>(a.z) + (long long)t * d.raw_cols() + h * vp;
+    // this thread's first column of v and z: requested here, used much later
+    const float v0 = tid < vp ? to_f32(row[2 * d.G * kp + h * vp + tid]) : 0.0f, z0 = DELTA && tid < vp ? to_f32(z[tid]) : 0.0f;
     float sums[5] = {0.f, 0.f, 0.f, 0.f, 0.f};  // q . q, k . k, q . k, b, a
     for (int i = tid; i < kp; i += RT_THREADS) {
         const float q = to_f32(row[g * kp + i]), k = to_f32(row[(d.G + g) * kp + i]);
@@ -565,6 +611,7 @@ __global__ void __launch_bounds__(RT_THREADS) rec_step_kernel(RecArgs a, RecDims
         const T* x = static_cast<const T*>(a.x) + (long long)t * a.x_pitch;
         const T* wb = static_cast<const T*>(a.ba_w) + (long long)h * a.x_pitch;
         const T* wa = wb + (long long)(d.ba_cols() / 2) * a.x_pitch;
+#pragma unroll 2
         for (int i = tid * 8; i < a.x_pitch; i += RT_THREADS * 8) {
             float xv[8], bv[8], av[8];
             load_f32x8(x + i, xv); load_f32x8(wb + i, bv); load_f32x8(wa + i, av);
@@ -584,81 +631,97 @@ __global__ void __launch_bounds__(RT_THREADS) rec_step_kernel(RecArgs a, RecDims
         for (int w = 0; w < RT_THREADS / 32; ++w) s += red[w][tid];
         tot[tid] = s;
     }
-    float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
-    auto take = [&](int r, const float4& s) {
-        const float k = ks[r], q = qs[r];
-        ak.x = fmaf(s.x, k, ak.x); ak.y = fmaf(s.y, k, ak.y); ak.z = fmaf(s.z, k, ak.z); ak.w = fmaf(s.w, k, ak.w);
-        aq.x = fmaf(s.x, q, aq.x); aq.y = fmaf(s.y, q, aq.y); aq.z = fmaf(s.z, q, aq.z); aq.w = fmaf(s.w, q, aq.w);
-    };
-    if (on) {
-        if (NR > 0) {
-#pragma unroll
-            for (int i = 0; i < NR; ++i)
-                if (rg + i * groups < kp) take(rg + i * groups, S[i]);
-        } else if (!fresh) {
-#pragma unroll 4
-            for (int r = rg; r < kp; r += groups) take(r, *reinterpret_cast<const float4*>(state + (long long)r * vp));
+    if (IN_SMEM && !fresh && !__syncthreads_and(tc::mbar_wait(&full, 0, &abort_flag, err, RT_ERR_FULL))) {
+        if (tid == 0) {  // let the copy in flight land (bounded); the host learns of it
+            const long long t0 = clock64();
+            while (!tc::mbar_try_wait(&full, 0) && clock64() - t0 < tc::WAIT_LIMIT_CYCLES) {}
         }
+        __syncthreads();
+        return;
+    }
+    const float* old = IN_SMEM ? rt_sm : state;
+    if (on) {
+        float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
+        if (IN_SMEM || !fresh)
+#pragma unroll 4
+            for (int r = rg; r < kp; r += groups) {
+                const float4 s = *reinterpret_cast<const float4*>(old + r * vp + c);
+                const float k = ks[r], q = qs[r];
+                ak.x = fmaf(s.x, k, ak.x); ak.y = fmaf(s.y, k, ak.y); ak.z = fmaf(s.z, k, ak.z); ak.w = fmaf(s.w, k, ak.w);
+                aq.x = fmaf(s.x, q, aq.x); aq.y = fmaf(s.y, q, aq.y); aq.z = fmaf(s.z, q, aq.z); aq.w = fmaf(s.w, q, aq.w);
+            }
         *reinterpret_cast<float4*>(pk + rg * vp + c) = ak;
         *reinterpret_cast<float4*>(pq + rg * vp + c) = aq;
     }
     __syncthreads();
     const float nq = DELTA ? a.q_scale / sqrtf(tot[0] + UNIT_EPS) : 1.0f, nk = DELTA ? 1.0f / sqrtf(tot[1] + UNIT_EPS) : 1.0f;
     const float beta = DELTA ? rec_sigmoid(tot[3]) : 1.0f;
-    const float gt = DELTA ? expf(a.A[h] * rec_softplus(tot[4] + a.dt_bias[h])) : a.decay[h];
+    const float gt = DELTA ? expf(A * rec_softplus(tot[4] + dt_bias)) : A;
     const float kq = tot[2] * nk * nq;
     // one thread per column: fold the row groups, the new value u and the output
+    float ss = 0.0f;
     for (int j = tid; j < vp; j += RT_THREADS) {
         float sk = 0.0f, sq = 0.0f;
         for (int r = 0; r < groups; ++r) { sk += pk[r * vp + j]; sq += pq[r * vp + j]; }
-        float u = to_f32(row[2 * d.G * kp + h * vp + j]);
+        float u = j == tid ? v0 : to_f32(row[2 * d.G * kp + h * vp + j]);
         if (DELTA) u = beta * (u - gt * nk * sk);
-        os[j] = fmaf(kq, u, gt * nq * sq);
+        const float o = fmaf(kq, u, gt * nq * sq);
+        os[j] = o;
+        ss = fmaf(o, o, ss);
         pk[j] = u * nk;  // (row group 0 of this column has been read)
+    }
+    if (DELTA) {
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp][0] = ss;
     }
     __syncthreads();
     if (on) {
         const float4 u = *reinterpret_cast<const float4*>(pk + c);
-        auto put = [&](int r, float4 s) {
+#pragma unroll 4
+        for (int r = rg; r < kp; r += groups) {
+            float4 s = IN_SMEM || !fresh ? *reinterpret_cast<const float4*>(old + r * vp + c) : make_float4(0.f, 0.f, 0.f, 0.f);
             const float k = ks[r];
             s.x = fmaf(k, u.x, gt * s.x); s.y = fmaf(k, u.y, gt * s.y); s.z = fmaf(k, u.z, gt * s.z); s.w = fmaf(k, u.w, gt * s.w);
-            *reinterpret_cast<float4*>(state + (long long)r * vp) = s;
-        };
-        if (NR > 0) {
-#pragma unroll
-            for (int i = 0; i < NR; ++i)
-                if (rg + i * groups < kp) put(rg + i * groups, S[i]);
-        } else {
-#pragma unroll 4
-            for (int r = rg; r < kp; r += groups)
-                put(r, fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(state + (long long)r * vp));
+            *reinterpret_cast<float4*>((IN_SMEM ? rt_sm : state) + r * vp + c) = s;
+        }
+    }
+    if (IN_SMEM) {
+        tc::fence_proxy_async_smem();
+        __syncthreads();
+        if (tid == 0) {
+            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(reinterpret_cast<uint64_t>(state)), "r"(smem_u32(rt_sm)), "r"(kp * vp * 4)
+                         : "memory");
+            asm volatile("cp.async.bulk.commit_group;" ::: "memory");
         }
     }
     T* out = static_cast<T*>(a.out) + (long long)t * d.H * vp + h * vp;
-    if (!DELTA) {
-        for (int j = tid; j < vp; j += RT_THREADS) out[j] = from_f32<T>(os[j]);
-        return;
-    }
-    float ss = 0.0f;
-    for (int j = tid; j < vp; j += RT_THREADS) ss = fmaf(os[j], os[j], ss);
-    ss = warp_sum(ss);
-    if (lane == 0) red[warp][0] = ss;
-    __syncthreads();
-    ss = 0.0f;
+    if (DELTA) {
+        ss = 0.0f;
 #pragma unroll
-    for (int w = 0; w < RT_THREADS / 32; ++w) ss += red[w][0];
-    const float rms = sqrtf(ss / (float)d.dv + a.eps);
-    const T* z = static_cast<const T*>(a.z) + (long long)t * d.raw_cols() + h * vp;
-    for (int j = tid; j < vp; j += RT_THREADS) {
-        const float zv = to_f32(z[j]);
-        out[j] = from_f32<T>(os[j] / rms * a.norm[j] * (zv * rec_sigmoid(zv)));
+        for (int w = 0; w < RT_THREADS / 32; ++w) ss += red[w][0];
     }
+    const float rms = DELTA ? sqrtf(ss / (float)d.dv + a.eps) : 1.0f;
+    for (int j = tid; j < vp; j += RT_THREADS) {
+        float o = os[j];
+        if (DELTA) {
+            const float zv = j == tid ? z0 : to_f32(z[j]);
+            o = o / rms * (j == tid ? gain : a.norm[j]) * (zv * rec_sigmoid(zv));
+        }
+        out[j] = from_f32<T>(o);
+    }
+    if (IN_SMEM && tid == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");  // the copy out reads this CTA's memory
 }
 
 // ---- norm and gate of the output ----------------------------------------------------------------------------------
 // PER_HEAD: every head by itself, weight [vp], gate silu(z); otherwise all heads together, weight [H vp], gate sigmoid(z).
-// In place.  One CTA per token.
-template <typename T, bool PER_HEAD>
+// In place.  One CTA per token; a thread holds MAXV vectors of eight columns (0: any number, read twice).  PER_HEAD with MAXV > 0
+// needs heads of 8 x 2^n <= 256 columns: a head is a group of neighbouring lanes.
+template <typename T>
+__device__ __forceinline__ float gate_sigmoid(float x) {
+    if constexpr (sizeof(T) == 4) return rec_sigmoid(x);
+    return fast_rcp(1.0f + fast_ex2(-LOG2E * x));
+}
+template <typename T, bool PER_HEAD, int MAXV>
 __global__ void __launch_bounds__(256) rec_norm_kernel(T* __restrict__ o, const T* __restrict__ z, long long z_pitch, const float* __restrict__ gain,
                                                        float eps, int H, int dv, int vp) {
     __shared__ float red[8];
@@ -666,8 +729,8 @@ __global__ void __launch_bounds__(256) rec_norm_kernel(T* __restrict__ o, const 
     chain_wait();
     T* row = o + (long long)blockIdx.x * H * vp;
     const T* zr = z + blockIdx.x * z_pitch;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    if (PER_HEAD) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = H * vp;
+    if constexpr (PER_HEAD && MAXV == 0) {
         for (int h = warp; h < H; h += 8) {
             float ss = 0.0f;
             for (int j = lane * 2; j < vp; j += 64) {
@@ -680,34 +743,63 @@ __global__ void __launch_bounds__(256) rec_norm_kernel(T* __restrict__ o, const 
                 float a, b, za, zb;
                 load_f32x2(row + h * vp + j, a, b);
                 load_f32x2(zr + h * vp + j, za, zb);
-                store_f32x2(row + h * vp + j, a / rms * gain[j] * (za * rec_sigmoid(za)), b / rms * gain[j + 1] * (zb * rec_sigmoid(zb)));
+                store_f32x2(row + h * vp + j, a / rms * gain[j] * (za * gate_sigmoid<T>(za)), b / rms * gain[j + 1] * (zb * gate_sigmoid<T>(zb)));
             }
         }
         return;
-    }
-    const int n = H * vp;
-    float ss = 0.0f;
-    for (int j = threadIdx.x * 8; j < n; j += 2048) {
-        float v[8];
-        load_f32x8(row + j, v);
+    } else {
+        float v[MAXV ? MAXV : 1][8], zv[MAXV ? MAXV : 1][8], ss[MAXV ? MAXV : 1], all = 0.0f;
+        if constexpr (MAXV > 0) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
-    }
-    ss = warp_sum(ss);
-    if (lane == 0) red[warp] = ss;
-    __syncthreads();
-    ss = 0.0f;
+            for (int i = 0; i < MAXV; ++i) {
+                const int j = (i * 256 + threadIdx.x) * 8;
+                ss[i] = 0.0f;
+                if (j < n) {
+                    load_f32x8(row + j, v[i]);
+                    load_f32x8(zr + j, zv[i]);
 #pragma unroll
-    for (int w = 0; w < 8; ++w) ss += red[w];
-    const float rms = sqrtf(ss / (float)(H * dv) + eps);
-    for (int j = threadIdx.x * 8; j < n; j += 2048) {
-        float v[8], zv[8], gv[8];
-        load_f32x8(row + j, v);
-        load_f32x8(zr + j, zv);
-        load_f32x8(gain + j, gv);
+                    for (int e = 0; e < 8; ++e) ss[i] = fmaf(v[i][e], v[i][e], ss[i]);
+                }
+                all += ss[i];
+            }
+        } else {
+            for (int j = threadIdx.x * 8; j < n; j += 2048) {
+                load_f32x8(row + j, v[0]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = v[e] / rms * gv[e] * rec_sigmoid(zv[e]);
-        store_f32x8(row + j, v);
+                for (int e = 0; e < 8; ++e) all = fmaf(v[0][e], v[0][e], all);
+            }
+        }
+        if (!PER_HEAD) {
+            all = warp_sum(all);
+            if (lane == 0) red[warp] = all;
+            __syncthreads();
+            all = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) all += red[w];
+        }
+        auto finish = [&](int j, float (&x)[8], const float (&zz)[8], float sum) {
+            const float inv = 1.0f / sqrtf(sum / (float)(PER_HEAD ? dv : H * dv) + eps);
+            float gv[8];
+            load_f32x8(gain + (PER_HEAD ? j % vp : j), gv);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = x[e] * inv * gv[e] * (PER_HEAD ? zz[e] * gate_sigmoid<T>(zz[e]) : gate_sigmoid<T>(zz[e]));
+            store_f32x8(row + j, x);
+        };
+        if constexpr (MAXV > 0) {
+#pragma unroll
+            for (int i = 0; i < MAXV; ++i) {
+                const int j = (i * 256 + threadIdx.x) * 8;
+                if (PER_HEAD)
+                    for (int x = 1; x < vp / 8; x <<= 1) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], x);
+                if (j < n) finish(j, v[i], zv[i], PER_HEAD ? ss[i] : all);
+            }
+        } else {
+            for (int j = threadIdx.x * 8; j < n; j += 2048) {
+                load_f32x8(row + j, v[0]);
+                load_f32x8(zr + j, zv[0]);
+                finish(j, v[0], zv[0], all);
+            }
+        }
     }
 }
 
@@ -742,7 +834,12 @@ static jsm_status norm_typed(const RecDims& d, const RecArgs& a, int n_tok, cuda
     auto go = [&](auto kernel) {
         return launch_chained(kernel, dim3(n_tok), dim3(256), 0, st, (T*)a.out, (const T*)a.z, (long long)d.raw_cols(), a.norm, a.eps, d.H, d.dv, d.vp());
     };
-    JSM_CUDA_CHECK(d.delta ? go(rec_norm_kernel<T, true>) : go(rec_norm_kernel<T, false>));
+    const int n = d.H * d.vp(), lanes = d.vp() / 8;
+    const bool groups = lanes <= 32 && (lanes & (lanes - 1)) == 0;
+    if (d.delta) JSM_CUDA_CHECK(n <= 2048 && groups ? go(rec_norm_kernel<T, true, 1>) : n <= 4096 && groups ? go(rec_norm_kernel<T, true, 2>)
+                                : n <= 8192 && groups ? go(rec_norm_kernel<T, true, 4>) : go(rec_norm_kernel<T, true, 0>));
+    else JSM_CUDA_CHECK(n <= 2048 ? go(rec_norm_kernel<T, false, 1>) : n <= 4096 ? go(rec_norm_kernel<T, false, 2>)
+                        : n <= 8192 ? go(rec_norm_kernel<T, false, 4>) : go(rec_norm_kernel<T, false, 0>));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
@@ -759,17 +856,17 @@ static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& 
     static bool attr_done = false;
     if (!attr_done) {
         JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_prep_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024));
-        JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_kernel<KT, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_kernel<KT, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         attr_done = true;
     }
     const int kw = KT * 16;
-    JSM_CUDA_CHECK(launch_chained(rec_chunk_prep_kernel<DELTA>, dim3(ch.n_chunks, d.H), dim3(256), (size_t)2 * RC_C * (kw + 8) * 2 + 2 * RC_C * 68 * 4, st, a, d,
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_prep_kernel<DELTA>, dim3(ch.n_chunks, d.H), dim3(256), (size_t)rc_prep_tiles(kw, DELTA) + (DELTA ? RC_C * 68 * 4 : 0), st, a, d,
                                   ch.chunk_seg, ch.chunk_t0, static_cast<uint8_t*>(ch.ws), kw));
     JSM_LAUNCH_CHECK();
-    // warps per CTA: a warp keeps a scheduler busy, so two while the SMs suffice and four beyond
-    const int warps = (d.vp() + 15) / 16, nw = std::min(warps, (long long)n_segs * d.H * ((warps + 1) / 2) > 2 * sm_count() ? 4 : 2);
-    const size_t smem = 2 * ((size_t)2 * RC_C * (kw + 8) * 2 + RC_C * (nw * 16 + 8) * 2 + rc_block(DELTA));
-    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((warps + nw - 1) / nw, d.H, n_segs), dim3(nw * 32), smem, st, a, d, ch.seg_chunk0,
+    // columns per CTA: 16 while that leaves SMs idle
+    const int cols = (long long)n_segs * d.H * ((d.vp() + 15) / 16) <= sm_count() || d.vp() <= 16 ? 16 : 32;
+    const size_t smem = 2 * ((size_t)2 * RC_C * (kw + 8) * 2 + RC_C * (cols + 8) * 2 + rc_block(DELTA)) + (size_t)cols * (2 * (kw + 8) + (DELTA ? 5 : 3) * RC_P) * 2;
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((d.vp() + cols - 1) / cols, d.H, n_segs), dim3(cols * 8), smem, st, a, d, ch.seg_chunk0,
                                   static_cast<const uint8_t*>(ch.ws), tc_error_word()));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
@@ -796,21 +893,23 @@ jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, cons
     return f32 ? norm_typed<float>(d, a, tk.T, st) : norm_typed<__nv_bfloat16>(d, a, tk.T, st);
 }
 
-template <typename T, int NR, bool DELTA>
-static jsm_status step_go(const RecArgs& a, const RecDims& d, int lpr, int n_segs, cudaStream_t st) {
-    const size_t smem = sizeof(float) * (2 * d.kp() + 2 * (size_t)(RT_THREADS / lpr) * d.vp() + d.vp());
-    JSM_CUDA_CHECK(launch_chained(rec_step_kernel<T, NR, DELTA>, dim3(d.H, n_segs), dim3(RT_THREADS), smem, st, a, d, lpr));
+template <typename T, bool IN_SMEM, bool DELTA>
+static jsm_status step_go(const RecArgs& a, const RecDims& d, int lpr, size_t smem, int n_segs, cudaStream_t st) {
+    static bool attr_done = false;
+    if (!attr_done) {
+        JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_step_kernel<T, IN_SMEM, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_MAX_SMEM));
+        attr_done = true;
+    }
+    JSM_CUDA_CHECK(launch_chained(rec_step_kernel<T, IN_SMEM, DELTA>, dim3(d.H, n_segs), dim3(RT_THREADS), smem, st, a, d, lpr, tc_error_word()));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
 template <typename T, bool DELTA>
 static jsm_status step_sized(const RecArgs& a, const RecDims& d, int n_segs, cudaStream_t st) {
-    int lpr = 1;
+    int lpr = 1;  // lanes per row of the state
     while (lpr * 4 < d.vp()) lpr *= 2;
-    const int groups = RT_THREADS / lpr, nr = (d.kp() + groups - 1) / groups;
-    return nr <= 1 ? step_go<T, 1, DELTA>(a, d, lpr, n_segs, st) : nr <= 2 ? step_go<T, 2, DELTA>(a, d, lpr, n_segs, st)
-         : nr <= 4 ? step_go<T, 4, DELTA>(a, d, lpr, n_segs, st) : nr <= 8 ? step_go<T, 8, DELTA>(a, d, lpr, n_segs, st)
-         : nr <= 16 ? step_go<T, 16, DELTA>(a, d, lpr, n_segs, st) : step_go<T, 0, DELTA>(a, d, lpr, n_segs, st);
+    const size_t base = sizeof(float) * (2 * d.kp() + 2 * (size_t)(RT_THREADS / lpr) * d.vp() + d.vp()), state = sizeof(float) * d.kp() * d.vp();
+    return base + state <= RT_MAX_SMEM ? step_go<T, true, DELTA>(a, d, lpr, base + state, n_segs, st) : step_go<T, false, DELTA>(a, d, lpr, base, n_segs, st);
 }
 
 jsm_status rec_step_launch(bool f32, const RecDims& d, const RecWeights& w, const RecState& s, float eps, const StepTokens& tk, const void* raw,

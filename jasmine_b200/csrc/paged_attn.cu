@@ -35,79 +35,111 @@ __device__ __forceinline__ T* cache_at(T* pool, const AttnDims& d, int page, int
 }
 
 // ---- bias, norm, rotation, append ---------------------------------------------------------------------------------
-// A warp per (token, unit): the query heads, then the key heads, the value heads (own_kv), and one unit for the gates.  wide
-// row of a token: [q | gates | k | v].
-template <typename T>
+// A warp takes one unit of TOK consecutive tokens: the query heads, then the key heads, the value heads (own_kv), and one unit
+// for the gates.  wide row of a token: [q | gates | k | v].  NP: pairs of components per lane (0: any number, read twice).
+template <typename T, int NP, int TOK>
 __global__ void __launch_bounds__(256) attn_prep_kernel(const float* __restrict__ wide, AttnDims d, AttnWeights w, float eps, T* __restrict__ pool,
                                                         const int32_t* __restrict__ block_table, int max_pages, const float2* __restrict__ rope,
                                                         const int32_t* __restrict__ tok_row, const int32_t* __restrict__ tok_pos, int own_kv, int n_tok,
                                                         T* __restrict__ q, float* __restrict__ gate) {
+    static_assert(NP > 0 || TOK == 1, "heads of any width take one token");
+    const int t0 = blockIdx.x * TOK, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int kv_units = own_kv ? 2 * d.G : 0;
+    const int off = d.q_cols() + pad8(d.H), pitch = d.wide_cols(own_kv != 0);
     chain_trigger();
     chain_wait();
-    const int t = blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    const int kv_units = own_kv ? 2 * d.G : 0;
-    const float* row = wide + (long long)t * d.wide_cols(own_kv != 0);
-    if (unit > d.H + kv_units) return;
+    if (unit >= d.H + kv_units + d.gated) return;
     if (unit == d.H + kv_units) {
-        for (int h = lane; h < d.H; h += 32) gate[(long long)t * d.H + h] = 1.0f / (1.0f + expf(-row[d.q_cols() + h]));
+        for (int t = t0; t < min(n_tok, t0 + TOK); ++t)
+            for (int h = lane; h < d.H; h += 32) gate[(long long)t * d.H + h] = 1.0f / (1.0f + expf(-wide[(long long)t * pitch + d.q_cols() + h]));
         return;
     }
-    const int pos = tok_pos[t];
-    const int page = own_kv ? block_table[(long long)tok_row[t] * max_pages + pos / PAGE] : 0;
-    const int off = d.q_cols() + pad8(d.H);
+    auto page_of = [&](int t, int pos) { return block_table[(long long)tok_row[t] * max_pages + pos / PAGE]; };
+    auto put = [](T* dst, const float2& v) {
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
+        else *reinterpret_cast<float2*>(dst) = v;
+    };
     if (unit >= d.H + d.G) {  // values
         const int g = unit - d.H - d.G, vh = pad8(d.vdim);
-        const float* src = row + off + d.G * d.qh() + g * vh;
         const float* b = w.v_bias ? w.v_bias + g * vh : nullptr;
-        for (int j = lane; j < d.vs() * 64; j += 32)
-            *cache_at(pool, d, page, g, 1, pos % PAGE, j) = from_f32<T>(j < d.vdim ? src[j] + (b ? b[j] : 0.0f) : 0.0f);
-        // last token of its portion, in a page that this portion opened: clear the rest of the page's values
-        const int in = pos % PAGE, r = tok_row[t];
-        const bool last = t + 1 == n_tok || tok_row[t + 1] != r;
-        const bool opened = t >= in && tok_row[t - in] == r && tok_pos[t - in] == pos - in;
-        if (last && opened)
-            for (int s = 0; s < d.vs(); ++s) {
-                T* slab = cache_at(pool, d, page, g, 1, 0, s * 64);
-                for (int i = (in + 1) * 64 + lane; i < SLAB; i += 32) slab[i] = from_f32<T>(0.0f);
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) {
+            const int t = t0 + i;
+            if (t >= n_tok) break;
+            const int pos = tok_pos[t], page = page_of(t, pos);
+            const float* src = wide + (long long)t * pitch + off + d.G * d.qh() + g * vh;
+            for (int j = lane * 2; j < d.vs() * 64; j += 64) {
+                float2 v = make_float2(0.0f, 0.0f);
+                if (j < d.vdim) {
+                    v = *reinterpret_cast<const float2*>(src + j);
+                    if (b) { const float2 bv = *reinterpret_cast<const float2*>(b + j); v.x += bv.x; v.y += bv.y; }
+                    if (j + 1 >= d.vdim) v.y = 0.0f;
+                }
+                put(cache_at(pool, d, page, g, 1, pos % PAGE, j), v);
             }
+            // last token of its portion, in a page that this portion opened: clear the rest of the page's values
+            const int in = pos % PAGE, r = tok_row[t];
+            const bool last = t + 1 == n_tok || tok_row[t + 1] != r;
+            if (last && t >= in && tok_row[t - in] == r && tok_pos[t - in] == pos - in)
+                for (int s = 0; s < d.vs(); ++s) {
+                    T* slab = cache_at(pool, d, page, g, 1, 0, s * 64);
+                    for (int k = (in + 1) * 64 + lane * 2; k < SLAB; k += 64) put(slab + k, make_float2(0.0f, 0.0f));
+                }
+        }
         return;
     }
     const bool key = unit >= d.H;
     const int hd = key ? unit - d.H : unit, qh = d.qh();
-    const float* src = row + (key ? off : 0) + hd * qh;
     const float* bias = key ? w.k_bias : w.q_bias;
     if (bias) bias += hd * qh;
     const float* gain = key ? w.k_norm : w.q_norm;
-    auto pair = [&](int p) {  // (the pitch of a head is a multiple of 8: a pair lies inside it, columns behind the head are zero)
+    const int end = key ? d.ks() * 32 : qh / 2;
+    // pair p of a row (the pitch of a head is a multiple of 8: a pair lies inside it; components behind the head are zero)
+    auto pair = [&](const float* src, int p) {
+        if (2 * p >= d.dim) return make_float2(0.0f, 0.0f);
         float2 v = *reinterpret_cast<const float2*>(src + 2 * p);
         if (bias) { const float2 b = *reinterpret_cast<const float2*>(bias + 2 * p); v.x += b.x; v.y += b.y; }
+        if (2 * p + 1 >= d.dim) v.y = 0.0f;
         return v;
     };
-    float rms = 1.0f;
-    if (gain) {
+    auto finish = [&](int t, int pos, T* dst_q, int page, int p, float2 v, float rms) {
+        if (gain && 2 * p < d.dim) {
+            const float2 gv = *reinterpret_cast<const float2*>(gain + 2 * p);
+            v.x = v.x / rms * gv.x; v.y = v.y / rms * gv.y;
+        }
+        if (2 * p < d.rot) {
+            const float2 e = rope[(long long)pos * (d.rot / 2) + p];
+            v = make_float2(v.x * e.x - v.y * e.y, v.y * e.x + v.x * e.y);
+        }
+        put(key ? cache_at(pool, d, page, hd, 0, pos % PAGE, 2 * p) : dst_q + 2 * p, v);
+    };
+    if constexpr (NP > 0) {
+        float2 v[TOK][NP];
+#pragma unroll
+        for (int i = 0; i < TOK; ++i)
+#pragma unroll
+            for (int k = 0; k < NP; ++k)
+                v[i][k] = t0 + i < n_tok ? pair(wide + (long long)(t0 + i) * pitch + (key ? off : 0) + hd * qh, k * 32 + lane) : make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) {
+            const int t = t0 + i;
+            if (t >= n_tok) break;
+            float ss = 0.0f;
+#pragma unroll
+            for (int k = 0; k < NP; ++k) ss = fmaf(v[i][k].x, v[i][k].x, fmaf(v[i][k].y, v[i][k].y, ss));
+            const float rms = sqrtf(warp_sum(ss) / (float)d.dim + eps);
+            const int pos = tok_pos[t], page = key ? page_of(t, pos) : 0;
+#pragma unroll
+            for (int k = 0; k < NP; ++k)
+                if (k * 32 + lane < end) finish(t, pos, q + (long long)t * d.q_cols() + hd * qh, page, k * 32 + lane, v[i][k], rms);
+        }
+    } else {
+        const float* src = wide + (long long)t0 * pitch + (key ? off : 0) + hd * qh;
         float ss = 0.0f;
-        for (int p = lane; 2 * p < d.dim; p += 32) {
-            const float2 v = pair(p);
-            ss = fmaf(v.x, v.x, ss);
-            if (2 * p + 1 < d.dim) ss = fmaf(v.y, v.y, ss);
-        }
-        rms = sqrtf(warp_sum(ss) / (float)d.dim + eps);
-    }
-    const int end = key ? d.ks() * 32 : qh / 2;
-    for (int p = lane; p < end; p += 32) {
-        float2 v = make_float2(0.0f, 0.0f);
-        if (2 * p < d.dim) {
-            v = pair(p);
-            if (gain) { v.x = v.x / rms * gain[2 * p]; v.y = v.y / rms * gain[2 * p + 1]; }
-            if (2 * p < d.rot) {
-                const float2 e = rope[(long long)pos * (d.rot / 2) + p];
-                v = make_float2(v.x * e.x - v.y * e.y, v.y * e.x + v.x * e.y);
-            }
-            if (2 * p + 1 >= d.dim) v.y = 0.0f;
-        }
-        T* dst = key ? cache_at(pool, d, page, hd, 0, pos % PAGE, 2 * p) : q + (long long)t * d.q_cols() + hd * qh + 2 * p;
-        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
-        else *reinterpret_cast<float2*>(dst) = v;
+        for (int p = lane; 2 * p < d.dim; p += 32) { const float2 v = pair(src, p); ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss)); }
+        const float rms = sqrtf(warp_sum(ss) / (float)d.dim + eps);
+        const int pos = tok_pos[t0], page = key ? page_of(t0, pos) : 0;
+        for (int p = lane; p < end; p += 32) finish(t0, pos, q + (long long)t0 * d.q_cols() + hd * qh, page, p, pair(src, p), rms);
     }
 }
 
@@ -437,19 +469,23 @@ __global__ void __launch_bounds__(AM_THREADS, 1) attn_paged_mma_kernel(AttnArgs 
 }
 
 // ---- launches -----------------------------------------------------------------------------------------------------
-jsm_status attn_prep_launch(bool f32, const float* wide, const AttnDims& d, const AttnWeights& w, float eps, const AttnCache& cache, bool own_kv,
-                            const StepTokens& tk, void* q, float* gate, cudaStream_t st) {
+template <typename T>
+static jsm_status prep_typed(const float* wide, const AttnDims& d, const AttnWeights& w, float eps, const AttnCache& cache, bool own_kv, const StepTokens& tk,
+                             void* q, float* gate, cudaStream_t st) {
     const int units = d.H + (own_kv ? 2 * d.G : 0) + (d.gated ? 1 : 0);
-    const dim3 grid(tk.T, (units + 7) / 8);
-    if (f32)
-        JSM_CUDA_CHECK(launch_chained(attn_prep_kernel<float>, grid, dim3(256), 0, st, wide, d, w, eps, (float*)cache.pool, cache.block_table,
-                                      cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, own_kv ? 1 : 0, tk.T, (float*)q, gate));
-    else
-        JSM_CUDA_CHECK(launch_chained(attn_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, wide, d, w, eps, (__nv_bfloat16*)cache.pool,
-                                      cache.block_table, cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, own_kv ? 1 : 0, tk.T,
-                                      (__nv_bfloat16*)q, gate));
+    auto go = [&](auto kernel, int tok) {
+        return launch_chained(kernel, dim3((tk.T + tok - 1) / tok, (units + 7) / 8), dim3(256), 0, st, wide, d, w, eps, (T*)cache.pool, cache.block_table,
+                              cache.max_pages, cache.rope, tk.tok_row, tk.tok_pos, own_kv ? 1 : 0, tk.T, (T*)q, gate);
+    };
+    const bool many = tk.T >= 512;
+    JSM_CUDA_CHECK(d.ks() == 1 ? many ? go(attn_prep_kernel<T, 1, 4>, 4) : go(attn_prep_kernel<T, 1, 1>, 1)
+                   : d.ks() == 2 ? many ? go(attn_prep_kernel<T, 2, 4>, 4) : go(attn_prep_kernel<T, 2, 1>, 1) : go(attn_prep_kernel<T, 0, 1>, 1));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
+}
+jsm_status attn_prep_launch(bool f32, const float* wide, const AttnDims& d, const AttnWeights& w, float eps, const AttnCache& cache, bool own_kv,
+                            const StepTokens& tk, void* q, float* gate, cudaStream_t st) {
+    return f32 ? prep_typed<float>(wide, d, w, eps, cache, own_kv, tk, q, gate, st) : prep_typed<__nv_bfloat16>(wide, d, w, eps, cache, own_kv, tk, q, gate, st);
 }
 
 bool attn_mma_usable(const AttnDims& d) { return d.ks() <= 4 && d.vs() <= 4; }
