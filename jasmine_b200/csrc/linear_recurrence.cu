@@ -259,33 +259,73 @@ __global__ void __launch_bounds__(256) rec_chunk_prep_kernel(RecArgs a, RecDims 
     }
     if (!DELTA) return;
     __syncthreads();
-    // column j of the inverse by forward substitution, x_t = [t = j] - sum_{i < t} A[t][i] x_i; four threads per column: thread p
-    // holds the rows 16 q + 4 p + e
-    const int j = tid >> 2, p = tid & 3;
-    float x[4][4];
+    // The inverse X of I + A in blocks: 16 x 16 diagonal blocks by forward substitution (a thread per column), then twice
+    //     [[D1, 0], [A21, D2]]^-1 = [[X1, 0], [-X2 A21 X1, X2]].
+    // The products A21 X1 rest in the upper triangle of As, which nothing else uses.
+    for (int i = tid; i < RC_C * 64; i += 256) {
+        const int r = i >> 6, c = i & 63;
+        if (r >> 4 < c >> 4) Xs[r * 68 + c] = 0.0f;
+    }
+    if (tid < RC_C) {
+        const int b = tid & 48, j = tid & 15;
+        float x[16];
 #pragma unroll
-    for (int q = 0; q < 4; ++q)
+        for (int t = 0; t < 16; ++t) {
+            float sum = 0.0f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) x[q][e] = 0.0f;
-#pragma unroll
-    for (int tq = 0; tq < 4; ++tq)
-#pragma unroll
-        for (int tr = 0; tr < 16; ++tr) {
-            const int t = tq * 16 + tr;
-            float s = 0.0f;
-#pragma unroll
-            for (int q = 0; q <= tq; ++q) {
-                const float4 r = *reinterpret_cast<const float4*>(As + t * 68 + q * 16 + p * 4);
-                s = fmaf(r.x, x[q][0], s); s = fmaf(r.y, x[q][1], s); s = fmaf(r.z, x[q][2], s); s = fmaf(r.w, x[q][3], s);
+            for (int i = 0; i < t; i += 4) {  // (entries of the row from t on are zero)
+                const float4 r = *reinterpret_cast<const float4*>(As + (b + t) * 68 + b + i);
+                sum = fmaf(r.x, x[i], sum);
+                if (i + 1 < t) sum = fmaf(r.y, x[i + 1], sum);
+                if (i + 2 < t) sum = fmaf(r.z, x[i + 2], sum);
+                if (i + 3 < t) sum = fmaf(r.w, x[i + 3], sum);
             }
-            s += __shfl_xor_sync(0xffffffffu, s, 1);
-            s += __shfl_xor_sync(0xffffffffu, s, 2);
-            if (p == tr / 4) x[tq][tr % 4] = (t == j ? 1.0f : 0.0f) - s;
+            x[t] = (t == j ? 1.0f : 0.0f) - sum;
+            Xs[(b + t) * 68 + b + j] = x[t];
         }
+    }
+    __syncthreads();
+    {
+        const int m = (tid >> 7) * 32, r = (tid & 127) >> 3, c = (tid & 7) * 2;
+        float y0 = 0.0f, y1 = 0.0f;
 #pragma unroll
-    for (int q = 0; q < 4; ++q)
+        for (int k = 0; k < 16; ++k) {
+            const float v = As[(m + 16 + r) * 68 + m + k];
+            const float2 x = *reinterpret_cast<const float2*>(Xs + (m + k) * 68 + m + c);
+            y0 = fmaf(v, x.x, y0); y1 = fmaf(v, x.y, y1);
+        }
+        *reinterpret_cast<float2*>(As + (m + r) * 68 + m + 16 + c) = make_float2(y0, y1);
+        __syncthreads();
+        y0 = y1 = 0.0f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) Xs[(q * 16 + p * 4 + e) * 68 + j] = x[q][e];
+        for (int k = 0; k < 16; ++k) {
+            const float v = Xs[(m + 16 + r) * 68 + m + 16 + k];
+            const float2 y = *reinterpret_cast<const float2*>(As + (m + k) * 68 + m + 16 + c);
+            y0 = fmaf(v, y.x, y0); y1 = fmaf(v, y.y, y1);
+        }
+        *reinterpret_cast<float2*>(Xs + (m + 16 + r) * 68 + m + c) = make_float2(-y0, -y1);
+    }
+    __syncthreads();
+    {
+        const int r = tid >> 3, c = (tid & 7) * 4;
+        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int k = 0; k < 32; ++k) {
+            const float v = As[(32 + r) * 68 + k];
+            const float4 x = *reinterpret_cast<const float4*>(Xs + k * 68 + c);
+            y.x = fmaf(v, x.x, y.x); y.y = fmaf(v, x.y, y.y); y.z = fmaf(v, x.z, y.z); y.w = fmaf(v, x.w, y.w);
+        }
+        *reinterpret_cast<float4*>(As + r * 68 + 32 + c) = y;
+        __syncthreads();
+        y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int k = 0; k < 32; ++k) {
+            const float v = Xs[(32 + r) * 68 + 32 + k];
+            const float4 x = *reinterpret_cast<const float4*>(As + k * 68 + 32 + c);
+            y.x = fmaf(v, x.x, y.x); y.y = fmaf(v, x.y, y.y); y.z = fmaf(v, x.z, y.z); y.w = fmaf(v, x.w, y.w);
+        }
+        *reinterpret_cast<float4*>(Xs + (32 + r) * 68 + c) = make_float4(-y.x, -y.y, -y.z, -y.w);
+    }
     __syncthreads();
     __nv_bfloat16* Th = reinterpret_cast<__nv_bfloat16*>(out);
     for (int i = tid; i < RC_C * 8; i += 256) {

@@ -54,72 +54,66 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const float* __restrict_
             for (int h = lane; h < d.H; h += 32) gate[(long long)t * d.H + h] = 1.0f / (1.0f + expf(-wide[(long long)t * pitch + d.q_cols() + h]));
         return;
     }
-    auto page_of = [&](int t, int pos) { return block_table[(long long)tok_row[t] * max_pages + pos / PAGE]; };
     auto put = [](T* dst, const float2& v) {
         if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(v.x, v.y);
         else *reinterpret_cast<float2*>(dst) = v;
     };
-    if (unit >= d.H + d.G) {  // values
-        const int g = unit - d.H - d.G, vh = pad8(d.vdim);
-        const float* b = w.v_bias ? w.v_bias + g * vh : nullptr;
-#pragma unroll
+    const bool value = unit >= d.H + d.G, key = unit >= d.H && !value;
+    const int hd = value ? unit - d.H - d.G : key ? unit - d.H : unit;
+    const int n = value ? d.vdim : d.dim;
+    const int col0 = value ? off + d.G * d.qh() + hd * pad8(d.vdim) : (key ? off : 0) + hd * d.qh();  // of the unit in a row
+    const int end = value ? d.vs() * 32 : key ? d.ks() * 32 : d.qh() / 2;                              // pairs to write
+    const float* bias = value ? w.v_bias : key ? w.k_bias : w.q_bias;
+    if (bias) bias += hd * (value ? pad8(d.vdim) : d.qh());
+    const float* gain = value ? nullptr : key ? w.k_norm : w.q_norm;
+    // (the pitch of a head is a multiple of 8: a pair lies inside it, and bias and gain are zero behind the head)
+    auto vec = [&](const float* p, int pr, float none) { return p && 2 * pr < n ? *reinterpret_cast<const float2*>(p + 2 * pr) : make_float2(none, none); };
+    auto pair = [&](int t, int pr, const float2& b) {
+        float2 v = vec(wide + (long long)t * pitch + col0, pr, 0.0f);
+        v.x += b.x; v.y += b.y;
+        if (2 * pr + 1 >= n) v.y = 0.0f;
+        return v;
+    };
+    // where pair pr of a token goes
+    auto entry = [&](int t, int pos) {  // keys and values: first element of the token's row in the first slab
+        return cache_at(pool, d, block_table[(long long)tok_row[t] * max_pages + pos / PAGE], hd, value ? 1 : 0, pos % PAGE, 0) - slab_index<T>(pos % PAGE, 0) + pos % PAGE * 64;
+    };
+    auto store = [&](T* row, int pos, int pr, const float2& v) {
+        put(key || value ? row + (pr >> 5) * SLAB + ((((pr >> 2) & 7) ^ (pos & 7)) << 3) + (pr & 3) * 2 : row + 2 * pr, v);
+    };
+    auto turn = [&](int pos, int pr, float2 v, float inv, const float2& g) {
+        v.x *= inv * g.x; v.y *= inv * g.y;
+        if (2 * pr < d.rot) {
+            const float2 e = rope[pos * (d.rot / 2) + pr];
+            v = make_float2(v.x * e.x - v.y * e.y, v.y * e.x + v.x * e.y);
+        }
+        return v;
+    };
+    auto length = [&](float ss) { return gain ? 1.0f / sqrtf(warp_sum(ss) / (float)n + eps) : 1.0f; };
+    if (value) {
         for (int i = 0; i < TOK; ++i) {
             const int t = t0 + i;
             if (t >= n_tok) break;
-            const int pos = tok_pos[t], page = page_of(t, pos);
-            const float* src = wide + (long long)t * pitch + off + d.G * d.qh() + g * vh;
-            for (int j = lane * 2; j < d.vs() * 64; j += 64) {
-                float2 v = make_float2(0.0f, 0.0f);
-                if (j < d.vdim) {
-                    v = *reinterpret_cast<const float2*>(src + j);
-                    if (b) { const float2 bv = *reinterpret_cast<const float2*>(b + j); v.x += bv.x; v.y += bv.y; }
-                    if (j + 1 >= d.vdim) v.y = 0.0f;
-                }
-                put(cache_at(pool, d, page, g, 1, pos % PAGE, j), v);
-            }
+            const int pos = tok_pos[t], in = pos % PAGE, r = tok_row[t];
+            T* row = entry(t, pos);
+            for (int pr = lane; pr < end; pr += 32) store(row, pos, pr, pair(t, pr, vec(bias, pr, 0.0f)));
             // last token of its portion, in a page that this portion opened: clear the rest of the page's values
-            const int in = pos % PAGE, r = tok_row[t];
             const bool last = t + 1 == n_tok || tok_row[t + 1] != r;
             if (last && t >= in && tok_row[t - in] == r && tok_pos[t - in] == pos - in)
-                for (int s = 0; s < d.vs(); ++s) {
-                    T* slab = cache_at(pool, d, page, g, 1, 0, s * 64);
-                    for (int k = (in + 1) * 64 + lane * 2; k < SLAB; k += 64) put(slab + k, make_float2(0.0f, 0.0f));
-                }
+                for (int s = 0; s < d.vs(); ++s)
+                    for (int k = 64 + lane * 2; k < SLAB - in * 64; k += 64) put(row + s * SLAB + k, make_float2(0.0f, 0.0f));
         }
-        return;
-    }
-    const bool key = unit >= d.H;
-    const int hd = key ? unit - d.H : unit, qh = d.qh();
-    const float* bias = key ? w.k_bias : w.q_bias;
-    if (bias) bias += hd * qh;
-    const float* gain = key ? w.k_norm : w.q_norm;
-    const int end = key ? d.ks() * 32 : qh / 2;
-    // pair p of a row (the pitch of a head is a multiple of 8: a pair lies inside it; components behind the head are zero)
-    auto pair = [&](const float* src, int p) {
-        if (2 * p >= d.dim) return make_float2(0.0f, 0.0f);
-        float2 v = *reinterpret_cast<const float2*>(src + 2 * p);
-        if (bias) { const float2 b = *reinterpret_cast<const float2*>(bias + 2 * p); v.x += b.x; v.y += b.y; }
-        if (2 * p + 1 >= d.dim) v.y = 0.0f;
-        return v;
-    };
-    auto finish = [&](int t, int pos, T* dst_q, int page, int p, float2 v, float rms) {
-        if (gain && 2 * p < d.dim) {
-            const float2 gv = *reinterpret_cast<const float2*>(gain + 2 * p);
-            v.x = v.x / rms * gv.x; v.y = v.y / rms * gv.y;
-        }
-        if (2 * p < d.rot) {
-            const float2 e = rope[(long long)pos * (d.rot / 2) + p];
-            v = make_float2(v.x * e.x - v.y * e.y, v.y * e.x + v.x * e.y);
-        }
-        put(key ? cache_at(pool, d, page, hd, 0, pos % PAGE, 2 * p) : dst_q + 2 * p, v);
-    };
-    if constexpr (NP > 0) {
-        float2 v[TOK][NP];
+    } else if constexpr (NP > 0) {
+        float2 v[TOK][NP], g[NP];
+        {
+            float2 b[NP];
 #pragma unroll
-        for (int i = 0; i < TOK; ++i)
+            for (int k = 0; k < NP; ++k) { b[k] = vec(bias, k * 32 + lane, 0.0f); g[k] = vec(gain, k * 32 + lane, 1.0f); }
 #pragma unroll
-            for (int k = 0; k < NP; ++k)
-                v[i][k] = t0 + i < n_tok ? pair(wide + (long long)(t0 + i) * pitch + (key ? off : 0) + hd * qh, k * 32 + lane) : make_float2(0.0f, 0.0f);
+            for (int i = 0; i < TOK; ++i)
+#pragma unroll
+                for (int k = 0; k < NP; ++k) v[i][k] = t0 + i < n_tok ? pair(t0 + i, k * 32 + lane, b[k]) : make_float2(0.0f, 0.0f);
+        }
 #pragma unroll
         for (int i = 0; i < TOK; ++i) {
             const int t = t0 + i;
@@ -127,19 +121,23 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const float* __restrict_
             float ss = 0.0f;
 #pragma unroll
             for (int k = 0; k < NP; ++k) ss = fmaf(v[i][k].x, v[i][k].x, fmaf(v[i][k].y, v[i][k].y, ss));
-            const float rms = sqrtf(warp_sum(ss) / (float)d.dim + eps);
-            const int pos = tok_pos[t], page = key ? page_of(t, pos) : 0;
+            const float inv = length(ss);
+            const int pos = tok_pos[t];
+            T* row = key ? entry(t, pos) : q + (long long)t * d.q_cols() + hd * d.qh();
 #pragma unroll
             for (int k = 0; k < NP; ++k)
-                if (k * 32 + lane < end) finish(t, pos, q + (long long)t * d.q_cols() + hd * qh, page, k * 32 + lane, v[i][k], rms);
+                if (k * 32 + lane < end) store(row, pos, k * 32 + lane, turn(pos, k * 32 + lane, v[i][k], inv, g[k]));
         }
     } else {
-        const float* src = wide + (long long)t0 * pitch + (key ? off : 0) + hd * qh;
         float ss = 0.0f;
-        for (int p = lane; 2 * p < d.dim; p += 32) { const float2 v = pair(src, p); ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss)); }
-        const float rms = sqrtf(warp_sum(ss) / (float)d.dim + eps);
-        const int pos = tok_pos[t0], page = key ? page_of(t0, pos) : 0;
-        for (int p = lane; p < end; p += 32) finish(t0, pos, q + (long long)t0 * d.q_cols() + hd * qh, page, p, pair(src, p), rms);
+        for (int pr = lane; 2 * pr < n; pr += 32) {
+            const float2 v = pair(t0, pr, vec(bias, pr, 0.0f));
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
+        }
+        const float inv = length(ss);
+        const int pos = tok_pos[t0];
+        T* row = key ? entry(t0, pos) : q + (long long)t0 * d.q_cols() + hd * d.qh();
+        for (int pr = lane; pr < end; pr += 32) store(row, pos, pr, turn(pos, pr, pair(t0, pr, vec(bias, pr, 0.0f)), inv, vec(gain, pr, 1.0f)));
     }
 }
 
