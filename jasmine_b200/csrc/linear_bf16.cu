@@ -40,7 +40,7 @@ static encode_tiled_fn get_encode() {
 }
 
 jsm_status make_tmap_bf16_2d(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint64_t row_stride_elems,
-                             uint32_t box_rows, uint32_t box_cols) {
+                             uint32_t box_rows, uint32_t box_cols, bool swizzle) {
     encode_tiled_fn enc = get_encode();
     if (!enc) JSM_FAIL(JSM_CUDA, "cuTensorMapEncodeTiled is not available (no CUDA driver)");
     if ((reinterpret_cast<uintptr_t>(base) & 15) || (row_stride_elems * 2) % 16)
@@ -50,7 +50,7 @@ jsm_status make_tmap_bf16_2d(CUtensorMap* map, const void* base, uint64_t rows, 
     cuuint32_t box[2] = {box_cols, box_rows};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                     CU_TENSOR_MAP_INTERLEAVE_NONE, swizzle ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                      CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) JSM_FAIL(JSM_CUDA, "cuTensorMapEncodeTiled failed with %d (rows %llu cols %llu)", (int)r,
                                     (unsigned long long)rows, (unsigned long long)cols);

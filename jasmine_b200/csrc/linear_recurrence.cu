@@ -130,6 +130,7 @@ constexpr int RC_C = REC_CHUNK;       // tokens per chunk
 constexpr int RC_P = RC_C + 8;        // pitch of a chunk matrix (bf16)
 constexpr int RC_MAT = RC_C * RC_P * 2;
 constexpr int RC_SCAL = 4 * RC_C * 4 + 16;  // per token: factors of v, K S0, Q S0 and k u^T; the chunk's decay
+constexpr int RC_SLAB = RC_C * 128;   // bytes of 64 key components of a chunk
 constexpr int RC_ERR_FULL = 71;
 constexpr float LOG_MIN = -120.0f;    // e^-120 is 0 in fp32
 __host__ __device__ inline int rc_block(bool delta) { return (delta ? 3 : 1) * RC_MAT + RC_SCAL; }  // bytes per (chunk, head): [T hi | T lo |] P | factors
@@ -139,6 +140,7 @@ __host__ __device__ inline int rc_prep_tiles(int kw, bool delta) {  // bytes of 
     return tiles > x ? tiles : x;
 }
 
+__host__ __device__ inline int rc_stage(int tile, int cols, bool delta) { return (2 * tile + RC_C * cols * 2 + rc_block(delta) + 1023) & ~1023; }
 // Per (chunk, head): the factors, P, and the inverse T of I + A.  Eight warps.
 template <bool DELTA>
 __global__ void __launch_bounds__(256) rec_chunk_prep_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ chunk_seg, const int32_t* __restrict__ chunk_t0,
@@ -354,18 +356,21 @@ __device__ __forceinline__ uint32_t rc_movmatrix(uint32_t x) {
 // state columns, 16 per group of four warps - so that the state, U and its right-hand side turn from accumulators into
 // left operands without a change of order: they pass through shared memory as bf16 pairs (hi, lo).  The four warps of a group
 // share the tokens of a chunk (16 each) for O and U and the key components (a quarter each) for the state, whose fp32 values
-// stay in their registers.  K, Q, V (16-byte copies by all threads) and the chunk matrices (one bulk copy, the wait for it is
-// bounded) come in two stages.  KT: 16-wide steps of the key components.
+// stay in their registers.  K and Q (slabs of 64 components in the 128-byte swizzle), V and the chunk matrices come in two
+// stages by bulk and TMA copies of one thread, whose waits are bounded; a segment's last, short chunk and heads that do not
+// fill their instance by 16-byte copies of all threads, which write zeros where there is nothing.  KT: 16-wide steps of the key components.
 template <int KT, bool DELTA>
-__global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
+__global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ CUtensorMap map_qk, const __grid_constant__ CUtensorMap map_v, RecArgs a, RecDims d,
+                                                       const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
     constexpr int KP = KT * 16 + 8, PAIRS = KT >= 4 ? KT / 4 : 1;  // pairs of 8 key components of the state per warp
-    extern __shared__ __align__(16) uint8_t rc_dyn[];
+    constexpr int SLABS = KT >= 4 ? KT / 4 : 1, TILE = SLABS * RC_SLAB;  // K or Q of a chunk
+    extern __shared__ uint8_t rc_raw[];
+    uint8_t* rc_dyn = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(rc_raw) + 1023) & ~uintptr_t(1023));
     __shared__ __align__(8) uint64_t full[2];
     __shared__ int abort_flag;
     chain_trigger();
     const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, cols = nthr / 8;
-    const int vpitch = cols + 8, block = rc_block(DELTA);
-    const int stage_bytes = 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + block;
+    const int block = rc_block(DELTA), v_bytes = RC_C * cols * 2, stage_bytes = rc_stage(TILE, cols, DELTA);
     __nv_bfloat16* Sh = reinterpret_cast<__nv_bfloat16*>(rc_dyn + 2 * stage_bytes);  // [cols][KP]: state, hi
     __nv_bfloat16* Sl = Sh + cols * KP;
     __nv_bfloat16* Uh = Sl + cols * KP;      // [cols][RC_P]: U
@@ -378,6 +383,8 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
         tc::mbar_init(&full[0], 1);
         tc::mbar_init(&full[1], 1);
         tc::mbar_fence_init();
+        tc::tma_prefetch_desc(&map_qk);
+        tc::tma_prefetch_desc(&map_v);
     }
     __syncthreads();
     chain_wait();
@@ -389,22 +396,34 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
     auto load = [&](int ci) {
         uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
         const int n = min(RC_C, len - ci * RC_C);
+        const bool tiles = n == RC_C && kp == KT * 16;
         if (tid == 0) {
-            tc::mbar_expect_tx(&full[ci & 1], (uint32_t)block);
-            tc::bulk_load(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2, blocks + (long long)ci * d.H * block, block, &full[ci & 1]);
+            uint64_t* bar = &full[ci & 1];
+            tc::mbar_expect_tx(bar, (uint32_t)(block + (tiles ? 2 * TILE + v_bytes : 0)));
+            if (tiles) {
+                const int y = start + ci * RC_C;
+#pragma unroll
+                for (int s = 0; s < SLABS; ++s) {
+                    tc::tma_load_2d(st + s * RC_SLAB, &map_qk, (d.G + g) * kp + s * 64, y, bar);
+                    tc::tma_load_2d(st + TILE + s * RC_SLAB, &map_qk, g * kp + s * 64, y, bar);
+                }
+                tc::tma_load_2d(st + 2 * TILE, &map_v, 2 * d.G * kp + h * vp + c0, y, bar);  // (columns behind the head end in state columns that do not exist)
+            }
+            tc::bulk_load(st + 2 * TILE + v_bytes, blocks + (long long)ci * d.H * block, block, bar);
         }
-        // (rows behind the segment and columns behind the head become zeros)
-        const __nv_bfloat16* rows = qkv + (long long)ci * RC_C * cc;
-#pragma unroll 4
-        for (int i = tid; i < 2 * RC_C * KT * 2; i += nthr) {  // k, then q
-            const int r = i / (KT * 2), c = i % (KT * 2) * 8;
-            const bool on = (r & (RC_C - 1)) < n && c < kp;
-            cp_async16(smem_u32(st + (r * KP + c) * 2), on ? rows + (long long)(r & (RC_C - 1)) * cc + (r < RC_C ? d.G * kp : 0) + g * kp + c : rows, on);
-        }
-        for (int i = tid; i < RC_C * (cols / 8); i += nthr) {
-            const int r = i / (cols / 8), c = i % (cols / 8) * 8;
-            const bool on = r < n && c < n_cols;
-            cp_async16(smem_u32(st + 2 * RC_C * KP * 2 + (r * vpitch + c) * 2), on ? rows + (long long)r * cc + 2 * d.G * kp + h * vp + c0 + c : rows, on);
+        if (!tiles) {
+            const __nv_bfloat16* rows = qkv + (long long)ci * RC_C * cc;
+            for (int i = tid; i < 2 * RC_C * KT * 2; i += nthr) {  // k, then q
+                const int q = i / (RC_C * KT * 2), r = i / (KT * 2) % RC_C, c = i % (KT * 2) * 8;
+                const bool on = r < n && c < kp;
+                cp_async16(smem_u32(st + q * TILE + (c >> 6) * RC_SLAB + r * 128 + ((((c >> 3) & 7) ^ (r & 7)) << 4)),
+                           on ? rows + (long long)r * cc + ((q ? 0 : d.G) + g) * kp + c : rows, on);
+            }
+            for (int i = tid; i < RC_C * (cols / 8); i += nthr) {
+                const int r = i / (cols / 8), c = i % (cols / 8) * 8;
+                const bool on = r < n && c < n_cols;
+                cp_async16(smem_u32(st + 2 * TILE + (r * cols + c) * 2), on ? rows + (long long)r * cc + 2 * d.G * kp + h * vp + c0 + c : rows, on);
+            }
         }
         cp_async_commit();
     };
@@ -450,9 +469,9 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
         if (ci + 1 < n_chunks) load(ci + 1);
         ok = tc::mbar_wait(&full[ci & 1], (ci >> 1) & 1, &abort_flag, err, RC_ERR_FULL);
         const uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
-        const uint32_t kb = smem_u32(st), qb = kb + RC_C * KP * 2, vb = qb + RC_C * KP * 2, tb = vb + RC_C * vpitch * 2;
+        const uint32_t kb = smem_u32(st), qb = kb + TILE, vb = qb + TILE, tb = vb + v_bytes;
         const uint32_t pm = tb + (DELTA ? 2 * RC_MAT : 0) + ((jp * 16 + b_row) * RC_P + b_col) * 2;
-        const float* f = reinterpret_cast<const float*>(st + 2 * RC_C * KP * 2 + RC_C * vpitch * 2 + (DELTA ? 3 : 1) * RC_MAT);
+        const float* f = reinterpret_cast<const float*>(st + 2 * TILE + v_bytes + (DELTA ? 3 : 1) * RC_MAT);
         float u[2][4], o[2][4];
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
@@ -460,19 +479,20 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
             o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.0f;
         }
         // S0^T K^T and S0^T Q^T of this warp's tokens
-        const uint32_t k_addr = kb + ((jp * 16 + b_row) * KP + b_col) * 2, q_addr = qb + ((jp * 16 + b_row) * KP + b_col) * 2;
+        const uint32_t k_addr = kb + (jp * 16 + b_row) * 128, q_addr = qb + (jp * 16 + b_row) * 128, x0 = (lm & 1) ^ lr;  // (the row's piece p lies at p ^ lr)
 #pragma unroll
         for (int kk = 0; kk < KT; ++kk) {
             uint32_t hi[4], lo[4], b[4];
             ldsm_x4(sh + kk * 32, hi);
             ldsm_x4(sl + kk * 32, lo);
-            ldsm_x4(q_addr + kk * 32, b);
+            const uint32_t piece = (kk >> 2) * RC_SLAB + ((((kk & 3) * 2) ^ x0) << 4);
+            ldsm_x4(q_addr + piece, b);
             mma_16816(o[0], hi, b[0], b[1]);
             mma_16816(o[1], hi, b[2], b[3]);
             mma_16816(o[0], lo, b[0], b[1]);
             mma_16816(o[1], lo, b[2], b[3]);
             if (DELTA) {
-                ldsm_x4(k_addr + kk * 32, b);
+                ldsm_x4(k_addr + piece, b);
                 mma_16816(u[0], hi, b[0], b[1]);
                 mma_16816(u[1], hi, b[2], b[3]);
                 mma_16816(u[0], lo, b[0], b[1]);
@@ -481,7 +501,7 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
         }
         {   // right-hand side: f0 v - f1 (K S0); the decayed sum has U = v
             uint32_t v[4];  // matrices: tokens 0-7 / 8-15 (lm >> 1), state columns + 8 (lm & 1); transposed
-            ldsm_x4_trans(vb + (jp * 16 + b_row) * vpitch * 2 + mt * 32 + b_col * 2, v);
+            ldsm_x4_trans(vb + (jp * 16 + b_row) * cols * 2 + mt * 32 + b_col * 2, v);
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
                 const int t = jp * 16 + x * 8;
@@ -541,7 +561,8 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(RecArgs a, RecDims d, co
 #pragma unroll
                 for (int i = 0; i < PAIRS; ++i) {
                     uint32_t b[4];  // matrices: tokens 0-7 / 8-15 (lm & 1), components + 8 (lm >> 1); transposed
-                    ldsm_x4_trans(kb + (kk * 16 + (lm & 1) * 8 + lr) * KP * 2 + (w * PAIRS + i) * 32 + (lm >> 1) * 16, b);
+                    const int pair = w * PAIRS + i;
+                    ldsm_x4_trans(kb + (pair >> 2) * RC_SLAB + (kk * 16 + (lm & 1) * 8 + lr) * 128 + ((((pair & 3) * 2) ^ (lm >> 1) ^ lr) << 4), b);
                     mma_16816(S[2 * i], hi, b[0], b[1]);
                     mma_16816(S[2 * i + 1], hi, b[2], b[3]);
                     mma_16816(S[2 * i], lo, b[0], b[1]);
@@ -892,7 +913,7 @@ bool rec_chunk_usable(const RecDims& d) { return d.dk <= 128 && d.dv <= 1024; }
 size_t rec_chunk_bytes(const RecDims& d) { return (size_t)d.H * rc_block(d.delta); }
 
 template <int KT, bool DELTA>
-static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, cudaStream_t st) {
+static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, int n_tok, cudaStream_t st) {
     static bool attr_done = false;
     if (!attr_done) {
         JSM_CUDA_CHECK(cudaFuncSetAttribute(rec_chunk_prep_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 80 * 1024));
@@ -905,18 +926,23 @@ static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& 
     JSM_LAUNCH_CHECK();
     // columns per CTA: 16 while that leaves SMs idle
     const int cols = (long long)n_segs * d.H * ((d.vp() + 15) / 16) <= sm_count() || d.vp() <= 16 ? 16 : 32;
-    const size_t smem = 2 * ((size_t)2 * RC_C * (kw + 8) * 2 + RC_C * (cols + 8) * 2 + rc_block(DELTA)) + (size_t)cols * (2 * (kw + 8) + (DELTA ? 5 : 3) * RC_P) * 2;
-    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((d.vp() + cols - 1) / cols, d.H, n_segs), dim3(cols * 8), smem, st, a, d, ch.seg_chunk0,
+    const size_t smem = 2 * (size_t)rc_stage((KT >= 4 ? KT / 4 : 1) * RC_SLAB, cols, DELTA) + (size_t)cols * (2 * (kw + 8) + (DELTA ? 5 : 3) * RC_P) * 2 + 1024;
+    CUtensorMap map_qk, map_v;
+    jsm_status s = make_tmap_bf16_2d(&map_qk, a.qkv, (uint64_t)n_tok, (uint64_t)d.conv_cols(), (uint64_t)d.conv_cols(), RC_C, 64);
+    if (s != JSM_OK) return s;
+    s = make_tmap_bf16_2d(&map_v, a.qkv, (uint64_t)n_tok, (uint64_t)d.conv_cols(), (uint64_t)d.conv_cols(), RC_C, cols, false);
+    if (s != JSM_OK) return s;
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((d.vp() + cols - 1) / cols, d.H, n_segs), dim3(cols * 8), smem, st, map_qk, map_v, a, d, ch.seg_chunk0,
                                   static_cast<const uint8_t*>(ch.ws), tc_error_word()));
     JSM_LAUNCH_CHECK();
     return JSM_OK;
 }
 template <bool DELTA>
-static jsm_status chunk_sized(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, cudaStream_t st) {
+static jsm_status chunk_sized(const RecArgs& a, const RecDims& d, const RecChunks& ch, int n_segs, int n_tok, cudaStream_t st) {
     switch (chunk_kt(d)) {
-        case 2: return chunk_go<2, DELTA>(a, d, ch, n_segs, st);
-        case 4: return chunk_go<4, DELTA>(a, d, ch, n_segs, st);
-        default: return chunk_go<8, DELTA>(a, d, ch, n_segs, st);
+        case 2: return chunk_go<2, DELTA>(a, d, ch, n_segs, n_tok, st);
+        case 4: return chunk_go<4, DELTA>(a, d, ch, n_segs, n_tok, st);
+        default: return chunk_go<8, DELTA>(a, d, ch, n_segs, n_tok, st);
     }
 }
 
@@ -926,7 +952,7 @@ jsm_status rec_scan_launch(bool f32, const RecDims& d, const RecWeights& w, cons
     RecArgs a = rec_args(f32, d, w, s, tk, raw, qkv, out, eps);
     a.ba = ba;
     jsm_status r;
-    if (!f32 && rec_chunk_usable(d)) r = d.delta ? chunk_sized<true>(a, d, ch, tk.n_segs, st) : chunk_sized<false>(a, d, ch, tk.n_segs, st);
+    if (!f32 && rec_chunk_usable(d)) r = d.delta ? chunk_sized<true>(a, d, ch, tk.n_segs, tk.T, st) : chunk_sized<false>(a, d, ch, tk.n_segs, tk.T, st);
     else r = f32 ? (d.delta ? scan_sized<float, true>(a, d, tk.n_segs, st) : scan_sized<float, false>(a, d, tk.n_segs, st))
                        : (d.delta ? scan_sized<__nv_bfloat16, true>(a, d, tk.n_segs, st) : scan_sized<__nv_bfloat16, false>(a, d, tk.n_segs, st));
     if (r != JSM_OK) return r;

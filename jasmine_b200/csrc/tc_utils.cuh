@@ -204,9 +204,9 @@ __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.
 }  // namespace tc
 
 // ---- host: tensor maps -----------------------------------------------------------------------
-// bf16 row-major [rows, cols] matrix, box = [box_rows, box_cols], 128-byte swizzle (box_cols * 2 == 128).
+// bf16 row-major [rows, cols] matrix, box = [box_rows, box_cols], 128-byte swizzle (box_cols * 2 == 128) or none.
 jsm_status make_tmap_bf16_2d(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint64_t row_stride_elems,
-                             uint32_t box_rows, uint32_t box_cols);
+                             uint32_t box_rows, uint32_t box_cols, bool swizzle = true);
 // bf16 [d2, d1, d0] tensor with element strides (s2, s1, 1)
 jsm_status make_tmap_bf16_3d(CUtensorMap* map, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1_elems,
                              uint64_t s2_elems, uint32_t b0, uint32_t b1, uint32_t b2);
