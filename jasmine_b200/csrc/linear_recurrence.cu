@@ -357,10 +357,10 @@ __device__ __forceinline__ uint32_t rc_movmatrix(uint32_t x) {
 // left operands without a change of order: they pass through shared memory as bf16 pairs (hi, lo).  The four warps of a group
 // share the tokens of a chunk (16 each) for O and U and the key components (a quarter each) for the state, whose fp32 values
 // stay in their registers.  K and Q (slabs of 64 components in the 128-byte swizzle), V and the chunk matrices come in two
-// stages by bulk and TMA copies of one thread, whose waits are bounded; a segment's last, short chunk and heads that do not
+// stages by bulk and TMA copies of a warp of its own (a copy takes its thread 140 cycles to issue), whose waits are bounded; a segment's last, short chunk and heads that do not
 // fill their instance by 16-byte copies of all threads, which write zeros where there is nothing.  KT: 16-wide steps of the key components.
 template <int KT, bool DELTA>
-__global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ CUtensorMap map_qk, const __grid_constant__ CUtensorMap map_v, RecArgs a, RecDims d,
+__global__ void __launch_bounds__(288) rec_chunk_kernel(const __grid_constant__ CUtensorMap map_qk, const __grid_constant__ CUtensorMap map_v, RecArgs a, RecDims d,
                                                        const int32_t* __restrict__ seg_chunk0, const uint8_t* __restrict__ ws, int* err) {
     constexpr int KP = KT * 16 + 8, PAIRS = KT >= 4 ? KT / 4 : 1;  // pairs of 8 key components of the state per warp
     constexpr int SLABS = KT >= 4 ? KT / 4 : 1, TILE = SLABS * RC_SLAB;  // K or Q of a chunk
@@ -369,7 +369,8 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ 
     __shared__ __align__(8) uint64_t full[2];
     __shared__ int abort_flag;
     chain_trigger();
-    const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, cols = nthr / 8;
+    const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, cols = (nthr - 32) / 8;
+    const bool loader = tid >= nthr - 32;
     const int block = rc_block(DELTA), v_bytes = RC_C * cols * 2, stage_bytes = rc_stage(TILE, cols, DELTA);
     __nv_bfloat16* Sh = reinterpret_cast<__nv_bfloat16*>(rc_dyn + 2 * stage_bytes);  // [cols][KP]: state, hi
     __nv_bfloat16* Sl = Sh + cols * KP;
@@ -397,7 +398,7 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ 
         uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
         const int n = min(RC_C, len - ci * RC_C);
         const bool tiles = n == RC_C && kp == KT * 16;
-        if (tid == 0) {
+        if (loader && lane == 0) {
             uint64_t* bar = &full[ci & 1];
             tc::mbar_expect_tx(bar, (uint32_t)(block + (tiles ? 2 * TILE + v_bytes : 0)));
             if (tiles) {
@@ -433,7 +434,7 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ 
     const int lm = lane >> 3, lr = lane & 7, kc = (lane & 3) * 2, ar = mt * 16 + (lane >> 2);
     // accumulators: row (lane / 4, + 8) = state column, columns (lane % 4) * 2, + 1 = token or key component
     float* state = a.S + ((long long)a.seg_slot[seg] * d.H + h) * kp * vp;
-    const bool fresh = a.seg_pos0[seg] == 0, keeps = w * PAIRS < KT;
+    const bool fresh = a.seg_pos0[seg] == 0, keeps = !loader && w * PAIRS < KT;
     float S[2 * PAIRS][4];
 #pragma unroll
     for (int j = 0; j < 2 * PAIRS; ++j)
@@ -467,6 +468,11 @@ __global__ void __launch_bounds__(256) rec_chunk_kernel(const __grid_constant__ 
         cp_async_wait<0>();
         __syncthreads();  // K, Q, V are here, the state is published, the other stage used up
         if (ci + 1 < n_chunks) load(ci + 1);
+        if (loader) {
+            if (DELTA && !__syncthreads_and(1)) { ok = false; break; }
+            if (!__syncthreads_and(1)) { ok = false; break; }
+            continue;
+        }
         ok = tc::mbar_wait(&full[ci & 1], (ci >> 1) & 1, &abort_flag, err, RC_ERR_FULL);
         const uint8_t* st = rc_dyn + (ci & 1) * stage_bytes;
         const uint32_t kb = smem_u32(st), qb = kb + TILE, vb = qb + TILE, tb = vb + v_bytes;
@@ -932,7 +938,7 @@ static jsm_status chunk_go(const RecArgs& a, const RecDims& d, const RecChunks& 
     if (s != JSM_OK) return s;
     s = make_tmap_bf16_2d(&map_v, a.qkv, (uint64_t)n_tok, (uint64_t)d.conv_cols(), (uint64_t)d.conv_cols(), RC_C, cols, false);
     if (s != JSM_OK) return s;
-    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((d.vp() + cols - 1) / cols, d.H, n_segs), dim3(cols * 8), smem, st, map_qk, map_v, a, d, ch.seg_chunk0,
+    JSM_CUDA_CHECK(launch_chained(rec_chunk_kernel<KT, DELTA>, dim3((d.vp() + cols - 1) / cols, d.H, n_segs), dim3(cols * 8 + 32), smem, st, map_qk, map_v, a, d, ch.seg_chunk0,
                                   static_cast<const uint8_t*>(ch.ws), tc_error_word()));
     JSM_LAUNCH_CHECK();
     return JSM_OK;

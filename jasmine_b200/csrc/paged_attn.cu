@@ -208,6 +208,7 @@ constexpr int AM_STAGES = 3;
 constexpr int AM_WARPS = 4;
 constexpr int AM_THREADS = (AM_WARPS + 1) * 32;
 constexpr int AM_MAX_SPLITS = 64;
+__host__ __device__ constexpr int am_pitch(int vp) { return vp + 4; }  // a row of partial sums: the columns, its maximum, its sum
 constexpr int AM_ERR_FULL = 61, AM_ERR_EMPTY = 62;
 
 struct AttnArgs {
@@ -418,10 +419,10 @@ __global__ void __launch_bounds__(AM_THREADS, 1) attn_paged_mma_kernel(AttnArgs 
         const float gv = a.gate ? a.gate[(long long)t * d.H + h] : 1.0f;
         a.out[(long long)t * d.out_cols() + h * d.vdim + c] = __float2bfloat16_rn(acc * f / fmaf(L, f, exp2f(s2 - top)) * gv);
     };
-    float* part = a.part + (long long)(tile * d.G + g) * a.splits * R * (VP + 2);
+    float* part = a.part + (long long)(tile * d.G + g) * a.splits * R * am_pitch(VP);
     for (int e = threadIdx.x; e < n_rows * VP; e += AM_THREADS) {
         const int r = e / VP, c = e % VP;
-        if (c >= d.vdim) continue;
+        if (live == 1 && c >= d.vdim) continue;
         float M = -INFINITY, acc = 0.0f, L = 0.0f;
 #pragma unroll
         for (int w = 0; w < AM_WARPS; ++w) M = fmaxf(M, sm_m[w][r]);
@@ -434,7 +435,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) attn_paged_mma_kernel(AttnArgs 
         if (live == 1) {
             finish(r, c, acc, L, M);
         } else {
-            float* dst = part + ((long long)sp * R + r) * (VP + 2);
+            float* dst = part + ((long long)sp * R + r) * am_pitch(VP);
             dst[c] = acc;
             if (c == 0) { dst[VP] = M; dst[VP + 1] = L; }
         }
@@ -450,19 +451,39 @@ __global__ void __launch_bounds__(AM_THREADS, 1) attn_paged_mma_kernel(AttnArgs 
     }
     __syncthreads();
     if (!is_last) return;
-    for (int e = threadIdx.x; e < n_rows * VP; e += AM_THREADS) {
-        const int r = e / VP, c = e % VP;
-        if (c >= d.vdim) continue;
-        const float* src = part + (long long)r * (VP + 2);
-        const long long stride = (long long)R * (VP + 2);
-        float M = -INFINITY, acc = 0.0f, L = 0.0f;
-        for (int s = 0; s < live; ++s) M = fmaxf(M, __ldcg(src + s * stride + VP));
-        for (int s = 0; s < live; ++s) {
-            const float ms = __ldcg(src + s * stride + VP), f = ms == -INFINITY ? 0.0f : exp2f(ms - M);
-            acc = fmaf(f, __ldcg(src + s * stride + c), acc);
-            L = fmaf(f, __ldcg(src + s * stride + VP + 1), L);
+    // weight of every split's partial sum per row, then four columns per thread
+    const long long stride = (long long)R * am_pitch(VP);
+    float* wts = reinterpret_cast<float*>(ring);  // [R][AM_MAX_SPLITS]
+    for (int r = warp; r < n_rows; r += AM_WARPS + 1) {
+        float ms[2], ls[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const float* src = part + (long long)(lane + 32 * i) * stride + r * am_pitch(VP) + VP;
+            const bool on = lane + 32 * i < live;
+            ms[i] = on ? __ldcg(src) : -INFINITY;
+            ls[i] = on ? __ldcg(src + 1) : 0.0f;
         }
-        finish(r, c, acc, L, M);
+        const float M = warp_max(fmaxf(ms[0], ms[1])), f0 = exp2f(ms[0] - M), f1 = exp2f(ms[1] - M);  // (M is finite: a row sees its own key)
+        const float L = warp_sum(fmaf(f0, ls[0], f1 * ls[1]));
+        wts[r * AM_MAX_SPLITS + lane] = f0;
+        wts[r * AM_MAX_SPLITS + lane + 32] = f1;
+        if (lane == 0) { sm_m[0][r] = M; sm_l[0][r] = L; }
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < n_rows * (VP / 4); e += AM_THREADS) {
+        const int r = e / (VP / 4), c = e % (VP / 4) * 4;
+        const float* src = part + r * am_pitch(VP) + c;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int s = 0; s < live; ++s) {
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(src + s * stride));
+            const float f = wts[r * AM_MAX_SPLITS + s];
+            acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
+        }
+        const float o4[4] = {acc.x, acc.y, acc.z, acc.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (c + i < d.vdim) finish(r, c + i, o4[i], sm_l[0][r], sm_m[0][r]);
     }
 }
 
@@ -492,7 +513,7 @@ static int attn_splits(const AttnDims& d, int n_tiles, int max_keys) {
     const int pages = max_keys / PAGE + 2, ctas = std::max(1, n_tiles * d.G);
     return std::max(1, std::min({2 * sm_count() / ctas, pages / 2, AM_MAX_SPLITS}));
 }
-size_t attn_part_floats(const AttnDims& d) { return (size_t)2 * sm_count() * 32 * (am_vp(d) + 2); }
+size_t attn_part_floats(const AttnDims& d) { return (size_t)2 * sm_count() * 32 * am_pitch(am_vp(d)); }
 int attn_counters() { return 2 * sm_count(); }
 
 template <int NB, int VT>
@@ -533,7 +554,7 @@ jsm_status attn_paged_launch(bool f32, const AttnDims& d, const AttnWeights& w, 
     a.max_pages = cache.max_pages;
     a.splits = attn_splits(d, tl.n_tiles, tl.max_keys);
     a.scale_log2 = d.scale * LOG2E;
-    if (a.splits > 1 && ((size_t)tl.n_tiles * d.G * a.splits * tl.rows * (am_vp(d) + 2) > sc.part_floats || tl.n_tiles * d.G > sc.n_counters))
+    if (a.splits > 1 && ((size_t)tl.n_tiles * d.G * a.splits * tl.rows * am_pitch(am_vp(d)) > sc.part_floats || tl.n_tiles * d.G > sc.n_counters))
         JSM_FAIL(JSM_INVALID_ARG, "attention: workspace of %zu floats for %d tiles x %d heads in %d splits", sc.part_floats, tl.n_tiles, d.G, a.splits);
     const int vs = d.vs();
     if (tl.rows == 8) return vs == 1 ? launch_attn_mma<1, 4>(a, d, tl.n_tiles, st) : vs == 2 ? launch_attn_mma<1, 8>(a, d, tl.n_tiles, st)
