@@ -179,7 +179,7 @@ jsm_status jsm_linear_bf16(const void* d_X, const void* d_W, const float* d_bias
  * forwards).  The packed image stores every 128-feature x 64-k tile as one contiguous 16 KB block in the
  * shared-memory layout of the tensor cores, tiles in stream order, so that the kernel reads the matrix as one linear
  * stream split evenly over all SMs.  paired != 0 packs a [2N, K] matrix of N gate rows followed by N up rows for
- * epilogue 3 (silu(gate)*up), N being the number of gate rows.
+ * epilogue 3 (silu(gate)*up) or 6 (gelu(gate)*up, the tanh form; bf16 output), N being the number of gate rows.
  * jsm_linear_packed_bytes: size of the packed image.  jsm_linear_pack / jsm_linear_unpack convert between the
  * reference's [out, in] layout and the packed image.  jsm_linear_bf16_packed: any T (chunks of 256 tokens);
  * N % 4 == 0, K % 8 == 0.  The tiles that several CTAs share are reduced through a per-device workspace that the calls

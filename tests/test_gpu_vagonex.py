@@ -286,6 +286,45 @@ def test_delta_rule_remembers_the_first_token(dtype):
     far_token(cfg, w, dtype)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_delta_rule_with_keys_that_repeat(dtype):
+    """The same token over and over, beta near 1: every write takes back the one before it, the chunk's triangular system is as
+    full as it gets; then two tokens in turn, and others."""
+    cfg = vu.config([vu.delta(heads=2, kv_heads=1, dim=32, vdim=32, conv=1)], alpha=0.4)
+    w = vu.random_weights(cfg, 65)
+    emb = vu.widen(w["embed"]).reshape(72, 48)
+    emb[:, 0] = 1.0
+    b = np.zeros((2, 48))
+    b[0, 0], b[1, 0] = 3.0, 1.0  # (x is three times the table)
+    w.update({"embed": vu.bf16_bits(emb), "l0.mix.b": vu.bf16_bits(b), "l0.mix.A_log": vu.bf16_bits(np.array([-9.0, -3.0]))})
+    toks = [5] * 150 + [6, 7] * 60 + vu.tokens(90, 72, 66)
+    want = want_logits(cfg, w, toks)
+    m = vu.build(cfg, w, dtype)
+    for sizes in ([360], [100, 1, 2, 257], [3]):
+        assert vu.error(vu.run_portions(m, toks, sizes), want) < TOL[dtype], sizes
+    m.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_decays_from_nothing_to_everything(dtype):
+    """Steps that forget the whole state beside steps that keep it: running sums of their logarithms must not drown the rest."""
+    cfg = vu.config([vu.delta(heads=2, kv_heads=1, dim=32, vdim=32, conv=2)], alpha=0.4)
+    w = vu.random_weights(cfg, 67)
+    emb = vu.widen(w["embed"]).reshape(72, 48)
+    emb[:, 0] = 0.0
+    emb[:4, 0] = 10.0  # tokens 0 .. 3 forget
+    a = np.zeros((2, 48))
+    a[:, 0] = 3.0
+    w.update({"embed": vu.bf16_bits(emb), "l0.mix.a": vu.bf16_bits(a), "l0.mix.A_log": vu.bf16_bits(np.array([2.0, 1.0])),
+              "l0.mix.dt_bias": vu.bf16_bits(np.array([-7.0, -8.0]))})
+    toks = vu.tokens(300, 72, 68)
+    want = want_logits(cfg, w, toks)
+    m = vu.build(cfg, w, dtype)
+    for sizes in ([300], [64, 7, 1], [1]):
+        assert vu.error(vu.run_portions(m, toks, sizes), want) < TOL[dtype], sizes
+    m.close()
+
+
 # ---- whole models -----------------------------------------------------------------------------------------------------
 def mixed_config():
     layers = [vu.delta(ff=88), vu.lightning(heads=2, dim=24, vdim=16, ff=40), vu.attention(heads=6, kv_heads=3, size=50, scaling=vu.YARN, ff=56),
